@@ -16,6 +16,7 @@ tree by the two functions below.
 from __future__ import annotations
 
 import concurrent.futures as cf
+import hashlib
 import os
 import shutil
 import subprocess
@@ -59,19 +60,20 @@ def _run(cmd: list[str]) -> None:
 
 
 def build_cuda(force: bool = False, verbose: bool = False, extra_flags: list[str] | None = None,
-               variant: str = "") -> Path:
+               variant: str = "", sources: tuple[str, ...] | None = None) -> Path:
     """Builds `_C/libzb_cuda.so`.  With `variant` (and usually `extra_flags`) the same sources are built into
     `_C/libzb_cuda_<variant>.so` with objects of their own - e.g. `variant="bc", extra_flags=["-DZB_BOUNDS_CHECK"]`,
-    the checking build that `ZB_CUDA_LIB` then selects."""
+    the checking build that `ZB_CUDA_LIB` then selects.  `sources` (stems of `csrc/*.cu`) restricts the library to a part
+    of the kernels; the objects are shared with the whole library's."""
     nvcc = _nvcc()
     if nvcc is None:
         raise RuntimeError("nvcc not found; cannot build libzb_cuda.so")
-    srcs = sorted(CSRC.glob("*.cu"))
+    srcs = sorted(CSRC.glob("*.cu")) if sources is None else [CSRC / f"{n}.cu" for n in sorted(sources)]
     hdrs = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
     target = OUT / (f"libzb_cuda_{variant}.so" if variant else "libzb_cuda.so")
     if not force and _newer(target, srcs + hdrs):
         return target
-    obj_dir = OBJ.parent / (f"obj_{variant}" if variant else "obj")
+    obj_dir = OBJ.parent / (f"obj_{variant}" if variant and sources is None else "obj")
     OUT.mkdir(parents=True, exist_ok=True)
     obj_dir.mkdir(parents=True, exist_ok=True)
     flags = NVCC_FLAGS + (extra_flags or []) + (["-Xptxas", "-v"] if verbose else [])
@@ -92,6 +94,18 @@ def build_cuda(force: bool = False, verbose: bool = False, extra_flags: list[str
     ctypes.CDLL(str(tmp), mode=getattr(os, "RTLD_NOW", 2))
     os.replace(tmp, target)
     return target
+
+
+def ensure_cuda(sources: tuple[str, ...] | None = None) -> Path:
+    """An up-to-date library with at least the kernels of `sources`: the whole one if it is built, else - in a fresh
+    checkout - one compiled from `sources` alone, so that a program that serves one model family compiles no more than
+    that family needs."""
+    hdrs = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
+    whole = OUT / "libzb_cuda.so"
+    if sources is None or _newer(whole, sorted(CSRC.glob("*.cu")) + hdrs):
+        return build_cuda()
+    name = hashlib.sha256(",".join(sorted(sources)).encode()).hexdigest()[:8]
+    return build_cuda(variant=f"part_{name}", sources=sources)
 
 
 def build_host(force: bool = False) -> Path:

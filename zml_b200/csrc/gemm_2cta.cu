@@ -258,7 +258,7 @@ zb_gemm_2cta_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
           for (int j = 0; j < 32; ++j)
             if (whole || q + j < prm.n) v[j] += __bfloat162float(prm.bias[q + j]);
         }
-        if (prm.epi.swiglu) {
+        if (prm.epi.swiglu == ZB_ACT_SWIGLU) {
           // columns interleave gate and up: 16 outputs at columns q / 2 ..
           __nv_bfloat16* op = reinterpret_cast<__nv_bfloat16*>(prm.out) + static_cast<size_t>(p) * prm.ldo + (q >> 1);
           if (whole) {
@@ -294,6 +294,10 @@ zb_gemm_2cta_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
             for (int j = 0; j < 32; ++j)
               if (q + j < prm.n) v[j] += __bfloat162float(prm.residual[o + j]);
           }
+        }
+        if (prm.epi.swiglu == ZB_ACT_RELU2) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = zb_plain_act(v[j], ZB_ACT_RELU2);
         }
         if (prm.out_f32) {
           float* op = reinterpret_cast<float*>(prm.out) + o;

@@ -102,7 +102,8 @@ zb_gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_p,
   constexpr bool kGeneric = PLAN != 1;      // whole-tile / stream-K code present
   const float* const epi_in_sumsq = kEpi ? prm.epi.in_sumsq : nullptr;
   float* const epi_out_sumsq = kEpi ? prm.epi.out_sumsq : nullptr;
-  const int epi_swiglu = kEpi ? prm.epi.swiglu : 0;
+  const bool epi_swiglu = kEpi && prm.epi.swiglu == ZB_ACT_SWIGLU;
+  const bool epi_relu2 = kEpi && prm.epi.swiglu == ZB_ACT_RELU2;
   const unsigned long long epi_pf_bytes = kEpi ? prm.epi.pf_bytes : 0ull;
   constexpr int kStages = stages_for(BN, SWAP);
   constexpr int kStageBytes = stage_bytes(BN);
@@ -684,6 +685,7 @@ zb_gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_p,
 #pragma unroll
               for (int c = 0; c < KC; ++c) v += tv[i][c];            // ascending rank: deterministic
               v = v * sc[i] + bs[i] + rsd[i];
+              if (epi_relu2) v = zb_plain_act(v, ZB_ACT_RELU2);
               const int col = off[i] / kBlockP, row = off[i] - col * kBlockP;
               const int pp = pt * kBlockP + row, qq = q0 + col;
               if (epi_swiglu) {
@@ -1069,6 +1071,10 @@ zb_gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_p,
           swiglu_store_chunk(c0, v);
         } else if (p < prm.rows_p) {
           finish_chunk(c0, v);
+          if (epi_relu2) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = zb_plain_act(v[j], ZB_ACT_RELU2);
+          }
           store_chunk(c0, v, prm.out);
         }
       };
@@ -1154,6 +1160,10 @@ zb_gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_p,
                 v4[2] += f1.x;
                 v4[3] += f1.y;
               }
+              if (epi_relu2) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) v4[e] = zb_plain_act(v4[e], ZB_ACT_RELU2);
+              }
               if (prm.out_f32) {
                 *reinterpret_cast<float4*>(reinterpret_cast<float*>(prm.out) + o) = make_float4(v4[0], v4[1], v4[2], v4[3]);
               } else {
@@ -1166,6 +1176,7 @@ zb_gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_p,
                 if (pb + e < prm.rows_p) {
                   float x = v4[e];
                   if (prm.residual) x += __bfloat162float(prm.residual[o + e]);
+                  if (epi_relu2) x = zb_plain_act(x, ZB_ACT_RELU2);
                   if (prm.out_f32) reinterpret_cast<float*>(prm.out)[o + e] = x;
                   else reinterpret_cast<__nv_bfloat16*>(prm.out)[o + e] = __float2bfloat16(x);
                 }
@@ -1730,7 +1741,7 @@ int launch_row_sumsq(const void* x, int rows, int d, long long ld, float* out, c
 int check_epi(const ZbGemmEpi* epi, int m, int n, int ldo, int out_f32, const void* residual, const void* bias) {
   if (epi == nullptr) return 0;
   if (epi->in_sumsq != nullptr && (epi->in_parts < 1 || epi->in_ld < m)) return -15;
-  if (epi->swiglu) {
+  if (epi->swiglu == ZB_ACT_SWIGLU) {
     // gate / up pairs: an even number of weight rows, bf16 output of n / 2 columns, no bias or residual
     if ((n % 2) != 0 || out_f32 || residual != nullptr || bias != nullptr || (ldo % 8) != 0 || epi->out_sumsq != nullptr) return -16;
   }
@@ -1883,7 +1894,7 @@ int zb_row_sumsq(const void* x, int rows, int d, long long ld, float* out, void*
 
 // zb_gemm_bf16 with the epilogue options of ZbGemmEpi (host_api.h) passed as scalars:
 //   in_sumsq [in_parts][in_ld], inv_d, eps  -> accumulators of token t scaled by rsqrt(sum * inv_d + eps)
-//   swiglu                                  -> interleaved gate / up rows, n / 2 output columns
+//   swiglu                                  -> 1: interleaved gate / up rows, n / 2 output columns; 4: relu(x)^2
 //   out_sumsq [..][out_ld], *out_parts      -> partial sums of squares of the output rows and how many parts
 //   pf_ptr, pf_bytes                        -> bytes to pull into L2 behind this kernel's own loads
 int zb_gemm_bf16_epi(const void* a, const void* w, void* out, const void* residual, const void* bias, int m, int n, int k,
@@ -1898,7 +1909,8 @@ int zb_gemm_bf16_epi(const void* a, const void* w, void* out, const void* residu
   epi.in_ld = in_ld;
   epi.in_inv_d = in_inv_d;
   epi.in_eps = in_eps;
-  epi.swiglu = swiglu ? 1 : 0;
+  if (swiglu != ZB_ACT_NONE && swiglu != ZB_ACT_SWIGLU && swiglu != ZB_ACT_RELU2) return -16;
+  epi.swiglu = swiglu;
   epi.out_sumsq = out_sumsq;
   epi.out_ld = out_ld;
   epi.pf_ptr = pf_bytes ? pf_ptr : nullptr;

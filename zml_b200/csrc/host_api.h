@@ -47,6 +47,7 @@ struct ZbArContext {
 //              compute rmsnorm(a) * w^T without a normalisation kernel (zml/nn.zig:486-493).
 //   swiglu   : the rows of `w` interleave gate and up (row 2 i = gate_i, row 2 i + 1 = up_i); the output has
 //              n / 2 columns, out[t][i] = silu(gate_i) * up_i (examples/llm/models/llama/model.zig:491-496).
+//              The value is a ZbMoeAct code: ZB_ACT_SWIGLU, or ZB_ACT_RELU2 for relu(x)^2 of a plain projection.
 //   out_sumsq: the kernel writes partial sums of squares of its (bf16-rounded) output rows, [parts][out_ld];
 //              `parts` is reported by the entry point.
 //   pf_ptr   : contiguous bytes (the next GEMM's weights) that the kernel pulls into L2 once its own operand

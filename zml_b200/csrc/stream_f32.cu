@@ -1,0 +1,354 @@
+// Layer glue of decoders that keep the residual stream in fp32:
+//
+//   zb_embedding_f32   gathers table rows (bf16 or fp32) into the fp32 stream
+//   zb_post_norm       x <- layernorm(alpha * x + y) * w, the normalisation behind a sublayer ("norm after the sum");
+//                      without y a plain layer norm.  For decode steps the same launch continues with the input
+//                      convolution of the next layer (one token per sequence: everything it needs is in the row and
+//                      in the sequence's state)
+//   zb_stream_conv     that input convolution over a varlen batch: h = x + conv(x), causal and per channel, and for
+//                      token-shift mixers the interpolations h + (h_prev - h) * mu of h with the previous token's h
+//
+// Sums, norms and convolutions are fp32; what a projection reads is written as bf16 or fp32.  The state of a sequence
+// is the last `rows` rows of x (taps - 1 of them, or taps when the previous token's h is needed: it is computed again
+// from x rather than stored).
+#include "act.cuh"
+#include "host_api.h"
+
+namespace {
+constexpr uint32_t kKernelEmbeddingF32 = 26;
+constexpr uint32_t kKernelStreamConv = 27;
+constexpr int kMaxMix = 5;
+constexpr int kMaxTaps = 8;
+
+template <typename W>
+__global__ void __launch_bounds__(256) zb_embedding_f32_kernel(const int32_t* __restrict__ ids, const W* __restrict__ table,
+                                                               float* __restrict__ out, int d, int vocab) {
+  zb_pdl_launch();
+  zb_pdl_wait();
+  const int t = blockIdx.x;
+  int id = ids[t];
+  if (id < 0 || id >= vocab) {
+    (void)ZB_BC_OK(id, vocab, kKernelEmbeddingF32, 1);
+    id = 0;
+  }
+  const W* src = table + static_cast<size_t>(id) * d;
+  float* dst = out + static_cast<size_t>(t) * d;
+  for (int i = threadIdx.x; i < d; i += 256) dst[i] = zb_ld_act(src + i);
+}
+
+// ------------------------------------------------------------------------------------------ convolution
+struct ConvArgs {
+  const float* w;          // [d, taps], tap taps - 1 on the current token
+  float* state;            // [slots, rows, d]: the last `rows` inputs, oldest first
+  const int32_t* slots;    // [num_seqs]
+  const float* mu;         // [nmix, d] or null
+  void* out;               // h [T, ld], or the nmix interpolations [nmix][T, ld]
+  long long ld;
+  long long plane;         // elements between interpolations
+  int taps;
+  int rows;
+  int nmix;                // 0: h itself
+  int d;
+};
+
+template <typename A>
+ZB_DEVICE void emit_h(const ConvArgs& a, long long t, int c, float h, float h_prev) {
+  A* out = reinterpret_cast<A*>(a.out) + t * a.ld + c;
+  if (a.nmix == 0) {
+    zb_st_act(out, h);
+    return;
+  }
+  const float delta = h_prev - h;
+  for (int m = 0; m < a.nmix; ++m) zb_st_act(out + m * a.plane, h + delta * a.mu[static_cast<size_t>(m) * a.d + c]);
+}
+
+// One thread owns a channel and walks a block of kConvRows tokens of one sequence.
+constexpr int kConvRows = 32;
+
+template <typename A>
+__global__ void __launch_bounds__(128) zb_stream_conv_kernel(const float* __restrict__ x, const ConvArgs a, const ZbVarlen b) {
+  zb_pdl_launch();
+  zb_pdl_wait();
+  const int c = blockIdx.x * 128 + threadIdx.x;
+  int s, blk;
+  if (c >= a.d || !zb_find_block(b, kConvRows, blockIdx.y, s, blk)) return;
+  const int slot = a.slots[s];
+  if (!ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelStreamConv, 1)) return;
+  const int t0 = b.q_start[s], n = b.q_start[s + 1] - t0;
+  const bool fresh = b.seq_lens[s] - n <= 0;
+  float* st = a.state + static_cast<size_t>(slot) * a.rows * a.d + c;
+  // input `i` tokens after the launch's first token of this sequence (negative: before it)
+  auto input = [&](int i) -> float {
+    if (i >= 0) return x[static_cast<size_t>(t0 + i) * a.d + c];
+    return fresh || i < -a.rows ? 0.f : st[static_cast<size_t>(a.rows + i) * a.d];
+  };
+  const int taps = a.taps;
+  float w[kMaxTaps], win[kMaxTaps];           // win[j]: the input `taps - 1 - j` tokens before the current one
+#pragma unroll
+  for (int j = 0; j < kMaxTaps; ++j) {
+    w[j] = j < taps ? a.w[static_cast<size_t>(c) * taps + j] : 0.f;
+    win[j] = 0.f;
+  }
+  const int i0 = blk * kConvRows, i1 = min(n, i0 + kConvRows);
+  auto conv = [&]() {
+    float acc = 0.f;
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j)
+      if (j < taps) acc += w[j] * win[j];
+    return acc;
+  };
+  float h_prev = 0.f;
+  if (a.nmix > 0) {
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j)
+      if (j < taps) win[j] = input(i0 - taps + j);
+    float cur = 0.f;
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j)
+      if (j == taps - 1) cur = win[j];
+    h_prev = cur + conv();
+  } else {
+#pragma unroll
+    for (int j = 1; j < kMaxTaps; ++j)
+      if (j < taps) win[j] = input(i0 - taps + j);
+  }
+  for (int i = i0; i < i1; ++i) {
+    const float cur = x[static_cast<size_t>(t0 + i) * a.d + c];
+#pragma unroll
+    for (int j = 0; j < kMaxTaps - 1; ++j) win[j] = win[j + 1];
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j)
+      if (j == taps - 1) win[j] = cur;
+    const float h = cur + conv();
+    emit_h<A>(a, t0 + i, c, h, h_prev);
+    h_prev = h;
+  }
+  // The block that reads the old state also writes the new one: no other thread touches this channel's state.
+  if (blk == 0) {
+    float keep[kMaxTaps];
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j)
+      if (j < a.rows) keep[j] = input(n - a.rows + j);
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j)
+      if (j < a.rows) st[static_cast<size_t>(j) * a.d] = keep[j];
+  }
+}
+
+// ------------------------------------------------------------------------------------------ post norm
+struct PostNormArgs {
+  const void* y;           // sublayer output, bf16 or fp32, or null
+  long long ldy;
+  int y_f32;
+  const float* x;          // [T, d]
+  float alpha;
+  const float* w;          // [d]
+  float eps;
+  float* x_out;            // [T, d] or null (may be x)
+  void* act;               // [T, ld_act] or null: the same rows in the activation type
+  long long ld_act;
+  int d;
+  int conv;                // 1: one token per sequence, continue with the convolution
+};
+
+ZB_DEVICE float block_sum_256(float v, float* red) {
+  v = zb_warp_sum(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) tot += red[i];
+  return tot;
+}
+
+// NV values per thread; VEC: groups of four consecutive channels (d a multiple of 4), else one channel each.
+template <typename A, int NV, bool VEC>
+__global__ void __launch_bounds__(256) zb_post_norm_kernel(const PostNormArgs p, const ConvArgs a, const ZbVarlen b) {
+  zb_pdl_launch();
+  zb_pdl_wait();
+  __shared__ float red[8];
+  const long long t = blockIdx.x;
+  const int d = p.d;
+  auto channel = [&](int i) { return VEC ? (threadIdx.x + 256 * (i >> 2)) * 4 + (i & 3) : threadIdx.x + 256 * i; };
+  const float* xr = p.x + t * d;
+  float v[NV];
+#pragma unroll
+  for (int i = 0; i < NV; i += VEC ? 4 : 1) {
+    const int c = channel(i);
+    if constexpr (VEC) {
+      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < d) {
+        f = *reinterpret_cast<const float4*>(xr + c);
+        f.x *= p.alpha; f.y *= p.alpha; f.z *= p.alpha; f.w *= p.alpha;
+        if (p.y != nullptr && p.y_f32) {
+          const float4 g = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.y) + t * p.ldy + c);
+          f.x += g.x; f.y += g.y; f.z += g.z; f.w += g.w;
+        } else if (p.y != nullptr) {
+          const uint2 g = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.y) + t * p.ldy + c);
+          const float2 lo = zb_unpack_bf16x2(g.x), hi = zb_unpack_bf16x2(g.y);
+          f.x += lo.x; f.y += lo.y; f.z += hi.x; f.w += hi.y;
+        }
+      }
+      v[i] = f.x; v[i + 1] = f.y; v[i + 2] = f.z; v[i + 3] = f.w;
+    } else {
+      v[i] = 0.f;
+      if (c < d) {
+        v[i] = p.alpha * xr[c];
+        if (p.y != nullptr)
+          v[i] += p.y_f32 ? reinterpret_cast<const float*>(p.y)[t * p.ldy + c]
+                          : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.y)[t * p.ldy + c]);
+      }
+    }
+  }
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) sum += v[i];
+  const float mean = block_sum_256(sum, red) / static_cast<float>(d);
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    if (channel(i) < d) {
+      v[i] -= mean;
+      sq += v[i] * v[i];
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum_256(sq, red) / static_cast<float>(d) + p.eps);
+#pragma unroll
+  for (int i = 0; i < NV; i += VEC ? 4 : 1) {
+    const int c = channel(i);
+    if (c >= d) continue;
+    if constexpr (VEC) {
+      const float4 g = *reinterpret_cast<const float4*>(p.w + c);
+      v[i] *= inv * g.x; v[i + 1] *= inv * g.y; v[i + 2] *= inv * g.z; v[i + 3] *= inv * g.w;
+      if (p.x_out != nullptr) *reinterpret_cast<float4*>(p.x_out + t * d + c) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+      if (p.act != nullptr) {
+        A* o = reinterpret_cast<A*>(p.act) + t * p.ld_act + c;
+        if constexpr (sizeof(A) == 2) {
+          if ((p.ld_act & 3) == 0) {
+            *reinterpret_cast<uint2*>(o) = make_uint2(zb_pack_bf16x2(v[i], v[i + 1]), zb_pack_bf16x2(v[i + 2], v[i + 3]));
+            continue;
+          }
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) zb_st_act(o + e, v[i + e]);
+      }
+    } else {
+      v[i] *= inv * p.w[c];
+      if (p.x_out != nullptr) p.x_out[t * d + c] = v[i];
+      if (p.act != nullptr) zb_st_act(reinterpret_cast<A*>(p.act) + t * p.ld_act + c, v[i]);
+    }
+  }
+  if (!p.conv) return;
+  const int s = static_cast<int>(t);
+  const int slot = a.slots[s];
+  if (!ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelStreamConv, 2)) return;
+  const bool fresh = b.seq_lens[s] - 1 <= 0;
+  float* st0 = a.state + static_cast<size_t>(slot) * a.rows * d;
+  const int taps = a.taps;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = channel(i);
+    if (c >= d) continue;
+    float* st = st0 + c;
+    float hist[kMaxTaps];                    // hist[j]: the j-th row of the state
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j) hist[j] = (j < a.rows && !fresh) ? st[static_cast<size_t>(j) * d] : 0.f;
+    const int off = a.rows - (taps - 1);     // 1 when the state also reaches the previous token's first tap
+    float h = 0.f, hp = 0.f;
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j) {
+      if (j < taps) {
+        const float w = a.w[static_cast<size_t>(c) * taps + j];
+        if (off == 1) hp += w * hist[j];
+        float in = v[i];
+        if (j < taps - 1) in = off == 1 ? hist[j + 1 < kMaxTaps ? j + 1 : j] : hist[j];
+        h += w * in;
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j)
+      if (off == 1 && j == taps - 1) hp += hist[j];
+    emit_h<A>(a, t, c, v[i] + h, hp);
+#pragma unroll
+    for (int j = 0; j < kMaxTaps; ++j) {
+      if (j < a.rows - 1) st[static_cast<size_t>(j) * d] = hist[j + 1 < kMaxTaps ? j + 1 : j];
+      else if (j == a.rows - 1) st[static_cast<size_t>(j) * d] = v[i];
+    }
+  }
+}
+
+template <typename A, bool VEC>
+int launch_post_norm(const PostNormArgs& p, const ConvArgs& a, const ZbVarlen& b, int tokens, cudaStream_t s) {
+  const int per = (p.d + 255) / 256;
+  cudaError_t e;
+  if (per <= 4) e = zb_launch(zb_post_norm_kernel<A, 4, VEC>, dim3(tokens), dim3(256), 0, s, p, a, b);
+  else if (per <= 8) e = zb_launch(zb_post_norm_kernel<A, 8, VEC>, dim3(tokens), dim3(256), 0, s, p, a, b);
+  else if (per <= 16) e = zb_launch(zb_post_norm_kernel<A, 16, VEC>, dim3(tokens), dim3(256), 0, s, p, a, b);
+  else if (per <= 32) e = zb_launch(zb_post_norm_kernel<A, 32, VEC>, dim3(tokens), dim3(256), 0, s, p, a, b);
+  else if (per <= 64) e = zb_launch(zb_post_norm_kernel<A, 64, VEC>, dim3(tokens), dim3(256), 0, s, p, a, b);
+  else return -70;
+  zb_count_launch(1);
+  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+}
+
+ConvArgs conv_args(const float* w, float* state, const int32_t* slots, const float* mu, void* out, long long ld, long long plane,
+                   int taps, int rows, int nmix, int d) {
+  return ConvArgs{w, state, slots, mu, out, ld, plane, taps, rows, nmix, d};
+}
+
+bool conv_ok(int taps, int rows, int nmix) {
+  return taps >= 1 && taps <= kMaxTaps && nmix >= 0 && nmix <= kMaxMix && rows == (nmix > 0 ? taps : taps - 1);
+}
+}  // namespace
+
+extern "C" {
+
+int zb_embedding_f32(const int32_t* ids, const void* table, int table_f32, float* out, int tokens, int d, int vocab, void* stream) {
+  if (tokens <= 0) return 0;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const cudaError_t e =
+      table_f32 ? zb_launch(zb_embedding_f32_kernel<float>, dim3(tokens), dim3(256), 0, s, ids, reinterpret_cast<const float*>(table), out, d, vocab)
+                : zb_launch(zb_embedding_f32_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, s, ids,
+                            reinterpret_cast<const __nv_bfloat16*>(table), out, d, vocab);
+  zb_count_launch(1);
+  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+}
+
+// h = x + conv(x) over a varlen batch; num_blocks >= sum over sequences of ceil(tokens / 32).
+int zb_stream_conv(const float* x, const float* w, float* state, const int32_t* slots, const float* mu, void* out, int act_f32,
+                   long long ld, long long plane, int taps, int rows, int nmix, int d, const int32_t* q_start,
+                   const int32_t* seq_lens, int num_seqs, int num_blocks, void* stream) {
+  if (num_seqs <= 0 || num_blocks <= 0) return 0;
+  if (!conv_ok(taps, rows, nmix)) return -70;
+  const ConvArgs a = conv_args(w, state, slots, mu, out, ld, plane, taps, rows, nmix, d);
+  const ZbVarlen b = {q_start, seq_lens, num_seqs};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid((d + 127) / 128, num_blocks);
+  const cudaError_t e = act_f32 ? zb_launch(zb_stream_conv_kernel<float>, grid, dim3(128), 0, s, x, a, b)
+                                : zb_launch(zb_stream_conv_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, x, a, b);
+  zb_count_launch(1);
+  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+}
+
+// x_out = layernorm(alpha * x + y) * w (row-wise); `conv_w` non-null: one token per sequence, and the row goes on
+// through the convolution described by the remaining arguments (see zb_stream_conv).
+int zb_post_norm(const void* y, long long ldy, int y_f32, const float* x, float alpha, const float* w, float eps, float* x_out,
+                 void* act, long long ld_act, int act_f32, int tokens, int d, const float* conv_w, float* state,
+                 const int32_t* slots, const float* mu, void* out, long long ld, long long plane, int taps, int rows, int nmix,
+                 const int32_t* seq_lens, void* stream) {
+  if (tokens <= 0) return 0;
+  const PostNormArgs p = {y, ldy, y_f32, x, alpha, w, eps, x_out, act, ld_act, d, conv_w != nullptr ? 1 : 0};
+  ConvArgs a = {};
+  ZbVarlen b = {nullptr, seq_lens, tokens};
+  if (conv_w != nullptr) {
+    if (!conv_ok(taps, rows, nmix)) return -70;
+    a = conv_args(conv_w, state, slots, mu, out, ld, plane, taps, rows, nmix, d);
+  }
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const bool vec = d % 4 == 0 && (y == nullptr || ldy % 4 == 0) && (reinterpret_cast<uintptr_t>(y) & 15) == 0;
+  if (act_f32) return vec ? launch_post_norm<float, true>(p, a, b, tokens, s) : launch_post_norm<float, false>(p, a, b, tokens, s);
+  return vec ? launch_post_norm<__nv_bfloat16, true>(p, a, b, tokens, s) : launch_post_norm<__nv_bfloat16, false>(p, a, b, tokens, s);
+}
+
+}  // extern "C"

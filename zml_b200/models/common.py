@@ -59,13 +59,16 @@ def parse_config(cls, source: Union[str, dict]):
 MODEL_TYPES = {
     "llama": "llama", "qwen3_5": "qwen3_5", "qwen3_5_text": "qwen3_5", "qwen3_5_moe": "qwen3_5_moe",
     "qwen3_5_moe_text": "qwen3_5_moe", "lfm2": "lfm2", "qwen3": "qwen3", "qwen2": "qwen3",
-    "qwen3_moe": "qwen3_moe", "mistral": "llama",
+    "qwen3_moe": "qwen3_moe", "mistral": "llama", "dopurax": "dopurax",
 }
 
 
 def detect_model_type(config: dict) -> str:
-    """examples/llm/models.zig:189-194: pick the implementation from `model_type`."""
+    """examples/llm/models.zig:189-194: pick the implementation from `model_type` (or, where a config names its design
+    instead, from `architecture`)."""
     mt = config.get("model_type")
+    if mt is None and isinstance(config.get("architecture"), str):
+        mt = config["architecture"].lower()
     if mt is None and "text_config" in config:
         mt = config["text_config"].get("model_type")
     if mt not in MODEL_TYPES:

@@ -26,6 +26,7 @@ from .. import ops
 from ..nn import rotary as rope_mod
 from ..parallel.comm import Comm
 from . import common
+from .decoder import AttnMeta, DecoderModel  # noqa: F401  (AttnMeta: part of this module's interface)
 
 
 @dataclass
@@ -116,25 +117,6 @@ PRESETS = {
 }
 
 
-@dataclass
-class AttnMeta:
-    """Per-step attention metadata in the shapes of the reference's paged API
-    (zml/attention/paged_attention.zig:19-293): block_table {b,p}, seq_lens {b},
-    query_start_len {b+1}, slot_mapping {tokens}."""
-    is_prefill: bool
-    positions: torch.Tensor
-    slot_mapping: torch.Tensor
-    block_table: torch.Tensor
-    seq_lens: torch.Tensor
-    q_start: Optional[torch.Tensor] = None
-    total_q_blocks: Optional[int] = None
-    num_splits: Optional[int] = None
-    max_seq_len: Optional[int] = None
-    logits_rows: Optional[torch.Tensor] = None    # rows of the hidden state that need logits
-    state_slots: Optional[torch.Tensor] = None    # {b} slot of every sequence in a model's recurrent-state pool
-    q_start_host: Optional[list] = None           # host copy of q_start (prefill), for splitting a chunk by sequences
-
-
 class LayerWeights:
     __slots__ = ("input_norm", "qkv", "qkv_bias", "q_norm", "k_norm", "o", "post_norm", "gate_up", "down",
                  "extra")
@@ -144,15 +126,12 @@ class LayerWeights:
             setattr(self, s, None)
 
 
-class LlamaModel:
+class LlamaModel(DecoderModel):
     """Weights of one tensor-parallel rank plus the forward pass over a flattened token batch."""
 
     def __init__(self, config: LlamaConfig, comm: Optional[Comm] = None, device="cpu",
                  dtype=torch.bfloat16):
-        self.config = config
-        self.comm = comm or Comm.single()
-        self.device = torch.device(device)
-        self.dtype = dtype
+        super().__init__(config, comm, device, dtype)
         c, p, r = config, self.comm.world, self.comm.rank
         if c.num_attention_heads % p != 0:
             raise ValueError(f"{c.num_attention_heads} heads not divisible by TP={p}")
@@ -162,20 +141,12 @@ class LlamaModel:
         self.hkv = self.kv_rng[1] - self.kv_rng[0]
         self.f_rng = common.shard_range(c.intermediate_size, r, p)
         self.f_local = self.f_rng[1] - self.f_rng[0]
-        # vocab-parallel lm_head: every rank holds v_per rows; rows past the vocabulary (last ranks, when the
-        # vocabulary does not divide) are zero rows whose logits are masked to -inf
-        self.v_per = (c.vocab_size + p - 1) // p
-        self.v_rng = (min(c.vocab_size, r * self.v_per), min(c.vocab_size, (r + 1) * self.v_per))
-        self.v_pad = self.v_per - (self.v_rng[1] - self.v_rng[0])
         self.fused_layout = False     # see prepare_fused
         opts = c.rope_opts()
         self.rope_layout = opts.layout.value
         self.rot_dim = opts.scaling.partial_rotary_dim(c.hd)
         self.attn_factor = opts.scaling.attention_scaling()
         self.inv_freq = rope_mod.inv_freq(c.hd, opts).to(self.device)
-        self.embed = None
-        self.final_norm = None
-        self.lm_head = None
         self.layers: list[LayerWeights] = []
 
     # ------------------------------------------------------------------ weights
@@ -218,11 +189,6 @@ class LlamaModel:
             lw.down = rw((d, c.intermediate_size), b + 6, cols=self.f_rng)
             self.layers.append(lw)
         return self
-
-    def _pad_lm_head(self) -> None:
-        if self.v_pad > 0 and self.comm.world > 1 and self.lm_head.shape[0] < self.v_per:
-            pad = torch.zeros((self.v_pad, self.lm_head.shape[1]), dtype=self.lm_head.dtype, device=self.lm_head.device)
-            self.lm_head = torch.cat([self.lm_head, pad], 0)
 
     def load(self, store, prefix: str = "", platform=None) -> "LlamaModel":
         """Loads this rank's shards from a TensorStore view (HF names).  Only the byte ranges
@@ -506,45 +472,4 @@ class LlamaModel:
         if rows is not None:
             x = x.index_select(0, rows.long() if rows.dtype != torch.int64 else rows)
         n = ops.rmsnorm(x, self.final_norm, self.config.rms_norm_eps)
-        if self.v_pad > 0 and self.comm.world > 1 and self.lm_head.shape[0] < self.v_per:
-            self._pad_lm_head()         # model families that fill `lm_head` themselves
-        lg = ops.gemm(n, self.lm_head, out_dtype=torch.float32, static_w=True)
-        if self.v_pad > 0 and self.comm.world > 1:
-            lg[:, self.v_per - self.v_pad:] = float("-inf")
-        return lg
-
-    def sample(self, logits, strategy: common.SamplingStrategy, seed: int = 0, step: int = 0, rng=None):
-        """Token ids int32 [B] from vocab-parallel logits.  `rng`: device-side {seed, draw counter} of
-        `ops.topk_sample` (the serving engine's, so that graph replays draw fresh noise)."""
-        comm = self.comm
-        rng = rng if (rng is not None and logits.is_cuda) else None
-        if comm.world == 1:
-            if strategy.topk <= 1:
-                return ops.argmax(logits)
-            return ops.topk_sample(logits, strategy.topk, strategy.temperature, seed, step, rng=rng)
-        if strategy.topk <= 1:
-            if comm.fused is not None and logits.is_cuda and comm.fused.can_argmax_tp(logits.shape[0]):
-                return comm.fused.argmax_tp(logits, comm.rank * self.v_per)     # candidates exchanged inside the kernel
-            idx = ops.argmax(logits)
-            val = logits.gather(1, idx.long()[:, None])[:, 0]
-            vals = comm.all_gather(val[None])                   # [P, B]
-            idxs = comm.all_gather((idx + self.comm.rank * self.v_per)[None])
-            best = vals.argmax(0)
-            return idxs.gather(0, best[None])[0].to(torch.int32)
-        # Every rank ranks its own columns (column j of rank r is token r * v_per + j; padding columns are -inf) and
-        # only the k best (value, token) pairs per row travel: the k best of their union are the k best of the whole
-        # vocabulary, in the same order, so the draw below equals the draw on gathered logits at 1 / (v_per / k) of the bytes.
-        k = min(strategy.topk, logits.shape[1])
-        vals, idx = ops.topk(logits, k)
-        cand_v = comm.all_gather(vals.contiguous(), dim=1).contiguous()
-        cand_i = comm.all_gather((idx + comm.rank * self.v_per).to(torch.int32).contiguous(), dim=1)
-        pos = ops.topk_sample(cand_v, strategy.topk if strategy.topk <= cand_v.shape[1] else cand_v.shape[1],
-                              strategy.temperature, seed, step, rng=rng)
-        return cand_i.gather(1, pos.long()[:, None])[:, 0].to(torch.int32)
-
-    def forward(self, ids, meta: AttnMeta, kv_cache, strategy: Optional[common.SamplingStrategy] = None,
-                seed: int = 0, step: int = 0, rng=None):
-        """ids int32 [T] -> sampled tokens int32 [rows] (one per sequence)."""
-        x = self.hidden_states(ids, meta, kv_cache)
-        lg = self.logits(x, meta.logits_rows)
-        return self.sample(lg, strategy or common.SamplingStrategy(), seed, step, rng)
+        return self.head_logits(n)

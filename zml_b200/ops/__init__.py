@@ -76,7 +76,7 @@ def interleave_gate_up(gate_up: torch.Tensor) -> torch.Tensor:
 
 def gemm(a, w, residual=None, bias=None, out=None, out_dtype=None, force_splits: int = 0, static_w: bool = False,
          row_stats: RowStats | None = None, eps: float = 1e-5, swiglu: bool = False, emit_stats: bool = False,
-         prefetch=None):
+         prefetch=None, act: str | None = None):
     """out[M,N] = a[M,K] @ w[N,K]^T (+ bias[N]) (+ residual[M,N]).
 
     `w` is stored [N, K] (the safetensors layout of every HF linear weight), so both
@@ -91,28 +91,46 @@ def gemm(a, w, residual=None, bias=None, out=None, out_dtype=None, force_splits:
     `swiglu` - the rows of `w` interleave gate and up (`interleave_gate_up`), the result is
     silu(gate) * up, [M, N / 2];
     `emit_stats` - also returns the RowStats of the (rounded) output: the call returns (out, stats);
-    `prefetch` - a tensor (the next GEMM's weights) pulled into L2 behind this kernel's own loads.
+    `prefetch` - a tensor (the next GEMM's weights) pulled into L2 behind this kernel's own loads;
+    `act` - "relu2": the square of relu of the result.
+
+    float32 operands run in fp32 throughout (gemm_f32.cu; no residual or row statistics).  K and N need not be multiples
+    of 8 (the copies of the bf16 kernels move 16 bytes): `w` may be stored with its columns padded with zeros
+    (`pad_k`), and `a` is padded to match.
     """
+    code = _ACTIVATIONS[act]
     if not _cuda(a):
         scale = row_stats.scale(a.shape[1], eps) if row_stats is not None else None
-        r = reference.gemm(a, w, residual, bias, out_dtype, scale, swiglu)
+        if w.shape[1] > a.shape[1]:
+            w = w[:, :a.shape[1]]
+        r = reference.gemm(a, w, residual, bias, out_dtype if act is None else torch.float32, scale, swiglu)
+        if act is not None:
+            r = torch.relu(r).square().to(out_dtype or a.dtype)
         if out is not None:
             out.copy_(r)
             r = out
         return (r, RowStats(reference.row_sumsq(r)[None], 1)) if emit_stats else r
+    if a.dtype == torch.float32:
+        return _gemm_f32(a, w, residual, bias, out, code, row_stats is not None or swiglu or emit_stats)
     _need_bf16(a, w, residual, bias)
+    if a.shape[1] % 8 or a.stride(0) % 8:
+        a = torch.nn.functional.pad(a, (0, -a.shape[1] % 8))
+        if w.shape[1] < a.shape[1]:
+            w = pad_k(w)
     m, k = a.shape
     n, k2 = w.shape
     assert k == k2, (a.shape, w.shape)
     assert a.stride(1) == 1 and w.stride(1) == 1
     odt = out_dtype or torch.bfloat16
     if out is None:
-        out = torch.empty((m, n // 2 if swiglu else n), dtype=odt, device=a.device)
+        cols = n // 2 if swiglu else n
+        ld = (cols + 3) // 4 * 4 if odt == torch.float32 else (cols + 7) // 8 * 8      # rows start on 16 bytes
+        out = torch.empty((m, ld), dtype=odt, device=a.device)[:, :cols]
     assert out.stride(1) == 1 and out.dtype in (torch.bfloat16, torch.float32)
     if residual is not None:
         assert residual.stride(0) == out.stride(0) and residual.stride(1) == 1
     flags = (1 if out.dtype == torch.float32 else 0) | (2 if static_w else 0)
-    if row_stats is None and not swiglu and not emit_stats and prefetch is None:
+    if row_stats is None and not swiglu and not emit_stats and prefetch is None and not code:
         rc = _lib.lib().zb_gemm_bf16(
             _ptr(a), _ptr(w), _ptr(out), _ptr(residual), _ptr(bias), m, n, k, a.stride(0), w.stride(0),
             out.stride(0), flags, force_splits, _lib.stream_ptr())
@@ -128,12 +146,33 @@ def gemm(a, w, residual=None, bias=None, out=None, out_dtype=None, force_splits:
     rc = _lib.lib().zb_gemm_bf16_epi(
         _ptr(a), _ptr(w), _ptr(out), _ptr(residual), _ptr(bias), m, n, k, a.stride(0), w.stride(0), out.stride(0), flags,
         force_splits, _ptr(row_stats.parts) if row_stats is not None else 0, row_stats.n if row_stats is not None else 0,
-        row_stats.parts.stride(0) if row_stats is not None else 0, 1.0 / k, float(eps), int(swiglu),
+        row_stats.parts.stride(0) if row_stats is not None else 0, 1.0 / k, float(eps), code or int(swiglu),
         _ptr(stats_out), m, C.byref(parts), _ptr(prefetch), pf_bytes, _lib.stream_ptr())
     _lib.check(rc, "zb_gemm_bf16_epi")
     if emit_stats:
         assert 0 < parts.value <= RowStats.MAX_PARTS, parts.value
         return out, RowStats(stats_out, parts.value)
+    return out
+
+
+# epilogue activation codes (csrc/common.cuh: ZbMoeAct); SwiGLU has an argument of its own because it halves the columns
+_ACTIVATIONS = {None: 0, "relu2": 4}
+
+
+def pad_k(w: torch.Tensor) -> torch.Tensor:
+    """[N, K] with zero columns up to a multiple of 8."""
+    return torch.nn.functional.pad(w, (0, -w.shape[1] % 8)) if w.shape[1] % 8 else w
+
+
+def _gemm_f32(a, w, residual, bias, out, act: int, unsupported: bool):
+    if unsupported or residual is not None:
+        raise TypeError("the fp32 GEMM has no residual, row-statistics or SwiGLU epilogue")
+    m, n, k = a.shape[0], w.shape[0], a.shape[1]
+    assert w.dtype == torch.float32 and a.stride(1) == 1 and w.stride(1) == 1 and k <= w.shape[1] <= k + 7, (a.shape, w.shape)
+    if out is None:
+        out = torch.empty((m, n), dtype=torch.float32, device=a.device)
+    _lib.check(_lib.lib().zb_gemm_f32(_ptr(a), a.stride(0), _ptr(w), w.stride(0), _ptr(bias), _ptr(out), out.stride(0), m, n, k, act,
+                                      _lib.stream_ptr()), "zb_gemm_f32")
     return out
 
 

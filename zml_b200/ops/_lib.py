@@ -67,6 +67,7 @@ _SIGS = {
     "zb_gemm_bf16_epi": (c_i, [c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_i, c_i, c_f, c_f,
                                c_i, c_p, c_i, c_p, c_p, c_ull, c_p]),
     "zb_gemm_scratch_needed": (c_sz, [c_i, c_i, c_i, c_i]),
+    "zb_gemm_f32": (c_i, [c_p, c_ll, c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_p]),
     "zb_row_sumsq": (c_i, [c_p, c_i, c_i, c_ll, c_p, c_p]),
     "zb_rmsnorm": (c_i, [c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_ll, c_ll, c_f, c_i, c_p]),
     "zb_rope_kvwrite": (c_i, [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_ll, c_i, c_i, c_i, c_i,
@@ -109,6 +110,14 @@ def path() -> Path:
     return _PATH
 
 
+def use(path: Path) -> None:
+    """Selects the library file; before the first call of `lib()`."""
+    global _PATH
+    if _LIB is not None and Path(path) != _PATH:
+        raise KernelError(f"{_PATH} is already loaded")
+    _PATH = Path(path)
+
+
 def lib():
     """Loads the library once.  Raises if it has not been built."""
     global _LIB
@@ -123,13 +132,13 @@ def lib():
             f"{_PATH} is missing: run `python -m zml_b200._build` (needs nvcc); "
             "ops on CUDA tensors never fall back to PyTorch")
     l = C.CDLL(str(_PATH))
-    for name, (res, args) in _SIGS.items():
+    # a library built for one model family exports a part of the symbols: calling one it lacks is an AttributeError
+    part = "_part_" in _PATH.name
+    for name, (res, args) in list(_OPTIONAL_SIGS.items()) + list(_SIGS.items()):
+        if (part or name in _OPTIONAL_SIGS) and not hasattr(l, name):
+            continue
         fn = getattr(l, name)
         fn.restype, fn.argtypes = res, args
-    for name, (res, args) in _OPTIONAL_SIGS.items():
-        if hasattr(l, name):
-            fn = getattr(l, name)
-            fn.restype, fn.argtypes = res, args
     _LIB = l
     return l
 
@@ -144,7 +153,9 @@ STATUS_NAMES = {0: "ok", 1: "mbarrier wait timed out", 2: "flag wait timed out",
 KERNEL_NAMES = {1: "gemm_bf16", 2: "paged_decode", 3: "paged_prefill", 4: "gemm_ar_fused",
                 5: "comm_barrier", 6: "moe_grouped_gemm", 7: "moe_a2a", 8: "wait_probe", 9: "moe_grouped_gemm_w4",
                 10: "moe_combine", 11: "allreduce_ll", 12: "allreduce_mm", 13: "paged_prefill_tc", 14: "gemm_2cta", 15: "argmax_tp",
-                20: "rope_kvwrite", 21: "embedding", 22: "decode_advance", 24: "causal_conv1d", 25: "gated_delta_scan"}
+                20: "rope_kvwrite", 21: "embedding", 22: "decode_advance", 24: "causal_conv1d", 25: "gated_delta_scan",
+                26: "embedding_f32", 27: "stream_conv", 28: "latent_prep", 29: "latent_attend", 30: "latent_gather", 31: "wkv_scan",
+                32: "latent_prefill_tc", 33: "latent_decode"}
 
 
 class BoundsError(KernelError):

@@ -1,0 +1,186 @@
+"""Latent attention: keys and values are per-head projections of one low-rank latent per token, and only the latent and
+one rotated key part shared by all heads are cached (libzb_cuda.so: latent_attention.cu).
+
+Two formulations of the same attention, chosen by `latent_attention`:
+
+* in the latent space: the queries are taken through the key projection (`absorb_q`), attend to the cached latents as
+  one key/value head, and the result goes through the value projection (`absorb_out`).  Reads each cached row once for
+  all heads: decode.
+* expanded (`prefill`): the visible latents of the batch are gathered from the pages and projected to keys and
+  values of every head, which costs a third of the products in the latent space when a chunk has many queries per key.
+
+bf16 runs on the tensor cores, fp32 on the FMA pipes; CPU tensors take the plain torch branch.
+"""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from . import _lib
+
+_p, _i, _ll, _f = C.c_void_p, C.c_int, C.c_longlong, C.c_float
+_lib.register_signature("zb_latent_prep", _i, [_p, _ll, _p, _p, _p, _p, _p, _p, _ll, _p, _ll, _ll, _f, _i, _i, _i, _i, _i, _i, _p])
+_lib.register_signature("zb_latent_absorb", _i, [_p, _ll, _ll, _p, _ll, _p, _ll, _ll, _p, _ll, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _p])
+_lib.register_signature("zb_latent_attend", _i, [_p, _p, _ll, _p, _ll, _p, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _i, _i, _p])
+_lib.register_signature("zb_latent_gather", _i, [_p, _ll, _p, _i, _i, _p, _p, _i, _p, _ll, _i, _i, _i, _i, _i, _p])
+_lib.register_signature("zb_latent_q_pack", _i, [_p, _ll, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p])
+
+
+def _ptr(t: Optional[torch.Tensor]):
+    return None if t is None else t.data_ptr()
+
+
+def _up(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+@dataclass(frozen=True)
+class LatentDims:
+    """Sizes and constants of one latent-attention layer (heads: this rank's)."""
+    heads: int
+    dim: int            # unrotated query / key dimensions per head
+    rot: int            # rotated ones (the key part is shared by all heads)
+    vdim: int
+    rank: int           # latent size
+    q_rank: int
+    window: int         # keys a position sees, itself included; <= 0: all
+    scale: float
+    base: float         # of the rotation frequencies
+
+    @property
+    def rot_off(self) -> int:
+        return _up(self.rank, 16)
+
+    @property
+    def row(self) -> int:
+        """Elements of a cache row: latent and rotated part, each padded to 16."""
+        return self.rot_off + _up(self.rot, 16)
+
+    def inv_freq(self, device) -> torch.Tensor:
+        i = torch.arange(0, self.rot, 2, dtype=torch.float64)
+        return (float(self.base) ** (-i / self.rot)).to(torch.float32).to(device)
+
+
+def rotate_reference(x, positions, inv_freq):
+    """Adjacent pairs of x [..., T, rot] (T second from the right or with heads between) turned by position * frequency."""
+    a = positions.float()[:, None] * inv_freq[None]
+    shape = (x.shape[0],) + (1,) * (x.dim() - 2) + (inv_freq.shape[0],)
+    cs, sn = torch.cos(a).reshape(shape), torch.sin(a).reshape(shape)
+    u, v = x[..., 0::2].float(), x[..., 1::2].float()
+    return torch.stack([u * cs - v * sn, v * cs + u * sn], -1).reshape(x.shape)
+
+
+def _rms(x, w, eps):
+    return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * w
+
+
+# ---------------------------------------------------------------------------- norms, rotation, cache write
+def prep(proj, q_norm, c_norm, inv_freq, positions, slots, cache, eps: float, d: LatentDims):
+    """proj [T, >= q_rank + rank + rot] (query latent | latent | shared key part): returns the normed query latent
+    [T, q_rank] and writes the normed latent and the rotated key part into cache [pages, page, row] at `slots`."""
+    t = proj.shape[0]
+    if not proj.is_cuda:
+        cq = _rms(proj[:, :d.q_rank].float(), q_norm, eps).to(proj.dtype)
+        c = _rms(proj[:, d.q_rank:d.q_rank + d.rank].float(), c_norm, eps)
+        kr = rotate_reference(proj[:, d.q_rank + d.rank:d.q_rank + d.rank + d.rot], positions, inv_freq)
+        flat = cache.view(-1, cache.shape[-1])
+        ok = slots >= 0
+        idx = slots[ok].long()
+        flat[idx, :d.rank] = c[ok].to(cache.dtype)
+        flat[idx, d.rot_off:d.rot_off + d.rot] = kr[ok].to(cache.dtype)
+        return cq
+    assert proj.stride(1) == 1 and cache.is_contiguous() and cache.dtype == proj.dtype and cache.shape[-1] == d.row
+    cq = torch.empty((t, d.q_rank), dtype=proj.dtype, device=proj.device)
+    _lib.check(_lib.lib().zb_latent_prep(
+        _ptr(proj), proj.stride(0), _ptr(q_norm), _ptr(c_norm), _ptr(inv_freq), _ptr(positions), _ptr(slots), _ptr(cq), cq.stride(0),
+        _ptr(cache), d.row, cache.shape[0] * cache.shape[1], float(eps), d.q_rank, d.rank, d.rot, d.rot_off,
+        int(proj.dtype == torch.float32), t, _lib.stream_ptr()), "zb_latent_prep")
+    return cq
+
+
+# ---------------------------------------------------------------------------- latent space
+def absorb_q(q, w_uk_t, inv_freq, positions, d: LatentDims):
+    """q [T, H * (dim + rot)] -> [T, H, row]: the unrotated part through w_uk_t [H, rank, dim], the rotated part rotated."""
+    t, hd = q.shape[0], d.dim + d.rot
+    new = torch.empty if d.rot_off == d.rank and d.row == d.rot_off + d.rot else torch.zeros
+    out = new((t, d.heads, d.row), dtype=q.dtype, device=q.device)
+    if not q.is_cuda:
+        qh = q.reshape(t, d.heads, hd)
+        out[..., :d.rank] = torch.einsum("thk,hnk->thn", qh[..., :d.dim].float(), w_uk_t.float()).to(q.dtype)
+        out[..., d.rot_off:d.rot_off + d.rot] = rotate_reference(qh[..., d.dim:], positions, inv_freq).to(q.dtype)
+        return out
+    assert q.stride(1) == 1 and w_uk_t.is_contiguous()
+    _lib.check(_lib.lib().zb_latent_absorb(
+        _ptr(q), q.stride(0), hd, _ptr(w_uk_t), d.dim, _ptr(out), out.stride(0), d.row, None, 0, _ptr(inv_freq), _ptr(positions), d.rot,
+        d.dim, d.rot_off, t, d.heads, d.rank, d.dim, int(q.dtype == torch.float32), _lib.stream_ptr()), "zb_latent_absorb")
+    return out
+
+
+def absorb_out(o, w_uv, gate, d: LatentDims):
+    """o [T, H, rot_off] (latent-space results) -> sigmoid(gate) * (o w_uv^T) [T, H * vdim]; w_uv [H, vdim, rank],
+    gate [T, H * vdim] (row stride free)."""
+    t = o.shape[0]
+    if not o.is_cuda:
+        y = torch.einsum("thk,hnk->thn", o[..., :d.rank].float(), w_uv.float()).reshape(t, -1)
+        return (y * torch.sigmoid(gate.float())).to(o.dtype)
+    out = torch.empty((t, d.heads * d.vdim), dtype=o.dtype, device=o.device)
+    assert gate.stride(1) == 1 and w_uv.is_contiguous() and gate.dtype == o.dtype
+    _lib.check(_lib.lib().zb_latent_absorb(
+        _ptr(o), o.stride(0), o.stride(1), _ptr(w_uv), d.rank, _ptr(out), out.stride(0), d.vdim, _ptr(gate), gate.stride(0), None, None, 0,
+        0, 0, t, d.heads, d.vdim, d.rank, int(o.dtype == torch.float32), _lib.stream_ptr()), "zb_latent_absorb")
+    return out
+
+
+def attend_reference(q, cache, block_table, q_start, seq_lens, d: LatentDims):
+    out = torch.zeros((q.shape[0], d.heads, d.rot_off), dtype=q.dtype, device=q.device)
+    flat = cache.view(-1, cache.shape[-1])
+    page = cache.shape[1]
+    qs, sl = q_start.tolist(), seq_lens.tolist()
+    for s in range(len(sl)):
+        a, b, n = qs[s], qs[s + 1], sl[s]
+        if b <= a or n <= 0:
+            continue
+        key = torch.arange(n)
+        rows = flat[block_table[s].long()[key // page] * page + key % page].float()
+        pos = torch.arange(n - (b - a), n)
+        vis = key[None] <= pos[:, None]
+        if d.window > 0:
+            vis &= key[None] > pos[:, None] - d.window
+        sc = torch.einsum("thc,kc->htk", q[a:b].float(), rows) * d.scale
+        pr = torch.softmax(sc.masked_fill(~vis[None], float("-inf")), -1)
+        out[a:b, :, :d.rank] = torch.einsum("htk,kc->thc", pr, rows[:, :d.rank]).to(q.dtype)
+    return out
+
+
+def attend(q, cache, block_table, q_start, seq_lens, d: LatentDims, decode: bool = False, num_splits: int = 1):
+    """Windowed causal attention of q [T, H, row] (`absorb_q`) against the cached rows; a sequence's queries are its last
+    tokens.  Returns [T, H, rot_off]."""
+    if not q.is_cuda:
+        return attend_reference(q, cache, block_table, q_start, seq_lens, d)
+    t = q.shape[0]
+    out = torch.empty((t, d.heads, d.rot_off), dtype=q.dtype, device=q.device)
+    assert block_table.is_contiguous() and cache.dtype == q.dtype and q.is_contiguous()
+    _lib.check(_lib.lib().zb_latent_attend(
+        _ptr(q), _ptr(cache), d.row, _ptr(out), d.rot_off, _ptr(block_table), block_table.shape[1], cache.shape[1], d.heads, d.rank, d.rot,
+        d.rot_off, d.window, float(d.scale), _ptr(q_start), _ptr(seq_lens), seq_lens.shape[0], t, int(q.dtype == torch.float32),
+        _lib.stream_ptr()), "zb_latent_attend")
+    return out
+
+
+def decode_plan_splits(batch: int, d: LatentDims, max_seq_len: int) -> int:
+    return 1
+
+
+# ---------------------------------------------------------------------------- the layer's attention
+def latent_attention(q, gate, w_uk_t, w_ukv, inv_freq, cache, meta, d: LatentDims):
+    """sigmoid(gate) * attention of one step: q [T, H * (dim + rot)] unrotated, gate [T, H * vdim], w_uk_t [H, rank, dim],
+    w_ukv [H dim + H vdim, rank]; `meta` is the step's AttnMeta, the new tokens' cache rows are already written."""
+    q_start = meta.q_start
+    if q_start is None:
+        q_start = torch.arange(q.shape[0] + 1, dtype=torch.int32, device=q.device)
+    ql = absorb_q(q, w_uk_t, inv_freq, meta.positions, d)
+    o = attend(ql, cache, meta.block_table, q_start, meta.seq_lens, d, decode=not meta.is_prefill, num_splits=meta.num_splits or 1)
+    return absorb_out(o, w_ukv[d.heads * d.dim:].view(d.heads, d.vdim, d.rank), gate, d)

@@ -1,7 +1,8 @@
 """Ops of the hybrid decoder layers: depthwise causal conv with a rolling cache, the gated
-delta rule scan, and the sigmoid output gate (libzb_cuda.so: linear_attn.cu).
+delta rule scan, and the sigmoid output gate (libzb_cuda.so: linear_attn.cu); the WKV
+recurrence with its low-rank decay (wkv.cu).
 
-All three run over the flattened varlen token batch the engine uses everywhere else:
+All of them run over the flattened varlen token batch the engine uses everywhere else:
 `q_start[S+1]` gives every sequence's token range in this launch, `seq_lens[S]` its length
 including those tokens (so `seq_lens - count == 0` marks a sequence that starts here and
 takes a zero state), `slots[S]` its row in the state pool.  On CPU tensors the functions
@@ -144,3 +145,92 @@ def sigmoid_gate_mul(x, gate):
                                         _lib.stream_ptr())
     _lib.check(rc, "zb_sigmoid_gate_mul")
     return x
+
+
+# ---------------------------------------------------------------------------- WKV
+_lib.register_signature("zb_wkv_can_fuse", _i, [_i])
+_lib.register_signature("zb_wkv_scan", _i, [_p, _p, _p, _p, _ll, _p, _ll, _p, _p, _p, _f, _p, _p, _p, _ll, _p, _i, _i, _i, _p, _p, _i,
+                                            _i, _p])
+_lib.register_signature("zb_tanh_linear", _i, [_p, _ll, _p, _ll, _i, _p, _ll, _i, _i, _i, _p])
+_lib.register_signature("zb_tanh_split", _i, [_p, _ll, _p, _i, _i, _i, _p])
+
+
+def wkv_scan_reference(r, k, v, g, z, w0, u, norm_w, eps, state, q_start, seq_lens, slots, heads, dim):
+    t = r.shape[0]
+    hd = lambda x: x.float().reshape(-1, heads, dim)
+    rf, kf, vf, gf = hd(r), hd(k), hd(v), hd(g)
+    decay = torch.exp(-torch.exp(hd(z) + w0.reshape(1, heads, dim)))
+    uu = u.reshape(heads, dim)
+    o = torch.zeros((t, heads, dim))
+    qs, sl, so = q_start.tolist(), seq_lens.tolist(), slots.tolist()
+    for s in range(len(sl)):
+        a, b = qs[s], qs[s + 1]
+        if b <= a:
+            continue
+        st = torch.zeros((heads, dim, dim)) if sl[s] - (b - a) <= 0 else state[so[s]].clone()     # [H, value, key]
+        for i in range(a, b):
+            kv = vf[i][:, :, None] * kf[i][:, None, :]
+            o[i] = torch.einsum("hvk,hk->hv", st + uu[:, None, :] * kv, rf[i])
+            st = st * decay[i][:, None, :] + kv
+        state[so[s]] = st
+    o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * norm_w.reshape(1, heads, dim) * (gf * torch.sigmoid(gf))
+    return o.reshape(t, heads * dim).to(r.dtype)
+
+
+# (sequence, head) pairs from which one CTA per pair fills the GPU (148 SMs, two CTAs each)
+WKV_FUSE_PAIRS = 296
+
+
+def wkv_scan(r, k, v, g, z, w0, u, norm_w, eps, state, q_start, seq_lens, slots, heads: int, dim: int, decode: bool = False, out=None):
+    """The WKV recurrence with its output norm and gate: r, k, v, g [T, heads * dim] (equal row strides), z fp32 the
+    decay's pre-activation (w = exp(-exp(z + w0))), u the current token's bonus, norm_w the output norm's weight (fp32
+    [heads * dim] each), state fp32 [slots, heads, dim (value), dim (key)] updated in place.  Returns [T, heads * dim]."""
+    if not r.is_cuda:
+        return wkv_scan_reference(r, k, v, g, z, w0, u, norm_w, eps, state, q_start, seq_lens, slots, heads, dim)
+    t, n = r.shape[0], heads * dim
+    if dim > 256:
+        raise ValueError(f"the WKV kernel takes heads of at most 256 channels, not {dim}")
+    assert r.stride(0) == k.stride(0) == v.stride(0) == g.stride(0) and r.dtype == k.dtype == v.dtype == g.dtype
+    assert z.dtype == torch.float32 and state.dtype == torch.float32 and state.is_contiguous()
+    if out is None:
+        out = torch.empty((t, n), dtype=r.dtype, device=r.device)
+    fuse = bool(_lib.lib().zb_wkv_can_fuse(dim)) and (decode or heads * seq_lens.shape[0] >= WKV_FUSE_PAIRS)
+    o = None if fuse else torch.empty((t, n), dtype=torch.float32, device=r.device)
+    _lib.check(_lib.lib().zb_wkv_scan(
+        _ptr(r), _ptr(k), _ptr(v), _ptr(g), r.stride(0), _ptr(z), z.stride(0), _ptr(w0), _ptr(u), _ptr(norm_w), float(eps), _ptr(state),
+        _ptr(slots), _ptr(out), out.stride(0), _ptr(o), int(r.dtype == torch.float32), heads, dim, _ptr(q_start), _ptr(seq_lens),
+        seq_lens.shape[0], t, _lib.stream_ptr()), "zb_wkv_scan")
+    return out
+
+
+# tokens up to which the low-rank product runs as fp32 dot products instead of a GEMM
+TANH_LINEAR_TOKENS = 64
+
+
+def split_weight(w: torch.Tensor) -> torch.Tensor:
+    """[N, R] -> [N, 2 R'] with R' = R rounded up to 8: the weight repeated, for `tanh_linear` on many tokens."""
+    half = (w.shape[1] + 7) // 8 * 8
+    p = torch.nn.functional.pad(w, (0, half - w.shape[1]))
+    return torch.cat([p, p], 1).contiguous()
+
+
+def tanh_linear(a, w, w_split=None):
+    """tanh(a) @ w^T with an fp32 result from a fp32 [T, R] and w [N, R]: the activation is not rounded to bf16.  On the
+    GPU few tokens take fp32 dot products, many take a bf16 GEMM over tanh(a) split into two bf16 pieces (`w_split`)."""
+    if not a.is_cuda:
+        return torch.tanh(a.float()) @ w.float().t()
+    t, rank = a.shape
+    n = w.shape[0]
+    l = _lib.lib()
+    if w.dtype == torch.bfloat16 and w_split is not None and t > TANH_LINEAR_TOKENS:
+        from . import gemm
+        half = w_split.shape[1] // 2
+        s = torch.empty((t, 2 * half), dtype=torch.bfloat16, device=a.device)
+        _lib.check(l.zb_tanh_split(_ptr(a), a.stride(0), _ptr(s), half, rank, t, _lib.stream_ptr()), "zb_tanh_split")
+        return gemm(s, w_split, out_dtype=torch.float32, static_w=True)
+    out = torch.empty((t, n), dtype=torch.float32, device=a.device)
+    for t0 in range(0, t, 32768):
+        t1 = min(t, t0 + 32768)
+        _lib.check(l.zb_tanh_linear(_ptr(a[t0:]), a.stride(0), _ptr(w), w.stride(0), int(w.dtype == torch.float32), _ptr(out[t0:]),
+                                    out.stride(0), t1 - t0, n, rank, _lib.stream_ptr()), "zb_tanh_linear")
+    return out

@@ -1,0 +1,148 @@
+"""Layer glue of decoders with an fp32 residual stream: embedding, the norm behind a sublayer, and the convolution in
+front of a mixer (libzb_cuda.so: stream_f32.cu).
+
+All of it works on the flattened varlen batch of the engine (`q_start`, `seq_lens`, `slots`, as in
+`ops.linear_attn`).  Activations that a projection reads are written in the model's dtype (bf16 or fp32); the stream,
+the norms, the convolution and its state are fp32.  CPU tensors take the plain torch branch of each function.
+"""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from . import _lib
+
+_p, _i, _ll, _f = C.c_void_p, C.c_int, C.c_longlong, C.c_float
+_lib.register_signature("zb_embedding_f32", _i, [_p, _p, _i, _p, _i, _i, _i, _p])
+_lib.register_signature("zb_stream_conv", _i, [_p, _p, _p, _p, _p, _p, _i, _ll, _ll, _i, _i, _i, _i, _p, _p, _i, _i, _p])
+_lib.register_signature("zb_post_norm", _i, [_p, _ll, _i, _p, _f, _p, _f, _p, _p, _ll, _i, _i, _i, _p, _p, _p, _p, _p, _ll, _ll,
+                                             _i, _i, _i, _p, _p])
+
+MAX_TAPS = 8
+CONV_BLOCK = 32          # tokens per block of the convolution kernel
+
+
+def _ptr(t: Optional[torch.Tensor]):
+    return None if t is None else t.data_ptr()
+
+
+def embedding_f32(ids, table):
+    """Rows of `table` (bf16 or fp32) as fp32 [T, d]."""
+    if not table.is_cuda:
+        return table[ids.long()].float()
+    assert ids.dtype == torch.int32 and table.is_contiguous()
+    out = torch.empty((ids.shape[0], table.shape[1]), dtype=torch.float32, device=table.device)
+    _lib.check(_lib.lib().zb_embedding_f32(_ptr(ids), _ptr(table), int(table.dtype == torch.float32), _ptr(out), ids.shape[0],
+                                           table.shape[1], table.shape[0], _lib.stream_ptr()), "zb_embedding_f32")
+    return out
+
+
+def layer_norm_reference(x, w, eps):
+    d = x.float() - x.float().mean(-1, keepdim=True)
+    return d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps) * w
+
+
+@dataclass
+class InputConv:
+    """The convolution in front of a mixer and what follows it: h = x + conv(x), and with `mu` [nmix, d] the
+    interpolations h + (h_prev - h) * mu_m of h with the previous token's h.  `state` is [slots, rows, d] fp32: the
+    last inputs x of every sequence, `rows_for(taps, nmix)` of them."""
+    w: torch.Tensor                       # [d, taps] fp32, tap taps - 1 on the current token
+    state: torch.Tensor
+    mu: Optional[torch.Tensor] = None
+
+    @staticmethod
+    def rows_for(taps: int, mixes: bool) -> int:
+        return taps if mixes else taps - 1
+
+    def nmix(self) -> int:
+        return 0 if self.mu is None else self.mu.shape[0]
+
+    def check(self) -> None:
+        d, taps = self.w.shape
+        if not 1 <= taps <= MAX_TAPS:
+            raise ValueError(f"the input convolution takes 1 to {MAX_TAPS} taps, not {taps}")
+        assert self.w.dtype == torch.float32 and self.w.is_contiguous() and self.state.is_contiguous()
+        assert self.state.shape[1:] == (self.rows_for(taps, self.mu is not None), d), self.state.shape
+
+    def alloc(self, tokens: int, dtype, device):
+        shape = (tokens, self.w.shape[0]) if self.mu is None else (self.nmix(), tokens, self.w.shape[0])
+        return torch.empty(shape, dtype=dtype, device=device)
+
+    def args(self, out):
+        """The trailing kernel arguments: out pointer, row stride, plane stride, taps, rows, nmix."""
+        return (_ptr(out), out.stride(-2), out.stride(0) if self.mu is not None else 0, self.w.shape[1], self.state.shape[1], self.nmix())
+
+
+def _stream_conv_reference(x, conv: InputConv, q_start, seq_lens, slots, dtype):
+    d, taps = conv.w.shape
+    rows = conv.state.shape[1]
+    out = conv.alloc(x.shape[0], dtype, x.device)
+    qs, sl, so = q_start.tolist(), seq_lens.tolist(), slots.tolist()
+    for s in range(len(sl)):
+        a, b = qs[s], qs[s + 1]
+        if b <= a:
+            continue
+        fresh = sl[s] - (b - a) <= 0
+        hist = torch.zeros((rows, d)) if fresh else conv.state[so[s]]
+        full = torch.cat([torch.zeros((taps - rows, d)), hist, x[a:b]], 0)             # [taps + n, d]
+        h = full[taps - 1:] + (full.unfold(0, taps, 1) * conv.w[None]).sum(-1)          # previous token's h, then n of them
+        if conv.mu is None:
+            out[a:b] = h[1:].to(dtype)
+        else:
+            out[:, a:b] = (h[None, 1:] + (h[:-1] - h[1:])[None] * conv.mu[:, None]).to(dtype)
+        conv.state[so[s]] = full[full.shape[0] - rows:]
+    return out
+
+
+def stream_conv(x, conv: InputConv, q_start, seq_lens, slots, dtype, num_blocks: Optional[int] = None):
+    """x [T, d] fp32 -> h [T, d] or the interpolations [nmix, T, d], in `dtype`; updates `conv.state`."""
+    conv.check()
+    if not x.is_cuda:
+        return _stream_conv_reference(x, conv, q_start, seq_lens, slots, dtype)
+    t, d = x.shape
+    assert x.is_contiguous() and x.dtype == torch.float32
+    out = conv.alloc(t, dtype, x.device)
+    nb = num_blocks if num_blocks is not None else t // CONV_BLOCK + seq_lens.shape[0]
+    ptr, ld, plane, taps, rows, nmix = conv.args(out)
+    _lib.check(_lib.lib().zb_stream_conv(_ptr(x), _ptr(conv.w), _ptr(conv.state), _ptr(slots), _ptr(conv.mu), ptr,
+                                         int(dtype == torch.float32), ld, plane, taps, rows, nmix, d, _ptr(q_start), _ptr(seq_lens),
+                                         seq_lens.shape[0], nb, _lib.stream_ptr()), "zb_stream_conv")
+    return out
+
+
+def post_norm(x, w, eps: float, y=None, alpha: float = 1.0, keep_x: bool = True, act_dtype=None,
+              conv: Optional[InputConv] = None, seq_lens=None, slots=None):
+    """layernorm(alpha * x + y) * w over rows of the fp32 stream x [T, d].  Returns (x_new or None, second):
+    `second` is the same rows in `act_dtype` when that is given, or - for a decode step, one token per sequence - what
+    `stream_conv` makes of them when `conv` is (then in `act_dtype` as well), all in one launch."""
+    t, d = x.shape
+    if not x.is_cuda:
+        z = alpha * x.float()
+        if y is not None:
+            z = z + y.float()
+        n = layer_norm_reference(z, w, eps)
+        if conv is not None:
+            q_start = torch.arange(t + 1, dtype=torch.int32)
+            return (n if keep_x else None), _stream_conv_reference(n, conv, q_start, seq_lens, slots, act_dtype)
+        return (n if keep_x else None), (n.to(act_dtype) if act_dtype is not None else None)
+    assert x.dtype == torch.float32 and x.is_contiguous() and w.dtype == torch.float32
+    assert y is None or (y.stride(1) == 1 and y.dtype in (torch.float32, torch.bfloat16))
+    x_new = torch.empty_like(x) if keep_x else None
+    act = out = None
+    cargs = (None, 0, 0, 0, 0, 0)
+    if conv is not None:
+        conv.check()
+        out = conv.alloc(t, act_dtype, x.device)
+        cargs = conv.args(out)
+    elif act_dtype is not None:
+        act = torch.empty((t, d), dtype=act_dtype, device=x.device)
+    c = conv
+    _lib.check(_lib.lib().zb_post_norm(
+        _ptr(y), y.stride(0) if y is not None else 0, int(y is not None and y.dtype == torch.float32), _ptr(x), float(alpha), _ptr(w),
+        float(eps), _ptr(x_new), _ptr(act), d, int(act_dtype == torch.float32), t, d, _ptr(c.w) if c else None,
+        _ptr(c.state) if c else None, _ptr(slots), _ptr(c.mu) if c else None, *cargs, _ptr(seq_lens), _lib.stream_ptr()), "zb_post_norm")
+    return x_new, (out if conv is not None else act)

@@ -26,7 +26,7 @@ import torch
 
 from .. import ops
 from ..models.common import SamplingStrategy
-from ..models.llama import AttnMeta
+from ..models.decoder import AttnMeta
 from ..ops import _lib
 
 
@@ -103,7 +103,7 @@ def _bucket(n: int) -> int:
 class Engine:
     def __init__(self, model, num_pages: int, page_size: int = 64, max_batch: int = 64,
                  max_seq_len: int = 4096, max_prefill_tokens: int = 8192, use_graphs: Optional[bool] = None,
-                 history_steps: int = 1024):
+                 history_steps: int = 1024, num_state_slots: Optional[int] = None):
         self.model = model
         self.device = model.device
         self.page_size = page_size
@@ -112,8 +112,7 @@ class Engine:
         self.max_pages = (max_seq_len + page_size - 1) // page_size
         self.max_prefill_tokens = max_prefill_tokens
         self.pool = PagePool(num_pages)
-        self.kv_cache = torch.zeros(model.kv_cache_shape(num_pages, page_size), dtype=model.dtype,
-                                    device=self.device)
+        self.kv_cache = model.alloc_kv_cache(num_pages, page_size)
         self.on_gpu = self.device.type == "cuda"
         self.use_graphs = self.on_gpu if use_graphs is None else (use_graphs and self.on_gpu)
         self.history_steps = history_steps
@@ -136,7 +135,7 @@ class Engine:
         self.d_rng = torch.zeros(2, dtype=torch.int64, device=self.device)
         # recurrent-state slots (models with per-sequence state besides KV pages); the last slot is a
         # scratch row for padding rows of a batch bucket and for graph warm-up passes
-        self.num_slots = 2 * mb
+        self.num_slots = num_state_slots if num_state_slots is not None else 2 * mb
         self.scratch_slot = self.num_slots
         self.slot_free = list(range(self.num_slots - 1, -1, -1))
         self.d_sslot = torch.full((mb,), self.scratch_slot, **i32)
@@ -171,12 +170,34 @@ class Engine:
         if need > self.max_pages:
             raise ValueError(f"request needs {need} pages, engine allows {self.max_pages} per sequence")
         r.pages = self.pool.alloc(need)
+        try:
+            self._take_slot(r)
+        except OutOfPages:
+            self.pool.release(r.pages)
+            raise
+        return r
+
+    def _take_slot(self, r: Request) -> None:
         if self.stateful:
             if not self.slot_free:
-                self.pool.release(r.pages)
                 raise OutOfPages("no free recurrent-state slot")
             r.slot = self.slot_free.pop()
+
+    def open_request(self) -> Request:
+        """A request whose tokens come in portions (`step`): it takes a state slot now and pages as it grows."""
+        r = Request([], 0, self._next_rid)
+        self._next_rid += 1
+        self._take_slot(r)
         return r
+
+    def append_tokens(self, r: Request, tokens: Seq[int]) -> None:
+        """Adds tokens to the request's prompt, with the pages they need."""
+        need = (len(r.prompt) + len(tokens) + self.page_size - 1) // self.page_size
+        if need > self.max_pages:
+            raise ValueError(f"request needs {need} pages, engine allows {self.max_pages} per sequence")
+        if need > len(r.pages):
+            r.pages = r.pages + self.pool.alloc(need - len(r.pages))
+        r.prompt.extend(int(t) for t in tokens)
 
     def release(self, r: Request) -> None:
         self.pool.release(r.pages)
@@ -204,10 +225,11 @@ class Engine:
             chunks.append(cur)
         return chunks
 
-    def _run_prefill_chunk(self, chunk, strategy, stats: Optional[GenerationStats]):
-        """Runs one flattened varlen prefill.  Returns (finishing requests, their first tokens)."""
+    def _varlen_meta(self, chunk, rows: list[int], stats: Optional[GenerationStats]):
+        """(token ids, AttnMeta) on the device of one flattened varlen batch of (request, start, end) token ranges;
+        `rows`: the rows of the batch whose logits are needed."""
         ps = self.page_size
-        ids, pos, slots, qs, sl, rows, done = [], [], [], [0], [], [], []
+        ids, pos, slots, qs, sl = [], [], [], [0], []
         bt = torch.zeros((len(chunk), self.max_pages), dtype=torch.int32)
         for i, (r, a, b) in enumerate(chunk):
             ids.extend(r.prompt[a:b])
@@ -217,10 +239,6 @@ class Engine:
             qs.append(qs[-1] + (b - a))
             sl.append(b)
             bt[i, :len(pg)] = torch.tensor(pg, dtype=torch.int32)
-            if b == len(r.prompt):
-                rows.append(qs[-1] - 1)
-                done.append(r)
-        t = len(ids)
         host = self._pin(torch.tensor([ids, pos, slots], dtype=torch.int32))
         sslots = [max(r.slot, 0) if self.stateful else 0 for r, _, _ in chunk]
         meta_h = self._pin(torch.tensor(qs + sl + sslots + rows, dtype=torch.int32))
@@ -231,18 +249,88 @@ class Engine:
         nb = len(chunk)
         meta = AttnMeta(True, dev[1], dev[2], bt_d, meta_d[nb + 1:2 * nb + 1], meta_d[:nb + 1],
                         total_q_blocks=sum((b - a + 63) // 64 for _, a, b in chunk),
-                        logits_rows=meta_d[3 * nb + 1:] if rows else None, q_start_host=list(qs),
+                        logits_rows=meta_d[3 * nb + 1:] if rows else None, q_start_host=qs, seq_lens_host=sl,
                         state_slots=meta_d[2 * nb + 1:3 * nb + 1] if self.stateful else None)
+        return dev[0], meta
+
+    def _run_prefill_chunk(self, chunk, strategy, stats: Optional[GenerationStats]):
+        """Runs one flattened varlen prefill.  Returns (finishing requests, their first tokens)."""
+        rows, done, t = [], [], 0
+        for r, a, b in chunk:
+            t += b - a
+            if b == len(r.prompt):
+                rows.append(t - 1)
+                done.append(r)
+        ids, meta = self._varlen_meta(chunk, rows, stats)
         if rows:
-            toks = self.model.forward(dev[0], meta, self.kv_cache, strategy, self.seed, 0, rng=self.d_rng)
+            toks = self.model.forward(ids, meta, self.kv_cache, strategy, self.seed, 0, rng=self.d_rng)
             if strategy is not None and strategy.topk > 1:
                 ops.advance_rng(self.d_rng)
         else:
-            self.model.hidden_states(dev[0], meta, self.kv_cache)
+            self.model.hidden_states(ids, meta, self.kv_cache)
             toks = None
         for r, a, b in chunk:
             r.computed = b
         return done, toks, t
+
+    # ------------------------------------------------------------------ given tokens
+    def step(self, entries, want=None) -> Optional[torch.Tensor]:
+        """One batch of given tokens through the model's step: `entries` is a list of (request, tokens), each request's
+        next tokens; `want` (one list of places per entry) selects the tokens whose logits come back, in that order, as
+        float32 [wanted, vocab] - None when nothing is wanted.  A batch of one token each, with a past, is a decode step
+        (the captured one `generate` replays); anything else runs as a varlen batch, portions beside single tokens."""
+        want = want if want is not None else [[] for _ in entries]
+        for r, tokens in entries:
+            if not tokens:
+                raise ValueError("an entry without tokens")
+            self.append_tokens(r, tokens)
+        chunk = [(r, r.computed, len(r.prompt)) for r, _ in entries]
+        if all(b - a == 1 and a > 0 for _, a, b in chunk) and len(chunk) <= self.max_batch:
+            lg = self._step_decode(chunk)
+            rows = [i for i, w in enumerate(want) for _ in w]
+            lg = lg[torch.tensor(rows, device=lg.device)] if rows else None
+        else:
+            rows, base = [], 0
+            for (r, a, b), w in zip(chunk, want):
+                rows.extend(base + p for p in w)
+                base += b - a
+            ids, meta = self._varlen_meta(chunk, rows, None)
+            x = self.model.hidden_states(ids, meta, self.kv_cache)
+            lg = self.model.logits(x, meta.logits_rows) if rows else None
+        for r, a, b in chunk:
+            r.computed = b
+        if lg is not None and self.model.comm.world > 1:
+            lg = self.model.comm.all_gather(lg.contiguous(), dim=1)
+        return lg[:, :self.model.config.vocab_size] if lg is not None else None
+
+    def _step_decode(self, chunk) -> torch.Tensor:
+        b, ps = len(chunk), self.page_size
+        bb = min(_bucket(b) if self.use_graphs else b, self.max_batch)
+        st = torch.zeros((5, bb), dtype=torch.int32)
+        st[3] = -1
+        st[4] = self.scratch_slot
+        bt = torch.zeros((bb, self.max_pages), dtype=torch.int32)
+        for i, (r, a, _) in enumerate(chunk):
+            st[:4, i] = torch.tensor([r.prompt[a], a, a + 1, r.pages[a // ps] * ps + a % ps], dtype=torch.int32)
+            if self.stateful:
+                st[4, i] = r.slot
+            bt[i, :len(r.pages)] = torch.tensor(r.pages, dtype=torch.int32)
+        self._upload_decode(bb, st, bt, None)
+        self.d_step.zero_()
+        max_total = self.max_pages * ps
+        return self._decode_step(bb, SamplingStrategy(), self._plan_splits(bb, max_total), max_total, None)[:b]
+
+    def _plan_splits(self, batch: int, max_seq_len: int) -> int:
+        return self.model.decode_splits(batch, max_seq_len) if self.on_gpu else 1
+
+    def _upload_decode(self, bb: int, st: torch.Tensor, bt: torch.Tensor, stats: Optional[GenerationStats]) -> None:
+        """Device state of the first bb batch rows: st [5, bb] = token, position, length, cache slot (negative: none) and
+        state slot; bt [bb, max_pages] block tables."""
+        st_d = self._to_dev(self._pin(st), stats)
+        self.d_ids[:bb].copy_(st_d[0]); self.d_pos[:bb].copy_(st_d[1]); self.d_seq[:bb].copy_(st_d[2]); self.d_slot[:bb].copy_(st_d[3])
+        if self.stateful:
+            self.d_sslot[:bb].copy_(st_d[4])
+        self.d_bt[:bb].copy_(self._to_dev(self._pin(bt), stats))
 
     # ------------------------------------------------------------------ decode
     def _decode_body(self, b: int, strategy, num_splits, max_seq_len):
@@ -250,7 +338,8 @@ class Engine:
                         num_splits=num_splits, max_seq_len=max_seq_len,
                         q_start=self.d_qs[:b + 1] if self.stateful else None,
                         state_slots=self.d_sslot[:b] if self.stateful else None)
-        toks = self.model.forward(self.d_ids[:b], meta, self.kv_cache, strategy, self.seed, 0, rng=self.d_rng)
+        lg = self.model.logits(self.model.hidden_states(self.d_ids[:b], meta, self.kv_cache))
+        toks = self.model.sample(lg, strategy, self.seed, 0, self.d_rng)
         from ..ops import baseline as _baseline
         if self.on_gpu and not _baseline.enabled():
             rc = _lib.lib().zb_decode_advance_rng(
@@ -271,11 +360,13 @@ class Engine:
             row = self.d_step.long().clamp_max(self.d_hist.shape[0] - 1)
             self.d_hist[:, :b].index_copy_(0, row, toks[None, :].to(self.d_hist.dtype))
             self.d_step += 1
+        return lg
 
     def _decode_step(self, b: int, strategy, num_splits, max_seq_len, stats):
+        """One decode step of the first b rows; returns its logits (with graphs: the capture's buffer, overwritten by the
+        next replay)."""
         if not self.use_graphs:
-            self._decode_body(b, strategy, num_splits, max_seq_len)
-            return
+            return self._decode_body(b, strategy, num_splits, max_seq_len)
         key = (b, strategy.topk, float(strategy.temperature), num_splits)
         g = self._graphs.get(key)
         if g is None:
@@ -294,7 +385,7 @@ class Engine:
             graph = torch.cuda.CUDAGraph()
             before = _lib.launch_count()
             with torch.cuda.graph(graph):
-                self._decode_body(b, strategy, num_splits, max_seq_len)
+                lg = self._decode_body(b, strategy, num_splits, max_seq_len)
             nodes = _lib.launch_count() - before
             # the warm-up and capture passes must not count as decode steps: restore the state
             # (the warm-up really ran; the capture pass did not execute anything)
@@ -303,10 +394,11 @@ class Engine:
                 dst.copy_(src)
             # the warm-up wrote one KV row per sequence at the slot of the next position; the
             # real step writes the same slot with the real values, so nothing needs undoing
-            g = (graph, nodes)
+            g = (graph, nodes, lg)
             self._graphs[key] = g
         g[0].replay()
         _lib.lib().zb_launch_count_add(g[1])
+        return g[2]
 
     # ------------------------------------------------------------------ public API
     def generate(self, prompts: Seq[Seq[int]], max_new_tokens: int,
@@ -357,26 +449,22 @@ class Engine:
         bb = min(bb, self.max_batch)
         ps = self.page_size
         pos = [len(r.prompt) for r in reqs]                # position of the first generated token
-        st = torch.zeros((4, bb), dtype=torch.int32)
+        st = torch.zeros((5, bb), dtype=torch.int32)
         st[3, :] = -1
+        st[4, :] = self.scratch_slot
         bt = torch.zeros((bb, self.max_pages), dtype=torch.int32)
         for i, r in enumerate(reqs):
             st[1, i] = pos[i]
             st[2, i] = pos[i] + 1
             st[3, i] = r.pages[pos[i] // ps] * ps + pos[i] % ps
+            if self.stateful:
+                st[4, i] = r.slot
             bt[i, :len(r.pages)] = torch.tensor(r.pages, dtype=torch.int32)
-        st_d = self._to_dev(self._pin(st), stats)
-        self.d_bt[:bb].copy_(self._to_dev(self._pin(bt), stats))
-        self.d_pos[:bb].copy_(st_d[1]); self.d_seq[:bb].copy_(st_d[2]); self.d_slot[:bb].copy_(st_d[3])
-        self.d_ids[:bb].zero_()
+        self._upload_decode(bb, st, bt, stats)
         self.d_ids[:b].copy_(torch.cat([first_tok[r.rid] for r in reqs]))
-        if self.stateful:
-            ss = torch.full((bb,), self.scratch_slot, dtype=torch.int32)
-            ss[:b] = torch.tensor([r.slot for r in reqs], dtype=torch.int32)
-            self.d_sslot[:bb].copy_(self._to_dev(self._pin(ss), stats))
         self.d_step.zero_()
         max_total = max(pos) + max_new_tokens
-        num_splits = ops.decode_plan_splits(bb, self.model.hkv, max_total) if self.on_gpu else 1
+        num_splits = self._plan_splits(bb, max_total)
         # ---------------- decode loop
         outputs = [[] for _ in reqs]
         first_host = self.d_ids[:b].cpu() if max_new_tokens > 0 else None
@@ -465,7 +553,7 @@ class Engine:
         cap = min(cap, bb)
         ps = self.page_size
         max_total = max((len(p) + m for p, m in zip(prompts, budget)), default=1)
-        num_splits = ops.decode_plan_splits(bb, self.model.hkv, max_total) if self.on_gpu else 1
+        num_splits = self._plan_splits(bb, max_total)
         launches0 = _lib.launch_count() if self.on_gpu else 0
         outputs: list[list[int]] = [[] for _ in range(n_req)]
         waiting = list(range(n_req))
@@ -564,12 +652,7 @@ class Engine:
                 live = torch.zeros(bb, dtype=torch.bool)
                 live[list(running)] = True
                 slot_h = torch.where(live, slot_h, torch.full_like(slot_h, -1))
-                st = self._to_dev(self._pin(torch.stack([ids_h, pos_h, pos_h + 1, slot_h.to(torch.int32), ss_h])), stats)
-                self.d_ids[:bb].copy_(st[0]); self.d_pos[:bb].copy_(st[1]); self.d_seq[:bb].copy_(st[2])
-                self.d_slot[:bb].copy_(st[3])
-                if self.stateful:
-                    self.d_sslot[:bb].copy_(st[4])
-                self.d_bt[:bb].copy_(self._to_dev(self._pin(bt_h), stats))
+                self._upload_decode(bb, torch.stack([ids_h, pos_h, pos_h + 1, slot_h.to(torch.int32), ss_h]), bt_h, stats)
             # ---------------- one decode block
             left = max(budget[idx] - len(outputs[idx]) for idx, _ in running.values())
             n = max(1, min(sync_interval, self.history_steps, left))
@@ -662,7 +745,7 @@ class Session:
         eng.d_bt[0, :len(self.req.pages)] = torch.tensor(self.req.pages, **i32)
         if eng.stateful:
             eng.d_sslot[:1] = torch.tensor([self.req.slot], **i32)
-        splits = ops.decode_plan_splits(1, eng.model.hkv, self.max_tokens) if eng.on_gpu else 1
+        splits = eng._plan_splits(1, self.max_tokens)
         pending = [self._next]
         done = False
         while not done:
