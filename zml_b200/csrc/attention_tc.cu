@@ -56,25 +56,6 @@ struct PrefillTcParams {
   ZbStatus* status;
 };
 
-ZB_DEVICE float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
-// Shared-memory descriptor of an MN-major bf16 operand written by TMA with the 128-byte swizzle: rows are K
-// (here: keys), 64 contiguous MN elements (128 bytes) per row; `lbo` = bytes between 64-element groups along MN,
-// `sbo` = bytes between groups of 8 rows along K.
-ZB_DEVICE uint64_t make_desc_sw128_mn(uint32_t smem_addr, uint32_t lbo, uint32_t sbo) {
-  uint64_t d = 0;
-  d |= static_cast<uint64_t>((smem_addr & 0x3ffffu) >> 4);
-  d |= static_cast<uint64_t>((lbo >> 4) & 0x3fffu) << 16;
-  d |= static_cast<uint64_t>((sbo >> 4) & 0x3fffu) << 32;
-  d |= static_cast<uint64_t>(1) << 46;
-  d |= static_cast<uint64_t>(2) << 61;
-  return d;
-}
-
 ZB_DEVICE void wg_bar_sync(int wg) {
   asm volatile("bar.sync %0, 128;" ::"r"(1 + wg) : "memory");
 }
@@ -241,7 +222,7 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
           const uint32_t va = zb_smem_u32(v_s + stage * kKvBytes);
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
-            const uint64_t dv = make_desc_sw128_mn(va + k * (16 * 128), p.v_lbo, p.v_sbo);
+            const uint64_t dv = zb_make_desc_sw128_mn(va + k * (16 * 128), p.v_lbo, p.v_sbo);
             zb_umma_f16_ts(tmem_base + kColO + w * kHD, tmem_base + kColP + w * 32 + 8 * k, dv, kIdescO, (jj > 0 || k > 0) ? 1u : 0u);
           }
           zb_umma_commit(&o_ready[w]);
@@ -310,7 +291,7 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       const float m_use = mx == -INFINITY ? 0.f : mx;             // a row without a visible key so far
       if (jj > 0) {
         // the output accumulated so far is relative to the old maximum: rescale it where the maximum moved
-        const float alpha = m == -INFINITY ? 1.f : ex2(m - m_use);
+        const float alpha = m == -INFINITY ? 1.f : zb_ex2(m - m_use);
         const bool moved = alpha != 1.f;
         if (__any_sync(0xffffffffu, moved)) {
           if (!zb_mbar_wait(&o_ready[w], (jj - 1u) & 1u, abort_flag)) {      // O += P V of the previous page is done
@@ -340,8 +321,8 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       float sum0 = 0.f, sum1 = 0.f;
 #pragma unroll
       for (int i = 0; i < 32; ++i) {
-        const float p0 = ex2(fmaf(__uint_as_float(sr[2 * i]), p.scale_log2, neg_m));
-        const float p1 = ex2(fmaf(__uint_as_float(sr[2 * i + 1]), p.scale_log2, neg_m));
+        const float p0 = zb_ex2(fmaf(__uint_as_float(sr[2 * i]), p.scale_log2, neg_m));
+        const float p1 = zb_ex2(fmaf(__uint_as_float(sr[2 * i + 1]), p.scale_log2, neg_m));
         pw[i] = zb_pack_bf16x2(p0, p1);
         sum0 += p0;
         sum1 += p1;

@@ -442,6 +442,19 @@ ZB_DEVICE uint64_t zb_make_desc_sw128(uint32_t smem_addr) {
   return d;
 }
 
+// Shared-memory descriptor of an MN-major bf16 operand written by TMA with the 128-byte swizzle: rows are K
+// (here: keys), 64 contiguous MN elements (128 bytes) per row; `lbo` = bytes between 64-element groups along MN,
+// `sbo` = bytes between groups of 8 rows along K.
+ZB_DEVICE uint64_t zb_make_desc_sw128_mn(uint32_t smem_addr, uint32_t lbo, uint32_t sbo) {
+  uint64_t d = 0;
+  d |= static_cast<uint64_t>((smem_addr & 0x3ffffu) >> 4);
+  d |= static_cast<uint64_t>((lbo >> 4) & 0x3fffu) << 16;
+  d |= static_cast<uint64_t>((sbo >> 4) & 0x3fffu) << 32;
+  d |= static_cast<uint64_t>(1) << 46;
+  d |= static_cast<uint64_t>(2) << 61;
+  return d;
+}
+
 // Instruction descriptor for kind::f16 with bf16 inputs, fp32 accumulate, A and B K-major.
 //   bits 4-5 D format (1 = f32), 7-9 A format (1 = bf16), 10-12 B format,
 //   15 A major, 16 B major (0 = K), 17-22 N >> 3, 24-28 M >> 4.
@@ -479,6 +492,12 @@ ZB_DEVICE uint32_t zb_pack_bf16x2(float lo, float hi) {
 ZB_DEVICE float2 zb_unpack_bf16x2(uint32_t u) {
   __nv_bfloat162 v = *reinterpret_cast<__nv_bfloat162*>(&u);
   return __bfloat1622float2(v);
+}
+
+ZB_DEVICE float zb_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 
 ZB_DEVICE float zb_warp_sum(float v) {

@@ -171,7 +171,8 @@ class _Layer:
 
 
 class DopuraxModel(DecoderModel):
-    KERNEL_SOURCES = ("runtime", "gemm_bf16", "gemm_2cta", "gemm_f32", "elementwise", "stream_f32", "latent_attention", "wkv", "moe")
+    KERNEL_SOURCES = ("runtime", "gemm_bf16", "gemm_2cta", "gemm_f32", "elementwise", "stream_f32", "latent_attention",
+                      "latent_prefill_tc", "latent_decode", "wkv", "moe")
     FP32_ON_GPU = True
 
     def __init__(self, config: DopuraxConfig, comm: Optional[Comm] = None, device="cpu", dtype=torch.bfloat16):

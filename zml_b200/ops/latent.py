@@ -27,6 +27,12 @@ _lib.register_signature("zb_latent_absorb", _i, [_p, _ll, _ll, _p, _ll, _p, _ll,
 _lib.register_signature("zb_latent_attend", _i, [_p, _p, _ll, _p, _ll, _p, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _i, _i, _p])
 _lib.register_signature("zb_latent_gather", _i, [_p, _ll, _p, _i, _i, _p, _p, _i, _p, _ll, _i, _i, _i, _i, _i, _p])
 _lib.register_signature("zb_latent_q_pack", _i, [_p, _ll, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p])
+_lib.register_signature("zb_latent_prefill_tc_supported", _i, [_i, _i, _i, _i])
+_lib.register_signature("zb_latent_prefill_tc", _i, [_p, _p, _ll, _p, _ll, _i, _p, _ll, _p, _ll, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _i,
+                                                     _i, _i, _f, _p])
+_lib.register_signature("zb_latent_decode_supported", _i, [_i, _i])
+_lib.register_signature("zb_latent_decode_groups", _i, [_i])
+_lib.register_signature("zb_latent_decode", _i, [_p, _p, _i, _p, _ll, _p, _i, _i, _p, _i, _i, _i, _i, _f, _i, _p])
 
 
 def _ptr(t: Optional[torch.Tensor]):
@@ -163,21 +169,86 @@ def attend(q, cache, block_table, q_start, seq_lens, d: LatentDims, decode: bool
     t = q.shape[0]
     out = torch.empty((t, d.heads, d.rot_off), dtype=q.dtype, device=q.device)
     assert block_table.is_contiguous() and cache.dtype == q.dtype and q.is_contiguous()
-    _lib.check(_lib.lib().zb_latent_attend(
+    l = _lib.lib()
+    if decode and q.dtype == torch.bfloat16 and l.zb_latent_decode_supported(d.row, d.rot_off):
+        _lib.check(l.zb_latent_decode(
+            _ptr(q), _ptr(cache), d.row, _ptr(out), d.rot_off, _ptr(block_table), block_table.shape[1], cache.shape[1], _ptr(seq_lens), t,
+            d.heads, d.rot_off, d.window, float(d.scale), int(num_splits), _lib.stream_ptr()), "zb_latent_decode")
+        return out
+    _lib.check(l.zb_latent_attend(
         _ptr(q), _ptr(cache), d.row, _ptr(out), d.rot_off, _ptr(block_table), block_table.shape[1], cache.shape[1], d.heads, d.rank, d.rot,
         d.rot_off, d.window, float(d.scale), _ptr(q_start), _ptr(seq_lens), seq_lens.shape[0], t, int(q.dtype == torch.float32),
         _lib.stream_ptr()), "zb_latent_attend")
     return out
 
 
+# tokens of a decode chunk: below this a chunk costs more in partial results than it gains in parallelism
+_MIN_CHUNK = 256
+
+
 def decode_plan_splits(batch: int, d: LatentDims, max_seq_len: int) -> int:
-    return 1
+    """Chunks a sequence's visible tokens are cut into by a decode step: enough to give every SM a CTA."""
+    l = _lib.lib()
+    visible = min(max_seq_len, d.window) if d.window > 0 else max_seq_len
+    ctas = max(1, batch * int(l.zb_latent_decode_groups(d.heads)))
+    return max(1, min(l.zb_num_sms() // ctas, (visible + _MIN_CHUNK - 1) // _MIN_CHUNK, 64))
+
+
+# ---------------------------------------------------------------------------- expanded keys and values
+def _visible_plan(meta, window: int):
+    """(first gathered row of every sequence and the total, position of that row's token) on the device, total rows: the
+    tokens that this batch's queries see.  One upload per step and window, kept in `meta.plans`."""
+    key = ("latent_visible", window)
+    plan = meta.plans.get(key)
+    if plan is None:
+        qs, sl = meta.q_start_host, meta.seq_lens_host
+        start, first = [0], []
+        for a, b, n in zip(qs, qs[1:], sl):
+            f = max(0, n - (b - a) - window + 1) if window > 0 else 0
+            first.append(f)
+            start.append(start[-1] + (n - f if b > a else 0))
+        dev = torch.tensor(start + first, dtype=torch.int32).pin_memory().to(meta.seq_lens.device, non_blocking=True)
+        plan = meta.plans[key] = (dev[:len(start)], dev[len(start):], start[-1])
+    return plan
+
+
+def prefill(q, gate, w_ukv, inv_freq, cache, meta, d: LatentDims):
+    """The expanded formulation on the tensor cores (bf16): gathers the visible latents, projects them to keys and values
+    of all heads, and runs the windowed prefill kernel with the output gate in its epilogue."""
+    from . import gemm
+    t, dev, l = q.shape[0], q.device, _lib.lib()
+    key_start, first_key, rows = _visible_plan(meta, d.window)
+    rot_out = _up(d.rot_off, 64)
+    lat = torch.empty((rows, rot_out + _up(d.rot, 64)), dtype=q.dtype, device=dev)
+    _lib.check(l.zb_latent_gather(_ptr(cache), d.row, _ptr(meta.block_table), meta.block_table.shape[1], cache.shape[1], _ptr(key_start),
+                                  _ptr(first_key), first_key.shape[0], _ptr(lat), lat.shape[1], rows, d.rank, d.rot, d.rot_off, rot_out,
+                                  _lib.stream_ptr()), "zb_latent_gather")
+    kv = gemm(lat[:, :d.rank], w_ukv, static_w=True)                               # [rows, H dim | H vdim]
+    dim_p, rot_p = _up(d.dim, 64), _up(d.rot, 64)
+    qp = torch.empty((t, d.heads, dim_p + rot_p), dtype=q.dtype, device=dev)
+    _lib.check(l.zb_latent_q_pack(_ptr(q), q.stride(0), _ptr(qp), _ptr(inv_freq), _ptr(meta.positions), t, d.heads, d.dim, d.rot, dim_p, rot_p,
+                                  _lib.stream_ptr()), "zb_latent_q_pack")
+    out = torch.empty((t, d.heads * d.vdim), dtype=q.dtype, device=dev)
+    blocks = sum((b - a + 255) // 256 for a, b in zip(meta.q_start_host, meta.q_start_host[1:]))
+    _lib.check(l.zb_latent_prefill_tc(
+        _ptr(qp), _ptr(kv), kv.stride(0), _ptr(lat), lat.stride(0), rot_out, _ptr(out), out.stride(0), _ptr(gate), gate.stride(0),
+        _ptr(meta.q_start), _ptr(meta.seq_lens), meta.seq_lens.shape[0], _ptr(key_start), _ptr(first_key), t, rows, blocks, d.heads, d.dim,
+        d.rot, d.vdim, d.window, float(d.scale), _lib.stream_ptr()), "zb_latent_prefill_tc")
+    return out
+
+
+def _expands(q, gate, meta, d: LatentDims) -> bool:
+    return (q.is_cuda and q.dtype == torch.bfloat16 and meta.is_prefill and meta.q_start_host is not None and meta.seq_lens_host is not None
+            and bool(_lib.lib().zb_latent_prefill_tc_supported(d.dim, d.rot, d.vdim, d.rank)) and q.stride(0) % 8 == 0
+            and gate.stride(0) % 8 == 0)
 
 
 # ---------------------------------------------------------------------------- the layer's attention
 def latent_attention(q, gate, w_uk_t, w_ukv, inv_freq, cache, meta, d: LatentDims):
     """sigmoid(gate) * attention of one step: q [T, H * (dim + rot)] unrotated, gate [T, H * vdim], w_uk_t [H, rank, dim],
     w_ukv [H dim + H vdim, rank]; `meta` is the step's AttnMeta, the new tokens' cache rows are already written."""
+    if _expands(q, gate, meta, d):
+        return prefill(q, gate, w_ukv, inv_freq, cache, meta, d)
     q_start = meta.q_start
     if q_start is None:
         q_start = torch.arange(q.shape[0] + 1, dtype=torch.int32, device=q.device)
