@@ -6,6 +6,10 @@
     python examples/benchmark/kernels.py --op=prefill_attention --batch=4 --seqlen=2048
     python examples/benchmark/kernels.py --op=moe --tokens=128 --experts=128 --topk=8 --n=768 --k=2048
     python examples/benchmark/kernels.py --op=gated_delta_scan --batch=32 --seqlen=1024
+    python examples/benchmark/kernels.py --op=latent_prefill --batch=2 --seqlen=2048 --hq=16 --window=4096
+    python examples/benchmark/kernels.py --op=latent_decode --batch=32 --seqlen=4096 --hq=32 --window=4096
+    python examples/benchmark/kernels.py --op=wkv_scan --batch=8 --seqlen=512 --hq=32 --hd=128
+    python examples/benchmark/kernels.py --op=stream --tokens=4096 --k=4096
     python examples/benchmark/kernels.py --op=decode_layers --model=llama-3.1-8b --batch=32 --seqlen=1344
     python examples/benchmark/kernels.py --op=gemm_chain_timeline --model=llama-3.1-8b --batch=32
     python examples/benchmark/kernels.py --op=moe_w4_timeline --tokens=128 --experts=128 --topk=8 --n=768 --k=2048
@@ -51,6 +55,7 @@ class Args:
     warmup: int = 3
     splits: int = 0          # decode_attention: KV chunks per sequence (0: the planner's choice)
     w4: int = 0              # moe: 1 = NVFP4 expert weights de-quantised inside the grouped GEMM
+    window: int = 4096       # latent attention: keys a position sees
     copies: int = 0          # operand copies to rotate through (0: enough to exceed the L2)
     help = __doc__
 
@@ -76,6 +81,18 @@ def timed(fns, iters: int, warmup: int) -> float:
     e.record()
     torch.cuda.synchronize()
     return s.elapsed_time(e) / iters
+
+
+def timed_graph(fns, iters: int, warmup: int) -> float:
+    """As `timed`, for launches shorter than their submission: the iterations are captured in one CUDA graph."""
+    for i in range(warmup):
+        fns[i % len(fns)]()
+    torch.cuda.synchronize()
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g):
+        for i in range(iters):
+            fns[i % len(fns)]()
+    return timed([g.replay], 5, 2) / iters
 
 
 def n_copies(args: Args, bytes_per_copy: int) -> int:
@@ -185,13 +202,107 @@ def bench_gated_delta_scan(a: Args) -> None:
     dtb = torch.zeros(hv, device="cuda")
     nw = torch.ones(dv, device="cuda").bfloat16()
     qs = (torch.arange(a.batch + 1, dtype=torch.int32, device="cuda") * a.seqlen).int()
-    sl = torch.full((a.batch,), a.seqlen, dtype=torch.int32, device="cuda")
+    # one token per sequence: a decode step, with a past; else whole sequences
+    sl = torch.full((a.batch,), a.seqlen + (a.seqlen == 1), dtype=torch.int32, device="cuda")
     slots = torch.arange(a.batch, dtype=torch.int32, device="cuda")
     oz, ob = 2 * hk * dk + hv * dv, 2 * hk * dk + 2 * hv * dv
     fn = lambda: la.gated_delta_scan(proj[:, :oz], proj[:, oz:ob], proj[:, ob + hv:ob + 2 * hv], proj[:, ob:ob + hv], a_log, dtb,
                                      nw, 1e-6, state, qs, sl, slots, hk, hv, dk, dv)
-    ms = timed([fn], a.iters, a.warmup)
+    ms = (timed_graph if a.seqlen == 1 else timed)([fn], a.iters, a.warmup)
     report(a, ms, t * cols * 2 + t * hv * dv * 2 + 2 * state.numel() * 4, 6.0 * t * hv * dk * dv, {"batch": a.batch, "seqlen": a.seqlen})
+
+
+def _latent(a: Args):
+    """Layer sizes of the latent-attention benchmarks and a filled cache with one block table per copy."""
+    from zml_b200.ops import latent as lat
+    d = lat.LatentDims(a.hq, 128, 64, 128, 512, 1536, a.window, 192 ** -0.5, 500000.0)
+    pages_per = (a.seqlen + 63) // 64
+    bt = (torch.arange(a.batch * pages_per, dtype=torch.int32, device="cuda") + 1).view(a.batch, pages_per)
+    c = n_copies(a, a.batch * min(a.seqlen, a.window) * d.row * 2)
+    caches = [torch.randn(a.batch * pages_per + 1, 64, d.row, device="cuda").bfloat16() for _ in range(c)]
+    return lat, d, bt, caches
+
+
+def bench_latent_prefill(a: Args) -> None:
+    """The prefill kernel alone, and the whole attention of a layer behind the query projection (gather, key / value
+    projection, query packing, attention with the gate)."""
+    from types import SimpleNamespace
+    lat, d, bt, caches = _latent(a)
+    t = a.batch * a.seqlen
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device="cuda")
+    qs, sl = [i * a.seqlen for i in range(a.batch + 1)], [a.seqlen] * a.batch
+    meta = SimpleNamespace(is_prefill=True, q_start_host=qs, seq_lens_host=sl, q_start=i32(qs), seq_lens=i32(sl), plans={}, block_table=bt,
+                           positions=torch.arange(a.seqlen, dtype=torch.int32, device="cuda").repeat(a.batch))
+    q = torch.randn(t, d.heads * 192, device="cuda").bfloat16()
+    gate = torch.randn(t, d.heads * 128, device="cuda").bfloat16()
+    w = torch.randn(d.heads * 256, 512, device="cuda").bfloat16() * 0.05
+    inv = d.inv_freq("cuda")
+    pairs = sum(min(i + 1, a.window) for i in range(a.seqlen)) * a.batch
+    flops = 2.0 * pairs * d.heads * (192 + 128)
+    ms = timed([lambda c=c: lat.prefill(q, gate, w, inv, c, meta, d) for c in caches], a.iters, a.warmup)
+    report(a, ms, t * d.heads * (192 + 256) * 2, flops + 2.0 * t * 512 * d.heads * 256, {"part": "whole", "batch": a.batch, "seqlen": a.seqlen, "heads": a.hq, "window": a.window})
+    shape = {"batch": a.batch, "seqlen": a.seqlen, "heads": a.hq, "window": a.window}
+    x, kv, rot_out, plan = lat.expand(caches[0], w, meta, d)
+    qp = lat.pack_q(q, inv, meta.positions, d)
+    ms = timed([lambda: lat.attend_expanded(qp, gate, x, kv, rot_out, plan, meta, d)], a.iters, a.warmup)
+    report(a, ms, t * d.heads * (192 + 192 + 128 + 128) * 2, flops, dict(shape, part="attention kernel"))
+    ms = timed([lambda: lat.pack_q(q, inv, meta.positions, d)], a.iters, a.warmup)
+    report(a, ms, t * d.heads * 192 * 4, 0, dict(shape, part="query packing"))
+    ms = timed([lambda c=c: lat.expand(c, w, meta, d) for c in caches], a.iters, a.warmup)
+    report(a, ms, t * (576 * 4 + 512 * 2 + d.heads * 512), 2.0 * t * 512 * d.heads * 256, dict(shape, part="gather and key / value projection"))
+
+
+def bench_latent_decode(a: Args) -> None:
+    lat, d, bt, caches = _latent(a)
+    q = torch.randn(a.batch, d.heads * 192, device="cuda").bfloat16()
+    gate = torch.randn(a.batch, d.heads * 128, device="cuda").bfloat16()
+    uk = [torch.randn(d.heads, 512, 128, device="cuda").bfloat16() for _ in range(8)]
+    uv = [torch.randn(d.heads, 128, 512, device="cuda").bfloat16() for _ in range(8)]
+    inv, pos = d.inv_freq("cuda"), torch.full((a.batch,), a.seqlen - 1, dtype=torch.int32, device="cuda")
+    qs, sl = torch.arange(a.batch + 1, dtype=torch.int32, device="cuda"), torch.full((a.batch,), a.seqlen, dtype=torch.int32, device="cuda")
+    ql = lat.absorb_q(q, uk[0], inv, pos, d)
+    splits = a.splits or lat.decode_plan_splits(a.batch, d, a.seqlen)
+    keys = a.batch * min(a.seqlen, a.window)
+    shape = {"batch": a.batch, "seqlen": a.seqlen, "heads": a.hq, "window": a.window, "splits": splits}
+    ms = timed_graph([lambda c=c: lat.attend(ql, c, bt, qs, sl, d, decode=True, num_splits=splits) for c in caches], a.iters, a.warmup)
+    report(a, ms, keys * d.row * 2, 2.0 * keys * d.heads * (576 + 512), dict(shape, part="attention kernel"))
+    o = lat.attend(ql, caches[0], bt, qs, sl, d, decode=True, num_splits=splits)
+    wb = d.heads * 512 * 128 * 2
+    ms = timed_graph([lambda w=w: lat.absorb_q(q, w, inv, pos, d) for w in uk], a.iters, a.warmup)
+    report(a, ms, wb, 2.0 * a.batch * d.heads * 512 * 128, dict(shape, part="queries into the latent space"))
+    ms = timed_graph([lambda w=w: lat.absorb_out(o, w, gate, d) for w in uv], a.iters, a.warmup)
+    report(a, ms, wb, 2.0 * a.batch * d.heads * 512 * 128, dict(shape, part="results out of it"))
+
+
+def bench_wkv_scan(a: Args) -> None:
+    from zml_b200.ops import linear_attn as la
+    H, D, t = a.hq, a.hd, a.batch * a.seqlen
+    x = [torch.randn(t, H * D, device="cuda").bfloat16() for _ in range(4)]
+    z = torch.randn(t, H * D, device="cuda")
+    v = [torch.randn(H * D, device="cuda") for _ in range(3)]
+    qs = (torch.arange(a.batch + 1, dtype=torch.int32, device="cuda") * a.seqlen).int()
+    sl = torch.full((a.batch,), a.seqlen + 1, dtype=torch.int32, device="cuda")
+    slots = torch.arange(a.batch, dtype=torch.int32, device="cuda")
+    states = [torch.zeros(a.batch, H, D, D, device="cuda") for _ in range(n_copies(a, a.batch * H * D * D * 8) if a.seqlen == 1 else 1)]
+    ms = (timed_graph if a.seqlen == 1 else timed)([lambda s=s: la.wkv_scan(*x, z, *v, 1e-5, s, qs, sl, slots, H, D, decode=a.seqlen == 1) for s in states], a.iters, a.warmup)
+    report(a, ms, t * H * D * (5 * 2 + 4) + 2 * states[0].numel() * 4, 6.0 * t * H * D * D, {"batch": a.batch, "seqlen": a.seqlen, "heads": H, "dim": D})
+
+
+def bench_stream(a: Args) -> None:
+    """The norm behind a sublayer, the input convolution (with and without interpolations) and the decode step's fusion."""
+    from zml_b200.ops import stream
+    t, d = a.tokens, a.k
+    c = max(2, math.ceil(256e6 / (t * d * 8)) + 1)
+    xs = [torch.randn(t, d, device="cuda") for _ in range(c)]
+    y, w = torch.randn(t, d, device="cuda"), torch.ones(d, device="cuda")
+    mu = torch.rand(5, d, device="cuda")
+    qs, sl, slots = torch.tensor([0, t], dtype=torch.int32, device="cuda"), torch.tensor([t], dtype=torch.int32, device="cuda"), torch.zeros(t, dtype=torch.int32, device="cuda")
+    ms = timed_graph([lambda x=x: stream.post_norm(x, w, 1e-5, y, 2.0, act_dtype=torch.bfloat16) for x in xs], a.iters, a.warmup)
+    report(a, ms, t * d * 14, 0, {"part": "post_norm", "tokens": t, "d": d})
+    for mixes in (False, True):
+        conv = stream.InputConv(torch.randn(d, 4, device="cuda"), torch.zeros(1, 4 if mixes else 3, d, device="cuda"), mu if mixes else None)
+        ms = timed_graph([lambda x=x: stream.stream_conv(x, conv, qs, sl, slots, torch.bfloat16) for x in xs], a.iters, a.warmup)
+        report(a, ms, t * d * (4 + (10 if mixes else 2)), 0, {"part": "stream_conv", "mixes": mixes, "tokens": t, "d": d})
 
 
 def bench_decode_layers(a: Args) -> None:
@@ -358,7 +469,8 @@ def bench_moe_w4_timeline(a: Args) -> None:
 
 
 OPS = {"moe_w4_timeline": bench_moe_w4_timeline, "gemm_chain_timeline": bench_gemm_chain_timeline, "gemm": bench_gemm, "decode_attention": bench_decode_attention, "prefill_attention": bench_prefill_attention,
-       "moe": bench_moe, "gated_delta_scan": bench_gated_delta_scan, "decode_layers": bench_decode_layers}
+       "moe": bench_moe, "gated_delta_scan": bench_gated_delta_scan, "decode_layers": bench_decode_layers,
+       "latent_prefill": bench_latent_prefill, "latent_decode": bench_latent_decode, "wkv_scan": bench_wkv_scan, "stream": bench_stream}
 
 
 def main(argv=None) -> int:

@@ -212,29 +212,45 @@ def _visible_plan(meta, window: int):
     return plan
 
 
-def prefill(q, gate, w_ukv, inv_freq, cache, meta, d: LatentDims):
-    """The expanded formulation on the tensor cores (bf16): gathers the visible latents, projects them to keys and values
-    of all heads, and runs the windowed prefill kernel with the output gate in its epilogue."""
+def expand(cache, w_ukv, meta, d: LatentDims):
+    """Gathers the latents that this batch's queries see and projects them: (latents [rows, ..] with the rotated part at the
+    returned column, kv [rows, H dim | H vdim], that column, the gather's plan)."""
     from . import gemm
-    t, dev, l = q.shape[0], q.device, _lib.lib()
-    key_start, first_key, rows = _visible_plan(meta, d.window)
+    plan = key_start, first_key, rows = _visible_plan(meta, d.window)
     rot_out = _up(d.rot_off, 64)
-    lat = torch.empty((rows, rot_out + _up(d.rot, 64)), dtype=q.dtype, device=dev)
-    _lib.check(l.zb_latent_gather(_ptr(cache), d.row, _ptr(meta.block_table), meta.block_table.shape[1], cache.shape[1], _ptr(key_start),
-                                  _ptr(first_key), first_key.shape[0], _ptr(lat), lat.shape[1], rows, d.rank, d.rot, d.rot_off, rot_out,
-                                  _lib.stream_ptr()), "zb_latent_gather")
-    kv = gemm(lat[:, :d.rank], w_ukv, static_w=True)                               # [rows, H dim | H vdim]
-    dim_p, rot_p = _up(d.dim, 64), _up(d.rot, 64)
-    qp = torch.empty((t, d.heads, dim_p + rot_p), dtype=q.dtype, device=dev)
-    _lib.check(l.zb_latent_q_pack(_ptr(q), q.stride(0), _ptr(qp), _ptr(inv_freq), _ptr(meta.positions), t, d.heads, d.dim, d.rot, dim_p, rot_p,
-                                  _lib.stream_ptr()), "zb_latent_q_pack")
-    out = torch.empty((t, d.heads * d.vdim), dtype=q.dtype, device=dev)
+    lat = torch.empty((rows, rot_out + _up(d.rot, 64)), dtype=cache.dtype, device=cache.device)
+    _lib.check(_lib.lib().zb_latent_gather(
+        _ptr(cache), d.row, _ptr(meta.block_table), meta.block_table.shape[1], cache.shape[1], _ptr(key_start), _ptr(first_key),
+        first_key.shape[0], _ptr(lat), lat.shape[1], rows, d.rank, d.rot, d.rot_off, rot_out, _lib.stream_ptr()), "zb_latent_gather")
+    return lat, gemm(lat[:, :d.rank], w_ukv, static_w=True), rot_out, plan
+
+
+def pack_q(q, inv_freq, positions, d: LatentDims):
+    """q [T, H * (dim + rot)] -> [T, H, dim | rot], the rotated part rotated and both padded with zeros to 64 columns."""
+    t, dim_p, rot_p = q.shape[0], _up(d.dim, 64), _up(d.rot, 64)
+    out = torch.empty((t, d.heads, dim_p + rot_p), dtype=q.dtype, device=q.device)
+    _lib.check(_lib.lib().zb_latent_q_pack(_ptr(q), q.stride(0), _ptr(out), _ptr(inv_freq), _ptr(positions), t, d.heads, d.dim, d.rot, dim_p,
+                                           rot_p, _lib.stream_ptr()), "zb_latent_q_pack")
+    return out
+
+
+def attend_expanded(qp, gate, lat, kv, rot_out: int, plan, meta, d: LatentDims):
+    """sigmoid(gate) * windowed causal attention of packed queries over expanded keys and values: [T, H * vdim]."""
+    key_start, first_key, rows = plan
+    t = qp.shape[0]
+    out = torch.empty((t, d.heads * d.vdim), dtype=qp.dtype, device=qp.device)
     blocks = sum((b - a + 255) // 256 for a, b in zip(meta.q_start_host, meta.q_start_host[1:]))
-    _lib.check(l.zb_latent_prefill_tc(
+    _lib.check(_lib.lib().zb_latent_prefill_tc(
         _ptr(qp), _ptr(kv), kv.stride(0), _ptr(lat), lat.stride(0), rot_out, _ptr(out), out.stride(0), _ptr(gate), gate.stride(0),
         _ptr(meta.q_start), _ptr(meta.seq_lens), meta.seq_lens.shape[0], _ptr(key_start), _ptr(first_key), t, rows, blocks, d.heads, d.dim,
         d.rot, d.vdim, d.window, float(d.scale), _lib.stream_ptr()), "zb_latent_prefill_tc")
     return out
+
+
+def prefill(q, gate, w_ukv, inv_freq, cache, meta, d: LatentDims):
+    """The expanded formulation on the tensor cores (bf16)."""
+    lat, kv, rot_out, plan = expand(cache, w_ukv, meta, d)
+    return attend_expanded(pack_q(q, inv_freq, meta.positions, d), gate, lat, kv, rot_out, plan, meta, d)
 
 
 def _expands(q, gate, meta, d: LatentDims) -> bool:
