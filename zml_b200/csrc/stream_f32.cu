@@ -62,77 +62,127 @@ ZB_DEVICE void emit_h(const ConvArgs& a, long long t, int c, float h, float h_pr
   for (int m = 0; m < a.nmix; ++m) zb_st_act(out + m * a.plane, h + delta * a.mu[static_cast<size_t>(m) * a.d + c]);
 }
 
-// One thread owns a channel and walks a block of kConvRows tokens of one sequence.
+template <int V>
+ZB_DEVICE void ld_vec(float (&v)[V], const float* p) {
+  if constexpr (V == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+  } else {
+    v[0] = *p;
+  }
+}
+template <typename A, int V>
+ZB_DEVICE void st_vec(A* p, const float (&v)[V]) {
+  if constexpr (V == 4 && sizeof(A) == 2) *reinterpret_cast<uint2*>(p) = make_uint2(zb_pack_bf16x2(v[0], v[1]), zb_pack_bf16x2(v[2], v[3]));
+  else if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else zb_st_act(p, v[0]);
+}
+
+// One thread owns V neighbouring channels and walks a block of kConvRows tokens of one sequence; T >= taps bounds the
+// unrolled window.
 constexpr int kConvRows = 32;
 
-template <typename A>
+template <typename A, int T, int V, bool MIX>
 __global__ void __launch_bounds__(128) zb_stream_conv_kernel(const float* __restrict__ x, const ConvArgs a, const ZbVarlen b) {
   zb_pdl_launch();
   zb_pdl_wait();
-  const int c = blockIdx.x * 128 + threadIdx.x;
+  const int c = (blockIdx.x * 128 + threadIdx.x) * V;
   int s, blk;
   if (c >= a.d || !zb_find_block(b, kConvRows, blockIdx.y, s, blk)) return;
   const int slot = a.slots[s];
   if (!ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelStreamConv, 1)) return;
   const int t0 = b.q_start[s], n = b.q_start[s + 1] - t0;
   const bool fresh = b.seq_lens[s] - n <= 0;
-  float* st = a.state + static_cast<size_t>(slot) * a.rows * a.d + c;
+  const int taps = a.taps, rows = a.rows;
+  float* st = a.state + static_cast<size_t>(slot) * rows * a.d + c;
+  const float* xs = x + static_cast<size_t>(t0) * a.d + c;
   // input `i` tokens after the launch's first token of this sequence (negative: before it)
-  auto input = [&](int i) -> float {
-    if (i >= 0) return x[static_cast<size_t>(t0 + i) * a.d + c];
-    return fresh || i < -a.rows ? 0.f : st[static_cast<size_t>(a.rows + i) * a.d];
-  };
-  const int taps = a.taps;
-  float w[kMaxTaps], win[kMaxTaps];           // win[j]: the input `taps - 1 - j` tokens before the current one
+  auto input = [&](int i, float (&v)[V]) {
 #pragma unroll
-  for (int j = 0; j < kMaxTaps; ++j) {
-    w[j] = j < taps ? a.w[static_cast<size_t>(c) * taps + j] : 0.f;
-    win[j] = 0.f;
+    for (int e = 0; e < V; ++e) v[e] = 0.f;
+    if (i >= 0) ld_vec<V>(v, xs + static_cast<size_t>(i) * a.d);
+    else if (!fresh && i >= -rows) ld_vec<V>(v, st + static_cast<size_t>(rows + i) * a.d);
+  };
+  float w[T][V], win[T][V];                   // win[j]: the input T - 1 - j tokens before the current one; the last taps count
+#pragma unroll
+  for (int j = 0; j < T; ++j)
+#pragma unroll
+    for (int e = 0; e < V; ++e) w[j][e] = j >= T - taps ? a.w[static_cast<size_t>(c + e) * taps + j - (T - taps)] : 0.f;
+  float mu[MIX ? kMaxMix : 1][V];
+  if constexpr (MIX) {
+#pragma unroll
+    for (int m = 0; m < kMaxMix; ++m)
+      if (m < a.nmix) ld_vec<V>(mu[m], a.mu + static_cast<size_t>(m) * a.d + c);
   }
   const int i0 = blk * kConvRows, i1 = min(n, i0 + kConvRows);
-  auto conv = [&]() {
-    float acc = 0.f;
+  auto conv = [&](float (&h)[V]) {            // the newest input plus the weighted window
 #pragma unroll
-    for (int j = 0; j < kMaxTaps; ++j)
-      if (j < taps) acc += w[j] * win[j];
-    return acc;
+    for (int e = 0; e < V; ++e) {
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < T; ++j) acc = fmaf(w[j][e], win[j][e], acc);
+      h[e] = win[T - 1][e] + acc;
+    }
   };
-  float h_prev = 0.f;
-  if (a.nmix > 0) {
 #pragma unroll
-    for (int j = 0; j < kMaxTaps; ++j)
-      if (j < taps) win[j] = input(i0 - taps + j);
-    float cur = 0.f;
+  for (int j = 0; j < T; ++j) {
+    if (j >= T - taps) input(i0 - T + j, win[j]);
+    else
 #pragma unroll
-    for (int j = 0; j < kMaxTaps; ++j)
-      if (j == taps - 1) cur = win[j];
-    h_prev = cur + conv();
-  } else {
-#pragma unroll
-    for (int j = 1; j < kMaxTaps; ++j)
-      if (j < taps) win[j] = input(i0 - taps + j);
+      for (int e = 0; e < V; ++e) win[j][e] = 0.f;
   }
+  float h_prev[V];
+  conv(h_prev);                               // (used with interpolations only: there the state reaches far enough back)
+  A* out = reinterpret_cast<A*>(a.out) + static_cast<long long>(t0) * a.ld + c;
+#pragma unroll 4
   for (int i = i0; i < i1; ++i) {
-    const float cur = x[static_cast<size_t>(t0 + i) * a.d + c];
+    float cur[V], h[V];
+    ld_vec<V>(cur, xs + static_cast<size_t>(i) * a.d);
 #pragma unroll
-    for (int j = 0; j < kMaxTaps - 1; ++j) win[j] = win[j + 1];
+    for (int j = 0; j < T; ++j)
 #pragma unroll
-    for (int j = 0; j < kMaxTaps; ++j)
-      if (j == taps - 1) win[j] = cur;
-    const float h = cur + conv();
-    emit_h<A>(a, t0 + i, c, h, h_prev);
-    h_prev = h;
+      for (int e = 0; e < V; ++e) win[j][e] = j + 1 < T ? win[j + 1 < T ? j + 1 : j][e] : cur[e];
+    conv(h);
+    A* o = out + i * a.ld;
+    if constexpr (MIX) {
+#pragma unroll
+      for (int m = 0; m < kMaxMix; ++m) {
+        if (m >= a.nmix) break;
+        float v[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = fmaf(h_prev[e] - h[e], mu[m][e], h[e]);
+        st_vec<A, V>(o + m * a.plane, v);
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) h_prev[e] = h[e];
+    } else {
+      st_vec<A, V>(o, h);
+    }
   }
-  // The block that reads the old state also writes the new one: no other thread touches this channel's state.
+  // The block that reads the old state also writes the new one: no other thread touches these channels' state.
   if (blk == 0) {
-    float keep[kMaxTaps];
+    float keep[kMaxTaps][V];
 #pragma unroll
     for (int j = 0; j < kMaxTaps; ++j)
-      if (j < a.rows) keep[j] = input(n - a.rows + j);
+      if (j < rows) input(n - rows + j, keep[j]);
 #pragma unroll
     for (int j = 0; j < kMaxTaps; ++j)
-      if (j < a.rows) st[static_cast<size_t>(j) * a.d] = keep[j];
+      if (j < rows) st_vec<float, V>(st + static_cast<size_t>(j) * a.d, keep[j]);
   }
+}
+
+template <typename A, int V, bool MIX>
+cudaError_t launch_conv(const float* x, const ConvArgs& a, const ZbVarlen& b, int num_blocks, cudaStream_t s) {
+  const dim3 grid((a.d + 128 * V - 1) / (128 * V), num_blocks);
+  if (a.taps <= 3) return zb_launch(zb_stream_conv_kernel<A, 3, V, MIX>, grid, dim3(128), 0, s, x, a, b);
+  if (a.taps == 4) return zb_launch(zb_stream_conv_kernel<A, 4, V, MIX>, grid, dim3(128), 0, s, x, a, b);
+  return zb_launch(zb_stream_conv_kernel<A, kMaxTaps, V, MIX>, grid, dim3(128), 0, s, x, a, b);
+}
+template <typename A>
+cudaError_t launch_conv(const float* x, const ConvArgs& a, const ZbVarlen& b, int num_blocks, cudaStream_t s) {
+  const bool vec = a.d % 4 == 0 && a.ld % 4 == 0 && a.plane % 4 == 0;
+  if (a.nmix > 0) return vec ? launch_conv<A, 4, true>(x, a, b, num_blocks, s) : launch_conv<A, 1, true>(x, a, b, num_blocks, s);
+  return vec ? launch_conv<A, 4, false>(x, a, b, num_blocks, s) : launch_conv<A, 1, false>(x, a, b, num_blocks, s);
 }
 
 // ------------------------------------------------------------------------------------------ post norm
@@ -324,9 +374,7 @@ int zb_stream_conv(const float* x, const float* w, float* state, const int32_t* 
   const ConvArgs a = conv_args(w, state, slots, mu, out, ld, plane, taps, rows, nmix, d);
   const ZbVarlen b = {q_start, seq_lens, num_seqs};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  const dim3 grid((d + 127) / 128, num_blocks);
-  const cudaError_t e = act_f32 ? zb_launch(zb_stream_conv_kernel<float>, grid, dim3(128), 0, s, x, a, b)
-                                : zb_launch(zb_stream_conv_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, x, a, b);
+  const cudaError_t e = act_f32 ? launch_conv<float>(x, a, b, num_blocks, s) : launch_conv<__nv_bfloat16>(x, a, b, num_blocks, s);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }

@@ -148,7 +148,7 @@ def sigmoid_gate_mul(x, gate):
 
 
 # ---------------------------------------------------------------------------- WKV
-_lib.register_signature("zb_wkv_can_fuse", _i, [_i])
+_lib.register_signature("zb_wkv_step_supported", _i, [_i])
 _lib.register_signature("zb_wkv_scan", _i, [_p, _p, _p, _p, _ll, _p, _ll, _p, _p, _p, _f, _p, _p, _p, _ll, _p, _i, _i, _i, _p, _p, _i,
                                             _i, _p])
 _lib.register_signature("zb_tanh_linear", _i, [_p, _ll, _p, _ll, _i, _p, _ll, _i, _i, _i, _p])
@@ -177,14 +177,11 @@ def wkv_scan_reference(r, k, v, g, z, w0, u, norm_w, eps, state, q_start, seq_le
     return o.reshape(t, heads * dim).to(r.dtype)
 
 
-# (sequence, head) pairs from which one CTA per pair fills the GPU (148 SMs, two CTAs each)
-WKV_FUSE_PAIRS = 296
-
-
 def wkv_scan(r, k, v, g, z, w0, u, norm_w, eps, state, q_start, seq_lens, slots, heads: int, dim: int, decode: bool = False, out=None):
     """The WKV recurrence with its output norm and gate: r, k, v, g [T, heads * dim] (equal row strides), z fp32 the
     decay's pre-activation (w = exp(-exp(z + w0))), u the current token's bonus, norm_w the output norm's weight (fp32
-    [heads * dim] each), state fp32 [slots, heads, dim (value), dim (key)] updated in place.  Returns [T, heads * dim]."""
+    [heads * dim] each), state fp32 [slots, heads, dim (value), dim (key)] updated in place.  `decode`: one token per
+    sequence.  Returns [T, heads * dim]."""
     if not r.is_cuda:
         return wkv_scan_reference(r, k, v, g, z, w0, u, norm_w, eps, state, q_start, seq_lens, slots, heads, dim)
     t, n = r.shape[0], heads * dim
@@ -194,8 +191,7 @@ def wkv_scan(r, k, v, g, z, w0, u, norm_w, eps, state, q_start, seq_lens, slots,
     assert z.dtype == torch.float32 and state.dtype == torch.float32 and state.is_contiguous()
     if out is None:
         out = torch.empty((t, n), dtype=r.dtype, device=r.device)
-    fuse = bool(_lib.lib().zb_wkv_can_fuse(dim)) and (decode or heads * seq_lens.shape[0] >= WKV_FUSE_PAIRS)
-    o = None if fuse else torch.empty((t, n), dtype=torch.float32, device=r.device)
+    o = None if decode and _lib.lib().zb_wkv_step_supported(dim) else torch.empty((t, n), dtype=torch.float32, device=r.device)
     _lib.check(_lib.lib().zb_wkv_scan(
         _ptr(r), _ptr(k), _ptr(v), _ptr(g), r.stride(0), _ptr(z), z.stride(0), _ptr(w0), _ptr(u), _ptr(norm_w), float(eps), _ptr(state),
         _ptr(slots), _ptr(out), out.stride(0), _ptr(o), int(r.dtype == torch.float32), heads, dim, _ptr(q_start), _ptr(seq_lens),
