@@ -42,6 +42,9 @@ WORKLOADS = {
     "tiny-llama-test": dict(batch=4, prompt=(16, 64), new_tokens=8),
     "tiny-qwen35-test": dict(batch=4, prompt=(16, 64), new_tokens=8),
     "tiny-lfm2-test": dict(batch=4, prompt=(16, 64), new_tokens=8),
+    "dopurax-1b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
+    "dopurax-8b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
+    "tiny-dopurax-test": dict(batch=4, prompt=(16, 64), new_tokens=8),
 }
 
 
@@ -208,6 +211,74 @@ def run_workload(name: str, comm, args, steps: int, warmup: int, sample_clocks: 
     return res
 
 
+# Designs whose prefill and decode throughput `--compare` sets beside the closest other family at equal size: a hybrid of
+# gated full attention (where the design has latent attention) and gated delta net (where it has WKV) with the same width,
+# depth, vocabulary, head sizes of the recurrent layers and feed-forward parameters (three matrices of 2/3 the units).
+COMPARE_SHAPES = [dict(batch=1, prompt=4096), dict(batch=8, prompt=1024), dict(batch=32, prompt=1024), dict(batch=64, prompt=2048)]
+
+
+def hybrid_twin(cfg) -> dict:
+    from zml_b200.models.dopurax import LATENT, WKV
+    lat = next(s for s in cfg.layers if s.kind == LATENT)
+    rec = next(s for s in cfg.layers if s.kind == WKV)
+    ff = max(s.ff for s in cfg.layers)
+    return dict(hidden_size=cfg.hidden_size, num_hidden_layers=len(cfg.layers), num_attention_heads=lat.heads,
+                num_key_value_heads=max(1, lat.heads // 4), head_dim=lat.dim, intermediate_size=ff * 2 // 3 // 64 * 64, vocab_size=cfg.vocab_size,
+                rms_norm_eps=cfg.norm_eps, rope_parameters=dict(rope_theta=lat.rot_base, partial_rotary_factor=0.5), linear_conv_kernel_dim=cfg.taps,
+                linear_key_head_dim=rec.dim, linear_num_key_heads=rec.heads, linear_value_head_dim=rec.dim, linear_num_value_heads=rec.heads,
+                layer_types=["full_attention" if s.kind == LATENT else "linear_attention" for s in cfg.layers], tie_word_embeddings=False)
+
+
+def compare(name: str, args) -> None:
+    """Prints one JSON line: prefill and decode tokens/s of preset `name` and of its equal-size hybrid, through
+    `Engine.generate` (device times), random weights and token ids; two untimed jobs per shape, then the timed ones."""
+    import gc
+
+    import torch
+    from zml_b200.models.dopurax import PRESETS, DopuraxConfig, DopuraxModel
+    from zml_b200.models.qwen3_5 import Qwen35Config, Qwen35Model
+    from zml_b200.serving import Engine
+    torch.cuda.set_device(0)
+    cfg = DopuraxConfig.from_hf(PRESETS[name])
+    twin = Qwen35Config.from_hf(hybrid_twin(cfg))
+    sampler = ClockSampler(True)
+    new, out = args.new_tokens or 128, {}
+    for label, build in ((name, lambda: DopuraxModel(cfg, device="cuda:0")), ("hybrid of equal size", lambda: Qwen35Model(twin, device="cuda:0"))):
+        model = build().init_random(args.seed)
+        model.SERIAL_PREFILL = True                  # the same launch mode for both
+        rows = []
+        for sh in COMPARE_SHAPES:
+            b, n = sh["batch"], sh["prompt"]
+            per = (n + new + 63) // 64 + 1
+            eng = Engine(model, num_pages=b * per + 8, max_batch=b, max_seq_len=per * 64, max_prefill_tokens=8192)
+            g = torch.Generator().manual_seed(args.seed + 1)
+            prompts = torch.randint(0, cfg.vocab_size, (b, n), generator=g).tolist()
+            for _ in range(2):
+                eng.generate(prompts, new)
+            pre = dec = 0.0
+            for _ in range(max(1, args.steps)):
+                _, st = eng.generate(prompts, new)
+                pre += st.prefill_ms
+                dec += st.decode_ms
+            k = max(1, args.steps)
+            rows.append({"batch": b, "prompt": n, "prefill_tok_s": round(k * b * n / pre * 1e3), "decode_tok_s": round(k * b * (new - 1) / dec * 1e3),
+                         "prefill_ms": round(pre / k, 2), "decode_ms_per_step": round(dec / k / (new - 1), 4)})
+            progress_plain(f"{label}: {rows[-1]}")
+            del eng
+            gc.collect()
+            torch.cuda.empty_cache()
+        out[label] = {"params": model.config.num_params(), "layers": len(cfg.layers), "width": cfg.hidden_size, "shapes": rows}
+        del model
+        gc.collect()
+        torch.cuda.empty_cache()
+    print(json.dumps({"compare": out, "new_tokens": new, "steps": args.steps, "dtype": "bf16", "data": "synthetic token ids, random-init weights",
+                      "clocks": sampler.stop(0)}), flush=True)
+
+
+def progress_plain(msg: str) -> None:
+    print(f"[bench +{time.perf_counter() - _T0:6.1f}s] {msg}", file=sys.stderr, flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -222,6 +293,9 @@ def main() -> None:
     ap.add_argument("--headline", default="auto", choices=["auto", "none"],
                     help="auto: after the scaling configuration also measure the headline configurations that fit this "
                          "number of GPUs (Llama-3.1-70B and the NVFP4 MoE at 8, the MoE at 2 and 4), 3 timed jobs each")
+    ap.add_argument("--compare", default="", choices=["", "dopurax-1b", "dopurax-8b"],
+                    help="instead of the benchmark: prefill and decode throughput of this design beside the closest other family at equal "
+                         "size, at a few batch shapes (1 GPU)")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -234,6 +308,9 @@ def main() -> None:
 
     if not torch.cuda.is_available():
         raise SystemExit("bench.py needs a CUDA device (B200)")
+    if args.compare:
+        compare(args.compare, args)
+        return
     import faulthandler
     # a run that takes this long prints the Python stack of every thread of every rank (and again later): a cut-off
     # log then shows where each rank was

@@ -165,6 +165,7 @@ inline int zb_config_smem_once(K kernel, int smem, bool (&done)[16]) {
 
 extern "C" {
 void zb_set_pdl(int on);
+int zb_get_pdl();
 int zb_init(int device);
 int zb_num_sms();
 int zb_status_read(uint32_t* out4);     // copies {code, kernel, where, detail}; synchronises the device

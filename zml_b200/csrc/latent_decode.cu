@@ -1,25 +1,26 @@
 // Decode of latent attention in the latent space (bf16, mma.sync): one query token per sequence, all heads share one key
 // vector [c | rotated part] per cached token, whose first `rank` elements are the value as well.
 //
-// A CTA takes up to 16 * MT heads of one sequence and a chunk of its visible tokens.  A producer warp brings 64 cache
-// rows at a time into a ring of padded shared-memory rows (one bulk copy per row, mbarrier completion); eight consumer
-// warps compute
-//   scores   warp (key group, K half): 16 keys x all heads over half of the row, the halves are added by the softmax
+// A CTA takes up to 16 * MT heads of one sequence and a chunk of its visible tokens.  A producer warp brings 32 cache
+// rows at a time into a ring of padded shared-memory rows (one bulk copy per row, mbarrier completion); small tiles keep
+// the ring deep enough for the copies to run without gaps.  Eight consumer warps compute
+//   scores   warp (key group, K quarter): 16 keys x all heads over a quarter of the row, added by the softmax
 //   softmax  fp32, rows spread over the 256 threads, running maximum and sum in registers
 //   values   warp w owns 8 * NT latent columns of the output accumulator for all heads
-// Every cache row is read once per group of heads.  A sequence's chunks leave partial results in scratch, and the last
-// chunk to finish merges them.  Every wait is bounded.
+// Every cache row is read once per group of heads.  A sequence's chunks leave partial results in scratch for a second
+// launch to merge (with all SMs: a partial is as large as 57 cache rows).  Every wait is bounded.
 #include "act.cuh"
 #include "host_api.h"
 
 namespace {
 constexpr uint32_t kKernelId = 33;
-constexpr int kKeys = 64;
+constexpr int kKeys = 32;
 constexpr int kConsumers = 256;
 constexpr int kThreads = kConsumers + 32;
 constexpr int kScoreLd = kKeys + 4;               // fp32 score rows
 constexpr int kProbLd = kKeys + 8;                // bf16 probability rows: an odd number of 16-byte chunks
-constexpr int kMaxStages = 4;
+constexpr int kMaxStages = 6;
+constexpr int kQuarters = 4;                      // K pieces of the score products
 constexpr int kMaxSplits = 64;
 
 struct DecodeParams {
@@ -31,7 +32,6 @@ struct DecodeParams {
   const int32_t* seq_lens;
   float* part_o;                // [B, groups, splits, 16 * MT, rank_p]
   float* part_ml;               // [B, groups, splits, 16 * MT, 2]
-  uint32_t* counters;           // [B * groups], zero between launches
   int max_pages, page_size, heads, row, rank_p, window, num_splits, stages;
   float scale_log2;
   ZbStatus* status;
@@ -69,13 +69,13 @@ __global__ void __launch_bounds__(kThreads, 1) zb_latent_decode_kernel(const Dec
   extern __shared__ __align__(16) uint8_t smem[];
   const int row_bytes = p.row * 2, ld = row_bytes + 16;      // 16-byte chunks per padded row: odd, so ldmatrix has no conflicts
   uint8_t* q_s = smem;                                       // [kRows][ld]
-  uint8_t* kv_s = q_s + kRows * ld;                          // [stages][64][ld]
-  float* s_s = reinterpret_cast<float*>(kv_s + p.stages * kKeys * ld);      // [2][kRows][kScoreLd]
-  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(s_s + 2 * kRows * kScoreLd);      // [kRows][kProbLd]
+  uint8_t* kv_s = q_s + kRows * ld;                          // [stages][kKeys][ld]
+  float* s_s = reinterpret_cast<float*>(kv_s + p.stages * kKeys * ld);      // [kQuarters][kRows][kScoreLd]
+  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(s_s + kQuarters * kRows * kScoreLd);      // [kRows][kProbLd]
   float* corr_s = reinterpret_cast<float*>(p_s + kRows * kProbLd);          // [kRows]
   float* ml_s = corr_s + kRows;                              // [kRows][2]
   __shared__ uint64_t full_bar[kMaxStages], empty_bar[kMaxStages];
-  __shared__ uint32_t abort_word, last_word;
+  __shared__ uint32_t abort_word;
   volatile uint32_t* abort_flag = &abort_word;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
@@ -107,25 +107,21 @@ __global__ void __launch_bounds__(kThreads, 1) zb_latent_decode_kernel(const Dec
     for (int n = 0; n < NT; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
 
   if (warp == 8) {
-    // ------------------------------------------------------------------ producer: 64 rows per tile, two per lane
+    // ------------------------------------------------------------------ producer: 32 rows per tile, one per lane
     const int32_t* bt = p.block_table + static_cast<long long>(seq) * p.max_pages;
     uint32_t stage = 0, phase = 0;
     for (int t = tile0; t < tile1; ++t) {
+      const int key = min(t * kKeys + lane, len - 1);        // past the end: a visible row again, masked by the softmax
+      int page = bt[key / p.page_size];
+      if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelId, 1)) page = 0;
+      const __nv_bfloat16* src = p.cache + (static_cast<long long>(page) * p.page_size + key % p.page_size) * p.row;
       if (t - tile0 >= p.stages) {
         const bool ok = zb_mbar_wait(&empty_bar[stage], phase ^ 1u, abort_flag);
         if (!__all_sync(0xffffffffu, ok)) break;
       }
       if (lane == 0) zb_mbar_expect_tx(&full_bar[stage], static_cast<uint32_t>(kKeys * row_bytes));
       __syncwarp();
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int r = lane + 32 * i;
-        const int key = min(t * kKeys + r, len - 1);         // past the end: a visible row again, masked by the softmax
-        int page = bt[key / p.page_size];
-        if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelId, 1)) page = 0;
-        const long long src = static_cast<long long>(page) * p.page_size + key % p.page_size;
-        zb_bulk_load(kv_s + (stage * kKeys + r) * ld, p.cache + src * p.row, row_bytes, &full_bar[stage]);
-      }
+      zb_bulk_load(kv_s + (stage * kKeys + lane) * ld, src, row_bytes, &full_bar[stage]);
       if (++stage == static_cast<uint32_t>(p.stages)) {
         stage = 0;
         phase ^= 1u;
@@ -140,9 +136,9 @@ __global__ void __launch_bounds__(kThreads, 1) zb_latent_decode_kernel(const Dec
       *reinterpret_cast<uint4*>(q_s + r * ld + c * 16) = v;
     }
     consumer_sync();
-    const int kgrp = warp & 3, khalf = warp >> 2;
-    const int steps = p.row / 16, half = (steps + 1) / 2;
-    const int st0 = khalf * half, st1 = min(steps, st0 + half);
+    const int kgrp = warp & 1, kq = warp >> 1;
+    const int steps = p.row / 16, quarter = (steps + kQuarters - 1) / kQuarters;
+    const int st0 = kq * quarter, st1 = min(steps, st0 + quarter);
     const int srow = tid / kTpr, scol = (tid % kTpr) * kKpt;
     const int g = lane >> 2, tq = lane & 3;
     // lane's row and 16-byte half for the three kinds of ldmatrix tiles
@@ -156,7 +152,8 @@ __global__ void __launch_bounds__(kThreads, 1) zb_latent_decode_kernel(const Dec
     bool fine = true;
     uint32_t stage = 0, phase = 0;
     for (int t = tile0; t < tile1; ++t) {
-      const bool ok = zb_mbar_wait(&full_bar[stage], phase, abort_flag);
+      const bool here = zb_mbar_wait(&full_bar[stage], phase, abort_flag);
+      const bool ok = __all_sync(0xffffffffu, here);
       const uint32_t tile = ka + stage * kKeys * ld;
       float sc[MT][2][4];
 #pragma unroll
@@ -182,7 +179,7 @@ __global__ void __launch_bounds__(kThreads, 1) zb_latent_decode_kernel(const Dec
           for (int n = 0; n < 2; ++n)
 #pragma unroll
             for (int e = 0; e < 2; ++e)
-              *reinterpret_cast<float2*>(s_s + (khalf * kRows + m * 16 + g + 8 * e) * kScoreLd + kgrp * 16 + n * 8 + 2 * tq) =
+              *reinterpret_cast<float2*>(s_s + (kq * kRows + m * 16 + g + 8 * e) * kScoreLd + kgrp * 16 + n * 8 + 2 * tq) =
                   make_float2(sc[m][n][2 * e], sc[m][n][2 * e + 1]);
       }
       if (!consumer_sync_and(ok)) {
@@ -191,25 +188,24 @@ __global__ void __launch_bounds__(kThreads, 1) zb_latent_decode_kernel(const Dec
       }
       {
         const float* r0 = s_s + srow * kScoreLd + scol;
-        const float* r1 = r0 + kRows * kScoreLd;
         const int key0 = t * kKeys + scol;
         float v[kKpt], mx = m_run;
 #pragma unroll
         for (int i = 0; i < kKpt; ++i) {
-          v[i] = (r0[i] + r1[i]) * p.scale_log2;
+          v[i] = ((r0[i] + r0[i + kRows * kScoreLd]) + (r0[i + 2 * kRows * kScoreLd] + r0[i + 3 * kRows * kScoreLd])) * p.scale_log2;
           if (key0 + i < first || key0 + i >= len) v[i] = -INFINITY;
           mx = fmaxf(mx, v[i]);
         }
 #pragma unroll
         for (int o = kTpr / 2; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
         const float use = mx == -INFINITY ? 0.f : mx;
-        const float corr = m_run == -INFINITY ? 0.f : exp2f(m_run - use);
+        const float corr = m_run == -INFINITY ? 0.f : zb_ex2(m_run - use);
         m_run = mx;
         float sum = 0.f;
         __nv_bfloat16* pr = p_s + srow * kProbLd + scol;
 #pragma unroll
         for (int i = 0; i < kKpt; i += 2) {
-          const float a = exp2f(v[i] - use), b = exp2f(v[i + 1] - use);
+          const float a = zb_ex2(v[i] - use), b = zb_ex2(v[i + 1] - use);
           sum += a + b;
           *reinterpret_cast<uint32_t*>(pr + i) = zb_pack_bf16x2(a, b);
         }
@@ -291,55 +287,57 @@ __global__ void __launch_bounds__(kThreads, 1) zb_latent_decode_kernel(const Dec
     while (zb_globaltimer() - t0 < 200000ull) {
     }
   }
-  // ------------------------------------------------------------------ the last chunk of a sequence merges
-  if (my_splits == 1) return;
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) {
-    uint32_t* c = p.counters + seq * gridDim.y + grp;
-    const uint32_t prev = atomicAdd(c, 1u);
-    last_word = prev == static_cast<uint32_t>(my_splits - 1) ? 1u : 0u;
-    if (last_word) *c = 0u;
-  }
-  __syncthreads();
-  if (last_word == 0u) return;
-  __threadfence();
-  const long long base = (static_cast<long long>(seq) * gridDim.y + grp) * p.num_splits;
-  float* f_s = s_s;                                          // [kRows][my_splits] weights of the chunks
-  for (int r = tid; r < nh; r += kThreads) {
-    float mm = -INFINITY, ll = 0.f;
-    for (int s = 0; s < my_splits; ++s) mm = fmaxf(mm, __ldcg(p.part_ml + ((base + s) * kRows + r) * 2));
+}
+
+// Merges the chunks of a sequence: one CTA per (head, sequence).
+template <int ROWS>
+__global__ void __launch_bounds__(128) zb_latent_merge_kernel(const DecodeParams p) {
+  zb_pdl_launch();
+  zb_pdl_wait();
+  __shared__ float f_s[kMaxSplits];
+  __shared__ float inv_s;
+  const int seq = blockIdx.y, head = blockIdx.x, r = head % ROWS;
+  const int len = p.seq_lens[seq];
+  const int first = p.window > 0 ? max(0, len - p.window) : 0;
+  const int tiles = (max(len, 0) + kKeys - 1) / kKeys - first / kKeys;
+  const int per = max(1, (tiles + p.num_splits - 1) / p.num_splits);
+  const int n = max(1, (tiles + per - 1) / per);
+  if (n == 1) return;                                        // written by the chunk itself
+  const long long base = (static_cast<long long>(seq) * ((p.heads + ROWS - 1) / ROWS) + head / ROWS) * p.num_splits;
+  if (threadIdx.x < 32) {
+    float m[kMaxSplits / 32], l[kMaxSplits / 32], mm = -INFINITY, ll = 0.f;
+#pragma unroll
+    for (int i = 0; i < kMaxSplits / 32; ++i) {
+      const int s = threadIdx.x + 32 * i;
+      m[i] = s < n ? p.part_ml[((base + s) * ROWS + r) * 2] : -INFINITY;
+      l[i] = s < n ? p.part_ml[((base + s) * ROWS + r) * 2 + 1] : 0.f;
+      mm = fmaxf(mm, m[i]);
+    }
+    mm = zb_warp_max(mm);
     const float use = mm == -INFINITY ? 0.f : mm;
-    for (int s = 0; s < my_splits; ++s) {
-      const float2 ml = __ldcg(reinterpret_cast<const float2*>(p.part_ml + ((base + s) * kRows + r) * 2));
-      const float f = exp2f(ml.x - use);
-      f_s[r * kMaxSplits + s] = f;
-      ll += f * ml.y;
+#pragma unroll
+    for (int i = 0; i < kMaxSplits / 32; ++i) {
+      const float f = exp2f(m[i] - use);
+      f_s[threadIdx.x + 32 * i] = f;
+      ll += f * l[i];
     }
-    ml_s[r] = ll > 0.f ? 1.f / ll : 0.f;
+    ll = zb_warp_sum(ll);
+    if (threadIdx.x == 0) inv_s = ll > 0.f ? 1.f / ll : 0.f;
   }
   __syncthreads();
-  const int pieces = p.rank_p / 4;
-  for (int i = tid; i < nh * pieces; i += kThreads) {
-    const int r = i / pieces, c = (i % pieces) * 4;
+  const float inv = inv_s;
+  for (int c = threadIdx.x * 4; c < p.rank_p; c += 512) {
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int s0 = 0; s0 < my_splits; s0 += 4) {
-      float4 v[4];
-#pragma unroll
-      for (int j = 0; j < 4; ++j)
-        v[j] = __ldcg(reinterpret_cast<const float4*>(p.part_o + ((base + min(s0 + j, my_splits - 1)) * kRows + r) * p.rank_p + c));
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        if (s0 + j >= my_splits) break;
-        const float f = f_s[r * kMaxSplits + s0 + j];
-        o.x += f * v[j].x;
-        o.y += f * v[j].y;
-        o.z += f * v[j].z;
-        o.w += f * v[j].w;
-      }
+#pragma unroll 4
+    for (int s = 0; s < n; ++s) {
+      const float4 v = *reinterpret_cast<const float4*>(p.part_o + ((base + s) * ROWS + r) * p.rank_p + c);
+      const float f = f_s[s];
+      o.x = fmaf(f, v.x, o.x);
+      o.y = fmaf(f, v.y, o.y);
+      o.z = fmaf(f, v.z, o.z);
+      o.w = fmaf(f, v.w, o.w);
     }
-    const float inv = ml_s[r];
-    *reinterpret_cast<uint2*>(p.out + (static_cast<long long>(seq) * p.heads + h0 + r) * p.ld_out + c) =
+    *reinterpret_cast<uint2*>(p.out + (static_cast<long long>(seq) * p.heads + head) * p.ld_out + c) =
         make_uint2(zb_pack_bf16x2(o.x * inv, o.y * inv), zb_pack_bf16x2(o.z * inv, o.w * inv));
   }
 }
@@ -348,7 +346,7 @@ constexpr int kMaxSmem = 232448 - 1024;           // static shared memory and th
 
 int smem_bytes(int rows, int row, int stages) {
   const int ld = row * 2 + 16;
-  return rows * ld + stages * kKeys * ld + 2 * rows * kScoreLd * 4 + rows * kProbLd * 2 + rows * 4 + rows * 8;
+  return rows * ld + stages * kKeys * ld + kQuarters * rows * kScoreLd * 4 + rows * kProbLd * 2 + rows * 4 + rows * 8;
 }
 int pick_stages(int rows, int row) {
   for (int s = kMaxStages; s >= 2; --s)
@@ -364,7 +362,10 @@ int launch(const DecodeParams& p, int batch, int groups, cudaStream_t s) {
   const cudaError_t e = zb_launch(zb_latent_decode_kernel<MT, NT>, dim3(p.num_splits, groups, batch), dim3(kThreads),
                                   smem_bytes(16 * MT, p.row, p.stages), s, p);
   zb_count_launch(1);
-  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+  if (e != cudaSuccess || p.num_splits == 1) return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+  const cudaError_t m = zb_launch(zb_latent_merge_kernel<16 * MT>, dim3(p.heads, batch), dim3(128), 0, s, p);
+  zb_count_launch(1);
+  return static_cast<int>(m != cudaSuccess ? m : cudaGetLastError());
 }
 }  // namespace
 
@@ -391,7 +392,6 @@ int zb_latent_decode(const void* q, const void* cache, int row, void* out, long 
   const size_t cells = static_cast<size_t>(batch) * groups;
   const size_t per_split = cells * rows * (static_cast<size_t>(rank_p) + 2) * sizeof(float);
   while (num_splits > 1 && per_split * num_splits > st->attn_scratch_bytes) --num_splits;
-  if (num_splits > 1 && cells > static_cast<size_t>(st->attn_counters_len)) num_splits = 1;
   DecodeParams p = {};
   p.q = reinterpret_cast<const __nv_bfloat16*>(q);
   p.cache = reinterpret_cast<const __nv_bfloat16*>(cache);
@@ -401,7 +401,6 @@ int zb_latent_decode(const void* q, const void* cache, int row, void* out, long 
   p.seq_lens = seq_lens;
   p.part_o = st->attn_scratch;
   p.part_ml = st->attn_scratch + cells * num_splits * rows * rank_p;
-  p.counters = st->attn_counters;
   p.max_pages = max_pages;
   p.page_size = page_size;
   p.heads = heads;

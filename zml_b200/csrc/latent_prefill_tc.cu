@@ -52,7 +52,6 @@ template <int NQ, int NV, int STAGES>
 __global__ void __launch_bounds__(kThreads, 1)
 zb_latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
                             const __grid_constant__ CUtensorMap tmap_shared, const LatentPrefillParams p) {
-  zb_pdl_launch();
   zb_pdl_wait();
   constexpr int kQBytes = NQ * kQSub;
   constexpr int kKBytes = NQ * kKvSub, kVBytes = NV * kKvSub;
@@ -124,6 +123,7 @@ zb_latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
   __syncthreads();
   zb_tc_fence_after();
   const uint32_t tmem_base = *tmem_holder;
+  zb_pdl_launch();       // only now: a dependent CTA that allocated its tensor memory first would block this one for good
 
   if (warp == 8) {
     // ------------------------------------------------------------------ TMA producer

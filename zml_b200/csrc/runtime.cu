@@ -44,6 +44,7 @@ bool zb_pdl_enabled() {
   return v != 0;
 }
 extern "C" void zb_set_pdl(int on) { g_pdl.store(on ? 1 : 0); }
+extern "C" int zb_get_pdl() { return zb_pdl_enabled() ? 1 : 0; }
 
 void zb_count_launch(int n) { g_launches.fetch_add(static_cast<unsigned long long>(n)); }
 

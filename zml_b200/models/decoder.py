@@ -42,6 +42,8 @@ class DecoderModel:
     KERNEL_SOURCES: Optional[tuple] = None
     # True when the model's kernels also run in fp32 on the GPU
     FP32_ON_GPU = False
+    # True: varlen batches (prompts and portions of them) run without programmatic dependent launch
+    SERIAL_PREFILL = False
 
     def __init__(self, config, comm: Optional[Comm] = None, device="cpu", dtype=torch.bfloat16):
         self.config = config

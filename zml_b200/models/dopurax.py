@@ -174,6 +174,9 @@ class DopuraxModel(DecoderModel):
     KERNEL_SOURCES = ("runtime", "gemm_bf16", "gemm_2cta", "gemm_f32", "elementwise", "stream_f32", "latent_attention",
                       "latent_prefill_tc", "latent_decode", "wkv", "moe")
     FP32_ON_GPU = True
+    # With overlapping launches a prefill of several chunks queued back to back has stopped making progress (some kernel of
+    # the chain waits for resources that a later one holds); serial launches cost nothing here, the kernels are long.
+    SERIAL_PREFILL = True
 
     def __init__(self, config: DopuraxConfig, comm: Optional[Comm] = None, device="cpu", dtype=torch.bfloat16):
         super().__init__(config, comm, device, dtype)

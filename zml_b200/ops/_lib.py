@@ -6,6 +6,7 @@ to PyTorch silently; `lib()` raises instead.
 """
 from __future__ import annotations
 
+import contextlib
 import ctypes as C
 import os
 from pathlib import Path
@@ -39,6 +40,8 @@ class CollectiveTimeout(KernelError):
 _SIGS = {
     "zb_init": (c_i, [c_i]),
     "zb_num_sms": (c_i, []),
+    "zb_set_pdl": (None, [c_i]),
+    "zb_get_pdl": (c_i, []),
     "zb_status_read": (c_i, [c_p]),
     "zb_status_reset": (c_i, []),
     "zb_status_ptr": (c_p, []),
@@ -198,6 +201,19 @@ def raise_on_status() -> None:
         if code == 3:
             raise BoundsError(msg, str(KERNEL_NAMES.get(kernel, kernel)), where, detail if detail < 2 ** 31 else detail - 2 ** 32)
         raise KernelError(msg)
+
+
+@contextlib.contextmanager
+def serial_launches():
+    """Kernels launched inside start only when their predecessor in the stream is complete (no programmatic dependent
+    launch)."""
+    l = lib()
+    on = l.zb_get_pdl()
+    l.zb_set_pdl(0)
+    try:
+        yield
+    finally:
+        l.zb_set_pdl(on)
 
 
 def stream_ptr(stream=None) -> int:

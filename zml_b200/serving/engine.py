@@ -18,6 +18,7 @@ schedule (SPMD), so no control traffic is needed.
 """
 from __future__ import annotations
 
+import contextlib
 import time
 from dataclasses import dataclass, field
 from typing import Optional, Sequence as Seq
@@ -225,6 +226,9 @@ class Engine:
             chunks.append(cur)
         return chunks
 
+    def _varlen_launches(self):
+        return _lib.serial_launches() if self.on_gpu and self.model.SERIAL_PREFILL else contextlib.nullcontext()
+
     def _varlen_meta(self, chunk, rows: list[int], stats: Optional[GenerationStats]):
         """(token ids, AttnMeta) on the device of one flattened varlen batch of (request, start, end) token ranges;
         `rows`: the rows of the batch whose logits are needed."""
@@ -262,13 +266,14 @@ class Engine:
                 rows.append(t - 1)
                 done.append(r)
         ids, meta = self._varlen_meta(chunk, rows, stats)
-        if rows:
-            toks = self.model.forward(ids, meta, self.kv_cache, strategy, self.seed, 0, rng=self.d_rng)
-            if strategy is not None and strategy.topk > 1:
-                ops.advance_rng(self.d_rng)
-        else:
-            self.model.hidden_states(ids, meta, self.kv_cache)
-            toks = None
+        with self._varlen_launches():
+            if rows:
+                toks = self.model.forward(ids, meta, self.kv_cache, strategy, self.seed, 0, rng=self.d_rng)
+                if strategy is not None and strategy.topk > 1:
+                    ops.advance_rng(self.d_rng)
+            else:
+                self.model.hidden_states(ids, meta, self.kv_cache)
+                toks = None
         for r, a, b in chunk:
             r.computed = b
         return done, toks, t
@@ -295,8 +300,9 @@ class Engine:
                 rows.extend(base + p for p in w)
                 base += b - a
             ids, meta = self._varlen_meta(chunk, rows, None)
-            x = self.model.hidden_states(ids, meta, self.kv_cache)
-            lg = self.model.logits(x, meta.logits_rows) if rows else None
+            with self._varlen_launches():
+                x = self.model.hidden_states(ids, meta, self.kv_cache)
+                lg = self.model.logits(x, meta.logits_rows) if rows else None
         for r, a, b in chunk:
             r.computed = b
         if lg is not None and self.model.comm.world > 1:
