@@ -300,7 +300,7 @@ def bench_stream(a: Args) -> None:
     ms = timed_graph([lambda x=x: stream.post_norm(x, w, 1e-5, y, 2.0, act_dtype=torch.bfloat16) for x in xs], a.iters, a.warmup)
     report(a, ms, t * d * 14, 0, {"part": "post_norm", "tokens": t, "d": d})
     for mixes in (False, True):
-        conv = stream.InputConv(torch.randn(d, 4, device="cuda"), torch.zeros(1, 4 if mixes else 3, d, device="cuda"), mu if mixes else None)
+        conv = stream.InputConv(torch.randn(4, d, device="cuda"), torch.zeros(1, 4 if mixes else 3, d, device="cuda"), mu if mixes else None)
         ms = timed_graph([lambda x=x: stream.stream_conv(x, conv, qs, sl, slots, torch.bfloat16) for x in xs], a.iters, a.warmup)
         report(a, ms, t * d * (4 + (10 if mixes else 2)), 0, {"part": "stream_conv", "mixes": mixes, "tokens": t, "d": d})
 

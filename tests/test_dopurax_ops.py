@@ -80,7 +80,7 @@ def test_input_convolution_in_portions_and_slots(target, taps, mixes):
         prev = np.concatenate([np.zeros_like(h[:1]), h[:-1]])
         want.append(h if mu is None else np.stack([h + (prev - h) * npd(mu[m]) for m in range(5)]))
     state = torch.full((4, stream.InputConv.rows_for(taps, mixes), d), 1e4, device=dev)       # whatever the slots held before
-    conv = stream.InputConv(w.to(dev), state, None if mu is None else mu.to(dev).contiguous())
+    conv = stream.InputConv(w.t().contiguous().to(dev), state, None if mu is None else mu.to(dev).contiguous())
     slots = i32([2, 1], dev)
     at = [0, 0]
     for ns in ((2, 3), (1, 1), (40, 2), (1, 33), (27, 1)):
@@ -98,14 +98,14 @@ def test_input_convolution_in_portions_and_slots(target, taps, mixes):
 @pytest.mark.parametrize("target", TARGETS)
 @pytest.mark.parametrize("taps", [1, 3, 8])
 @pytest.mark.parametrize("mixes", [False, True])
-@pytest.mark.parametrize("d", [64, 70])
+@pytest.mark.parametrize("d", [64, 70, 2500])
 def test_decode_step_norm_and_convolution_in_one_launch(target, taps, mixes, d):
     dev, dt = target
     w, nw = rnd((d, taps), 1), rnd((d,), 2)
     mu = rnd((5, d), 3).to(dev).contiguous() if mixes else None
     rows = stream.InputConv.rows_for(taps, mixes)
-    a = stream.InputConv(w.to(dev), torch.zeros((3, rows, d), device=dev), mu)
-    b = stream.InputConv(w.to(dev), torch.full((3, rows, d), 7.0, device=dev), mu)
+    a = stream.InputConv(w.t().contiguous().to(dev), torch.zeros((3, rows, d), device=dev), mu)
+    b = stream.InputConv(w.t().contiguous().to(dev), torch.full((3, rows, d), 7.0, device=dev), mu)
     slots = i32([2, 0], dev)
     for t in range(taps + 3):
         x, y = rnd((2, d), 10 + t).to(dev), rnd((2, d), 50 + t).to(dev)
@@ -162,7 +162,7 @@ def test_wkv_recurrence(target, heads, dim):
 def test_low_rank_decay_keeps_more_than_bf16(target, t, rank, n):
     dev, dt = target
     a, w = torch.randn((t, rank), generator=torch.Generator().manual_seed(1)).to(dev), rnd((n, rank), 2).to(dev, dt)
-    got = la.tanh_linear(a, w, la.split_weight(w))
+    got = la.tanh_linear(a, w.t().contiguous(), la.split_weight(w))
     close(got, np.tanh(npd(a)) @ npd(w).T, 2e-5)
 
 

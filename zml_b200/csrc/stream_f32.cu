@@ -38,7 +38,7 @@ __global__ void __launch_bounds__(256) zb_embedding_f32_kernel(const int32_t* __
 
 // ------------------------------------------------------------------------------------------ convolution
 struct ConvArgs {
-  const float* w;          // [d, taps], tap taps - 1 on the current token
+  const float* w;          // [taps, d], tap taps - 1 on the current token
   float* state;            // [slots, rows, d]: the last `rows` inputs, oldest first
   const int32_t* slots;    // [num_seqs]
   const float* mu;         // [nmix, d] or null
@@ -107,7 +107,7 @@ __global__ void __launch_bounds__(128) zb_stream_conv_kernel(const float* __rest
 #pragma unroll
   for (int j = 0; j < T; ++j)
 #pragma unroll
-    for (int e = 0; e < V; ++e) w[j][e] = j >= T - taps ? a.w[static_cast<size_t>(c + e) * taps + j - (T - taps)] : 0.f;
+    for (int e = 0; e < V; ++e) w[j][e] = j >= T - taps ? a.w[static_cast<size_t>(j - (T - taps)) * a.d + c + e] : 0.f;
   float mu[MIX ? kMaxMix : 1][V];
   if constexpr (MIX) {
 #pragma unroll
@@ -309,7 +309,7 @@ __global__ void __launch_bounds__(256) zb_post_norm_kernel(const PostNormArgs p,
 #pragma unroll
     for (int j = 0; j < kMaxTaps; ++j) {
       if (j < taps) {
-        const float w = a.w[static_cast<size_t>(c) * taps + j];
+        const float w = a.w[static_cast<size_t>(j) * d + c];
         if (off == 1) hp += w * hist[j];
         float in = v[i];
         if (j < taps - 1) in = off == 1 ? hist[j + 1 < kMaxTaps ? j + 1 : j] : hist[j];
@@ -326,6 +326,144 @@ __global__ void __launch_bounds__(256) zb_post_norm_kernel(const PostNormArgs p,
       else if (j == a.rows - 1) st[static_cast<size_t>(j) * d] = v[i];
     }
   }
+}
+
+// The decode step's form of the above for d a multiple of 4: 512 threads, NG groups of four channels each.  Everything
+// that the convolution reads is requested before the norm's reductions, the parameters even before the preceding kernel
+// has finished; T >= taps.
+template <int N>
+ZB_DEVICE float block_sum_warps(float v, float* red) {
+  v = zb_warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int i = 0; i < N; ++i) tot += red[i];
+  return tot;
+}
+
+template <typename A, int NG, int T, bool MIX>
+__global__ void __launch_bounds__(512) zb_post_norm_conv_kernel(const PostNormArgs p, const ConvArgs a, const ZbVarlen b) {
+  constexpr int R = MIX ? T : T - 1;                     // rows of state the window can need
+  __shared__ float red[2][16];
+  zb_pdl_launch();
+  const int d = p.d, taps = a.taps, rows = a.rows;
+  float w[NG][T][4], mu[NG][MIX ? kMaxMix : 1][4], nw[NG][4];
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + 512 * i) * 4;
+    if (c >= d) continue;
+    ld_vec<4>(nw[i], p.w + c);
+#pragma unroll
+    for (int j = 0; j < T; ++j) {                        // the last taps of the window count
+      if (j >= T - taps) ld_vec<4>(w[i][j], a.w + static_cast<size_t>(j - (T - taps)) * d + c);
+      else w[i][j][0] = w[i][j][1] = w[i][j][2] = w[i][j][3] = 0.f;
+    }
+    if constexpr (MIX) {
+#pragma unroll
+      for (int m = 0; m < kMaxMix; ++m)
+        if (m < a.nmix) ld_vec<4>(mu[i][m], a.mu + static_cast<size_t>(m) * d + c);
+    }
+  }
+  zb_pdl_wait();
+  const int s = blockIdx.x;
+  const long long t = s;
+  const int slot = a.slots[s];
+  const bool slot_ok = ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelStreamConv, 2);
+  const bool fresh = b.seq_lens[s] - 1 <= 0 || !slot_ok;
+  float* st0 = a.state + static_cast<size_t>(slot_ok ? slot : 0) * rows * d;
+  float v[NG][4], hist[NG][R > 0 ? R : 1][4];             // hist[R - 1]: the newest past input
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + 512 * i) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[i][e] = 0.f;
+    if (c >= d) continue;
+    ld_vec<4>(v[i], p.x + t * d + c);
+    float y[4] = {0.f, 0.f, 0.f, 0.f};
+    if (p.y != nullptr && p.y_f32) {
+      ld_vec<4>(y, reinterpret_cast<const float*>(p.y) + t * p.ldy + c);
+    } else if (p.y != nullptr) {
+      const uint2 g = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.y) + t * p.ldy + c);
+      const float2 lo = zb_unpack_bf16x2(g.x), hi = zb_unpack_bf16x2(g.y);
+      y[0] = lo.x; y[1] = lo.y; y[2] = hi.x; y[3] = hi.y;
+    }
+#pragma unroll
+    for (int j = 0; j < R; ++j) {
+      if (j >= R - rows && !fresh) ld_vec<4>(hist[i][j], st0 + static_cast<size_t>(j - (R - rows)) * d + c);
+      else hist[i][j][0] = hist[i][j][1] = hist[i][j][2] = hist[i][j][3] = 0.f;
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[i][e] = fmaf(p.alpha, v[i][e], y[e]);
+  }
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < NG; ++i) sum += (v[i][0] + v[i][1]) + (v[i][2] + v[i][3]);
+  const float mean = block_sum_warps<16>(sum, red[0]) / static_cast<float>(d);
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    if ((threadIdx.x + 512 * i) * 4 >= d) continue;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      v[i][e] -= mean;
+      sq = fmaf(v[i][e], v[i][e], sq);
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum_warps<16>(sq, red[1]) / static_cast<float>(d) + p.eps);
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + 512 * i) * 4;
+    if (c >= d) continue;
+    float h[4], hp[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      v[i][e] *= inv * nw[i][e];
+      float acc = w[i][T - 1][e] * v[i][e], prev = 0.f;
+#pragma unroll
+      for (int j = 0; j + 1 < T; ++j) acc = fmaf(w[i][j][e], hist[i][j + R - (T - 1)][e], acc);
+      if constexpr (MIX) {
+#pragma unroll
+        for (int j = 0; j < T; ++j) prev = fmaf(w[i][j][e], hist[i][j][e], prev);
+        prev += hist[i][R - 1][e];
+      }
+      h[e] = v[i][e] + acc;
+      hp[e] = prev;
+    }
+    if (p.x_out != nullptr) st_vec<float, 4>(p.x_out + t * d + c, v[i]);
+    A* out = reinterpret_cast<A*>(a.out) + t * a.ld + c;
+    if constexpr (MIX) {
+#pragma unroll
+      for (int m = 0; m < kMaxMix; ++m) {
+        if (m >= a.nmix) break;
+        float o[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[e] = fmaf(hp[e] - h[e], mu[i][m][e], h[e]);
+        st_vec<A, 4>(out + m * a.plane, o);
+      }
+    } else {
+      st_vec<A, 4>(out, h);
+    }
+    if (!slot_ok) continue;
+#pragma unroll
+    for (int j = 0; j < R; ++j) {
+      if (j < R - rows) continue;
+      float* dst = st0 + static_cast<size_t>(j - (R - rows)) * d + c;
+      if (j + 1 < R) st_vec<float, 4>(dst, hist[i][j + 1 < R ? j + 1 : j]);
+      else st_vec<float, 4>(dst, v[i]);
+    }
+  }
+}
+
+template <typename A, int NG, bool MIX>
+cudaError_t launch_post_norm_conv(const PostNormArgs& p, const ConvArgs& a, const ZbVarlen& b, int tokens, cudaStream_t s) {
+  if (a.taps <= 4) return zb_launch(zb_post_norm_conv_kernel<A, NG, 4, MIX>, dim3(tokens), dim3(512), 0, s, p, a, b);
+  return zb_launch(zb_post_norm_conv_kernel<A, NG, kMaxTaps, MIX>, dim3(tokens), dim3(512), 0, s, p, a, b);
+}
+template <typename A>
+cudaError_t launch_post_norm_conv(const PostNormArgs& p, const ConvArgs& a, const ZbVarlen& b, int tokens, cudaStream_t s) {
+  if (p.d <= 2048) return a.nmix > 0 ? launch_post_norm_conv<A, 1, true>(p, a, b, tokens, s) : launch_post_norm_conv<A, 1, false>(p, a, b, tokens, s);
+  return a.nmix > 0 ? launch_post_norm_conv<A, 2, true>(p, a, b, tokens, s) : launch_post_norm_conv<A, 2, false>(p, a, b, tokens, s);
 }
 
 template <typename A, bool VEC>
@@ -395,6 +533,11 @@ int zb_post_norm(const void* y, long long ldy, int y_f32, const float* x, float 
   }
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const bool vec = d % 4 == 0 && (y == nullptr || ldy % 4 == 0) && (reinterpret_cast<uintptr_t>(y) & 15) == 0;
+  if (conv_w != nullptr && vec && d <= 4096 && ld % 4 == 0 && plane % 4 == 0 && act == nullptr) {
+    const cudaError_t e = act_f32 ? launch_post_norm_conv<float>(p, a, b, tokens, s) : launch_post_norm_conv<__nv_bfloat16>(p, a, b, tokens, s);
+    zb_count_launch(1);
+    return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+  }
   if (act_f32) return vec ? launch_post_norm<float, true>(p, a, b, tokens, s) : launch_post_norm<float, false>(p, a, b, tokens, s);
   return vec ? launch_post_norm<__nv_bfloat16, true>(p, a, b, tokens, s) : launch_post_norm<__nv_bfloat16, false>(p, a, b, tokens, s);
 }

@@ -321,23 +321,41 @@ __global__ void __launch_bounds__(256) zb_wkv_finish_kernel(const WkvArgs p, lon
   }
 }
 
-// out[t, n] = sum_r tanh(a[t, r]) * w[n, r], fp32 sums: the second half of a low-rank pre-activation for few tokens.
-// One CTA: one token, 256 outputs.
+// out[t, n] = sum_r tanh(a[t, r]) * w[r, n], fp32 sums: the second half of a low-rank pre-activation for few tokens.
+// One CTA: eight tokens, 64 outputs.
+constexpr int kTlTokens = 8;
+
 template <typename W>
-__global__ void __launch_bounds__(256) zb_tanh_linear_kernel(const float* __restrict__ a, long long lda, const W* __restrict__ w, long long ldw,
-                                                             float* __restrict__ out, long long ldo, int n, int rank) {
+__global__ void __launch_bounds__(64) zb_tanh_linear_kernel(const float* __restrict__ a, long long lda, const W* __restrict__ w, long long ldw,
+                                                            float* __restrict__ out, long long ldo, int tokens, int n, int rank) {
   zb_pdl_launch();
   zb_pdl_wait();
-  extern __shared__ float tl_smem[];
-  const long long t = blockIdx.y;
-  for (int i = threadIdx.x; i < rank; i += 256) tl_smem[i] = tanhf(a[t * lda + i]);
+  extern __shared__ __align__(16) float tl_smem[];        // [rank][kTlTokens]
+  const int t0 = blockIdx.y * kTlTokens, nt = min(kTlTokens, tokens - t0);
+  for (int i = threadIdx.x; i < rank * kTlTokens; i += 64) {
+    const int t = i / rank, r = i - t * rank;
+    tl_smem[r * kTlTokens + t] = t < nt ? tanhf(a[(t0 + t) * lda + r]) : 0.f;
+  }
   __syncthreads();
-  const int c = blockIdx.x * 256 + threadIdx.x;
+  const int c = blockIdx.x * 64 + threadIdx.x;
   if (c >= n) return;
-  const W* row = w + c * ldw;
-  float acc = 0.f;
-  for (int i = 0; i < rank; ++i) acc = fmaf(tl_smem[i], zb_ld_act(row + i), acc);
-  out[t * ldo + c] = acc;
+  float acc[kTlTokens] = {};
+#pragma unroll 16
+  for (int r = 0; r < rank; ++r) {
+    const float wv = zb_ld_act(w + r * ldw + c);
+    const float4 lo = *reinterpret_cast<const float4*>(tl_smem + r * kTlTokens), hi = *reinterpret_cast<const float4*>(tl_smem + r * kTlTokens + 4);
+    acc[0] = fmaf(lo.x, wv, acc[0]);
+    acc[1] = fmaf(lo.y, wv, acc[1]);
+    acc[2] = fmaf(lo.z, wv, acc[2]);
+    acc[3] = fmaf(lo.w, wv, acc[3]);
+    acc[4] = fmaf(hi.x, wv, acc[4]);
+    acc[5] = fmaf(hi.y, wv, acc[5]);
+    acc[6] = fmaf(hi.z, wv, acc[6]);
+    acc[7] = fmaf(hi.w, wv, acc[7]);
+  }
+#pragma unroll
+  for (int t = 0; t < kTlTokens; ++t)
+    if (t < nt) out[(t0 + t) * ldo + c] = acc[t];
 }
 
 // tanh(a) as two bf16 pieces, [hi | lo] side by side: a bf16 product with the weights repeated twice along K then has
@@ -425,13 +443,14 @@ int zb_wkv_scan(const void* r, const void* k, const void* v, const void* g, long
 int zb_tanh_linear(const float* a, long long lda, const void* w, long long ldw, int w_f32, float* out, long long ldo, int tokens, int n,
                    int rank, void* stream) {
   if (tokens <= 0 || n <= 0) return 0;
-  if (rank > 8192 || tokens > 65535) return -70;
-  const dim3 grid((n + 255) / 256, tokens);
+  const size_t smem = static_cast<size_t>(rank) * kTlTokens * sizeof(float);
+  if (smem > 48 * 1024 || tokens > 65535 * kTlTokens) return -70;
+  const dim3 grid((n + 63) / 64, (tokens + kTlTokens - 1) / kTlTokens);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  const size_t smem = static_cast<size_t>(rank) * sizeof(float);
-  const cudaError_t e = w_f32 ? zb_launch(zb_tanh_linear_kernel<float>, grid, dim3(256), smem, s, a, lda, reinterpret_cast<const float*>(w), ldw, out, ldo, n, rank)
-                              : zb_launch(zb_tanh_linear_kernel<__nv_bfloat16>, grid, dim3(256), smem, s, a, lda,
-                                          reinterpret_cast<const __nv_bfloat16*>(w), ldw, out, ldo, n, rank);
+  const cudaError_t e =
+      w_f32 ? zb_launch(zb_tanh_linear_kernel<float>, grid, dim3(64), smem, s, a, lda, reinterpret_cast<const float*>(w), ldw, out, ldo, tokens, n, rank)
+            : zb_launch(zb_tanh_linear_kernel<__nv_bfloat16>, grid, dim3(64), smem, s, a, lda, reinterpret_cast<const __nv_bfloat16*>(w), ldw, out,
+                        ldo, tokens, n, rank);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }

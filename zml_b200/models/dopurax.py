@@ -200,9 +200,9 @@ class DopuraxModel(DecoderModel):
             L, t = _Layer(s), f"l{i}."
             h0, h1 = common.shard_range(s.heads, r, p)
             L.norm1 = get(t + "norm1", f32=True)
-            L.conv_w = get(t + "canon1", f32=True).contiguous()
-            if L.conv_w.shape[1] != c.taps:
-                raise ValueError(f"layer {i}: {L.conv_w.shape[1]} convolution taps in the checkpoint, {c.taps} in config.json")
+            L.conv_w = get(t + "canon1", f32=True).t().contiguous()                              # [taps, d]
+            if L.conv_w.shape[0] != c.taps:
+                raise ValueError(f"layer {i}: {L.conv_w.shape[0]} convolution taps in the checkpoint, {c.taps} in config.json")
             m = t + "mix."
             if s.kind == LATENT:
                 self._assemble_latent(L, get, m, h0, h1)
@@ -239,9 +239,10 @@ class DopuraxModel(DecoderModel):
         L.mix["mu"] = torch.stack([get(m + "mu." + x, f32=True) for x in MIX_ORDER]).contiguous()
         L.mix["rkvg"] = torch.stack([ops.pad_k(get(m + x, rows=n)) for x in MIX_ORDER[:4]]).contiguous()     # [4, H dim, d]
         L.mix["w1"] = ops.pad_k(get(m + "w1"))
-        L.mix["w2"] = get(m + "w2", rows=n).contiguous()
+        w2 = get(m + "w2", rows=n)
+        L.mix["w2_t"] = w2.t().contiguous()
         if self.dtype == torch.bfloat16:
-            L.mix["w2_split"] = la.split_weight(L.mix["w2"])
+            L.mix["w2_split"] = la.split_weight(w2)
         for name, key in (("w0", "w0"), ("norm", "norm")):
             L.mix[name] = get(m + key, f32=True)[n[0]:n[1]].contiguous()
         L.mix["u"] = get(m + "u", f32=True)[h0:h1].reshape(-1).contiguous()
@@ -309,7 +310,7 @@ class DopuraxModel(DecoderModel):
         out = {"embed": self.embed, "final.norm": self.final_norm, "head": self.lm_head[:self.v_rng[1] - self.v_rng[0], :d]}
         for i, L in enumerate(self.layers):
             s, t, m, x = L.spec, f"l{i}.", f"l{i}.mix.", L.mix
-            out.update({t + "norm1": L.norm1, t + "canon1": L.conv_w})
+            out.update({t + "norm1": L.norm1, t + "canon1": L.conv_w.t()})
             if s.kind == LATENT:
                 H, down = L.dims.heads, s.q_rank + s.rank + s.rot
                 out.update({m + "dq": x["proj"][:s.q_rank, :d], m + "dkv": x["proj"][s.q_rank:down, :d], m + "g": x["proj"][down + -down % 8:, :d],
@@ -319,7 +320,7 @@ class DopuraxModel(DecoderModel):
                 n = x["w0"].shape[0]
                 out.update({m + "mu." + k: x["mu"][j] for j, k in enumerate(MIX_ORDER)})
                 out.update({m + k: x["rkvg"][j][:, :d] for j, k in enumerate(MIX_ORDER[:4])})
-                out.update({m + "w1": x["w1"][:, :d], m + "w2": x["w2"], m + "w0": x["w0"], m + "u": x["u"].reshape(-1, s.dim), m + "norm": x["norm"],
+                out.update({m + "w1": x["w1"][:, :d], m + "w2": x["w2_t"].t(), m + "w0": x["w0"], m + "u": x["u"].reshape(-1, s.dim), m + "norm": x["norm"],
                             m + "o": x["o"][:, :n]})
             if L.ff is not None:
                 out.update({t + "norm2": L.norm2, t + "mlp.up": L.ff.up[:, :d], t + "mlp.down": L.ff.down[:, :s.ff // self.comm.world]})
@@ -389,7 +390,7 @@ class DopuraxModel(DecoderModel):
         s, m = L.spec, L.mix
         r, k, v, g = self._stacked(mix[:4], m["rkvg"])
         low = ops.gemm(mix[4], m["w1"], out_dtype=torch.float32, static_w=True)
-        z = la.tanh_linear(low, m["w2"], m.get("w2_split"))
+        z = la.tanh_linear(low, m["w2_t"], m.get("w2_split"))
         a = la.wkv_scan(r, k, v, g, z, m["w0"], m["u"], m["norm"], self.config.norm_eps, L.wkv_state, q_start, meta.seq_lens, meta.state_slots,
                         s.heads // self.comm.world, s.dim, decode=not meta.is_prefill)
         return self._out_proj(a, m["o"])

@@ -183,7 +183,7 @@ def attend(q, cache, block_table, q_start, seq_lens, d: LatentDims, decode: bool
 
 
 # tokens of a decode chunk: below this a chunk costs more in partial results than it gains in parallelism
-_MIN_CHUNK = 256
+_MIN_CHUNK = 64
 
 
 def decode_plan_splits(batch: int, d: LatentDims, max_seq_len: int) -> int:

@@ -210,23 +210,23 @@ def split_weight(w: torch.Tensor) -> torch.Tensor:
     return torch.cat([p, p], 1).contiguous()
 
 
-def tanh_linear(a, w, w_split=None):
-    """tanh(a) @ w^T with an fp32 result from a fp32 [T, R] and w [N, R]: the activation is not rounded to bf16.  On the
-    GPU few tokens take fp32 dot products, many take a bf16 GEMM over tanh(a) split into two bf16 pieces (`w_split`)."""
+def tanh_linear(a, w_t, w_split=None):
+    """tanh(a) @ w_t with an fp32 result from a fp32 [T, R] and w_t [R, N]: the activation is not rounded to bf16.  On the
+    GPU few tokens take fp32 dot products, many take a bf16 GEMM over tanh(a) split into two bf16 pieces (`w_split`, see
+    `split_weight`)."""
     if not a.is_cuda:
-        return torch.tanh(a.float()) @ w.float().t()
+        return torch.tanh(a.float()) @ w_t.float()
     t, rank = a.shape
-    n = w.shape[0]
+    n = w_t.shape[1]
     l = _lib.lib()
-    if w.dtype == torch.bfloat16 and w_split is not None and t > TANH_LINEAR_TOKENS:
+    if w_t.dtype == torch.bfloat16 and w_split is not None and t > TANH_LINEAR_TOKENS:
         from . import gemm
         half = w_split.shape[1] // 2
         s = torch.empty((t, 2 * half), dtype=torch.bfloat16, device=a.device)
         _lib.check(l.zb_tanh_split(_ptr(a), a.stride(0), _ptr(s), half, rank, t, _lib.stream_ptr()), "zb_tanh_split")
         return gemm(s, w_split, out_dtype=torch.float32, static_w=True)
+    assert w_t.stride(1) == 1
     out = torch.empty((t, n), dtype=torch.float32, device=a.device)
-    for t0 in range(0, t, 32768):
-        t1 = min(t, t0 + 32768)
-        _lib.check(l.zb_tanh_linear(_ptr(a[t0:]), a.stride(0), _ptr(w), w.stride(0), int(w.dtype == torch.float32), _ptr(out[t0:]),
-                                    out.stride(0), t1 - t0, n, rank, _lib.stream_ptr()), "zb_tanh_linear")
+    _lib.check(l.zb_tanh_linear(_ptr(a), a.stride(0), _ptr(w_t), w_t.stride(0), int(w_t.dtype == torch.float32), _ptr(out), out.stride(0), t, n,
+                                rank, _lib.stream_ptr()), "zb_tanh_linear")
     return out

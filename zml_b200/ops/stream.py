@@ -50,7 +50,7 @@ class InputConv:
     """The convolution in front of a mixer and what follows it: h = x + conv(x), and with `mu` [nmix, d] the
     interpolations h + (h_prev - h) * mu_m of h with the previous token's h.  `state` is [slots, rows, d] fp32: the
     last inputs x of every sequence, `rows_for(taps, nmix)` of them."""
-    w: torch.Tensor                       # [d, taps] fp32, tap taps - 1 on the current token
+    w: torch.Tensor                       # [taps, d] fp32, tap taps - 1 on the current token
     state: torch.Tensor
     mu: Optional[torch.Tensor] = None
 
@@ -62,23 +62,23 @@ class InputConv:
         return 0 if self.mu is None else self.mu.shape[0]
 
     def check(self) -> None:
-        d, taps = self.w.shape
+        taps, d = self.w.shape
         if not 1 <= taps <= MAX_TAPS:
             raise ValueError(f"the input convolution takes 1 to {MAX_TAPS} taps, not {taps}")
         assert self.w.dtype == torch.float32 and self.w.is_contiguous() and self.state.is_contiguous()
         assert self.state.shape[1:] == (self.rows_for(taps, self.mu is not None), d), self.state.shape
 
     def alloc(self, tokens: int, dtype, device):
-        shape = (tokens, self.w.shape[0]) if self.mu is None else (self.nmix(), tokens, self.w.shape[0])
+        shape = (tokens, self.w.shape[1]) if self.mu is None else (self.nmix(), tokens, self.w.shape[1])
         return torch.empty(shape, dtype=dtype, device=device)
 
     def args(self, out):
         """The trailing kernel arguments: out pointer, row stride, plane stride, taps, rows, nmix."""
-        return (_ptr(out), out.stride(-2), out.stride(0) if self.mu is not None else 0, self.w.shape[1], self.state.shape[1], self.nmix())
+        return (_ptr(out), out.stride(-2), out.stride(0) if self.mu is not None else 0, self.w.shape[0], self.state.shape[1], self.nmix())
 
 
 def _stream_conv_reference(x, conv: InputConv, q_start, seq_lens, slots, dtype):
-    d, taps = conv.w.shape
+    taps, d = conv.w.shape
     rows = conv.state.shape[1]
     out = conv.alloc(x.shape[0], dtype, x.device)
     qs, sl, so = q_start.tolist(), seq_lens.tolist(), slots.tolist()
@@ -89,7 +89,7 @@ def _stream_conv_reference(x, conv: InputConv, q_start, seq_lens, slots, dtype):
         fresh = sl[s] - (b - a) <= 0
         hist = torch.zeros((rows, d)) if fresh else conv.state[so[s]]
         full = torch.cat([torch.zeros((taps - rows, d)), hist, x[a:b]], 0)             # [taps + n, d]
-        h = full[taps - 1:] + (full.unfold(0, taps, 1) * conv.w[None]).sum(-1)          # previous token's h, then n of them
+        h = full[taps - 1:] + (full.unfold(0, taps, 1) * conv.w.t()[None]).sum(-1)          # previous token's h, then n of them
         if conv.mu is None:
             out[a:b] = h[1:].to(dtype)
         else:
