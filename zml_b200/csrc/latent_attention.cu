@@ -21,14 +21,6 @@ constexpr uint32_t kKernelPrep = 28;
 constexpr uint32_t kKernelAttend = 29;
 constexpr uint32_t kKernelGather = 30;
 
-ZB_DEVICE float block_sum_128(float v, float* red) {
-  v = zb_warp_sum(v);
-  __syncthreads();
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  return red[0] + red[1] + red[2] + red[3];
-}
-
 // ------------------------------------------------------------------------------------------ prep
 struct PrepArgs {
   const void* in;            // [T, ld_in]: query latent | c | shared key part
@@ -47,42 +39,77 @@ struct PrepArgs {
   int q_rank, rank, rot, rot_off;
 };
 
-template <typename A>
-__global__ void __launch_bounds__(128) zb_latent_prep_kernel(const PrepArgs p) {
+// NV values per thread; the input row is read once, and both norms are reduced together.
+template <typename A, int NV>
+__global__ void __launch_bounds__(256) zb_latent_prep_kernel(const PrepArgs p) {
+  __shared__ float red[2][8];
+  __shared__ float rot_s[2048];
   zb_pdl_launch();
+  const int cols = p.q_rank + p.rank + p.rot;
+  float w[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {                 // the norm weights are parameters
+    const int c = threadIdx.x + 256 * i;
+    w[i] = c < p.q_rank ? p.q_norm[c] : (c < p.q_rank + p.rank ? p.c_norm[c - p.q_rank] : 0.f);
+  }
   zb_pdl_wait();
-  __shared__ float red[4];
   const long long t = blockIdx.x;
   const A* in = reinterpret_cast<const A*>(p.in) + t * p.ld_in;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < p.q_rank; i += 128) {
-    const float v = zb_ld_act(in + i);
-    ss += v * v;
-  }
-  float inv = 1.f / sqrtf(block_sum_128(ss, red) / static_cast<float>(p.q_rank) + p.eps);
-  A* cq = reinterpret_cast<A*>(p.cq) + t * p.ld_cq;
-  for (int i = threadIdx.x; i < p.q_rank; i += 128) zb_st_act(cq + i, zb_ld_act(in + i) * inv * p.q_norm[i]);
-
   const long long slot = p.slots[t];
-  if (slot >= p.num_rows) (void)ZB_BC_OK(slot, p.num_rows, kKernelPrep, 1);
-  if (slot < 0 || slot >= p.num_rows) return;              // uniform over the block
-  const A* c = in + p.q_rank;
-  ss = 0.f;
-  for (int i = threadIdx.x; i < p.rank; i += 128) {
-    const float v = zb_ld_act(c + i);
-    ss += v * v;
-  }
-  inv = 1.f / sqrtf(block_sum_128(ss, red) / static_cast<float>(p.rank) + p.eps);
-  A* row = reinterpret_cast<A*>(p.cache) + slot * p.ld_cache;
-  for (int i = threadIdx.x; i < p.rank; i += 128) zb_st_act(row + i, zb_ld_act(c + i) * inv * p.c_norm[i]);
   const float pos = static_cast<float>(p.positions[t]);
-  for (int i = threadIdx.x; i < p.rot / 2; i += 128) {
+  A raw[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) raw[i] = in[min(threadIdx.x + 256 * i, cols - 1)];
+  float v[NV], sq = 0.f, sc = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = threadIdx.x + 256 * i;
+    v[i] = zb_ld_act(&raw[i]);
+    if (c < p.q_rank) sq = fmaf(v[i], v[i], sq);
+    else if (c < p.q_rank + p.rank) sc = fmaf(v[i], v[i], sc);
+    else if (c < cols) rot_s[c - p.q_rank - p.rank] = v[i];
+  }
+  sq = zb_warp_sum(sq);
+  sc = zb_warp_sum(sc);
+  if ((threadIdx.x & 31) == 0) {
+    red[0][threadIdx.x >> 5] = sq;
+    red[1][threadIdx.x >> 5] = sc;
+  }
+  __syncthreads();
+  sq = sc = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    sq += red[0][i];
+    sc += red[1][i];
+  }
+  const float iq = 1.f / sqrtf(sq / static_cast<float>(p.q_rank) + p.eps), ic = 1.f / sqrtf(sc / static_cast<float>(p.rank) + p.eps);
+  if (slot >= p.num_rows) (void)ZB_BC_OK(slot, p.num_rows, kKernelPrep, 1);
+  const bool write = slot >= 0 && slot < p.num_rows;
+  A* cq = reinterpret_cast<A*>(p.cq) + t * p.ld_cq;
+  A* row = reinterpret_cast<A*>(p.cache) + (write ? slot : 0) * p.ld_cache;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = threadIdx.x + 256 * i;
+    if (c < p.q_rank) zb_st_act(cq + c, v[i] * iq * w[i]);
+    else if (c < p.q_rank + p.rank && write) zb_st_act(row + c - p.q_rank, v[i] * ic * w[i]);
+  }
+  if (!write) return;
+  for (int i = threadIdx.x; i < p.rot / 2; i += 256) {
     float sn, cs;
     sincosf(pos * p.inv_freq[i], &sn, &cs);
-    const float u = zb_ld_act(c + p.rank + 2 * i), v = zb_ld_act(c + p.rank + 2 * i + 1);
-    zb_st_act(row + p.rot_off + 2 * i, u * cs - v * sn);
-    zb_st_act(row + p.rot_off + 2 * i + 1, v * cs + u * sn);
+    const float u = rot_s[2 * i], x = rot_s[2 * i + 1];
+    zb_st_act(row + p.rot_off + 2 * i, u * cs - x * sn);
+    zb_st_act(row + p.rot_off + 2 * i + 1, x * cs + u * sn);
   }
+}
+
+template <typename A>
+cudaError_t launch_prep(const PrepArgs& p, int tokens, cudaStream_t s) {
+  const int per = (p.q_rank + p.rank + p.rot + 255) / 256;
+  if (per <= 2) return zb_launch(zb_latent_prep_kernel<A, 2>, dim3(tokens), dim3(256), 0, s, p);
+  if (per <= 4) return zb_launch(zb_latent_prep_kernel<A, 4>, dim3(tokens), dim3(256), 0, s, p);
+  if (per <= 9) return zb_launch(zb_latent_prep_kernel<A, 9>, dim3(tokens), dim3(256), 0, s, p);
+  return zb_launch(zb_latent_prep_kernel<A, 32>, dim3(tokens), dim3(256), 0, s, p);
 }
 
 // ------------------------------------------------------------------------------------------ per-head products
@@ -386,11 +413,10 @@ int zb_latent_prep(const void* in, long long ld_in, const float* q_norm, const f
                    const int32_t* positions, const int32_t* slots, void* cq, long long ld_cq, void* cache, long long ld_cache,
                    long long num_rows, float eps, int q_rank, int rank, int rot, int rot_off, int act_f32, int tokens, void* stream) {
   if (tokens <= 0) return 0;
-  if (rot % 2 != 0 || rot_off < rank || rot_off + rot > ld_cache) return -70;
+  if (rot % 2 != 0 || rot_off < rank || rot_off + rot > ld_cache || rot > 2048 || q_rank + rank + rot > 32 * 256) return -70;
   const PrepArgs p = {in, ld_in, q_norm, c_norm, inv_freq, positions, slots, cq, ld_cq, cache, ld_cache, num_rows, eps, q_rank, rank, rot, rot_off};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  const cudaError_t e = act_f32 ? zb_launch(zb_latent_prep_kernel<float>, dim3(tokens), dim3(128), 0, s, p)
-                                : zb_launch(zb_latent_prep_kernel<__nv_bfloat16>, dim3(tokens), dim3(128), 0, s, p);
+  const cudaError_t e = act_f32 ? launch_prep<float>(p, tokens, s) : launch_prep<__nv_bfloat16>(p, tokens, s);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }

@@ -328,7 +328,12 @@ constexpr int kTlTokens = 8;
 template <typename W>
 __global__ void __launch_bounds__(64) zb_tanh_linear_kernel(const float* __restrict__ a, long long lda, const W* __restrict__ w, long long ldw,
                                                             float* __restrict__ out, long long ldo, int tokens, int n, int rank) {
+  constexpr int kFirst = 64;
   zb_pdl_launch();
+  const int c = blockIdx.x * 64 + threadIdx.x;
+  W first[kFirst];                                        // the weights are parameters: on their way before the input is there
+#pragma unroll
+  for (int r = 0; r < kFirst; ++r) first[r] = w[min(r, rank - 1) * ldw + min(c, n - 1)];
   zb_pdl_wait();
   extern __shared__ __align__(16) float tl_smem[];        // [rank][kTlTokens]
   const int t0 = blockIdx.y * kTlTokens, nt = min(kTlTokens, tokens - t0);
@@ -337,12 +342,9 @@ __global__ void __launch_bounds__(64) zb_tanh_linear_kernel(const float* __restr
     tl_smem[r * kTlTokens + t] = t < nt ? tanhf(a[(t0 + t) * lda + r]) : 0.f;
   }
   __syncthreads();
-  const int c = blockIdx.x * 64 + threadIdx.x;
   if (c >= n) return;
   float acc[kTlTokens] = {};
-#pragma unroll 16
-  for (int r = 0; r < rank; ++r) {
-    const float wv = zb_ld_act(w + r * ldw + c);
+  auto add = [&](int r, float wv) {
     const float4 lo = *reinterpret_cast<const float4*>(tl_smem + r * kTlTokens), hi = *reinterpret_cast<const float4*>(tl_smem + r * kTlTokens + 4);
     acc[0] = fmaf(lo.x, wv, acc[0]);
     acc[1] = fmaf(lo.y, wv, acc[1]);
@@ -352,7 +354,12 @@ __global__ void __launch_bounds__(64) zb_tanh_linear_kernel(const float* __restr
     acc[5] = fmaf(hi.y, wv, acc[5]);
     acc[6] = fmaf(hi.z, wv, acc[6]);
     acc[7] = fmaf(hi.w, wv, acc[7]);
-  }
+  };
+#pragma unroll
+  for (int r = 0; r < kFirst; ++r)
+    if (r < rank) add(r, zb_ld_act(&first[r]));
+#pragma unroll 8
+  for (int r = kFirst; r < rank; ++r) add(r, zb_ld_act(w + r * ldw + c));
 #pragma unroll
   for (int t = 0; t < kTlTokens; ++t)
     if (t < nt) out[(t0 + t) * ldo + c] = acc[t];

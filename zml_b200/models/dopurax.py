@@ -141,7 +141,7 @@ PRESETS = {
     # the 1B- and 8B-class shapes of the benchmark (random-init): latent attention and WKV in turn
     "dopurax-1b": _preset(2048, 65536, "LW" * 8, 8192, _latent(16, 128, 64, 128, 512, 1536, 4096), dict(heads=32, dim=64)),
     "dopurax-8b": _preset(4096, 65536, "LW" * 16, 16384, _latent(32, 128, 64, 128, 512, 1536, 4096), dict(heads=32, dim=128)),
-    "tiny-dopurax-test": _preset(192, 320, "WlL", 384, _latent(4, 40, 16, 24, 56, 72, 100, 10000.0), dict(heads=3, dim=40), taps=3,
+    "tiny-dopurax-test": _preset(192, 320, "WlL", 384, _latent(4, 40, 16, 24, 56, 72, 100, 10000.0), dict(heads=4, dim=40), taps=3,
                                  decay_rank=24),
 }
 
