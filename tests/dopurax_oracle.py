@@ -41,7 +41,7 @@ def silu(z):
 
 
 def rms(z, eps):
-    """z divided by its root mean square over the last axis."""
+    """z at unit root mean square over the last axis."""
     return z / np.sqrt((z * z).mean(-1, keepdims=True) + eps)
 
 

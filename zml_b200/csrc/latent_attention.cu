@@ -1,6 +1,6 @@
 // Latent attention (multi-head attention whose keys and values are projections of one low-rank latent per token), as
 // Dopurax layers use it: the paged cache holds, per token, the normalised latent c [rank] and one rotated key part
-// [rot] shared by all heads.  A cache row is [c | pad | rotated part | pad] with both parts padded to 16 elements.
+// [rot] for every head.  A cache row is [c | pad | rotated part | pad] with both parts padded to 16 elements.
 //
 //   zb_latent_prep     one token per CTA: RMS norm of the query latent, RMS norm of c, rotation of the shared key
 //                      part, cache write

@@ -1,7 +1,7 @@
 // Layer glue of decoders that keep the residual stream in fp32:
 //
 //   zb_embedding_f32   gathers table rows (bf16 or fp32) into the fp32 stream
-//   zb_post_norm       x <- layernorm(alpha * x + y) * w, the normalisation behind a sublayer ("norm after the sum");
+//   zb_post_norm       x <- layernorm(alpha * x + y) * w, the normalisation behind a sublayer;
 //                      without y a plain layer norm.  For decode steps the same launch continues with the input
 //                      convolution of the next layer (one token per sequence: everything it needs is in the row and
 //                      in the sequence's state)

@@ -1,4 +1,4 @@
-// WKV recurrence (RWKV-style time mixing) over a varlen batch with the per-head state in registers:
+// WKV recurrence (the token mixing of RWKV models) over a varlen batch with the per-head state in registers:
 //
 //   o_t = (S_{t-1} + diag(u) k_t v_t^T)^T r_t,   S_t = diag(w_t) S_{t-1} + k_t v_t^T,   w_t = exp(-exp(z_t + w0))
 //

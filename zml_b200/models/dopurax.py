@@ -1,10 +1,10 @@
 """Dopurax: a decoder whose layers mix tokens by latent attention or by a WKV recurrence, in any order.
 
 * The residual stream is fp32 and normalised behind every sublayer: x <- layernorm(alpha x + mixer(h)), then, where the
-  layer has a feed-forward, x <- layernorm(alpha x + ff(x)); the sublayers read x itself.
+  layer has a feed-forward, x <- layernorm(alpha x + ff(x)); there is no norm in front of a sublayer.
 * What a mixer reads is h = x + conv(x), a short causal convolution per channel over time.
 * Latent attention (`ops.latent`): queries through a low-rank latent, keys and values from one cached latent per token
-  plus a rotated key part shared by all heads, a sliding window, a sigmoid output gate.
+  plus a rotary key vector common to the heads, a sliding window, a sigmoid gate on the result.
 * WKV (`ops.linear_attn.wkv_scan`): per-head matrix state with a data-dependent decay, a bonus for the current token, token
   shift in front of every projection, a per-head RMS norm and a silu gate behind.
 * Feed-forward: down(relu(up x)^2).

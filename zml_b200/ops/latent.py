@@ -1,5 +1,5 @@
-"""Latent attention: keys and values are per-head projections of one low-rank latent per token, and only the latent and
-one rotated key part shared by all heads are cached (libzb_cuda.so: latent_attention.cu).
+"""Latent attention: keys and values are per-head projections of one low-rank latent per token.  The cache holds that
+latent and a single rotary key vector, common to the heads (libzb_cuda.so: latent_attention.cu).
 
 Two formulations of the same attention, chosen by `latent_attention`:
 
@@ -48,7 +48,7 @@ class LatentDims:
     """Sizes and constants of one latent-attention layer (heads: this rank's)."""
     heads: int
     dim: int            # unrotated query / key dimensions per head
-    rot: int            # rotated ones (the key part is shared by all heads)
+    rot: int            # rotated ones (keys: one such part for every head)
     vdim: int
     rank: int           # latent size
     q_rank: int

@@ -4,7 +4,7 @@
 
 Steps come on standard input, one JSON object a line:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "x", "tokens": [41, 8], "want": [1]}, {"id": "y", "tokens": [12], "want": []}], "end": ["y"]}
 
 The entries of a step are one batch (`Engine.step`): each brings its request's next tokens and the places among them whose
 logits are wanted; a request is admitted at its first entry.  `end` names the requests that are finished after the step:
