@@ -18,6 +18,7 @@
 // to finish merges them in chunk order, in the same launch.
 #include <cuda.h>
 
+#include "attention_tiles.cuh"
 #include "common.cuh"
 #include "host_api.h"
 
@@ -98,17 +99,49 @@ struct AttnParams {
   int window;                   // sliding window (keys), <= 0: none
   float scale_log2;             // softmax scale * log2(e)
   ZbStatus* status;
+  // what the EXT instantiations add (ZbAttnExt)
+  int keep;                     // keys 0 .. keep - 1 stay visible beyond the window
+  float cap_log2;               // score cap * log2(e), 0: no cap
+  float cap_in;                 // raw score -> exponent of the cap's exponential: 2 * scale * log2(e) / cap
+  int sink;                     // 1: the softmax denominator has an additional exp(0)
+  int vdim;                     // value columns written per head; the output is [tokens, num_q_heads, vdim]
+  const __nv_bfloat16* gate;    // [tokens, ldg]: output *= sigmoid(gate), or null
+  long long ldg;
 };
+
+// Score of a raw dot product in units of log2: scaled, and with a cap c * tanh(s * scale / c) as c * (1 - 2 / (1 + e^(2x))).
+template <bool EXT>
+ZB_DEVICE float attn_score(const AttnParams& p, float s) {
+  if constexpr (EXT) {
+    if (p.cap_log2 > 0.f) return p.cap_log2 - __fdividef(2.f * p.cap_log2, 1.f + exp2f(s * p.cap_in));
+  }
+  return s * p.scale_log2;
+}
+
+// Writes one output element, gated and only as far as the values reach.
+template <int HD, bool EXT>
+ZB_DEVICE void attn_store(const AttnParams& p, size_t tok, int head, int c, float v) {
+  if constexpr (EXT) {
+    if (c >= p.vdim) return;
+    if (p.gate != nullptr) {
+      const float g = __bfloat162float(p.gate[tok * p.ldg + static_cast<size_t>(head) * p.vdim + c]);
+      v *= __fdividef(1.f, 1.f + __expf(-g));
+    }
+    p.out[(tok * p.num_q_heads + head) * p.vdim + c] = __float2bfloat16(v);
+  } else {
+    p.out[(tok * p.num_q_heads + head) * HD + c] = __float2bfloat16(v);
+  }
+}
 
 // One 16-key block: S = Q K^T (16 x 16), online softmax update, O += P V.
 //   qf     : Q fragments, HD/16 k-steps
 //   k_base : shared address of the 16 K rows of this block (tile-relative row0)
 //   row0   : first row of the block inside its swizzled tile
-//   mask0/mask1 : per-row predicate producers are inlined by the callers via `visible`
-template <int HD, int LAYOUT = 0, typename Visible>
+//   score(raw), visible(half, col): the callers' score in units of log2 and mask, inlined
+template <int HD, int LAYOUT, typename Score, typename Visible>
 ZB_DEVICE void attn_block16(const uint32_t (&qf)[HD / 16][4], uint32_t k_tile, uint32_t v_tile,
                             int row0, float (&o)[HD / 8][4], float (&m)[2], float (&l)[2],
-                            float scale_log2, Visible visible) {
+                            Score score, Visible visible) {
   const int lane = threadIdx.x & 31;
   const int mi = lane >> 3;
   const int r8 = lane & 7;
@@ -130,7 +163,7 @@ ZB_DEVICE void attn_block16(const uint32_t (&qf)[HD / 16][4], uint32_t k_tile, u
     for (int j = 0; j < 4; ++j) {
       const int col = nt * 8 + 2 * t + (j & 1);
       const int half = j >> 1;
-      float v = s[nt][j] * scale_log2;
+      float v = score(s[nt][j]);
       if (!visible(half, col)) v = -INFINITY;
       s[nt][j] = v;
       mx[half] = fmaxf(mx[half], v);
@@ -190,7 +223,7 @@ ZB_DEVICE void attn_block16(const uint32_t (&qf)[HD / 16][4], uint32_t k_tile, u
 // memory, writes the chunk's partial (or the final output when the sequence has one chunk), and
 // lets the last chunk of a (sequence, kv head) to finish merge all of them.  Every thread of the
 // CTA calls it (warps beyond the fourth only take part in the barriers and the element loops).
-template <int HD>
+template <int HD, bool EXT>
 ZB_DEVICE void decode_tail(const AttnParams& p, uint8_t* smem, const float (&o)[HD / 8][4], const float (&m)[2],
                            const float (&l)[2], int seq, int kvh, int split, int my_splits, int group) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -233,7 +266,7 @@ ZB_DEVICE void decode_tail(const AttnParams& p, uint8_t* smem, const float (&o)[
     const int head = kvh * group + r;
     if (my_splits == 1) {
       const float inv = ll > 0.f ? 1.f / ll : 0.f;
-      p.out[(static_cast<size_t>(seq) * p.num_q_heads + head) * HD + c] = __float2bfloat16(acc * inv);
+      attn_store<HD, EXT>(p, seq, head, c, acc * inv);
     } else {
       const size_t pi = (static_cast<size_t>(seq) * p.num_q_heads + head) * p.num_splits + split;
       p.part_o[pi * HD + c] = acc;
@@ -291,14 +324,14 @@ ZB_DEVICE void decode_tail(const AttnParams& p, uint8_t* smem, const float (&o)[
         }
       }
     }
-    p.out[(static_cast<size_t>(seq) * p.num_q_heads + head) * HD + c] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+    attn_store<HD, EXT>(p, seq, head, c, ll > 0.f ? acc / ll : 0.f);
   }
 }
 
 // ---------------------------------------------------------------------- decode
 constexpr int kDecStages = 3;
 
-template <int HD>
+template <int HD, bool EXT>
 __global__ void __launch_bounds__(128) zb_paged_decode_kernel(const AttnParams p) {
   zb_pdl_launch();
   zb_pdl_wait();
@@ -312,7 +345,10 @@ __global__ void __launch_bounds__(128) zb_paged_decode_kernel(const AttnParams p
   const int split = blockIdx.y;
   const int group = p.num_q_heads / p.num_kv_heads;
   const int len = p.seq_lens[seq];
-  const int nblk = (len + 15) >> 4;
+  const int first_visible = p.window > 0 ? max(0, len - p.window) : 0;
+  ZbTileList tiles = {0, 0, (len + 15) >> 4};
+  if constexpr (EXT) tiles = zb_visible_tiles(first_visible, p.keep, tiles.count, 16);
+  const int nblk = tiles.count;
   // the sequence is cut into chunks of `chunk_blocks` 16-key blocks; CTAs beyond the
   // last chunk of a short sequence have nothing to do
   const int per = p.chunk_blocks;
@@ -320,7 +356,6 @@ __global__ void __launch_bounds__(128) zb_paged_decode_kernel(const AttnParams p
   if (split >= my_splits) return;
   const int blk0 = split * per;
   const int blk1 = min(nblk, blk0 + per);
-  const int first_visible = p.window > 0 ? max(0, len - p.window) : 0;
 
   const uint32_t wbase = zb_smem_u32(smem) + warp * kWarpBytes;
   const int32_t* bt = p.block_table + static_cast<size_t>(seq) * p.max_pages;
@@ -347,10 +382,11 @@ __global__ void __launch_bounds__(128) zb_paged_decode_kernel(const AttnParams p
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  if (EXT && p.sink && split == 0 && warp == 0) m[0] = m[1] = 0.f, l[0] = l[1] = 1.f;
 
   auto issue = [&](int blk, int stage) {
     if (blk < blk1) {
-      const int tok0 = blk << 4;
+      const int tok0 = tiles.at(blk) << 4;
       int page = bt[tok0 / p.page_size];
       if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelDecode, 10)) page = 0;      // checking build: reported, page 0 read instead
       const int off0 = tok0 % p.page_size;
@@ -390,18 +426,18 @@ __global__ void __launch_bounds__(128) zb_paged_decode_kernel(const AttnParams p
     issue(nxt, fill);
     nxt += 4;
     const uint32_t ks = wbase + stage * 2 * kBlkBytes;
-    const int tok0 = blk << 4;
-    attn_block16<HD>(qf, ks, ks + kBlkBytes, 0, o, m, l, p.scale_log2,
-                     [&](int /*half*/, int col) {
-                       const int kidx = tok0 + col;
-                       return kidx < len && kidx >= first_visible;
-                     });
+    const int tok0 = tiles.at(blk) << 4;
+    attn_block16<HD, 0>(qf, ks, ks + kBlkBytes, 0, o, m, l, [&](float v) { return attn_score<EXT>(p, v); },
+                        [&](int /*half*/, int col) {
+                          const int kidx = tok0 + col;
+                          return kidx < len && (kidx >= first_visible || (EXT && kidx < p.keep));
+                        });
     __syncwarp();
     if (++stage == kDecStages) stage = 0;
   }
   cp_async_wait<0>();
   __syncthreads();
-  decode_tail<HD>(p, smem, o, m, l, seq, kvh, split, my_splits, group);
+  decode_tail<HD, EXT>(p, smem, o, m, l, seq, kvh, split, my_splits, group);
 }
 
 // ------------------------------------------------------- decode, tensor-map fed
@@ -412,7 +448,7 @@ __global__ void __launch_bounds__(128) zb_paged_decode_kernel(const AttnParams p
 template <int HD>
 constexpr int dec_tma_stages() { return HD >= 256 ? 2 : 3; }
 
-template <int HD>
+template <int HD, bool EXT>
 __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tmap_k,
                                                                   const __grid_constant__ CUtensorMap tmap_v,
                                                                   const AttnParams p) {
@@ -442,27 +478,30 @@ __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_c
   const int split = blockIdx.y;
   const int group = p.num_q_heads / p.num_kv_heads;
   const int len = p.seq_lens[seq];
-  const int nblk = (len + 15) >> 4;
+  const int first_visible = p.window > 0 ? max(0, len - p.window) : 0;
+  ZbTileList tiles = {0, 0, (len + 63) >> 6};
+  if constexpr (EXT) tiles = zb_visible_tiles(first_visible, p.keep, tiles.count, 64);
+  const int nblk = EXT ? tiles.count * 4 : (len + 15) >> 4;
   const int per = p.chunk_blocks;                          // a multiple of 4 (64 keys)
   const int my_splits = max(1, (nblk + per - 1) / per);
   if (split >= my_splits) return;
   const int blk0 = split * per;
   const int blk1 = min(nblk, blk0 + per);
   const int tile0 = blk0 >> 2, tile1 = (blk1 + 3) >> 2;
-  const int first_visible = p.window > 0 ? max(0, len - p.window) : 0;
   const int32_t* bt = p.block_table + static_cast<size_t>(seq) * p.max_pages;
 
   float o[HD / 8][4];
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  if (EXT && p.sink && split == 0 && warp == 0) m[0] = m[1] = 0.f, l[0] = l[1] = 1.f;
 
   if (warp == 4) {
     if (lane == 0) {
       uint32_t stage = 0, phase = 0;
       for (int t = tile0; t < tile1; ++t) {
         if (!zb_mbar_wait(&empty_bar[stage], phase ^ 1u, abort_flag)) break;
-        int page = bt[t];
+        int page = bt[tiles.at(t)];
         if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelDecode, 11)) page = 0;
         uint8_t* ks = smem + stage * 2 * kTileBytes;
         zb_mbar_expect_tx(&full_bar[stage], 2 * kTileBytes);
@@ -493,8 +532,8 @@ __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_c
     uint32_t stage = 0, phase = 0;
     for (int t = tile0; t < tile1; ++t) {
       if (!zb_mbar_wait(&full_bar[stage], phase, abort_flag)) break;
-      const int tok0 = t * 64 + warp * 16;                 // this warp's 16 keys of the tile
-      if (tok0 < len && (tok0 >> 4) >= blk0 && (tok0 >> 4) < blk1) {
+      const int key0 = tiles.at(t) * 64, tok0 = key0 + warp * 16;      // the tile's first key, this warp's 16 keys of it
+      if (tok0 < len && (EXT || ((tok0 >> 4) >= blk0 && (tok0 >> 4) < blk1))) {
         const uint32_t ks = zb_smem_u32(smem + stage * 2 * kTileBytes);
         const uint32_t vs = ks + kTileBytes;
         if (tok0 + 16 > len) {
@@ -502,16 +541,17 @@ __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_c
           // probabilities are zero, but 0 x NaN would still poison the sum - clear those V rows
           for (int idx = lane; idx < 16 * (HD / 8); idx += 32) {
             const int row = warp * 16 + idx / (HD / 8), chunk = idx % (HD / 8);
-            if (t * 64 + row >= len)
+            if (key0 + row >= len)
               *reinterpret_cast<uint4*>(smem + stage * 2 * kTileBytes + kTileBytes + tile_off_tma<HD>(row, chunk)) =
                   make_uint4(0u, 0u, 0u, 0u);
           }
           __syncwarp();
         }
-        attn_block16<HD, 1>(qf, ks, vs, warp * 16, o, m, l, p.scale_log2, [&](int /*half*/, int col) {
-          const int kidx = tok0 + col;
-          return kidx < len && kidx >= first_visible;
-        });
+        attn_block16<HD, 1>(qf, ks, vs, warp * 16, o, m, l, [&](float v) { return attn_score<EXT>(p, v); },
+                            [&](int /*half*/, int col) {
+                              const int kidx = tok0 + col;
+                              return kidx < len && (kidx >= first_visible || (EXT && kidx < p.keep));
+                            });
       }
       __syncwarp();
       if (lane == 0) zb_mbar_arrive(&empty_bar[stage]);
@@ -531,11 +571,11 @@ __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_c
     __syncthreads();
     return;
   }
-  decode_tail<HD>(p, smem, o, m, l, seq, kvh, split, my_splits, group);
+  decode_tail<HD, EXT>(p, smem, o, m, l, seq, kvh, split, my_splits, group);
 }
 
 // --------------------------------------------------------------------- prefill
-template <int HD>
+template <int HD, bool EXT>
 __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams p) {
   zb_pdl_launch();
   zb_pdl_wait();
@@ -570,9 +610,8 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
   const int tok_base = p.q_start[seq] + row_base;     // its token index
   const int rows_valid = min(64, q_len - row_base);
   const int last_key = min(len, ctx + row_base + 64);  // exclusive
-  const int n_tiles = (last_key + 63) >> 6;
-  int first_tile = 0;
-  if (p.window > 0) first_tile = max(0, ctx + row_base - p.window + 1) >> 6;
+  const int first_key = p.window > 0 ? max(0, ctx + row_base - p.window + 1) : 0;
+  const ZbTileList tiles = zb_visible_tiles(first_key, EXT ? p.keep : 0, (last_key + 63) >> 6, 64);
 
   const uint32_t q_s = zb_smem_u32(smem);
   const uint32_t kv_s = q_s + kTileBytes;             // 2 stages x (K tile, V tile)
@@ -603,7 +642,7 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
       cp_async16(vs + tile_off<HD>(row, chunk), p.v_cache + goff, valid ? 16u : 0u);
     }
   };
-  issue_kv(first_tile, 0);
+  issue_kv(tiles.at(0), 0);
   cp_async_commit();
 
   uint32_t qf[HD / 16][4];
@@ -611,14 +650,15 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  if (EXT && p.sink) m[0] = m[1] = 0.f, l[0] = l[1] = 1.f;
   const int g = lane >> 2;
   const int qpos0 = ctx + row_base + warp * 16 + g;   // key position limit of row g (row g+8: +8)
 
-  for (int tile = first_tile; tile < n_tiles; ++tile) {
-    const int stage = (tile - first_tile) & 1;
+  for (int it = 0; it < tiles.count; ++it) {
+    const int tile = tiles.at(it), stage = it & 1;
     cp_async_wait<0>();
     __syncthreads();
-    if (tile == first_tile) {
+    if (it == 0) {
       const int mi = lane >> 3, r8 = lane & 7;
 #pragma unroll
       for (int kk = 0; kk < HD / 16; ++kk) {
@@ -626,7 +666,7 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
         ldmatrix_x4(qf[kk], q_s + tile_off<HD>(row, 2 * kk + (mi >> 1)));
       }
     }
-    if (tile + 1 < n_tiles) issue_kv(tile + 1, stage ^ 1);
+    if (it + 1 < tiles.count) issue_kv(tiles.at(it + 1), stage ^ 1);
     cp_async_commit();
     const uint32_t ks = kv_s + stage * 2 * kTileBytes;
     const uint32_t vs = ks + kTileBytes;
@@ -636,11 +676,11 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
     for (int sub = 0; sub < 4; ++sub) {
       const int key0 = tile * 64 + sub * 16;
       if (key0 > warp_max_q) break;
-      attn_block16<HD>(qf, ks, vs, sub * 16, o, m, l, p.scale_log2, [&](int half, int col) {
+      attn_block16<HD, 0>(qf, ks, vs, sub * 16, o, m, l, [&](float v) { return attn_score<EXT>(p, v); }, [&](int half, int col) {
         const int kidx = key0 + col;
         const int qp = qpos0 + half * 8;
         bool vis = kidx <= qp && kidx < len;
-        if (p.window > 0) vis = vis && (kidx > qp - p.window);
+        if (p.window > 0) vis = vis && (kidx > qp - p.window || (EXT && kidx < p.keep));
         return vis;
       });
     }
@@ -654,6 +694,14 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
     const int row = warp * 16 + g + half * 8;
     if (row < rows_valid) {
       const float inv = l[half] > 0.f ? 1.f / l[half] : 0.f;
+      if constexpr (EXT) {
+#pragma unroll
+        for (int nt = 0; nt < HD / 8; ++nt) {
+          attn_store<HD, true>(p, tok_base + row, head, nt * 8 + 2 * t, o[nt][half * 2] * inv);
+          attn_store<HD, true>(p, tok_base + row, head, nt * 8 + 2 * t + 1, o[nt][half * 2 + 1] * inv);
+        }
+        continue;
+      }
       __nv_bfloat16* orow = p.out + (static_cast<size_t>(tok_base + row) * p.num_q_heads + head) * HD;
 #pragma unroll
       for (int nt = 0; nt < HD / 8; ++nt) {
@@ -664,26 +712,26 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
   }
 }
 
-template <int HD>
+template <int HD, bool EXT>
 int launch_decode(const AttnParams& p, cudaStream_t stream) {
   constexpr int pipe = 4 * kDecStages * 2 * 16 * HD * 2;
   constexpr int merge = 4 * 16 * HD * 4 + 4 * 16 * 2 * 4;
   constexpr int smem = pipe > merge ? pipe : merge;
   static bool configured[16] = {};
-  if (const int rc = zb_config_smem_once(zb_paged_decode_kernel<HD>, smem, configured)) return rc;
+  if (const int rc = zb_config_smem_once(zb_paged_decode_kernel<HD, EXT>, smem, configured)) return rc;
   dim3 grid(p.batch * p.num_kv_heads, p.num_splits);
-  zb_launch(zb_paged_decode_kernel<HD>, dim3(grid), dim3(128), smem, stream, p);
+  zb_launch(zb_paged_decode_kernel<HD, EXT>, dim3(grid), dim3(128), smem, stream, p);
   zb_count_launch(1);
   return static_cast<int>(cudaGetLastError());
 }
 
 int g_decode_tma = 1;
 
-template <int HD>
+template <int HD, bool EXT>
 int launch_decode_tma(const AttnParams& p, cudaStream_t stream) {
   constexpr int smem = dec_tma_stages<HD>() * 2 * 64 * HD * 2 + 1024 + 256;
   static bool configured[16] = {};
-  if (const int rc = zb_config_smem_once(zb_paged_decode_tma_kernel<HD>, smem, configured)) return rc;
+  if (const int rc = zb_config_smem_once(zb_paged_decode_tma_kernel<HD, EXT>, smem, configured)) return rc;
   CUtensorMap tk, tv;
   const long long slots = 1ll << 30;      // bound only: pages are addressed through the block table
   int rc = zb_make_tmap_kv_cache(&tk, p.k_cache, slots, p.num_kv_heads, HD, 64);
@@ -691,20 +739,49 @@ int launch_decode_tma(const AttnParams& p, cudaStream_t stream) {
   rc = zb_make_tmap_kv_cache(&tv, p.v_cache, slots, p.num_kv_heads, HD, 64);
   if (rc != 0) return rc;
   dim3 grid(p.batch * p.num_kv_heads, p.num_splits);
-  zb_launch(zb_paged_decode_tma_kernel<HD>, dim3(grid), dim3(160), smem, stream, tk, tv, p);
+  zb_launch(zb_paged_decode_tma_kernel<HD, EXT>, dim3(grid), dim3(160), smem, stream, tk, tv, p);
   zb_count_launch(1);
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int HD>
+template <int HD, bool EXT>
 int launch_prefill(const AttnParams& p, int num_q_blocks, cudaStream_t stream) {
   constexpr int smem = 5 * 64 * HD * 2;
   static bool configured[16] = {};
-  if (const int rc = zb_config_smem_once(zb_paged_prefill_kernel<HD>, smem, configured)) return rc;
+  if (const int rc = zb_config_smem_once(zb_paged_prefill_kernel<HD, EXT>, smem, configured)) return rc;
   dim3 grid(num_q_blocks, p.num_q_heads);
-  zb_launch(zb_paged_prefill_kernel<HD>, dim3(grid), dim3(128), smem, stream, p);
+  zb_launch(zb_paged_prefill_kernel<HD, EXT>, dim3(grid), dim3(128), smem, stream, p);
   zb_count_launch(1);
   return static_cast<int>(cudaGetLastError());
+}
+
+template <bool EXT>
+int dispatch_decode(const AttnParams& p, int head_dim, bool tma, cudaStream_t stream) {
+  switch (head_dim) {
+    case 64: return tma ? launch_decode_tma<64, EXT>(p, stream) : launch_decode<64, EXT>(p, stream);
+    case 128: return tma ? launch_decode_tma<128, EXT>(p, stream) : launch_decode<128, EXT>(p, stream);
+    case 256: return tma ? launch_decode_tma<256, EXT>(p, stream) : launch_decode<256, EXT>(p, stream);
+  }
+  return -32;
+}
+template <bool EXT>
+int dispatch_prefill(const AttnParams& p, int head_dim, int num_q_blocks, cudaStream_t stream) {
+  switch (head_dim) {
+    case 64: return launch_prefill<64, EXT>(p, num_q_blocks, stream);
+    case 128: return launch_prefill<128, EXT>(p, num_q_blocks, stream);
+    case 256: return launch_prefill<256, EXT>(p, num_q_blocks, stream);
+  }
+  return -32;
+}
+
+void set_ext(AttnParams& p, const ZbAttnExt& x, float scale) {
+  p.keep = x.keep;
+  p.cap_log2 = x.cap > 0.f ? x.cap * 1.4426950408889634f : 0.f;
+  p.cap_in = x.cap > 0.f ? 2.f * scale * 1.4426950408889634f / x.cap : 0.f;
+  p.sink = x.sink;
+  p.vdim = x.vdim;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(x.gate);
+  p.ldg = x.ldg;
 }
 
 }  // namespace
@@ -764,7 +841,7 @@ int zb_paged_decode_ex(const void* q, const void* k_cache, const void* v_cache, 
                        int num_q_heads, int num_kv_heads, int head_dim, int page_size, int max_pages,
                        long long q_stride, float scale, int window, int num_splits, float* scratch,
                        size_t scratch_bytes, uint32_t* counters, int counters_len, ZbStatus* status,
-                       cudaStream_t stream) {
+                       const ZbAttnExt* ext, cudaStream_t stream) {
   if (batch <= 0) return 0;
   if (num_q_heads % num_kv_heads != 0 || num_q_heads / num_kv_heads > 16) return -30;
   if (page_size % 16 != 0) return -31;
@@ -775,7 +852,12 @@ int zb_paged_decode_ex(const void* q, const void* k_cache, const void* v_cache, 
          zb_decode_scratch_bytes(batch, num_q_heads, head_dim, num_splits) > scratch_bytes)
     --num_splits;
   // chunk length that lets `num_splits` chunks cover the longest sequence the block table allows
-  const int max_blocks = (max_pages * page_size + 15) / 16;
+  int max_blocks = (max_pages * page_size + 15) / 16;
+  if (ext != nullptr && window > 0) {          // the longest list of visible tiles: the kept ones and a window that starts inside a tile
+    const int tile = page_size == 64 ? 64 : 16;
+    const int visible = ((ext->keep + tile - 1) / tile + (window + tile - 2) / tile + 1) * (tile / 16);
+    if (visible < max_blocks) max_blocks = visible;
+  }
   int chunk_blocks = (max_blocks + num_splits - 1) / num_splits;
   if (page_size == 64) chunk_blocks = (chunk_blocks + 3) / 4 * 4;      // whole pages per chunk (tensor-map fed kernel)
   AttnParams p = {};
@@ -804,24 +886,21 @@ int zb_paged_decode_ex(const void* q, const void* k_cache, const void* v_cache, 
   // 64-token pages and chunks of whole pages: the tensor-map fed kernel; otherwise per-warp cp.async
   const bool tma = g_decode_tma != 0 && page_size == 64 && (p.chunk_blocks % 4) == 0 &&
                    (reinterpret_cast<uintptr_t>(k_cache) & 15) == 0 && (reinterpret_cast<uintptr_t>(v_cache) & 15) == 0;
-  switch (head_dim) {
-    case 64: return tma ? launch_decode_tma<64>(p, stream) : launch_decode<64>(p, stream);
-    case 128: return tma ? launch_decode_tma<128>(p, stream) : launch_decode<128>(p, stream);
-    case 256: return tma ? launch_decode_tma<256>(p, stream) : launch_decode<256>(p, stream);
-  }
-  return -32;
+  if (ext == nullptr) return dispatch_decode<false>(p, head_dim, tma, stream);
+  set_ext(p, *ext, scale);
+  return dispatch_decode<true>(p, head_dim, tma, stream);
 }
 
 int zb_paged_decode(const void* q, const void* k_cache, const void* v_cache, void* out,
                     const int32_t* block_table, const int32_t* seq_lens, int batch, int num_q_heads,
                     int num_kv_heads, int head_dim, int page_size, int max_pages,
-                    long long q_stride, float scale, int window, int num_splits, void* stream) {
+                    long long q_stride, float scale, int window, int num_splits, const ZbAttnExt* ext, void* stream) {
   ZbDeviceState* st = zb_device_state();
   if (!st) return -20;
   return zb_paged_decode_ex(q, k_cache, v_cache, out, block_table, seq_lens, batch, num_q_heads,
                             num_kv_heads, head_dim, page_size, max_pages, q_stride, scale, window,
                             num_splits, st->attn_scratch, st->attn_scratch_bytes, st->attn_counters,
-                            st->attn_counters_len, st->status, reinterpret_cast<cudaStream_t>(stream));
+                            st->attn_counters_len, st->status, ext, reinterpret_cast<cudaStream_t>(stream));
 }
 
 // total_q_blocks >= sum over sequences of ceil(q_len / 64); a safe bound is
@@ -830,7 +909,7 @@ int zb_paged_prefill(const void* q, const void* k_cache, const void* v_cache, vo
                      const int32_t* block_table, const int32_t* seq_lens, const int32_t* q_start,
                      int batch, int total_q_blocks, int num_q_heads, int num_kv_heads, int head_dim,
                      int page_size, int max_pages, long long q_stride, float scale, int window,
-                     void* stream) {
+                     const ZbAttnExt* ext, void* stream) {
   if (batch <= 0 || total_q_blocks <= 0) return 0;
   if (num_q_heads % num_kv_heads != 0) return -30;
   ZbDeviceState* st = zb_device_state();
@@ -854,12 +933,9 @@ int zb_paged_prefill(const void* q, const void* k_cache, const void* v_cache, vo
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = st->status;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  switch (head_dim) {
-    case 64: return launch_prefill<64>(p, total_q_blocks, s);
-    case 128: return launch_prefill<128>(p, total_q_blocks, s);
-    case 256: return launch_prefill<256>(p, total_q_blocks, s);
-  }
-  return -32;
+  if (ext == nullptr) return dispatch_prefill<false>(p, head_dim, total_q_blocks, s);
+  set_ext(p, *ext, scale);
+  return dispatch_prefill<true>(p, head_dim, total_q_blocks, s);
 }
 
 }  // extern "C"

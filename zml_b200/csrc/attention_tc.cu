@@ -18,9 +18,13 @@
 // P = exp2(S - m) as bf16 straight back into tensor memory -> O += P V (A = P from tensor memory,
 // B = V from shared memory in its natural [key][head_dim] layout, i.e. MN-major).
 // Tensor memory columns: S_A 0-63 | S_B 64-127 | P_A 128-159 | P_B 160-191 | O_A 192-319 | O_B 320-447.
+// With a score cap c (EXT; at most kMaxCap) the running maximum goes: every score lies in [-c, c], so P = exp2(S') needs no
+// reference and O no rescaling.  Kept first keys join the window's tiles as one list, a sink is one more term of the sum,
+// and the output gate is applied as the rows are stored.
 // Every wait is bounded; a wait that runs out records a status and the CTA leaves through its normal exit.
 #include <cuda.h>
 
+#include "attention_tiles.cuh"
 #include "common.cuh"
 #include "host_api.h"
 
@@ -38,6 +42,7 @@ constexpr int kKvBytes = kKeys * kHD * 2;          // one K or V page of one KV 
 constexpr int kThreads = 320;
 constexpr uint32_t kKernelId = 13;
 constexpr uint32_t kTmemCols = 512;
+constexpr float kMaxCap = 60.f;                    // exp(cap) times the number of keys stays far inside fp32
 constexpr uint32_t kColS = 0, kColP = 128, kColO = 192;
 
 struct PrefillTcParams {
@@ -54,12 +59,61 @@ struct PrefillTcParams {
   uint32_t v_lbo;               // byte offsets of the MN-major descriptor of V (between 64-column groups / 8-key groups)
   uint32_t v_sbo;
   ZbStatus* status;
+  // EXT only (ZbAttnExt)
+  int keep;
+  float cap_log2;               // cap * log2(e)
+  float cap_in;                 // 2 * scale * log2(e) / cap
+  int sink;
+  int vdim;                     // output [tokens, num_q_heads, vdim]
+  const __nv_bfloat16* gate;    // [tokens, ldg] or null
+  long long ldg;
 };
 
 ZB_DEVICE void wg_bar_sync(int wg) {
   asm volatile("bar.sync %0, 128;" ::"r"(1 + wg) : "memory");
 }
 
+// Eight output values of one row at column c: gated, and cut at vdim.
+ZB_DEVICE void store_ext8(const PrefillTcParams& p, size_t tok, int head, int c, const uint32_t* o, float inv) {
+  if (c >= p.vdim) return;
+  __nv_bfloat16* dst = p.out + (tok * p.num_q_heads + head) * p.vdim + c;
+  const __nv_bfloat16* gate = p.gate != nullptr ? p.gate + tok * p.ldg + static_cast<size_t>(head) * p.vdim + c : nullptr;
+  const bool vec = (p.vdim & 7) == 0 && (p.ldg & 7) == 0 && (reinterpret_cast<uintptr_t>(p.gate) & 15) == 0;
+  float v[8], g[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    v[i] = __uint_as_float(o[i]) * inv;
+    g[i] = 0.f;
+  }
+  if (gate != nullptr) {
+    if (vec) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(gate);
+      const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 f = zb_unpack_bf16x2(w[i]);
+        g[2 * i] = f.x;
+        g[2 * i + 1] = f.y;
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (c + i < p.vdim) g[i] = __bfloat162float(gate[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] *= __fdividef(1.f, 1.f + __expf(-g[i]));
+  }
+  if (vec) {
+    *reinterpret_cast<uint4*>(dst) = make_uint4(zb_pack_bf16x2(v[0], v[1]), zb_pack_bf16x2(v[2], v[3]), zb_pack_bf16x2(v[4], v[5]),
+                                                zb_pack_bf16x2(v[6], v[7]));
+  } else {
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (c + i < p.vdim) dst[i] = __float2bfloat16(v[i]);
+  }
+}
+
+template <bool EXT>
 __global__ void __launch_bounds__(kThreads, 1)
 zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                            const __grid_constant__ CUtensorMap tmap_v, const PrefillTcParams p) {
@@ -111,9 +165,9 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
   const int tok_base = p.q_start[seq] + row_base;
   const int rows_valid = min(kQRows, q_len - row_base);
   const int last_key = min(len, ctx + row_base + kQRows);     // exclusive
-  const int n_tiles = (last_key + kKeys - 1) / kKeys;
-  int first_tile = 0;
-  if (p.window > 0) first_tile = max(0, ctx + row_base - p.window + 1) / kKeys;
+  const int first_key = p.window > 0 ? max(0, ctx + row_base - p.window + 1) : 0;
+  const ZbTileList tiles = zb_visible_tiles(first_key, EXT ? p.keep : 0, (last_key + kKeys - 1) / kKeys, kKeys);
+  const int n_tiles = tiles.count;
 
   if (threadIdx.x == 0) {
     zb_mbar_init(q_full, 1);
@@ -152,14 +206,14 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
           zb_tma_load_2d(q_s + w * kQBytes + c * (kQRows * 128), &tmap_q, q_full, (head0 + w) * kHD + c * 64, tok_base);
       const int32_t* bt = p.block_table + static_cast<size_t>(seq) * p.max_pages;
       uint32_t stage = 0, phase = 0;
-      for (int j = first_tile; j < n_tiles; ++j) {
-        if (j - first_tile >= kStages) {
+      for (int j = 0; j < n_tiles; ++j) {
+        if (j >= kStages) {
           if (!zb_mbar_wait(&kv_empty[stage], phase ^ 1u, abort_flag)) {
             *abort_where = 1u;
             break;
           }
         }
-        int page = bt[j];
+        int page = bt[tiles.at(j)];
         if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelId, 10)) page = 0;
         zb_mbar_expect_tx(&k_full[stage], kKvBytes);
         zb_tma_load_4d(k_s + stage * kKvBytes, &tmap_k, &k_full[stage], 0, page * kKeys, 0, kvh);
@@ -191,7 +245,7 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
         zb_umma_commit(&s_full[w]);
       };
       uint32_t stage = 0, phase = 0;                 // ring position of tile j
-      if (ok && first_tile < n_tiles) {
+      if (ok && n_tiles > 0) {
         ok = zb_mbar_wait(&k_full[0], 0u, abort_flag);
         if (!ok) *abort_where = 3u;
         if (ok) {
@@ -200,8 +254,8 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
           mma_s(1, 0);
         }
       }
-      for (int j = first_tile; ok && j < n_tiles; ++j) {
-        const uint32_t jj = static_cast<uint32_t>(j - first_tile);
+      for (int j = 0; ok && j < n_tiles; ++j) {
+        const uint32_t jj = static_cast<uint32_t>(j);
         uint32_t nstage = stage + 1, nphase = phase;
         if (nstage == kStages) {
           nstage = 0;
@@ -254,10 +308,10 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
     const uint32_t t_s = tmem_base + kColS + w * kKeys + lane_off;
     const uint32_t t_p = tmem_base + kColP + w * 32 + lane_off;
     const uint32_t t_o = tmem_base + kColO + w * kHD + lane_off;
-    float m = -INFINITY, l = 0.f;
+    float m = -INFINITY, l = EXT && p.sink ? 1.f : 0.f;
     bool ok = true;
-    for (int j = first_tile; j < n_tiles; ++j) {
-      const uint32_t jj = static_cast<uint32_t>(j - first_tile);
+    for (int j = 0; j < n_tiles; ++j) {
+      const uint32_t jj = static_cast<uint32_t>(j);
       if (!zb_mbar_wait(&s_full[w], jj & 1u, abort_flag)) {
         *abort_where = 10u + w;
         ok = false;
@@ -268,64 +322,91 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       zb_tmem_ld32(t_s, reinterpret_cast<uint32_t(&)[32]>(sr[0]));
       zb_tmem_ld32(t_s + 32, reinterpret_cast<uint32_t(&)[32]>(sr[32]));
       zb_tmem_ld_wait();
-      const int key0 = j * kKeys;
+      const int key0 = tiles.at(j) * kKeys;
       // pages below the block's first row and inside every row's window need no mask (a branch per page, not a
       // predicate per score: predicated-off instructions still take issue slots, and this loop is issue-bound)
       const bool full = (key0 + kKeys - 1 <= ctx + row_base) && (key0 + kKeys <= len) &&
                         (p.window <= 0 || key0 > ctx + row_base + kQRows - 1 - p.window);
-      float mx_raw = -INFINITY;                      // maximum of the raw (unscaled) scores of this page
-      if (full) {
-#pragma unroll
-        for (int i = 0; i < 64; ++i) mx_raw = fmaxf(mx_raw, __uint_as_float(sr[i]));
-      } else {
-#pragma unroll
-        for (int i = 0; i < 64; ++i) {
-          const int kidx = key0 + i;
-          bool vis = kidx <= qpos && kidx < len;
-          if (p.window > 0) vis = vis && (kidx > qpos - p.window);
-          if (!vis) sr[i] = 0xff800000u;             // -inf
-          mx_raw = fmaxf(mx_raw, __uint_as_float(sr[i]));
-        }
-      }
-      const float mx = fmaxf(m, mx_raw * p.scale_log2);           // running maximum, in units of log2
-      const float m_use = mx == -INFINITY ? 0.f : mx;             // a row without a visible key so far
-      if (jj > 0) {
-        // the output accumulated so far is relative to the old maximum: rescale it where the maximum moved
-        const float alpha = m == -INFINITY ? 1.f : zb_ex2(m - m_use);
-        const bool moved = alpha != 1.f;
-        if (__any_sync(0xffffffffu, moved)) {
-          if (!zb_mbar_wait(&o_ready[w], (jj - 1u) & 1u, abort_flag)) {      // O += P V of the previous page is done
-            *abort_where = 12u + w;
-            ok = false;
-            break;
-          }
-          zb_tc_fence_after();
-#pragma unroll 1
-          for (int c0 = 0; c0 < kHD; c0 += 32) {
-            uint32_t o[32];
-            zb_tmem_ld32(t_o + c0, o);
-            zb_tmem_ld_wait();
-#pragma unroll
-            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
-            zb_tmem_st16(t_o + c0, o);
-            zb_tmem_st16(t_o + c0 + 16, o + 16);
-          }
-          zb_tmem_st_wait();
-        }
-        l *= alpha;
-      }
-      m = mx;
-      // p = 2^(s * scale - m): one fused multiply-add and one exponential per score
-      const float neg_m = -m_use;
       uint32_t pw[32];
       float sum0 = 0.f, sum1 = 0.f;
+      if constexpr (EXT) {
+        // c * tanh(x) = c - 2 c / (1 + e^(2x)) in units of log2
+        const float c2 = -2.f * p.cap_log2;
+        if (!full) {
 #pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        const float p0 = zb_ex2(fmaf(__uint_as_float(sr[2 * i]), p.scale_log2, neg_m));
-        const float p1 = zb_ex2(fmaf(__uint_as_float(sr[2 * i + 1]), p.scale_log2, neg_m));
-        pw[i] = zb_pack_bf16x2(p0, p1);
-        sum0 += p0;
-        sum1 += p1;
+          for (int i = 0; i < 64; ++i) {
+            const int kidx = key0 + i;
+            const bool vis = kidx <= qpos && kidx < len && (p.window <= 0 || kidx > qpos - p.window || kidx < p.keep);
+            if (!vis) sr[i] = 0x7fc00000u;           // marks a masked score
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          float pv[2];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const float s = __uint_as_float(sr[2 * i + e]);
+            const float r = zb_rcp(1.f + zb_ex2(s * p.cap_in));
+            pv[e] = zb_ex2(fmaf(c2, r, p.cap_log2));
+            if (!full && sr[2 * i + e] == 0x7fc00000u) pv[e] = 0.f;
+          }
+          pw[i] = zb_pack_bf16x2(pv[0], pv[1]);
+          sum0 += pv[0];
+          sum1 += pv[1];
+        }
+      } else {
+        float mx_raw = -INFINITY;                      // maximum of the raw (unscaled) scores of this page
+        if (full) {
+#pragma unroll
+          for (int i = 0; i < 64; ++i) mx_raw = fmaxf(mx_raw, __uint_as_float(sr[i]));
+        } else {
+#pragma unroll
+          for (int i = 0; i < 64; ++i) {
+            const int kidx = key0 + i;
+            bool vis = kidx <= qpos && kidx < len;
+            if (p.window > 0) vis = vis && (kidx > qpos - p.window);
+            if (!vis) sr[i] = 0xff800000u;             // -inf
+            mx_raw = fmaxf(mx_raw, __uint_as_float(sr[i]));
+          }
+        }
+        const float mx = fmaxf(m, mx_raw * p.scale_log2);           // running maximum, in units of log2
+        const float m_use = mx == -INFINITY ? 0.f : mx;             // a row without a visible key so far
+        if (jj > 0) {
+          // the output accumulated so far is relative to the old maximum: rescale it where the maximum moved
+          const float alpha = m == -INFINITY ? 1.f : zb_ex2(m - m_use);
+          const bool moved = alpha != 1.f;
+          if (__any_sync(0xffffffffu, moved)) {
+            if (!zb_mbar_wait(&o_ready[w], (jj - 1u) & 1u, abort_flag)) {      // O += P V of the previous page is done
+              *abort_where = 12u + w;
+              ok = false;
+              break;
+            }
+            zb_tc_fence_after();
+#pragma unroll 1
+            for (int c0 = 0; c0 < kHD; c0 += 32) {
+              uint32_t o[32];
+              zb_tmem_ld32(t_o + c0, o);
+              zb_tmem_ld_wait();
+#pragma unroll
+              for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
+              zb_tmem_st16(t_o + c0, o);
+              zb_tmem_st16(t_o + c0 + 16, o + 16);
+            }
+            zb_tmem_st_wait();
+          }
+          l *= alpha;
+        }
+        m = mx;
+        // p = 2^(s * scale - m): one fused multiply-add and one exponential per score
+        const float neg_m = -m_use;
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          const float p0 = zb_ex2(fmaf(__uint_as_float(sr[2 * i]), p.scale_log2, neg_m));
+          const float p1 = zb_ex2(fmaf(__uint_as_float(sr[2 * i + 1]), p.scale_log2, neg_m));
+          pw[i] = zb_pack_bf16x2(p0, p1);
+          sum0 += p0;
+          sum1 += p1;
+        }
       }
       l += sum0 + sum1;
       zb_tmem_st16(t_p, pw);
@@ -334,8 +415,8 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       zb_tc_fence_before();
       zb_mbar_arrive(&p_full[w]);
     }
-    if (ok && first_tile < n_tiles) {
-      const uint32_t last = static_cast<uint32_t>(n_tiles - 1 - first_tile);
+    if (ok && n_tiles > 0) {
+      const uint32_t last = static_cast<uint32_t>(n_tiles - 1);
       if (zb_mbar_wait(&o_ready[w], last & 1u, abort_flag)) {
         zb_tc_fence_after();
         const float inv = l > 0.f ? 1.f / l : 0.f;
@@ -346,6 +427,11 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
           zb_tmem_ld32(t_o + c0, o);
           zb_tmem_ld_wait();
           if (r < rows_valid) {
+            if constexpr (EXT) {
+#pragma unroll
+              for (int i = 0; i < 4; ++i) store_ext8(p, tok_base + r, head0 + w, c0 + 8 * i, o + 8 * i, inv);
+              continue;
+            }
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
               uint32_t wd[4];
@@ -359,7 +445,7 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       } else {
         *abort_where = 14u + w;
       }
-    } else if (ok && r < rows_valid) {
+    } else if (!EXT && ok && r < rows_valid) {
       // no key at all (cannot happen for a causal prefill, kept for completeness): zeros
       __nv_bfloat16* orow = p.out + (static_cast<size_t>(tok_base + r) * p.num_q_heads + head0 + w) * kHD;
       for (int c = 0; c < kHD; c += 8) *reinterpret_cast<uint4*>(orow + c) = make_uint4(0u, 0u, 0u, 0u);
@@ -395,24 +481,24 @@ int zb_paged_prefill_tc_supported(int num_q_heads, int num_kv_heads, int head_di
   return ((num_q_heads / num_kv_heads) % 2) == 0 ? 1 : 0;
 }
 
+// 1 when the kernel takes a call with ZbAttnExt: it needs a cap whose exponential fp32 holds.
+int zb_paged_prefill_tc_ext_supported(float cap) { return cap > 0.f && cap <= kMaxCap ? 1 : 0; }
+
 // Same contract as zb_paged_prefill.  total_q_blocks128 >= sum over sequences of ceil(q_len / 128).
 // `v_lbo` / `v_sbo` = 0 select the defaults of the V descriptor (8192 / 1024 bytes).
 int zb_paged_prefill_tc(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* block_table,
                         const int32_t* seq_lens, const int32_t* q_start, int batch, int total_q_blocks128, int total_tokens,
                         int num_q_heads, int num_kv_heads, int max_pages, long long q_stride, float scale, int window,
-                        unsigned v_lbo, unsigned v_sbo, void* stream) {
+                        unsigned v_lbo, unsigned v_sbo, const ZbAttnExt* ext, void* stream) {
   if (batch <= 0 || total_q_blocks128 <= 0) return 0;
   if (!zb_paged_prefill_tc_supported(num_q_heads, num_kv_heads, kHD, kKeys)) return -32;
   ZbDeviceState* st = zb_device_state();
   if (!st) return -20;
-  static bool configured[16] = {};
-  int dev = 0;
-  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 16) return -21;
-  if (!configured[dev]) {
-    cudaError_t e = zb_config_smem(zb_paged_prefill_tc_kernel, kSmemBytes);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    configured[dev] = true;
-  }
+  if (ext != nullptr && !zb_paged_prefill_tc_ext_supported(ext->cap)) return -34;
+  static bool configured[2][16] = {};
+  if (const int rc = ext != nullptr ? zb_config_smem_once(zb_paged_prefill_tc_kernel<true>, kSmemBytes, configured[1])
+                                    : zb_config_smem_once(zb_paged_prefill_tc_kernel<false>, kSmemBytes, configured[0]))
+    return rc;
   CUtensorMap tq, tk, tv;
   // q as a [tokens, heads * 128] matrix with leading dimension q_stride: boxes of 128 rows x 64 columns
   int rc = zb_make_tmap_bf16_2d(&tq, q, total_tokens, num_q_heads * kHD, static_cast<int>(q_stride), kQRows);
@@ -436,7 +522,17 @@ int zb_paged_prefill_tc(const void* q, const void* k_cache, const void* v_cache,
   p.v_lbo = v_lbo ? v_lbo : 8192u;
   p.v_sbo = v_sbo ? v_sbo : 1024u;
   p.status = st->status;
-  const cudaError_t le = zb_launch(zb_paged_prefill_tc_kernel, dim3(total_q_blocks128, num_q_heads / 2), dim3(kThreads), kSmemBytes,
+  if (ext != nullptr) {
+    p.keep = ext->keep;
+    p.cap_log2 = ext->cap * 1.4426950408889634f;
+    p.cap_in = 2.f * scale * 1.4426950408889634f / ext->cap;
+    p.sink = ext->sink;
+    p.vdim = ext->vdim;
+    p.gate = reinterpret_cast<const __nv_bfloat16*>(ext->gate);
+    p.ldg = ext->ldg;
+  }
+  const cudaError_t le = zb_launch(ext != nullptr ? zb_paged_prefill_tc_kernel<true> : zb_paged_prefill_tc_kernel<false>,
+                                   dim3(total_q_blocks128, num_q_heads / 2), dim3(kThreads), kSmemBytes,
                                    reinterpret_cast<cudaStream_t>(stream), tq, tk, tv, p);
   zb_count_launch(1);
   return static_cast<int>(le != cudaSuccess ? le : cudaGetLastError());

@@ -1,0 +1,692 @@
+// Gated delta rule with one decay per key channel, over a varlen batch with the per-head state in registers.  Per head, with
+// decay g, unit keys k and queries q, write gate beta:
+//
+//   S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q;   out = o / rms(o) * norm * sigmoid(gate)
+//
+// q, k and v come from a projection through a short causal convolution and silu; everything behind that is fp32.
+//
+//   zb_delta_prep_kernel    portions: convolutions, unit norms and decays of blocks of eight tokens, and what lets the scan
+//                           work on a block at once.  With P_t the product of the decays of the block's tokens up to t and
+//                           R_t the product of those behind t, the block's updates are, on the state S in front of it,
+//                             a_t = S^T (P_t k_t),  b_t = S^T (P_t q_t)
+//                             u_t = beta_t (v_t - a_t - sum_{j<t} L_tj u_j),  o_t = b_t + sum_{j<=t} Q_tj u_j
+//                             S <- diag(P_7) S + sum_t (R_t k_t) u_t^T
+//                           with L_tj = k_t^T diag(decays of j+1..t) k_j and Q_tj the same with q_t.  All factors are products
+//                           of decays, none a quotient, so nothing overflows however fast a channel forgets
+//   zb_delta_scan_kernel    walks the blocks of a (sequence, head): a warp owns eight columns of S (value channels), bulk
+//                           copies bring the blocks in through a ring of stages
+//   zb_delta_finish_kernel  norm and gate, and the convolution inputs that later tokens need
+//   zb_delta_step_kernel    one token per sequence: everything above in one launch, the whole state of the head requested
+//                           before anything else
+//
+// State pools: S as [slots, H, value, key padded to 4] fp32; the convolution's inputs as a ring [slots, taps, channels] in
+// which position p has row p % taps (a step reads the taps - 1 rows of earlier positions and writes the remaining one, so
+// heads that share key channels do not disturb each other).
+#include "act.cuh"
+#include "host_api.h"
+
+namespace {
+constexpr uint32_t kKernelDelta = 36;
+constexpr int kB = 8;                       // tokens per block
+constexpr int kMaxTaps = 8;                 // at most kB: only a sequence's first block reaches back into the ring
+constexpr int kColsPerCta = 32;
+constexpr int kScanWarps = 4;               // eight columns each
+constexpr int kScanStages = 3;
+
+struct DeltaArgs {
+  const void* in;            // [T, ld_in]: q (G dk) | k (G dk) | v (H dv) at 0, write-gate logits (H) at beta_off
+  long long ld_in;
+  int beta_off;
+  const float* low;          // [T, ld_low]: decay pre-activation (H dk) | output-gate logits (H dv)
+  long long ld_low;
+  const float* conv_w;       // [taps, 2 G dk + H dv], the last tap on the current token
+  int taps;
+  const float* a_log;        // [H]
+  const float* dt_bias;      // [H dk]
+  const float* norm;         // [dv]
+  float eps;
+  void* ring;                // [slots, taps, 2 G dk + H dv]
+  float* state;              // [slots, H, dv, dk4]
+  const int32_t* slots;
+  float* blocks;             // scratch of the portion path: see BlockLayout
+  float* o;                  // scratch [T, H dv]
+  void* out;                 // [T, ld_out]
+  long long ld_out;
+  int H, G, dk, dv, dk4;
+};
+
+// One (block of tokens, head) as the scan reads it, in floats: key-side part, then the values in groups of kColsPerCta
+// columns, [group][token][column].
+struct BlockLayout {
+  int DK, groups;            // padded key channels, groups of value columns
+  __host__ __device__ int pk() const { return 0; }                       // P_t k_t   [8][DK]
+  __host__ __device__ int pq() const { return kB * DK; }                 // P_t q_t   [8][DK]
+  __host__ __device__ int rk() const { return 2 * kB * DK; }             // R_t k_t   [8][DK]
+  __host__ __device__ int p7() const { return 3 * kB * DK; }             // P_7       [DK]
+  __host__ __device__ int bl() const { return p7() + DK; }               // beta_t L  [8][8]
+  __host__ __device__ int ql() const { return bl() + kB * kB; }          // Q         [8][8]
+  __host__ __device__ int beta() const { return ql() + kB * kB; }        // beta      [8]
+  __host__ __device__ int head() const { return beta() + kB; }           // floats of the key-side part
+  __host__ __device__ int vals(int group) const { return head() + group * kB * kColsPerCta; }
+  __host__ __device__ int total() const { return vals(groups); }
+};
+
+ZB_DEVICE float silu(float z) { return z / (1.f + expf(-z)); }
+ZB_DEVICE float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+// exp(-exp(a_log) softplus(z)).  Decays close to one act over many tokens, so their last bit counts: 1 + expm1 is correctly
+// rounded there, expf is not.
+ZB_DEVICE float decay_of(float a_log, float z) {
+  const float x = -expf(a_log) * (z > 20.f ? z : log1pf(expf(z)));
+  return x > -0.5f ? 1.f + expm1f(x) : expf(x);
+}
+
+// ------------------------------------------------------------------------------------------ portions: blocks
+template <typename A, int KI>      // KI = DK / 32
+__global__ void __launch_bounds__(128) zb_delta_prep_kernel(const DeltaArgs p, const BlockLayout bl, const ZbVarlen b) {
+  constexpr int DK = KI * 32;
+  constexpr int RC = (DK + 127) / 128;
+  __shared__ float sk[kB][DK], sq[kB][DK], sg[kB][DK];
+  __shared__ float red[4][2 * kB], sbeta[kB];
+  zb_pdl_launch();
+  zb_pdl_wait();
+  const int h = blockIdx.y, g = h / (p.H / p.G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  int s, blk;
+  if (!zb_find_block(b, kB, blockIdx.x, s, blk)) return;
+  const int t0 = b.q_start[s], n = b.q_start[s + 1] - t0, i0 = blk * kB, cn = min(kB, n - i0);
+  const int pos0 = b.seq_lens[s] - n;
+  const int slot = p.slots[s];
+  if (!ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelDelta, 1)) return;
+  const int C = 2 * p.G * p.dk + p.H * p.dv;
+  const A* in = reinterpret_cast<const A*>(p.in) + t0 * p.ld_in;
+  const A* ring = reinterpret_cast<const A*>(p.ring) + static_cast<long long>(slot) * p.taps * C;
+  float* blob = p.blocks + (static_cast<long long>(blockIdx.x) * p.H + h) * bl.total();
+
+  // convolution and silu of one channel for the block's tokens (zero past the last one)
+  auto conv = [&](int col, float (&y)[kB]) {
+    float x[kMaxTaps - 1 + kB], w[kMaxTaps];               // w[d]: the tap on the input d tokens back
+#pragma unroll
+    for (int d = 0; d < kMaxTaps; ++d) w[d] = d < p.taps ? p.conv_w[static_cast<long long>(p.taps - 1 - d) * C + col] : 0.f;
+#pragma unroll
+    for (int e = 0; e < kMaxTaps - 1 + kB; ++e) {
+      const int i = i0 + e - (kMaxTaps - 1);
+      x[e] = 0.f;
+      if (e < kMaxTaps - 1 && kMaxTaps - 1 - e >= p.taps) continue;      // further back than the taps reach
+      if (i >= n) continue;
+      if (i >= 0) x[e] = zb_ld_act(in + i * p.ld_in + col);
+      else if (pos0 + i >= 0) x[e] = zb_ld_act(ring + static_cast<long long>((pos0 + i) % p.taps) * C + col);
+    }
+#pragma unroll
+    for (int t = 0; t < kB; ++t) {
+      float acc = 0.f;
+#pragma unroll
+      for (int d = 0; d < kMaxTaps; ++d) acc = fmaf(w[d], x[kMaxTaps - 1 + t - d], acc);
+      y[t] = t < cn ? silu(acc) : 0.f;
+    }
+  };
+
+  if (tid < kB) sbeta[tid] = tid < cn ? sigmoid(zb_ld_act(in + (i0 + tid) * p.ld_in + p.beta_off + h)) : 0.f;
+  float q[RC][kB], k[RC][kB], ss[2 * kB];
+#pragma unroll
+  for (int j = 0; j < 2 * kB; ++j) ss[j] = 0.f;
+#pragma unroll
+  for (int r = 0; r < RC; ++r) {
+    const int c = tid + 128 * r;
+#pragma unroll
+    for (int t = 0; t < kB; ++t) q[r][t] = k[r][t] = 0.f;
+    if (c < p.dk) {
+      conv(g * p.dk + c, q[r]);
+      conv((p.G + g) * p.dk + c, k[r]);
+    }
+#pragma unroll
+    for (int t = 0; t < kB; ++t) {
+      ss[t] = fmaf(q[r][t], q[r][t], ss[t]);
+      ss[kB + t] = fmaf(k[r][t], k[r][t], ss[kB + t]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 2 * kB; ++j) {
+    ss[j] = zb_warp_sum(ss[j]);
+    if (lane == 0) red[warp][j] = ss[j];
+  }
+  __syncthreads();
+  const float q_scale = 1.f / sqrtf(static_cast<float>(p.dk));
+#pragma unroll
+  for (int j = 0; j < 2 * kB; ++j) {
+    const float tot = red[0][j] + red[1][j] + red[2][j] + red[3][j];
+    ss[j] = (j < kB ? q_scale : 1.f) / sqrtf(tot + 1e-6f);
+  }
+  const float a_log = p.a_log[h];
+#pragma unroll
+  for (int r = 0; r < RC; ++r) {
+    const int c = tid + 128 * r;
+    if (c >= DK) continue;
+    float dec[kB];
+    const float bias = c < p.dk ? p.dt_bias[h * p.dk + c] : 0.f;
+#pragma unroll
+    for (int t = 0; t < kB; ++t) {
+      q[r][t] *= ss[t];
+      k[r][t] *= ss[kB + t];
+      dec[t] = 1.f;                                       // a token past the end leaves the state as it is
+      if (t < cn && c < p.dk) dec[t] = decay_of(a_log, p.low[(t0 + i0 + t) * p.ld_low + h * p.dk + c] + bias);
+      sq[t][c] = q[r][t];
+      sk[t][c] = k[r][t];
+      sg[t][c] = dec[t];
+    }
+    float prod = 1.f;
+#pragma unroll
+    for (int t = 0; t < kB; ++t) {
+      prod *= dec[t];
+      blob[bl.pk() + t * DK + c] = prod * k[r][t];
+      blob[bl.pq() + t * DK + c] = prod * q[r][t];
+    }
+    blob[bl.p7() + c] = prod;
+    prod = 1.f;
+#pragma unroll
+    for (int t = kB - 1; t >= 0; --t) {
+      blob[bl.rk() + t * DK + c] = prod * k[r][t];
+      prod *= dec[t];
+    }
+  }
+  for (int c = tid; c < bl.groups * kColsPerCta; c += 128) {
+    float v[kB];
+#pragma unroll
+    for (int t = 0; t < kB; ++t) v[t] = 0.f;
+    if (c < p.dv) conv(2 * p.G * p.dk + h * p.dv + c, v);
+    float* dst = blob + bl.vals(c / kColsPerCta) + c % kColsPerCta;
+#pragma unroll
+    for (int t = 0; t < kB; ++t) dst[t * kColsPerCta] = v[t];
+  }
+  __syncthreads();
+  // L and Q, a warp per column j (two of them, so that all warps have nine pairs)
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int j = half == 0 ? warp : kB - 1 - warp;
+    float kp[KI];
+#pragma unroll
+    for (int i = 0; i < KI; ++i) kp[i] = sk[j][lane + 32 * i];
+    for (int t = 0; t < kB; ++t) {
+      float l = 0.f, qq = 0.f;
+      if (t >= j) {
+#pragma unroll
+        for (int i = 0; i < KI; ++i) {
+          const int c = lane + 32 * i;
+          if (t > j) kp[i] *= sg[t][c];
+          l = fmaf(kp[i], sk[t][c], l);
+          qq = fmaf(kp[i], sq[t][c], qq);
+        }
+        l = zb_warp_sum(l);
+        qq = zb_warp_sum(qq);
+      }
+      if (lane == 0) {
+        blob[bl.bl() + t * kB + j] = t > j ? sbeta[t] * l : 0.f;
+        blob[bl.ql() + t * kB + j] = t >= j ? qq : 0.f;
+      }
+    }
+  }
+  if (tid < kB) blob[bl.beta() + tid] = sbeta[tid];
+}
+
+// ------------------------------------------------------------------------------------------ portions: scan
+using F2 = unsigned long long;              // two packed fp32
+ZB_DEVICE F2 fma2(F2 a, F2 b, F2 c) {
+  F2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+ZB_DEVICE F2 mul2(F2 a, F2 b) {
+  F2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+ZB_DEVICE F2 pack2(float a, float b) {
+  F2 d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(a), "f"(b));
+  return d;
+}
+ZB_DEVICE float sum2(F2 a) {
+  float x, y;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a));
+  return x + y;
+}
+
+// Sums N values over the G lanes of a group; lane kl of the group ends up with values kl * N / G .. in v[0 .. N / G - 1].
+template <int N, int G>
+ZB_DEVICE void reduce_scatter(float (&v)[N], int kl) {
+  int n = N;
+#pragma unroll
+  for (int m = G / 2; m > 0; m >>= 1) {
+    n >>= 1;
+    const bool up = kl & m;
+#pragma unroll
+    for (int i = 0; i < N / 2; ++i) {
+      if (i >= n) break;
+      const float give = up ? v[i] : v[i + n], keep = up ? v[i + n] : v[i];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, m);
+    }
+  }
+}
+
+// G lanes share a column, each with KT key channels (float4 number i at channel (i G + lane) 4); C columns per lane, TB
+// tokens summed over the lanes at a time.
+template <int G, int KT, int C, int TB>
+__global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(const DeltaArgs p, const BlockLayout bl, const ZbVarlen b,
+                                                                              ZbStatus* status) {
+  constexpr int DK = G * KT;
+  constexpr int CW = 32 / G * C;
+  static_assert(CW == 8 && CW * kScanWarps == kColsPerCta && kB % TB == 0, "");
+  extern __shared__ __align__(128) float delta_smem[];
+  __shared__ uint64_t full_bar[kScanStages], empty_bar[kScanStages];
+  __shared__ uint32_t abort_word;
+  __shared__ __align__(16) float sa[kScanWarps][kB][8], sb[kScanWarps][kB][8], su[kScanWarps][kB][8];
+  volatile uint32_t* abort_flag = &abort_word;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.x, s = blockIdx.y, group = blockIdx.z;
+  const int stage_floats = bl.head() + kB * kColsPerCta;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < kScanStages; ++i) {
+      zb_mbar_init(&full_bar[i], 1);
+      zb_mbar_init(&empty_bar[i], kScanWarps);
+    }
+    abort_word = 0u;
+    zb_mbar_fence_init();
+  }
+  __syncthreads();
+  zb_pdl_launch();
+  zb_pdl_wait();
+  const int t0 = b.q_start[s], n = b.q_start[s + 1] - t0;
+  const int slot = p.slots[s];
+  if (n <= 0 || !ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelDelta, 2)) return;          // uniform over the block
+  int first = 0;
+  for (int i = 0; i < s; ++i) first += (b.q_start[i + 1] - b.q_start[i] + kB - 1) / kB;
+  const int nblk = (n + kB - 1) / kB;
+  if (warp == kScanWarps) {
+    if (lane == 0) {
+      uint32_t stage = 0, phase = 0;
+      const uint32_t head_bytes = bl.head() * 4, val_bytes = kB * kColsPerCta * 4;
+      for (int i = 0; i < nblk; ++i) {
+        if (!zb_mbar_wait(&empty_bar[stage], phase ^ 1u, abort_flag)) break;
+        const float* src = p.blocks + (static_cast<long long>(first + i) * p.H + h) * bl.total();
+        float* dst = delta_smem + stage * stage_floats;
+        zb_mbar_expect_tx(&full_bar[stage], head_bytes + val_bytes);
+        zb_bulk_load(dst, src, head_bytes, &full_bar[stage]);
+        zb_bulk_load(dst + bl.head(), src + bl.vals(group), val_bytes, &full_bar[stage]);
+        if (++stage == kScanStages) {
+          stage = 0;
+          phase ^= 1u;
+        }
+      }
+    }
+  } else {
+    const int kl = lane % G, grp = lane / G, c8 = lane & 7, r = lane >> 3;
+    const int col_w = group * kColsPerCta + warp * CW;              // the warp's first column
+    const bool fresh = b.seq_lens[s] - n <= 0;
+    float* st = p.state + ((static_cast<long long>(slot) * p.H + h) * p.dv + col_w + grp * C) * p.dk4;
+    F2 S[C][KT / 2];
+#pragma unroll
+    for (int c = 0; c < C; ++c)
+#pragma unroll
+      for (int i = 0; i < KT / 4; ++i) {
+        const int key = (i * G + kl) * 4;
+        float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (!fresh && key < p.dk4 && col_w + grp * C + c < p.dv) f = *reinterpret_cast<const float4*>(st + c * p.dk4 + key);
+        S[c][2 * i] = pack2(f.x, f.y);
+        S[c][2 * i + 1] = pack2(f.z, f.w);
+      }
+    uint32_t stage = 0, phase = 0;
+    for (int blk = 0; blk < nblk; ++blk) {
+      if (!__all_sync(0xffffffffu, zb_mbar_wait(&full_bar[stage], phase, abort_flag))) break;
+      const float* d = delta_smem + stage * stage_floats;
+      auto keys = [&](const float* row, F2 (&v)[KT / 2]) {
+#pragma unroll
+        for (int i = 0; i < KT / 4; ++i) {
+          const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(row + (i * G + kl) * 4);
+          v[2 * i] = x.x;
+          v[2 * i + 1] = x.y;
+        }
+      };
+#pragma unroll
+      for (int tb = 0; tb < kB; tb += TB) {
+        float part[2 * TB * C];
+#pragma unroll
+        for (int t = 0; t < TB; ++t)
+#pragma unroll
+          for (int ab = 0; ab < 2; ++ab) {
+            F2 v[KT / 2];
+            keys(d + (ab == 0 ? bl.pk() : bl.pq()) + (tb + t) * DK, v);
+#pragma unroll
+            for (int c = 0; c < C; ++c) {
+              F2 acc = mul2(v[0], S[c][0]);
+#pragma unroll
+              for (int i = 1; i < KT / 2; ++i) acc = fma2(v[i], S[c][i], acc);
+              part[(t * 2 + ab) * C + c] = sum2(acc);
+            }
+          }
+        reduce_scatter<2 * TB * C, G>(part, kl);
+#pragma unroll
+        for (int i = 0; i < 2 * TB * C / G; ++i) {
+          const int idx = kl * (2 * TB * C / G) + i, c = idx % C, ab = idx / C % 2, t = idx / (2 * C);
+          (ab == 0 ? sa : sb)[warp][tb + t][grp * C + c] = part[i];
+        }
+      }
+      __syncwarp();
+      // every lane solves for the block's u of column c8; lanes r = 0 .. 3 of a column then take outputs r and r + 4
+      float u[kB];
+      const float* vals = d + bl.head() + warp * CW + c8;
+#pragma unroll
+      for (int t = 0; t < kB; ++t) {
+        float acc = d[bl.beta() + t] * (vals[t * kColsPerCta] - sa[warp][t][c8]);
+#pragma unroll
+        for (int j = 0; j < t; ++j) acc = fmaf(-d[bl.bl() + t * kB + j], u[j], acc);
+        u[t] = acc;
+        if ((t & 3) == r) su[warp][t][c8] = acc;
+      }
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int t = r + 4 * e;
+        float o = sb[warp][t][c8];
+#pragma unroll
+        for (int j = 0; j < kB; ++j) o = fmaf(d[bl.ql() + t * kB + j], u[j], o);
+        const int i = blk * kB + t;
+        if (i < n && col_w + c8 < p.dv) p.o[static_cast<long long>(t0 + i) * p.H * p.dv + h * p.dv + col_w + c8] = o;
+      }
+      __syncwarp();
+      F2 v[KT / 2];
+      keys(d + bl.p7(), v);
+#pragma unroll
+      for (int c = 0; c < C; ++c)
+#pragma unroll
+        for (int i = 0; i < KT / 2; ++i) S[c][i] = mul2(S[c][i], v[i]);
+#pragma unroll
+      for (int t = 0; t < kB; ++t) {
+        keys(d + bl.rk() + t * DK, v);
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          const float uc = su[warp][t][grp * C + c];
+          const F2 uu = pack2(uc, uc);
+#pragma unroll
+          for (int i = 0; i < KT / 2; ++i) S[c][i] = fma2(v[i], uu, S[c][i]);
+        }
+      }
+      __syncwarp();
+      if (lane == 0) zb_mbar_arrive(&empty_bar[stage]);
+      if (++stage == kScanStages) {
+        stage = 0;
+        phase ^= 1u;
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < C; ++c)
+#pragma unroll
+      for (int i = 0; i < KT / 4; ++i) {
+        const int key = (i * G + kl) * 4;
+        if (key < p.dk4 && col_w + grp * C + c < p.dv)
+          *reinterpret_cast<ulonglong2*>(st + c * p.dk4 + key) = make_ulonglong2(S[c][2 * i], S[c][2 * i + 1]);
+      }
+  }
+  __syncthreads();
+  if (*abort_flag != 0u) {
+    if (threadIdx.x == 0) zb_record_error(status, ZB_ERR_MBAR_TIMEOUT, kKernelDelta, 2u, blockIdx.x);
+    const uint64_t w0 = zb_globaltimer();            // copies still in flight must land before the shared memory is reused
+    while (zb_globaltimer() - w0 < 200000ull) {
+    }
+    __syncthreads();
+  }
+}
+
+// out = o / rms(o) * norm * sigmoid(gate), one warp per (token, head); the last tokens of a sequence leave their convolution
+// inputs in the ring.
+template <typename A>
+__global__ void __launch_bounds__(256) zb_delta_finish_kernel(const DeltaArgs p, const ZbVarlen b, long long rows) {
+  zb_pdl_launch();
+  zb_pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const long long row = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  if (row >= rows) return;
+  const int t = static_cast<int>(row / p.H), h = static_cast<int>(row % p.H);
+  const float* o = p.o + row * p.dv;
+  const float* gate = p.low + t * p.ld_low + p.H * p.dk + h * p.dv;
+  A* out = reinterpret_cast<A*>(p.out) + t * p.ld_out + h * p.dv;
+  float ss = 0.f;
+  for (int c = lane; c < p.dv; c += 32) ss = fmaf(o[c], o[c], ss);
+  const float inv = 1.f / sqrtf(zb_warp_sum(ss) / static_cast<float>(p.dv) + p.eps);
+  for (int c = lane; c < p.dv; c += 32) zb_st_act(out + c, o[c] * inv * p.norm[c] * sigmoid(gate[c]));
+  int s = 0;
+  while (s + 1 < b.num_seqs && b.q_start[s + 1] <= t) ++s;
+  const int n = b.q_start[s + 1] - b.q_start[s], left = b.q_start[s + 1] - t;      // left: tokens from here to the portion's end
+  if (left > p.taps || left <= 0) return;
+  const int slot = p.slots[s], pos = b.seq_lens[s] - left;
+  if (!ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelDelta, 3) || n <= 0) return;
+  const int C = 2 * p.G * p.dk + p.H * p.dv, rep = p.H / p.G, g = h / rep;
+  const A* in = reinterpret_cast<const A*>(p.in) + t * p.ld_in;
+  A* ring = reinterpret_cast<A*>(p.ring) + (static_cast<long long>(slot) * p.taps + pos % p.taps) * C;
+  for (int c = lane; c < p.dv; c += 32) ring[2 * p.G * p.dk + h * p.dv + c] = in[2 * p.G * p.dk + h * p.dv + c];
+  if (h % rep == 0)
+    for (int c = lane; c < p.dk; c += 32) {
+      ring[g * p.dk + c] = in[g * p.dk + c];
+      ring[(p.G + g) * p.dk + c] = in[(p.G + g) * p.dk + c];
+    }
+}
+
+// ------------------------------------------------------------------------------------------ one token
+// SG lanes share a column, KT key channels each; the columns of a head in passes of NT / SG.
+template <typename A, int KT, int SG>
+__global__ void __launch_bounds__(512) zb_delta_step_kernel(const DeltaArgs p, const ZbVarlen b) {
+  constexpr int DP = KT * SG;
+  __shared__ __align__(16) float s_gk[DP], s_gq[DP], s_k[DP], s_g[DP];
+  extern __shared__ float step_smem[];                       // [dv] values, then outputs
+  __shared__ float red[4][16];
+  zb_pdl_launch();
+  const int h = blockIdx.x, s = blockIdx.y, tid = threadIdx.x, NT = blockDim.x, warps = NT / 32;
+  const int kg = tid % SG, rep = p.H / p.G, g = h / rep;
+  const int C = 2 * p.G * p.dk + p.H * p.dv;
+  const float a_log = p.a_log[h];
+  zb_pdl_wait();
+  const int t = b.q_start[s];
+  if (b.q_start[s + 1] <= t) return;
+  const int slot = p.slots[s];
+  if (!ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelDelta, 4)) return;
+  const int pos = max(0, b.seq_lens[s] - 1);
+  float* st0 = p.state + (static_cast<long long>(slot) * p.H + h) * p.dv * p.dk4;
+  F2 S[KT / 2];
+  auto load = [&](int col) {
+#pragma unroll
+    for (int i = 0; i < KT / 4; ++i) {
+      const int key = (i * SG + kg) * 4;
+      ulonglong2 f = make_ulonglong2(0ull, 0ull);
+      if (pos > 0 && key < p.dk4 && col < p.dv) f = *reinterpret_cast<const ulonglong2*>(st0 + static_cast<long long>(col) * p.dk4 + key);
+      S[2 * i] = f.x;
+      S[2 * i + 1] = f.y;
+    }
+  };
+  load(tid / SG);
+  const A* in = reinterpret_cast<const A*>(p.in) + t * p.ld_in;
+  A* ring = reinterpret_cast<A*>(p.ring) + static_cast<long long>(slot) * p.taps * C;
+  auto conv = [&](int col, bool keep) {
+    float acc = 0.f;
+    const A cur = in[col];
+#pragma unroll
+    for (int d = 0; d < kMaxTaps; ++d) {
+      if (d >= p.taps) break;
+      float x = 0.f;
+      if (d == 0) x = zb_ld_act(&cur);
+      else if (pos - d >= 0) x = zb_ld_act(ring + static_cast<long long>((pos - d) % p.taps) * C + col);
+      acc = fmaf(p.conv_w[static_cast<long long>(p.taps - 1 - d) * C + col], x, acc);
+    }
+    if (keep) ring[static_cast<long long>(pos % p.taps) * C + col] = cur;
+    return silu(acc);
+  };
+  float qq = 0.f, kk = 0.f, qk = 0.f;
+  for (int c = tid; c < DP; c += NT) {
+    float q = 0.f, k = 0.f, dec = 1.f;
+    if (c < p.dk) {
+      q = conv(g * p.dk + c, h % rep == 0);
+      k = conv((p.G + g) * p.dk + c, h % rep == 0);
+      dec = decay_of(a_log, p.low[t * p.ld_low + h * p.dk + c] + p.dt_bias[h * p.dk + c]);
+    }
+    qq = fmaf(q, q, qq);
+    kk = fmaf(k, k, kk);
+    qk = fmaf(q, k, qk);
+    s_gq[c] = q;
+    s_k[c] = k;
+    s_g[c] = dec;
+  }
+  float* sy = step_smem;
+  for (int c = tid; c < p.dv; c += NT) sy[c] = conv(2 * p.G * p.dk + h * p.dv + c, true);
+  const float beta = sigmoid(zb_ld_act(in + p.beta_off + h));
+  qq = zb_warp_sum(qq);
+  kk = zb_warp_sum(kk);
+  qk = zb_warp_sum(qk);
+  if ((tid & 31) == 0) {
+    red[0][tid >> 5] = qq;
+    red[1][tid >> 5] = kk;
+    red[2][tid >> 5] = qk;
+  }
+  __syncthreads();
+  qq = kk = qk = 0.f;
+  for (int i = 0; i < warps; ++i) {
+    qq += red[0][i];
+    kk += red[1][i];
+    qk += red[2][i];
+  }
+  const float qi = 1.f / (sqrtf(qq + 1e-6f) * sqrtf(static_cast<float>(p.dk))), ki = 1.f / sqrtf(kk + 1e-6f);
+  qk *= qi * ki;
+  for (int c = tid; c < DP; c += NT) {
+    const float k = s_k[c] * ki, dec = s_g[c];
+    s_k[c] = k;
+    s_gk[c] = dec * k;
+    s_gq[c] *= dec * qi;
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c0 = 0; c0 < p.dv; c0 += NT / SG) {
+    const int col = c0 + tid / SG;
+    if (c0 > 0) load(col);
+    const float v = col < p.dv ? sy[col] : 0.f;
+    F2 a2 = 0ull, b2 = 0ull;
+#pragma unroll
+    for (int i = 0; i < KT / 4; ++i) {
+      const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(s_gk + (i * SG + kg) * 4), y = *reinterpret_cast<const ulonglong2*>(s_gq + (i * SG + kg) * 4);
+      a2 = fma2(S[2 * i], x.x, a2);
+      b2 = fma2(S[2 * i], y.x, b2);
+      a2 = fma2(S[2 * i + 1], x.y, a2);
+      b2 = fma2(S[2 * i + 1], y.y, b2);
+    }
+    float a = sum2(a2), o = sum2(b2);
+#pragma unroll
+    for (int m = 1; m < SG; m <<= 1) {
+      a += __shfl_xor_sync(0xffffffffu, a, m);
+      o += __shfl_xor_sync(0xffffffffu, o, m);
+    }
+    const float u = beta * (v - a);
+    o = fmaf(qk, u, o);
+    const F2 uu = pack2(u, u);
+    if (col < p.dv) {
+#pragma unroll
+      for (int i = 0; i < KT / 4; ++i) {
+        const int key = (i * SG + kg) * 4;
+        const ulonglong2 gg = *reinterpret_cast<const ulonglong2*>(s_g + key), k = *reinterpret_cast<const ulonglong2*>(s_k + key);
+        S[2 * i] = fma2(S[2 * i], gg.x, mul2(k.x, uu));
+        S[2 * i + 1] = fma2(S[2 * i + 1], gg.y, mul2(k.y, uu));
+        if (key < p.dk4) *reinterpret_cast<ulonglong2*>(st0 + static_cast<long long>(col) * p.dk4 + key) = make_ulonglong2(S[2 * i], S[2 * i + 1]);
+      }
+      if (kg == 0) {
+        sy[col] = o;                                         // this thread and its SG - 1 neighbours alone have read it
+        ss = fmaf(o, o, ss);
+      }
+    }
+  }
+  ss = zb_warp_sum(ss);
+  if ((tid & 31) == 0) red[3][tid >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+  for (int i = 0; i < warps; ++i) ss += red[3][i];
+  const float inv = 1.f / sqrtf(ss / static_cast<float>(p.dv) + p.eps);
+  const float* gate = p.low + t * p.ld_low + p.H * p.dk + h * p.dv;
+  A* out = reinterpret_cast<A*>(p.out) + t * p.ld_out + h * p.dv;
+  for (int c = tid; c < p.dv; c += NT) zb_st_act(out + c, sy[c] * inv * p.norm[c] * sigmoid(gate[c]));
+}
+
+// ------------------------------------------------------------------------------------------ launches
+template <typename A, int KI>
+cudaError_t launch_prep(const DeltaArgs& p, const BlockLayout& bl, const ZbVarlen& b, int num_blocks, cudaStream_t s) {
+  return zb_launch(zb_delta_prep_kernel<A, KI>, dim3(num_blocks, p.H), dim3(128), 0, s, p, bl, b);
+}
+template <typename A>
+cudaError_t launch_prep(const DeltaArgs& p, const BlockLayout& bl, const ZbVarlen& b, int num_blocks, cudaStream_t s) {
+  if (bl.DK == 32) return launch_prep<A, 1>(p, bl, b, num_blocks, s);
+  if (bl.DK == 64) return launch_prep<A, 2>(p, bl, b, num_blocks, s);
+  if (bl.DK == 128) return launch_prep<A, 4>(p, bl, b, num_blocks, s);
+  return launch_prep<A, 8>(p, bl, b, num_blocks, s);
+}
+template <int G, int KT, int C, int TB>
+int launch_scan(const DeltaArgs& p, const BlockLayout& bl, const ZbVarlen& b, ZbStatus* status, cudaStream_t s) {
+  const int smem = kScanStages * (bl.head() + kB * kColsPerCta) * 4;
+  static bool configured[16] = {};
+  if (const int rc = zb_config_smem_once(zb_delta_scan_kernel<G, KT, C, TB>, smem, configured)) return rc;
+  const cudaError_t e = zb_launch(zb_delta_scan_kernel<G, KT, C, TB>, dim3(p.H, b.num_seqs, bl.groups), dim3(32 * (kScanWarps + 1)), smem, s, p, bl, b, status);
+  return static_cast<int>(e);
+}
+int launch_scan(const DeltaArgs& p, const BlockLayout& bl, const ZbVarlen& b, ZbStatus* status, cudaStream_t s) {
+  if (bl.DK == 32) return launch_scan<8, 4, 2, 8>(p, bl, b, status, s);
+  if (bl.DK == 64) return launch_scan<16, 4, 4, 8>(p, bl, b, status, s);
+  if (bl.DK == 128) return launch_scan<16, 8, 4, 8>(p, bl, b, status, s);
+  return launch_scan<32, 8, 8, 4>(p, bl, b, status, s);
+}
+template <typename A, int KT, int SG>
+cudaError_t launch_step(const DeltaArgs& p, const ZbVarlen& b, cudaStream_t s) {
+  int threads = (p.dv * SG + 31) / 32 * 32;
+  if (threads > 512) threads = 512;
+  return zb_launch(zb_delta_step_kernel<A, KT, SG>, dim3(p.H, b.num_seqs), dim3(threads), p.dv * sizeof(float), s, p, b);
+}
+template <typename A>
+cudaError_t launch_step(const DeltaArgs& p, const ZbVarlen& b, cudaStream_t s) {
+  if (p.dk <= 32) return launch_step<A, 8, 4>(p, b, s);
+  if (p.dk <= 64) return launch_step<A, 16, 4>(p, b, s);
+  if (p.dk <= 128) return launch_step<A, 32, 4>(p, b, s);
+  return launch_step<A, 32, 8>(p, b, s);
+}
+BlockLayout layout_of(int dk, int dv) {
+  return BlockLayout{dk <= 32 ? 32 : dk <= 64 ? 64 : dk <= 128 ? 128 : 256, (dv + kColsPerCta - 1) / kColsPerCta};
+}
+}  // namespace
+
+extern "C" {
+
+// Floats of the portion path's block scratch per (block of eight tokens, head).
+int zb_channel_delta_block_floats(int dk, int dv) { return layout_of(dk, dv).total(); }
+
+// The mixer behind its input projections over a varlen batch; see the top of the file.  `blocks` null: one token per
+// sequence; else scratch for num_blocks >= sum of ceil(tokens / 8) blocks x H heads, and `o` scratch [tokens, H dv].
+// dk <= 256, dv <= 4096, taps <= 8.
+int zb_channel_delta(const void* in, long long ld_in, int beta_off, const float* low, long long ld_low, const float* conv_w, int taps,
+                     const float* a_log, const float* dt_bias, const float* norm, float eps, void* ring, float* state, const int32_t* slots,
+                     float* blocks, float* o, void* out, long long ld_out, int H, int G, int dk, int dv, int act_f32, const int32_t* q_start,
+                     const int32_t* seq_lens, int num_seqs, int tokens, int num_blocks, void* stream) {
+  if (num_seqs <= 0 || tokens <= 0) return 0;
+  if (G <= 0 || H % G != 0 || taps < 1 || taps > kMaxTaps) return -71;
+  if (dk > 256 || dv > 4096) return -72;
+  const DeltaArgs p = {in, ld_in, beta_off, low, ld_low, conv_w, taps, a_log, dt_bias, norm, eps, ring, state, slots, blocks, o, out, ld_out,
+                       H, G, dk, dv, (dk + 3) / 4 * 4};
+  const ZbVarlen b = {q_start, seq_lens, num_seqs};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (blocks == nullptr) {
+    if (tokens > num_seqs) return -73;
+    const cudaError_t e = act_f32 ? launch_step<float>(p, b, s) : launch_step<__nv_bfloat16>(p, b, s);
+    zb_count_launch(1);
+    return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+  }
+  ZbDeviceState* st = zb_device_state();
+  if (!st) return -20;
+  const BlockLayout bl = layout_of(dk, dv);
+  cudaError_t e = act_f32 ? launch_prep<float>(p, bl, b, num_blocks, s) : launch_prep<__nv_bfloat16>(p, bl, b, num_blocks, s);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  if (const int rc = launch_scan(p, bl, b, st->status, s)) return rc;
+  const long long rows = static_cast<long long>(tokens) * H;
+  const dim3 grid(static_cast<unsigned>((rows + 7) / 8));
+  e = act_f32 ? zb_launch(zb_delta_finish_kernel<float>, grid, dim3(256), 0, s, p, b, rows)
+              : zb_launch(zb_delta_finish_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, p, b, rows);
+  zb_count_launch(3);
+  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+}
+
+}  // extern "C"

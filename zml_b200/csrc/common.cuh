@@ -500,6 +500,12 @@ ZB_DEVICE float zb_ex2(float x) {
   return y;
 }
 
+ZB_DEVICE float zb_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 ZB_DEVICE float zb_warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -98,6 +98,16 @@ struct ZbBandPipe {
   const __nv_bfloat16* residual;   // local [tokens, d] or null
 };
 
+// What a paged attention call may add to causal attention within a window (attention.cu, attention_tc.cu).
+struct ZbAttnExt {
+  int keep;                    // keys 0 .. keep - 1 stay visible beyond the window
+  float cap;                   // score -> cap * tanh(score / cap); 0: none
+  int sink;                    // 1: the softmax denominator has an additional exp(0)
+  int vdim;                    // value columns of a head that are written (heads are stored padded to the kernel's size)
+  const void* gate;            // bf16 [tokens, ldg]: the output times sigmoid(gate), or null
+  long long ldg;
+};
+
 ZbDeviceState* zb_device_state();       // state of the current device, or nullptr before zb_init
 void zb_count_launch(int n);            // adds to the process-wide kernel-launch counter
 

@@ -1,10 +1,13 @@
 // Layer glue of decoders that keep the residual stream in fp32:
 //
-//   zb_embedding_f32   gathers table rows (bf16 or fp32) into the fp32 stream
+//   zb_embedding_f32   gathers table rows (bf16 or fp32), times a constant, into the fp32 stream
 //   zb_post_norm       x <- layernorm(alpha * x + y) * w, the normalisation behind a sublayer;
 //                      without y a plain layer norm.  For decode steps the same launch continues with the input
 //                      convolution of the next layer (one token per sequence: everything it needs is in the row and
 //                      in the sequence's state)
+//   zb_sandwich_norm   x <- x + m * rmsnorm(y) * w, the residual sum of a sublayer with a norm behind it, and in the same
+//                      launch rmsnorm(x) * w_next, what the next sublayer reads.  y is a row, or the weighted sum of a
+//                      token's expert rows
 //   zb_stream_conv     that input convolution over a varlen batch: h = x + conv(x), causal and per channel, and for
 //                      token-shift mixers the interpolations h + (h_prev - h) * mu of h with the previous token's h
 //
@@ -22,7 +25,7 @@ constexpr int kMaxTaps = 8;
 
 template <typename W>
 __global__ void __launch_bounds__(256) zb_embedding_f32_kernel(const int32_t* __restrict__ ids, const W* __restrict__ table,
-                                                               float* __restrict__ out, int d, int vocab) {
+                                                               float* __restrict__ out, int d, int vocab, float scale) {
   zb_pdl_launch();
   zb_pdl_wait();
   const int t = blockIdx.x;
@@ -33,7 +36,7 @@ __global__ void __launch_bounds__(256) zb_embedding_f32_kernel(const int32_t* __
   }
   const W* src = table + static_cast<size_t>(id) * d;
   float* dst = out + static_cast<size_t>(t) * d;
-  for (int i = threadIdx.x; i < d; i += 256) dst[i] = zb_ld_act(src + i);
+  for (int i = threadIdx.x; i < d; i += 256) dst[i] = scale * zb_ld_act(src + i);
 }
 
 // ------------------------------------------------------------------------------------------ convolution
@@ -455,6 +458,140 @@ __global__ void __launch_bounds__(512) zb_post_norm_conv_kernel(const PostNormAr
   }
 }
 
+// ------------------------------------------------------------------------------------------ sandwich norm
+struct SandwichArgs {
+  const void* y;               // sublayer output [T, ldy], or expert rows [*, ldy] with pair_pos, or null: no residual sum
+  long long ldy;
+  const int32_t* pair_pos;     // [T, k]: row of y of every (token, chosen expert) pair, negative: held by another rank
+  const float* pair_w;         // [T, k]
+  int k;
+  const float* x;              // [T, d]
+  float mult;
+  const float* w;              // [d]: norm behind the sublayer
+  const float* w_next;         // [d] or null: no second norm
+  float eps;
+  float* x_out;                // [T, d] or null (may be x)
+  void* act;                   // [T, ld_act]: columns d .. ld_act are zero
+  long long ld_act;
+  int d;
+};
+
+// Four values of a row at column c.
+ZB_DEVICE void ld_row4(float (&v)[4], const float* p) { ld_vec<4>(v, p); }
+ZB_DEVICE void ld_row4(float (&v)[4], const __nv_bfloat16* p) {
+  const uint2 g = *reinterpret_cast<const uint2*>(p);
+  const float2 lo = zb_unpack_bf16x2(g.x), hi = zb_unpack_bf16x2(g.y);
+  v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+}
+
+// Y: type of y, A: type of act.  NT threads, NG groups of V neighbouring channels per thread.
+template <typename Y, typename A, int NT, int NG, int V>
+__global__ void __launch_bounds__(NT) zb_sandwich_norm_kernel(const SandwichArgs p) {
+  constexpr int kSlots = 32;                             // expert slots read through shared memory at a time
+  __shared__ float red[2][NT / 32];
+  __shared__ float sw[kSlots];
+  __shared__ int spos[kSlots];
+  zb_pdl_launch();
+  const int d = p.d;
+  float w[NG][V], wn[NG][V];                             // parameters: on their way before the input is there
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + NT * i) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) w[i][e] = wn[i][e] = 0.f;
+    if (c < d && p.y != nullptr) ld_vec<V>(w[i], p.w + c);
+    if (c < d && p.w_next != nullptr) ld_vec<V>(wn[i], p.w_next + c);
+  }
+  zb_pdl_wait();
+  const long long t = blockIdx.x;
+  float x[NG][V], y[NG][V];
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + NT * i) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[i][e] = y[i][e] = 0.f;
+    if (c < d) ld_vec<V>(x[i], p.x + t * d + c);
+  }
+  if (p.y != nullptr) {
+    const Y* ys = reinterpret_cast<const Y*>(p.y);
+    auto add = [&](long long row, float wt) {
+#pragma unroll
+      for (int i = 0; i < NG; ++i) {
+        const int c = (threadIdx.x + NT * i) * V;
+        if (c >= d) continue;
+        float v[V];
+        if constexpr (V == 4) ld_row4(v, ys + row * p.ldy + c);
+        else v[0] = zb_ld_act(ys + row * p.ldy + c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[i][e] = fmaf(wt, v[e], y[i][e]);
+      }
+    };
+    if (p.pair_pos == nullptr) {
+      add(t, 1.f);
+    } else {
+      for (int j0 = 0; j0 < p.k; j0 += kSlots) {
+        const int n = min(kSlots, p.k - j0);
+        __syncthreads();
+        if (threadIdx.x < n) {
+          spos[threadIdx.x] = p.pair_pos[t * p.k + j0 + threadIdx.x];
+          sw[threadIdx.x] = p.pair_w[t * p.k + j0 + threadIdx.x];
+        }
+        __syncthreads();
+#pragma unroll 4
+        for (int j = 0; j < n; ++j)
+          if (spos[j] >= 0) add(spos[j], sw[j]);
+      }
+    }
+    float sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < NG; ++i)
+#pragma unroll
+      for (int e = 0; e < V; ++e) sq = fmaf(y[i][e], y[i][e], sq);
+    const float inv = p.mult / sqrtf(block_sum_warps<NT / 32>(sq, red[0]) / static_cast<float>(d) + p.eps);
+#pragma unroll
+    for (int i = 0; i < NG; ++i) {
+      const int c = (threadIdx.x + NT * i) * V;
+      if (c >= d) continue;
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[i][e] = fmaf(inv * y[i][e], w[i][e], x[i][e]);
+      if (p.x_out != nullptr) st_vec<float, V>(p.x_out + t * d + c, x[i]);
+    }
+  }
+  if (p.act == nullptr) return;
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < NG; ++i)
+#pragma unroll
+    for (int e = 0; e < V; ++e) sq = fmaf(x[i][e], x[i][e], sq);
+  const float inv = 1.f / sqrtf(block_sum_warps<NT / 32>(sq, red[1]) / static_cast<float>(d) + p.eps);
+  A* act = reinterpret_cast<A*>(p.act) + t * p.ld_act;
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + NT * i) * V;
+    if (c >= p.ld_act) continue;
+    float v[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = inv * x[i][e] * wn[i][e];       // columns past d: zero
+    st_vec<A, V>(act + c, v);
+  }
+}
+
+template <typename Y, typename A, int V>
+cudaError_t launch_sandwich(const SandwichArgs& p, int tokens, cudaStream_t s) {
+  const long long groups = ((p.act != nullptr && p.ld_act > p.d ? p.ld_act : p.d) + V - 1) / V;
+  if (groups <= 128) return zb_launch(zb_sandwich_norm_kernel<Y, A, 128, 1, V>, dim3(tokens), dim3(128), 0, s, p);
+  if (groups <= 512) return zb_launch(zb_sandwich_norm_kernel<Y, A, 512, 1, V>, dim3(tokens), dim3(512), 0, s, p);
+  if (groups <= 1024) return zb_launch(zb_sandwich_norm_kernel<Y, A, 512, 2, V>, dim3(tokens), dim3(512), 0, s, p);
+  if (groups <= 4096) return zb_launch(zb_sandwich_norm_kernel<Y, A, 512, 8, V>, dim3(tokens), dim3(512), 0, s, p);
+  return cudaErrorInvalidValue;
+}
+template <typename Y>
+cudaError_t launch_sandwich(const SandwichArgs& p, int act_f32, int tokens, cudaStream_t s) {
+  const bool vec = p.d % 4 == 0 && p.ld_act % 4 == 0 && p.ldy % 4 == 0 && (reinterpret_cast<uintptr_t>(p.y) & 15) == 0;
+  if (act_f32) return vec ? launch_sandwich<Y, float, 4>(p, tokens, s) : launch_sandwich<Y, float, 1>(p, tokens, s);
+  return vec ? launch_sandwich<Y, __nv_bfloat16, 4>(p, tokens, s) : launch_sandwich<Y, __nv_bfloat16, 1>(p, tokens, s);
+}
+
 template <typename A, int NG, bool MIX>
 cudaError_t launch_post_norm_conv(const PostNormArgs& p, const ConvArgs& a, const ZbVarlen& b, int tokens, cudaStream_t s) {
   if (a.taps <= 4) return zb_launch(zb_post_norm_conv_kernel<A, NG, 4, MIX>, dim3(tokens), dim3(512), 0, s, p, a, b);
@@ -492,13 +629,14 @@ bool conv_ok(int taps, int rows, int nmix) {
 
 extern "C" {
 
-int zb_embedding_f32(const int32_t* ids, const void* table, int table_f32, float* out, int tokens, int d, int vocab, void* stream) {
+int zb_embedding_f32(const int32_t* ids, const void* table, int table_f32, float* out, int tokens, int d, int vocab, float scale,
+                     void* stream) {
   if (tokens <= 0) return 0;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const cudaError_t e =
-      table_f32 ? zb_launch(zb_embedding_f32_kernel<float>, dim3(tokens), dim3(256), 0, s, ids, reinterpret_cast<const float*>(table), out, d, vocab)
+      table_f32 ? zb_launch(zb_embedding_f32_kernel<float>, dim3(tokens), dim3(256), 0, s, ids, reinterpret_cast<const float*>(table), out, d, vocab, scale)
                 : zb_launch(zb_embedding_f32_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, s, ids,
-                            reinterpret_cast<const __nv_bfloat16*>(table), out, d, vocab);
+                            reinterpret_cast<const __nv_bfloat16*>(table), out, d, vocab, scale);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }
@@ -540,6 +678,21 @@ int zb_post_norm(const void* y, long long ldy, int y_f32, const float* x, float 
   }
   if (act_f32) return vec ? launch_post_norm<float, true>(p, a, b, tokens, s) : launch_post_norm<float, false>(p, a, b, tokens, s);
   return vec ? launch_post_norm<__nv_bfloat16, true>(p, a, b, tokens, s) : launch_post_norm<__nv_bfloat16, false>(p, a, b, tokens, s);
+}
+
+// x_out = x + mult * rmsnorm(y) * w; act = rmsnorm(x_out) * w_next.  y null: act alone, of x.  pair_pos null: y [tokens, ldy];
+// else y's rows are expert outputs and a token's value is sum_j pair_w[t, j] * y[pair_pos[t, j]].  d <= 4096 channels when
+// it is not a multiple of 4, else 16384.
+int zb_sandwich_norm(const void* y, long long ldy, int y_f32, const int32_t* pair_pos, const float* pair_w, int k, const float* x, float mult,
+                     const float* w, const float* w_next, float eps, float* x_out, void* act, long long ld_act, int act_f32, int tokens,
+                     int d, void* stream) {
+  if (tokens <= 0) return 0;
+  if (act != nullptr && (w_next == nullptr || ld_act < d)) return -70;
+  const SandwichArgs p = {y, ldy, pair_pos, pair_w, k, x, mult, w, w_next, eps, x_out, act, ld_act, d};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const cudaError_t e = y_f32 ? launch_sandwich<float>(p, act_f32, tokens, s) : launch_sandwich<__nv_bfloat16>(p, act_f32, tokens, s);
+  zb_count_launch(1);
+  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }
 
 }  // extern "C"

@@ -16,13 +16,15 @@ from .llama import PRESETS as LLAMA_PRESETS, LlamaConfig, LlamaModel
 def _families():
     """(presets, config class, model class) of every model family, imported lazily."""
     from .dopurax import PRESETS as P_DOP, DopuraxConfig, DopuraxModel
+    from .kirisun import PRESETS as P_KIR, KirisunConfig, KirisunModel
     from .lfm2 import PRESETS as P_LFM2, Lfm2Config, Lfm2Model
     from .qwen3_5 import PRESETS as P_Q35, Qwen35Config, Qwen35Model
     from .qwen3_5_moe import PRESETS as P_Q35M, Qwen35MoeConfig, Qwen35MoeModel
     from .qwen3_moe import PRESETS as P_MOE, Qwen3MoeConfig, Qwen3MoeModel
     return [(LLAMA_PRESETS, LlamaConfig, LlamaModel), (P_MOE, Qwen3MoeConfig, Qwen3MoeModel),
             (P_Q35, Qwen35Config, Qwen35Model), (P_Q35M, Qwen35MoeConfig, Qwen35MoeModel),
-            (P_LFM2, Lfm2Config, Lfm2Model), (P_DOP, DopuraxConfig, DopuraxModel)]
+            (P_LFM2, Lfm2Config, Lfm2Model), (P_DOP, DopuraxConfig, DopuraxModel),
+            (P_KIR, KirisunConfig, KirisunModel)]
 
 
 def preset_names() -> list[str]:
@@ -71,4 +73,7 @@ def model_class_for(config: dict):
     if kind == "dopurax":
         from .dopurax import DopuraxConfig, DopuraxModel
         return DopuraxConfig, DopuraxModel
+    if kind == "kirisun":
+        from .kirisun import KirisunConfig, KirisunModel
+        return KirisunConfig, KirisunModel
     raise ValueError(kind)

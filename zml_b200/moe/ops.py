@@ -19,6 +19,8 @@ _lib.register_signature("zb_moe_finalize", C.c_int, [C.c_void_p, C.c_void_p, C.c
 _lib.register_signature("zb_moe_grouped_gemm", C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int,
                                                           C.c_int, C.c_int, C.c_int, C.c_int, C.c_int, C.c_void_p],
                         optional=False)
+_lib.register_signature("zb_moe_grouped_f32", C.c_int, [C.c_void_p, C.c_longlong, C.c_void_p, C.c_int, C.c_void_p, C.c_void_p, C.c_longlong,
+                                                         C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_int, C.c_int, C.c_void_p])
 
 
 class Backend(enum.Enum):
@@ -171,11 +173,24 @@ def grouped_gemm(xs: torch.Tensor, w: torch.Tensor, meta: torch.Tensor, swiglu=F
             else:
                 out[a:b] = (x @ w[e].float().t()).to(xs.dtype)
         return out
+    if xs.dtype == torch.float32:
+        return _grouped_f32(xs, None, 1, w, meta, cap, cap, code)
     assert xs.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and xs.is_contiguous() and w.is_contiguous()
     out = torch.empty((cap, n_out), dtype=xs.dtype, device=xs.device)
     _lib.check(_lib.lib().zb_moe_grouped_gemm(xs.data_ptr(), w.data_ptr(), out.data_ptr(), meta.data_ptr(), e_local, n, k,
                                               cap, n_out, code, int(avg_tokens), _lib.stream_ptr()),
                "zb_moe_grouped_gemm")
+    return out
+
+
+def _grouped_f32(x, pair, per: int, w, meta, cap: int, max_rows: int, code: int):
+    """The fp32 grouped GEMM (libzb_cuda.so: moe_f32.cu); with `pair` the rows are gathered by its loads."""
+    e, n, k = w.shape
+    assert x.dtype == torch.float32 and w.dtype == torch.float32 and w.is_contiguous() and x.stride(1) == 1 and x.shape[1] == k
+    out = torch.empty((cap, n // 2 if 1 <= code <= 3 else n), dtype=torch.float32, device=x.device)
+    _lib.check(_lib.lib().zb_moe_grouped_f32(x.data_ptr(), x.stride(0), pair.data_ptr() if pair is not None else None, per, w.data_ptr(),
+                                             out.data_ptr(), out.stride(0), meta.data_ptr(), e, n, k, max_rows, code, _lib.stream_ptr()),
+               "zb_moe_grouped_f32")
     return out
 
 
@@ -451,6 +466,33 @@ def fp4_activations() -> bool:
     the default) or with bf16 activations after de-quantising the weights inside the kernel (`ZB_MOE_FP4=a16`)."""
     import os
     return os.environ.get("ZB_MOE_FP4", "a4") != "a16"
+
+
+def pad_experts(gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor):
+    """Expert weights of any sizes (gate, up [E, F, D], down [E, D, F]) as the grouped GEMM takes them: zero hidden units up
+    to a multiple of 64, gate and up interleaved ([E, 2 F', D8], D8 = D up to a multiple of 8), zero output rows up to a
+    multiple of 128 ([E, D', F']).  The extra columns of the result are zero."""
+    pad = torch.nn.functional.pad
+    _, f, d = gate.shape
+    fp, d8, dp = -f % 64, -d % 8, -d % 128
+    return interleave_gate_up(pad(gate, (0, d8, 0, fp)), pad(up, (0, d8, 0, fp))), pad(down, (0, fp, 0, dp)).contiguous()
+
+
+def expert_rows(x: torch.Tensor, topk_ids: torch.Tensor, w_gate_up_il: torch.Tensor, w_down: torch.Tensor, e0: int = 0,
+                num_experts_total: Optional[int] = None, activation: str = "swiglu"):
+    """The LOCAL experts' outputs before they are summed: (rows [T * k, D'], pair_pos [T * k]), bf16 or fp32 as x is.  Pair
+    t * k + j has its row at pair_pos (-1: another rank's expert); routing weights are applied by whoever sums them."""
+    t = x.shape[0]
+    k = topk_ids.shape[1]
+    e_local = w_gate_up_il.shape[0]
+    avg = max(1, (t * k) // max(num_experts_total or e_local, 1))
+    meta, sorted_pair, pair_pos = moe_align(topk_ids, e0, e_local)
+    if x.is_cuda and x.dtype == torch.float32:
+        h = _grouped_f32(x, sorted_pair, k, w_gate_up_il, meta, t * k, t, activation_code(activation))
+        return _grouped_f32(h, None, 1, w_down, meta, t * k, t, 0), pair_pos
+    xs = gather(x, sorted_pair, meta, e_local, k, t * k)
+    h = grouped_gemm(xs, w_gate_up_il, meta, swiglu=activation, avg_tokens=avg)
+    return grouped_gemm(h, w_down, meta, swiglu=False, avg_tokens=avg), pair_pos
 
 
 def fused_experts(x: torch.Tensor, topk_ids: torch.Tensor, topk_w: torch.Tensor, w_gate_up_il: torch.Tensor,

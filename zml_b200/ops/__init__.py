@@ -359,8 +359,9 @@ def decode_plan_splits(batch: int, num_kv_heads: int, max_seq_len: int) -> int:
 
 def paged_decode(q, k_cache, v_cache, block_table, seq_lens, scale: float | None = None,
                  window: int = 0, num_splits: int | None = None, max_seq_len: int | None = None,
-                 out=None):
-    """One query token per sequence against its paged KV.  q [B, hq, hd] -> [B, hq, hd]."""
+                 out=None, ext=None):
+    """One query token per sequence against its paged KV.  q [B, hq, hd] -> [B, hq, hd].  `ext` (CUDA only, with `out`): a
+    `gqa.AttnExt`, see `ops.gqa`."""
     if not _cuda(q):
         return reference.paged_decode(q, k_cache, v_cache, block_table, seq_lens, scale, window)
     _need_bf16(q, k_cache, v_cache)
@@ -378,9 +379,14 @@ def paged_decode(q, k_cache, v_cache, block_table, seq_lens, scale: float | None
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(seq_lens), b, hq,
         hkv, hd, page, block_table.shape[1], q.stride(0),
         float(scale if scale is not None else 1.0 / math.sqrt(hd)), int(window), int(num_splits),
-        _lib.stream_ptr())
+        _ext(ext), _lib.stream_ptr())
     _lib.check(rc, "zb_paged_decode")
     return out
+
+
+def _ext(ext):
+    import ctypes as C
+    return None if ext is None else C.addressof(ext)
 
 
 # ZB_ATTN_TC=0: prefill attention always on the mma.sync kernel (the tensor-core kernel takes head_dim 128,
@@ -390,11 +396,12 @@ _ATTN_TC = _os.environ.get("ZB_ATTN_TC", "1") != "0"
 
 
 def paged_prefill(q, k_cache, v_cache, block_table, seq_lens, q_start, scale: float | None = None,
-                  window: int = 0, out=None, total_q_blocks: int | None = None, impl: str = "auto"):
+                  window: int = 0, out=None, total_q_blocks: int | None = None, impl: str = "auto", ext=None):
     """Varlen causal attention of new tokens against the paged KV (which already holds them).
 
     q [T, hq, hd]; q_start int32 [B+1] (device); seq_lens int32 [B] = keys per sequence.
-    `impl`: "auto" (the tcgen05 kernel where it applies), "tc" (require it) or "mma" (the mma.sync kernel).
+    `impl`: "auto" (the tcgen05 kernel where it applies), "tc" (require it) or "mma" (the mma.sync kernel).  `ext` (CUDA
+    only, with `out`): a `gqa.AttnExt`, see `ops.gqa`.
     """
     if not _cuda(q):
         return reference.paged_attention(q, k_cache, v_cache, block_table, seq_lens.tolist(),
@@ -411,19 +418,20 @@ def paged_prefill(q, k_cache, v_cache, block_table, seq_lens, q_start, scale: fl
     nqb = total_q_blocks if total_q_blocks is not None else t // 64 + b
     l = _lib.lib()
     tc_ok = bool(l.zb_paged_prefill_tc_supported(hq, hkv, hd, page)) and q.stride(0) % 8 == 0
+    tc_ok = tc_ok and (ext is None or bool(l.zb_paged_prefill_tc_ext_supported(ext.cap)))
     if impl == "tc" and not tc_ok:
         raise ValueError(f"the tensor-core prefill kernel does not take hq={hq} hkv={hkv} hd={hd} page={page}")
     if tc_ok and (impl == "tc" or (impl == "auto" and _ATTN_TC)):
         rc = l.zb_paged_prefill_tc(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(seq_lens), _ptr(q_start), b, nqb, t,
             hq, hkv, block_table.shape[1], q.stride(0), float(scale if scale is not None else 1.0 / math.sqrt(hd)), int(window),
-            int(_os.environ.get("ZB_ATTN_V_LBO", "0")), int(_os.environ.get("ZB_ATTN_V_SBO", "0")), _lib.stream_ptr())
+            int(_os.environ.get("ZB_ATTN_V_LBO", "0")), int(_os.environ.get("ZB_ATTN_V_SBO", "0")), _ext(ext), _lib.stream_ptr())
         _lib.check(rc, "zb_paged_prefill_tc")
         return out
     rc = _lib.lib().zb_paged_prefill(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _ptr(seq_lens),
         _ptr(q_start), b, nqb, hq, hkv, hd, page, block_table.shape[1], q.stride(0),
-        float(scale if scale is not None else 1.0 / math.sqrt(hd)), int(window), _lib.stream_ptr())
+        float(scale if scale is not None else 1.0 / math.sqrt(hd)), int(window), _ext(ext), _lib.stream_ptr())
     _lib.check(rc, "zb_paged_prefill")
     return out
 

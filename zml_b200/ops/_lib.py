@@ -85,12 +85,13 @@ _SIGS = {
     "zb_decode_plan_splits": (c_i, [c_i, c_i, c_i, c_i]),
     "zb_decode_scratch_bytes": (c_sz, [c_i, c_i, c_i, c_i]),
     "zb_paged_decode": (c_i, [c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_ll, c_f,
-                              c_i, c_i, c_p]),
+                              c_i, c_i, c_p, c_p]),
+    "zb_paged_prefill_tc_ext_supported": (c_i, [c_f]),
     "zb_paged_prefill_tc_supported": (c_i, [c_i, c_i, c_i, c_i]),
     "zb_paged_prefill_tc": (c_i, [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_ll, c_f, c_i,
-                                  C.c_uint, C.c_uint, c_p]),
+                                  C.c_uint, C.c_uint, c_p, c_p]),
     "zb_paged_prefill": (c_i, [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
-                               c_ll, c_f, c_i, c_p]),
+                               c_ll, c_f, c_i, c_p, c_p]),
 }
 
 # Symbols added by later source files; bound only if the library exports them.
@@ -158,7 +159,7 @@ KERNEL_NAMES = {1: "gemm_bf16", 2: "paged_decode", 3: "paged_prefill", 4: "gemm_
                 10: "moe_combine", 11: "allreduce_ll", 12: "allreduce_mm", 13: "paged_prefill_tc", 14: "gemm_2cta", 15: "argmax_tp",
                 20: "rope_kvwrite", 21: "embedding", 22: "decode_advance", 24: "causal_conv1d", 25: "gated_delta_scan",
                 26: "embedding_f32", 27: "stream_conv", 28: "latent_prep", 29: "latent_attend", 30: "latent_gather", 31: "wkv_scan",
-                32: "latent_prefill_tc", 33: "latent_decode"}
+                32: "latent_prefill_tc", 33: "latent_decode", 34: "gqa_prep", 35: "gqa_attend", 36: "channel_delta"}
 
 
 class BoundsError(KernelError):

@@ -1,6 +1,7 @@
 """Ops of the hybrid decoder layers: depthwise causal conv with a rolling cache, the gated
 delta rule scan, and the sigmoid output gate (libzb_cuda.so: linear_attn.cu); the WKV
-recurrence with its low-rank decay (wkv.cu).
+recurrence with its low-rank decay (wkv.cu); the delta rule with a decay per key channel, with its
+convolutions, norms and gate (channel_delta.cu).
 
 All of them run over the flattened varlen token batch the engine uses everywhere else:
 `q_start[S+1]` gives every sequence's token range in this launch, `seq_lens[S]` its length
@@ -14,6 +15,7 @@ examples/llm/models/lfm2/model.zig:441-500.
 from __future__ import annotations
 
 import ctypes as C
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -229,4 +231,116 @@ def tanh_linear(a, w_t, w_split=None):
     out = torch.empty((t, n), dtype=torch.float32, device=a.device)
     _lib.check(l.zb_tanh_linear(_ptr(a), a.stride(0), _ptr(w_t), w_t.stride(0), int(w_t.dtype == torch.float32), _ptr(out), out.stride(0), t, n,
                                 rank, _lib.stream_ptr()), "zb_tanh_linear")
+    return out
+
+
+# ---------------------------------------------------------------------------- delta rule with a decay per key channel
+_lib.register_signature("zb_channel_delta_block_floats", _i, [_i, _i])
+_lib.register_signature("zb_channel_delta", _i, [_p, _ll, _i, _p, _ll, _p, _i, _p, _p, _p, _f, _p, _p, _p, _p, _p, _p, _ll, _i, _i, _i, _i, _i, _p, _p,
+                                                 _i, _i, _i, _p])
+
+DELTA_MAX_TAPS, DELTA_MAX_KEY, DELTA_BLOCK = 8, 256, 8
+
+
+@dataclass
+class ChannelDelta:
+    """Parameters and state pools of one layer: `heads` value heads of `vdim` channels, `kv_heads` query / key heads of `dim`
+    (head h uses h // (heads / kv_heads)).  Per head, with unit keys and queries (queries also times dim^-1/2):
+    S <- g S by key channel, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, out = o / rms(o) * norm * sigmoid(gate), where
+    g = exp(-exp(a_log) softplus(z + dt_bias)).  q, k and v pass a causal convolution and silu first."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv_w: torch.Tensor                  # fp32 [taps, channels], channels = q | k | v, the last tap on the current token
+    a_log: torch.Tensor                   # fp32 [heads]
+    dt_bias: torch.Tensor                 # fp32 [heads dim]
+    norm: torch.Tensor                    # fp32 [vdim]
+    eps: float
+    ring: Optional[torch.Tensor] = None   # [slots, taps, channels]: the input of position p at row p % taps
+    state: Optional[torch.Tensor] = None  # fp32 [slots, heads, vdim, dim up to a multiple of 4]
+
+    def __post_init__(self):
+        if self.kv_heads < 1 or self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} heads do not share {self.kv_heads} query / key heads")
+        if not 1 <= self.taps <= DELTA_MAX_TAPS:
+            raise ValueError(f"the convolution takes 1 to {DELTA_MAX_TAPS} taps, not {self.taps}")
+        if self.dim > DELTA_MAX_KEY:
+            raise ValueError(f"the delta rule takes at most {DELTA_MAX_KEY} key channels, not {self.dim}")
+        assert self.conv_w.shape[1] == self.channels and self.conv_w.is_contiguous()
+
+    @property
+    def taps(self) -> int:
+        return self.conv_w.shape[0]
+
+    @property
+    def channels(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    def alloc(self, num_slots: int, dtype, device) -> None:
+        self.ring = torch.zeros((num_slots, self.taps, self.channels), dtype=dtype, device=device)
+        self.state = torch.zeros((num_slots, self.heads, self.vdim, (self.dim + 3) // 4 * 4), dtype=torch.float32, device=device)
+
+    def slot_bytes(self) -> int:
+        return sum(t[0].numel() * t.element_size() for t in (self.ring, self.state))
+
+
+def channel_delta_reference(proj, beta_col, low, m: ChannelDelta, q_start, seq_lens, slots):
+    t, H, G, dk, dv, taps = proj.shape[0], m.heads, m.kv_heads, m.dim, m.vdim, m.taps
+    ch, rep = m.channels, m.heads // m.kv_heads
+    z = low[:, :H * dk].float() + m.dt_bias
+    decay = torch.exp(-torch.exp(m.a_log)[None, :, None] * torch.nn.functional.softplus(z).reshape(t, H, dk))
+    beta = torch.sigmoid(proj[:, beta_col:beta_col + H].float())
+    gate = torch.sigmoid(low[:, H * dk:H * (dk + dv)].float()).reshape(t, H, dv)
+    out = torch.zeros((t, H, dv))
+    unit = lambda v: v / torch.sqrt((v * v).sum(-1, keepdim=True) + 1e-6)
+    qs, sl, so = q_start.tolist(), seq_lens.tolist(), slots.tolist()
+    for s in range(len(sl)):
+        a, b = qs[s], qs[s + 1]
+        if b <= a:
+            continue
+        n, p0 = b - a, sl[s] - (b - a)
+        raw = proj[a:b, :ch]
+        hist = [m.ring[so[s], p % taps].float() if p >= 0 else torch.zeros(ch) for p in range(p0 - taps + 1, p0)]
+        full = torch.cat([torch.stack(hist) if hist else torch.zeros((0, ch)), raw.float()], 0)
+        x = (full.unfold(0, taps, 1) * m.conv_w.t()[None]).sum(-1)
+        x = x * torch.sigmoid(x)
+        q = unit(x[:, :G * dk].reshape(n, G, dk)).repeat_interleave(rep, 1) * dk ** -0.5
+        k = unit(x[:, G * dk:2 * G * dk].reshape(n, G, dk)).repeat_interleave(rep, 1)
+        v = x[:, 2 * G * dk:].reshape(n, H, dv)
+        st = torch.zeros((H, dv, dk)) if p0 <= 0 else m.state[so[s], ..., :dk].clone()
+        for i in range(n):
+            st = st * decay[a + i][:, None, :]
+            u = beta[a + i][:, None] * (v[i] - torch.einsum("hvk,hk->hv", st, k[i]))
+            st = st + u[:, :, None] * k[i][:, None, :]
+            out[a + i] = torch.einsum("hvk,hk->hv", st, q[i])
+        m.state[so[s], ..., :dk] = st
+        for i in range(max(0, n - taps), n):
+            m.ring[so[s], (p0 + i) % taps] = raw[i]
+    out = out / torch.sqrt((out * out).mean(-1, keepdim=True) + m.eps) * m.norm * gate
+    return out.reshape(t, H * dv).to(proj.dtype)
+
+
+def channel_delta(proj, beta_col: int, low, m: ChannelDelta, q_start, seq_lens, slots, decode: bool = False,
+                  num_blocks: Optional[int] = None):
+    """The mixer of `ChannelDelta` behind its input projections: proj [T, *] = q | k | v columns first, the write gates' logits
+    at column `beta_col`; low fp32 [T, heads dim + heads vdim] = the decays' pre-activations and the output gates' logits.
+    `decode`: one token per sequence; else `num_blocks` (optional) is the sum of ceil(tokens / 8) over the sequences.
+    Updates the layer's ring and state at `slots`; returns [T, heads vdim]."""
+    if not proj.is_cuda:
+        return channel_delta_reference(proj, beta_col, low, m, q_start, seq_lens, slots)
+    t, n, dev = proj.shape[0], m.heads * m.vdim, proj.device
+    assert proj.stride(1) == 1 and low.stride(1) == 1 and low.dtype == torch.float32 and m.ring.dtype == proj.dtype
+    l = _lib.lib()
+    out = torch.empty((t, (n + 7) // 8 * 8), dtype=proj.dtype, device=dev)[:, :n]
+    blocks = o = None
+    nb = 0
+    if not decode:
+        nb = num_blocks if num_blocks is not None else t // DELTA_BLOCK + seq_lens.shape[0]
+        blocks = torch.empty((nb, m.heads, l.zb_channel_delta_block_floats(m.dim, m.vdim)), dtype=torch.float32, device=dev)
+        o = torch.empty((t, n), dtype=torch.float32, device=dev)
+    _lib.check(l.zb_channel_delta(
+        _ptr(proj), proj.stride(0), beta_col, _ptr(low), low.stride(0), _ptr(m.conv_w), m.taps, _ptr(m.a_log), _ptr(m.dt_bias), _ptr(m.norm),
+        float(m.eps), _ptr(m.ring), _ptr(m.state), _ptr(slots), _ptr(blocks), _ptr(o), _ptr(out), out.stride(0), m.heads, m.kv_heads, m.dim,
+        m.vdim, int(proj.dtype == torch.float32), _ptr(q_start), _ptr(seq_lens), seq_lens.shape[0], t, nb, _lib.stream_ptr()), "zb_channel_delta")
     return out

@@ -1,5 +1,5 @@
-"""Layer glue of decoders with an fp32 residual stream: embedding, the norm behind a sublayer, and the convolution in
-front of a mixer (libzb_cuda.so: stream_f32.cu).
+"""Layer glue of decoders with an fp32 residual stream: embedding, the norms behind and in front of a sublayer, and the
+convolution in front of a mixer (libzb_cuda.so: stream_f32.cu).
 
 All of it works on the flattened varlen batch of the engine (`q_start`, `seq_lens`, `slots`, as in
 `ops.linear_attn`).  Activations that a projection reads are written in the model's dtype (bf16 or fp32); the stream,
@@ -16,7 +16,8 @@ import torch
 from . import _lib
 
 _p, _i, _ll, _f = C.c_void_p, C.c_int, C.c_longlong, C.c_float
-_lib.register_signature("zb_embedding_f32", _i, [_p, _p, _i, _p, _i, _i, _i, _p])
+_lib.register_signature("zb_embedding_f32", _i, [_p, _p, _i, _p, _i, _i, _i, _f, _p])
+_lib.register_signature("zb_sandwich_norm", _i, [_p, _ll, _i, _p, _p, _i, _p, _f, _p, _p, _f, _p, _p, _ll, _i, _i, _i, _p])
 _lib.register_signature("zb_stream_conv", _i, [_p, _p, _p, _p, _p, _p, _i, _ll, _ll, _i, _i, _i, _i, _p, _p, _i, _i, _p])
 _lib.register_signature("zb_post_norm", _i, [_p, _ll, _i, _p, _f, _p, _f, _p, _p, _ll, _i, _i, _i, _p, _p, _p, _p, _p, _ll, _ll,
                                              _i, _i, _i, _p, _p])
@@ -29,14 +30,14 @@ def _ptr(t: Optional[torch.Tensor]):
     return None if t is None else t.data_ptr()
 
 
-def embedding_f32(ids, table):
-    """Rows of `table` (bf16 or fp32) as fp32 [T, d]."""
+def embedding_f32(ids, table, scale: float = 1.0):
+    """Rows of `table` (bf16 or fp32) times `scale`, as fp32 [T, d]."""
     if not table.is_cuda:
-        return table[ids.long()].float()
+        return table[ids.long()].float() * scale
     assert ids.dtype == torch.int32 and table.is_contiguous()
     out = torch.empty((ids.shape[0], table.shape[1]), dtype=torch.float32, device=table.device)
     _lib.check(_lib.lib().zb_embedding_f32(_ptr(ids), _ptr(table), int(table.dtype == torch.float32), _ptr(out), ids.shape[0],
-                                           table.shape[1], table.shape[0], _lib.stream_ptr()), "zb_embedding_f32")
+                                           table.shape[1], table.shape[0], float(scale), _lib.stream_ptr()), "zb_embedding_f32")
     return out
 
 
@@ -146,3 +147,55 @@ def post_norm(x, w, eps: float, y=None, alpha: float = 1.0, keep_x: bool = True,
         float(eps), _ptr(x_new), _ptr(act), d, int(act_dtype == torch.float32), t, d, _ptr(c.w) if c else None,
         _ptr(c.state) if c else None, _ptr(slots), _ptr(c.mu) if c else None, *cargs, _ptr(seq_lens), _lib.stream_ptr()), "zb_post_norm")
     return x_new, (out if conv is not None else act)
+
+
+# ------------------------------------------------------------------ norms on both sides of a sublayer
+def rms_norm_reference(x, w, eps):
+    return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * w
+
+
+def pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+@dataclass
+class ExpertRows:
+    """Outputs of a routed mixture before they are summed: token t's value is sum_j weights[t, j] * rows[pair_pos[t, j]]
+    over the pairs with a row here (`moe.expert_rows`).  `rows` may be wider than the stream."""
+    rows: torch.Tensor                    # [*, >= d]
+    pair_pos: torch.Tensor                # int32 [T * k]
+    weights: torch.Tensor                 # float32 [T, k]
+
+    def sum(self, d: int) -> torch.Tensor:
+        t, k = self.weights.shape
+        pos = self.pair_pos.reshape(t, k).long()
+        w = self.weights.float() * (pos >= 0)
+        return (self.rows[pos.clamp_min(0)][..., :d].float() * w[..., None]).sum(1)
+
+
+def sandwich_norm(x, y=None, w=None, mult: float = 1.0, w_next=None, eps: float = 1e-6, act_dtype=None, keep_x: bool = True):
+    """The residual sum of a sublayer with a norm behind it, and the norm in front of the next one, in one launch:
+    x_new = x + mult * rmsnorm(y) * w and act = rmsnorm(x_new) * w_next in `act_dtype` ([T, d] with zero columns up to a
+    multiple of 8).  x fp32 [T, d]; y [T, d] (bf16 or fp32) or `ExpertRows`; without y, act of x itself; without w_next,
+    no act.  Returns (x_new or None, act or None); x is overwritten on CUDA."""
+    t, d = x.shape
+    if not x.is_cuda:
+        if y is not None:
+            v = y.sum(d) if isinstance(y, ExpertRows) else y[:, :d].float()
+            x = x + mult * rms_norm_reference(v, w, eps)
+        act = None
+        if w_next is not None:
+            act = torch.nn.functional.pad(rms_norm_reference(x, w_next, eps), (0, pad8(d) - d)).to(act_dtype)
+        return (x if keep_x else None), act
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    rows, pos, pw, k = y, None, None, 0
+    if isinstance(y, ExpertRows):
+        rows, pos, pw, k = y.rows, y.pair_pos, y.weights, y.weights.shape[1]
+        assert pw.dtype == torch.float32 and pw.is_contiguous()
+    assert rows is None or (rows.stride(1) == 1 and rows.shape[1] >= d and rows.dtype in (torch.float32, torch.bfloat16) and w.dtype == torch.float32)
+    act = torch.empty((t, pad8(d)), dtype=act_dtype, device=x.device) if w_next is not None else None
+    _lib.check(_lib.lib().zb_sandwich_norm(
+        _ptr(rows), rows.stride(0) if rows is not None else 0, int(rows is not None and rows.dtype == torch.float32), _ptr(pos), _ptr(pw), k,
+        _ptr(x), float(mult), _ptr(w), _ptr(w_next), float(eps), _ptr(x) if keep_x and rows is not None else None, _ptr(act), pad8(d),
+        int(act_dtype == torch.float32), t, d, _lib.stream_ptr()), "zb_sandwich_norm")
+    return (x if keep_x else None), act
