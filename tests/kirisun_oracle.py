@@ -28,12 +28,12 @@ def turn_halves(v, pos, dims, base, factor=1.0):
 
 
 def soft_cap(s, cap):
-    return cap * np.tanh(s / cap)
+    return cap * np.tanh(s / cap) if cap else s
 
 
 def sees(i, j, window, keep):
-    """Whether position i looks at position j."""
-    return j <= i and (i - j < window or j < keep)
+    """Whether position i looks at position j (window 0: no window)."""
+    return j <= i and (window == 0 or i - j < window or j < keep)
 
 
 def sink_softmax(s):
@@ -48,10 +48,22 @@ def unit(z):
 
 
 # ------------------------------------------------------------------ mixers
+def attend(q, k, v, scale, cap, window, keep, first=0):
+    """Rows first .. of a sequence: q [n, H, dk] at positions first + row, k, v [>= first + n, G, *] of all positions."""
+    n, H, G = q.shape[0], q.shape[1], k.shape[1]
+    out = np.zeros((n, H, v.shape[-1]))
+    for r in range(n):
+        i = first + r
+        js = [j for j in range(i + 1) if sees(i, j, window, keep)]
+        for a in range(H):
+            g = a // (H // G)
+            out[r, a] = sink_softmax(soft_cap(k[js, g] @ q[r, a] * scale, cap)) @ v[js, g]
+    return out
+
+
 def attention(h, W, m, eps):
     """W: tensors of the mixer by short name; m: its sizes.  Returns [T, width]."""
     T, H, G, dk, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    window, keep = m["mask"]["size"], m["mask"]["keep_first"]
     rot = m["rot"]
     q = rms_norm((h @ W["q"].T).reshape(T, H, dk), W["q.norm"], eps)
     k = rms_norm((h @ W["k"].T).reshape(T, G, dk), W["k.norm"], eps)
@@ -59,26 +71,13 @@ def attention(h, W, m, eps):
     factor = rot["scaling"]["factor"]
     q = np.stack([turn_halves(q[t], t, rot["dims"], rot["base"], factor) for t in range(T)])
     k = np.stack([turn_halves(k[t], t, rot["dims"], rot["base"], factor) for t in range(T)])
-    out = np.zeros((T, H, dv))
-    for t in range(T):
-        js = [j for j in range(t + 1) if sees(t, j, window, keep)]
-        for a in range(H):
-            g = a // (H // G)
-            p = sink_softmax(soft_cap(k[js, g] @ q[t, a] * m["scale"], m["softcap"]))
-            out[t, a] = p @ v[js, g]
+    out = attend(q, k, v, m["scale"], m["softcap"], m["mask"]["size"], m["mask"]["keep_first"])
     return (out.reshape(T, H * dv) * sigmoid(h @ W["g"].T)) @ W["o"].T
 
 
-def channel_delta(h, W, m, eps):
-    T, H, G, dk, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    assert W["q.conv"].shape[1] == W["k.conv"].shape[1] == W["v.conv"].shape[1] == m["conv"]
-    q, k, v = (silu(causal_taps(h @ W[n].T, W[n + ".conv"])) for n in "qkv")
-    q = unit(q.reshape(T, G, dk)) * dk ** -0.5
-    k = unit(k.reshape(T, G, dk))
-    v = v.reshape(T, H, dv)
-    beta = sigmoid(h @ W["b"].T)
-    rate = softplus((h @ W["a1"].T) @ W["a2"].T + W["dt_bias"]).reshape(T, H, dk)
-    decay = np.exp(-np.exp(W["A_log"])[None, :, None] * rate)
+def delta_rule(q, k, v, beta, decay):
+    """q, k [T, G, dk], v [T, H, dv], beta [T, H], decay [T, H, dk], one token after the other from a zero state."""
+    (T, G, dk), (H, dv) = k.shape, v.shape[1:]
     S = np.zeros((H, dk, dv))
     o = np.zeros((T, H, dv))
     for t in range(T):
@@ -88,8 +87,27 @@ def channel_delta(h, W, m, eps):
             u = beta[t, a] * (v[t, a] - S[a].T @ k[t, g])
             S[a] = S[a] + np.outer(k[t, g], u)
             o[t, a] = S[a].T @ q[t, g]
-    gate = sigmoid((h @ W["g1"].T) @ W["g2"].T)
-    return ((rms(o, eps) * W["norm"]).reshape(T, H * dv) * gate) @ W["o"].T
+    return o
+
+
+def delta_core(q, k, v, convs, beta, pre, a_log, dt_bias, gate, norm, sizes, eps):
+    """Everything between the input projections and the output projection: q, k, v before their convolutions, logits of the
+    write gates [T, H] and of the output gates [T, H dv], pre-activations of the decays [T, H dk]."""
+    H, G, dk, dv = sizes
+    T = q.shape[0]
+    q, k, v = (silu(causal_taps(x, w)) for x, w in zip((q, k, v), convs))
+    q = unit(q.reshape(T, G, dk)) * dk ** -0.5
+    k = unit(k.reshape(T, G, dk))
+    rate = softplus(pre + dt_bias).reshape(T, H, dk)
+    o = delta_rule(q, k, v.reshape(T, H, dv), sigmoid(beta), np.exp(-np.exp(a_log)[None, :, None] * rate))
+    return (rms(o, eps) * norm).reshape(T, H * dv) * sigmoid(gate)
+
+
+def channel_delta(h, W, m, eps):
+    assert W["q.conv"].shape[1] == W["k.conv"].shape[1] == W["v.conv"].shape[1] == m["conv"]
+    o = delta_core(*(h @ W[n].T for n in "qkv"), [W[n + ".conv"] for n in "qkv"], h @ W["b"].T, (h @ W["a1"].T) @ W["a2"].T, W["A_log"],
+                   W["dt_bias"], (h @ W["g1"].T) @ W["g2"].T, W["norm"], (m["heads"], m["kv_heads"], m["dim"], m["vdim"]), eps)
+    return o @ W["o"].T
 
 
 MIXERS = {"attention": attention, "channel_delta": channel_delta}
