@@ -45,6 +45,9 @@ WORKLOADS = {
     "dopurax-1b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
     "dopurax-8b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
     "tiny-dopurax-test": dict(batch=4, prompt=(16, 64), new_tokens=8),
+    "kirisun-3b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
+    "kirisun-10b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
+    "tiny-kirisun-test": dict(batch=4, prompt=(16, 64), new_tokens=8),
 }
 
 
@@ -212,9 +215,22 @@ def run_workload(name: str, comm, args, steps: int, warmup: int, sample_clocks: 
 
 
 # Designs whose prefill and decode throughput `--compare` sets beside the closest other family at equal size: a hybrid of
-# gated full attention (where the design has latent attention) and gated delta net (where it has WKV) with the same width,
-# depth, vocabulary, head sizes of the recurrent layers and feed-forward parameters (three matrices of 2/3 the units).
+# gated full attention (where the design has attention) and gated delta net (where it has a recurrence) with the same width,
+# depth, vocabulary, head sizes of the recurrent layers and feed-forward parameters (Dopurax: three matrices of 2/3 the
+# units; Kirisun: the same experts, and the shared expert that the family always has at its smallest size).
 COMPARE_SHAPES = [dict(batch=1, prompt=4096), dict(batch=8, prompt=1024), dict(batch=32, prompt=1024), dict(batch=64, prompt=2048)]
+
+
+def moe_hybrid_twin(cfg) -> dict:
+    from zml_b200.models.kirisun import ATTENTION, DELTA
+    att = next(s for s in cfg.layers if s.kind == ATTENTION)
+    rec = next(s for s in cfg.layers if s.kind == DELTA)
+    return dict(hidden_size=cfg.hidden_size, num_hidden_layers=len(cfg.layers), num_attention_heads=att.heads, num_key_value_heads=att.kv_heads,
+                head_dim=att.dim, vocab_size=cfg.vocab_size, rms_norm_eps=cfg.norm_eps,
+                rope_parameters=dict(rope_theta=att.attn["base"], partial_rotary_factor=att.attn["rot"] / att.dim), linear_conv_kernel_dim=rec.taps,
+                linear_key_head_dim=rec.dim, linear_num_key_heads=rec.kv_heads, linear_value_head_dim=rec.vdim, linear_num_value_heads=rec.heads,
+                layer_types=["full_attention" if s.kind == ATTENTION else "linear_attention" for s in cfg.layers], num_experts=att.experts,
+                num_experts_per_tok=att.top, moe_intermediate_size=att.ff, shared_expert_intermediate_size=64, tie_word_embeddings=False)
 
 
 def hybrid_twin(cfg) -> dict:
@@ -235,15 +251,21 @@ def compare(name: str, args) -> None:
     import gc
 
     import torch
-    from zml_b200.models.dopurax import PRESETS, DopuraxConfig, DopuraxModel
-    from zml_b200.models.qwen3_5 import Qwen35Config, Qwen35Model
     from zml_b200.serving import Engine
     torch.cuda.set_device(0)
-    cfg = DopuraxConfig.from_hf(PRESETS[name])
-    twin = Qwen35Config.from_hf(hybrid_twin(cfg))
+    if name.startswith("kirisun"):
+        from zml_b200.models.kirisun import PRESETS, KirisunConfig as Config, KirisunModel as Model
+        from zml_b200.models.qwen3_5_moe import Qwen35MoeConfig as TwinConfig, Qwen35MoeModel as TwinModel
+        to_twin = moe_hybrid_twin
+    else:
+        from zml_b200.models.dopurax import PRESETS, DopuraxConfig as Config, DopuraxModel as Model
+        from zml_b200.models.qwen3_5 import Qwen35Config as TwinConfig, Qwen35Model as TwinModel
+        to_twin = hybrid_twin
+    cfg = Config.from_hf(PRESETS[name])
+    twin = TwinConfig.from_hf(to_twin(cfg))
     sampler = ClockSampler(True)
     new, out = args.new_tokens or 128, {}
-    for label, build in ((name, lambda: DopuraxModel(cfg, device="cuda:0")), ("hybrid of equal size", lambda: Qwen35Model(twin, device="cuda:0"))):
+    for label, build in ((name, lambda: Model(cfg, device="cuda:0")), ("hybrid of equal size", lambda: TwinModel(twin, device="cuda:0"))):
         model = build().init_random(args.seed)
         model.SERIAL_PREFILL = True                  # the same launch mode for both
         rows = []
@@ -293,7 +315,7 @@ def main() -> None:
     ap.add_argument("--headline", default="auto", choices=["auto", "none"],
                     help="auto: after the scaling configuration also measure the headline configurations that fit this "
                          "number of GPUs (Llama-3.1-70B and the NVFP4 MoE at 8, the MoE at 2 and 4), 3 timed jobs each")
-    ap.add_argument("--compare", default="", choices=["", "dopurax-1b", "dopurax-8b"],
+    ap.add_argument("--compare", default="", choices=["", "dopurax-1b", "dopurax-8b", "kirisun-3b", "kirisun-10b"],
                     help="instead of the benchmark: prefill and decode throughput of this design beside the closest other family at equal "
                          "size, at a few batch shapes (1 GPU)")
     args = ap.parse_args()

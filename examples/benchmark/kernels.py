@@ -10,6 +10,10 @@
     python examples/benchmark/kernels.py --op=latent_decode --batch=32 --seqlen=4096 --hq=32 --window=4096
     python examples/benchmark/kernels.py --op=wkv_scan --batch=8 --seqlen=512 --hq=32 --hd=128
     python examples/benchmark/kernels.py --op=stream --tokens=4096 --k=4096
+    python examples/benchmark/kernels.py --op=gqa_prefill --batch=2 --seqlen=2048 --window=4096
+    python examples/benchmark/kernels.py --op=gqa_decode --batch=32 --seqlen=1344 --window=4096
+    python examples/benchmark/kernels.py --op=channel_delta --batch=8 --seqlen=512 --hq=32 --hd=128
+    python examples/benchmark/kernels.py --op=mixture --tokens=32 --experts=32 --topk=4 --n=1024 --k=2048
     python examples/benchmark/kernels.py --op=decode_layers --model=llama-3.1-8b --batch=32 --seqlen=1344
     python examples/benchmark/kernels.py --op=gemm_chain_timeline --model=llama-3.1-8b --batch=32
     python examples/benchmark/kernels.py --op=moe_w4_timeline --tokens=128 --experts=128 --topk=8 --n=768 --k=2048
@@ -55,7 +59,7 @@ class Args:
     warmup: int = 3
     splits: int = 0          # decode_attention: KV chunks per sequence (0: the planner's choice)
     w4: int = 0              # moe: 1 = NVFP4 expert weights de-quantised inside the grouped GEMM
-    window: int = 4096       # latent attention: keys a position sees
+    window: int = 4096       # latent and gated attention: keys a position sees
     copies: int = 0          # operand copies to rotate through (0: enough to exceed the L2)
     help = __doc__
 
@@ -288,6 +292,104 @@ def bench_wkv_scan(a: Args) -> None:
     report(a, ms, t * H * D * (5 * 2 + 4) + 2 * states[0].numel() * 4, 6.0 * t * H * D * D, {"batch": a.batch, "seqlen": a.seqlen, "heads": H, "dim": D})
 
 
+def _gqa(a: Args):
+    """A capped, sunk, windowed and gated attention at the sizes of the plain paged benchmarks, with filled caches."""
+    from types import SimpleNamespace
+    from zml_b200.ops import gqa
+    s = gqa.GqaSpec(a.hq, a.hkv, a.hd, a.hd, a.hd // 2, scale=a.hd ** -0.5, cap=50.0, window=a.window, keep=16, sink=True)
+    c = n_copies(a, a.batch * a.seqlen * a.hkv * a.hd * 4) if a.op == "gqa_decode" else 2
+    caches, bt = _kv(a, c)
+    n = a.seqlen if a.op == "gqa_prefill" else 1
+    t = a.batch * n
+    qs = (torch.arange(a.batch + 1, dtype=torch.int32, device="cuda") * n).int()
+    sl = torch.full((a.batch,), a.seqlen, dtype=torch.int32, device="cuda")
+    splits = a.splits or ops.decode_plan_splits(a.batch, a.hkv, s.visible(a.seqlen))
+    meta = SimpleNamespace(is_prefill=n > 1, q_start=qs, seq_lens=sl, block_table=bt, total_q_blocks=a.batch * ((n + 63) // 64), num_splits=splits,
+                           max_seq_len=a.seqlen)
+    nq = (a.hq + 2 * a.hkv) * a.hd
+    proj = torch.randn(t, nq + a.hq * a.hd, device="cuda").bfloat16()
+    return gqa, s, caches, meta, proj, nq, t
+
+
+def bench_gqa_prefill(a: Args) -> None:
+    gqa, s, caches, meta, proj, nq, t = _gqa(a)
+    q = torch.randn(t, a.hq, a.hd, device="cuda").bfloat16()
+    ms = timed([lambda c=c: gqa.attention(q, proj[:, nq:], c, meta, s) for c in caches], a.iters, a.warmup)
+    pairs = a.seqlen * (a.seqlen + 1) / 2 if a.window >= a.seqlen else a.window * (a.seqlen - (a.window - 1) / 2)
+    shape = {"batch": a.batch, "seqlen": a.seqlen, "hq": a.hq, "hkv": a.hkv, "hd": a.hd, "window": a.window}
+    report(a, ms, (3 * t * a.hq * a.hd + 2 * t * a.hkv * a.hd) * 2, 4.0 * a.batch * a.hq * a.hd * pairs, dict(shape, part="attention"))
+    slots = (torch.arange(t, dtype=torch.int32, device="cuda") + 64).int()
+    pos = (torch.arange(t, device="cuda") % a.seqlen).int()
+    w, f = torch.ones(a.hd, device="cuda"), s.inv_freq("cuda")
+    ms = timed([lambda c=c: gqa.prep(proj, w, w, f, pos, slots, c, 1e-6, s) for c in caches], a.iters, a.warmup)
+    report(a, ms, 2 * t * nq * 2, 0, dict(shape, part="norms, rotation, cache write"))
+    pos_full, lay = pos, dict(q_norm_w=w.bfloat16(), k_norm_w=w.bfloat16())
+    ms = timed([lambda c=c: ops.rope_kvwrite(proj[:, :nq], pos_full, slots, f, c[0], c[1], a.hq, a.hkv, a.hd, 0, a.hd // 2, **lay) for c in caches], a.iters,
+               a.warmup)
+    report(a, ms, 2 * t * nq * 2, 0, dict(shape, part="the same in the other families"))
+
+
+def bench_gqa_decode(a: Args) -> None:
+    gqa, s, caches, meta, proj, nq, t = _gqa(a)
+    q = torch.randn(t, a.hq, a.hd, device="cuda").bfloat16()
+    ms = timed_graph([lambda c=c: gqa.attention(q, proj[:, nq:], c, meta, s) for c in caches], a.iters, a.warmup)
+    kvb = a.batch * min(a.seqlen, a.window + 16) * a.hkv * a.hd * 4
+    report(a, ms, kvb, 4.0 * a.batch * a.hq * min(a.seqlen, a.window) * a.hd, {"batch": a.batch, "seqlen": a.seqlen, "window": a.window, "splits": meta.num_splits})
+    sl = meta.seq_lens
+    ms = timed_graph([lambda c=c: ops.paged_decode(q, *c, meta.block_table, sl, num_splits=meta.num_splits, max_seq_len=a.seqlen) for c in caches], a.iters, a.warmup)
+    kvb = a.batch * a.seqlen * a.hkv * a.hd * 4
+    report(a, ms, kvb, 4.0 * a.batch * a.hq * a.seqlen * a.hd, {"batch": a.batch, "seqlen": a.seqlen, "part": "the plain kernel"})
+
+
+def bench_channel_delta(a: Args) -> None:
+    from zml_b200.ops import linear_attn as la
+    H, D, t = a.hq, a.hd, a.batch * a.seqlen
+    decode = a.seqlen == 1
+    qs = (torch.arange(a.batch + 1, dtype=torch.int32, device="cuda") * a.seqlen).int()
+    sl = torch.full((a.batch,), a.seqlen + decode, dtype=torch.int32, device="cuda")
+    slots = torch.arange(a.batch, dtype=torch.int32, device="cuda")
+    layers = []
+    for _ in range(n_copies(a, a.batch * H * D * D * 4) if decode else 1):
+        m = la.ChannelDelta(H, H, D, D, torch.randn(4, 3 * H * D, device="cuda"), torch.rand(H, device="cuda"), torch.rand(H * D, device="cuda") * 4 - 5,
+                            torch.ones(D, device="cuda"), 1e-6)
+        m.alloc(a.batch, torch.bfloat16, "cuda")
+        layers.append(m)
+    proj = torch.randn(t, 3 * H * D + (H + 7) // 8 * 8, device="cuda").bfloat16()
+    low = torch.randn(t, 2 * H * D, device="cuda")
+    fns = [lambda m=m: la.channel_delta(proj, m.channels, low, m, qs, sl, slots, decode, a.batch * ((a.seqlen + 7) // 8)) for m in layers]
+    ms = (timed_graph if decode else timed)(fns, a.iters, a.warmup)
+    nbytes = t * H * D * (3 * 2 + 2 * 4 + 2) + a.batch * H * D * D * 8
+    report(a, ms, nbytes, 6.0 * t * H * D * D, {"batch": a.batch, "seqlen": a.seqlen, "heads": H, "dim": D})
+
+
+def bench_mixture(a: Args) -> None:
+    """Router, experts and the norm that sums their rows; the same with the other families' mixture and norm kernels."""
+    from zml_b200.moe import ops as mops
+    from zml_b200.ops import stream
+    e, k, f, d, t = a.experts, a.topk, a.n, a.k, a.tokens
+    c = max(2, min(8, math.ceil(300e6 / (e * f * d * 6)) + 1))
+    ws = [mops.pad_experts(*(torch.randn(e, *s, device="cuda").bfloat16() * 0.02 for s in ((f, d), (f, d), (d, f)))) for _ in range(c)]
+    router, bias = torch.randn(e, d, device="cuda").bfloat16() * 0.05, torch.zeros(e, device="cuda").bfloat16()
+    h, x, res = torch.randn(t, d, device="cuda").bfloat16(), torch.randn(t, d, device="cuda"), torch.randn(t, d, device="cuda").bfloat16()
+    nw, nb = torch.ones(d, device="cuda"), torch.ones(d, device="cuda").bfloat16()
+
+    def mine(w):
+        z = ops.gemm(h, router, bias=bias, out_dtype=torch.float32, static_w=True)
+        ids, wt = mops.router_topk(z, k)
+        rows, pos = mops.expert_rows(h, ids, *w, 0, e)
+        return stream.sandwich_norm(x, stream.ExpertRows(rows, pos, wt), nw, 0.5, nw, 1e-6, act_dtype=torch.bfloat16)
+
+    def theirs(w):
+        z = ops.gemm(h, router, out_dtype=torch.float32, static_w=True)
+        ids, wt = mops.router_topk(z, k)
+        return ops.rmsnorm(mops.fused_experts(h, ids, wt, *w, 0, e, residual=res), nb)
+
+    active = min(e, t * k)
+    for part, fn in (("mixture", mine), ("other families", theirs)):
+        ms = timed_graph([lambda w=w, fn=fn: fn(w) for w in ws], a.iters, a.warmup)
+        report(a, ms, active * 3 * f * d * 2, 6.0 * t * k * f * d, {"part": part, "tokens": t, "experts": e, "top": k, "ff": f, "d": d})
+
+
 def bench_stream(a: Args) -> None:
     """The norm behind a sublayer, the input convolution (with and without interpolations) and the decode step's fusion."""
     from zml_b200.ops import stream
@@ -299,6 +401,8 @@ def bench_stream(a: Args) -> None:
     qs, sl, slots = torch.tensor([0, t], dtype=torch.int32, device="cuda"), torch.tensor([t], dtype=torch.int32, device="cuda"), torch.zeros(t, dtype=torch.int32, device="cuda")
     ms = timed_graph([lambda x=x: stream.post_norm(x, w, 1e-5, y, 2.0, act_dtype=torch.bfloat16) for x in xs], a.iters, a.warmup)
     report(a, ms, t * d * 14, 0, {"part": "post_norm", "tokens": t, "d": d})
+    ms = timed_graph([lambda x=x: stream.sandwich_norm(x, y, w, 0.5, w, 1e-5, act_dtype=torch.bfloat16) for x in xs], a.iters, a.warmup)
+    report(a, ms, t * d * 14, 0, {"part": "sandwich_norm", "tokens": t, "d": d})
     for mixes in (False, True):
         conv = stream.InputConv(torch.randn(4, d, device="cuda"), torch.zeros(1, 4 if mixes else 3, d, device="cuda"), mu if mixes else None)
         ms = timed_graph([lambda x=x: stream.stream_conv(x, conv, qs, sl, slots, torch.bfloat16) for x in xs], a.iters, a.warmup)
@@ -470,7 +574,8 @@ def bench_moe_w4_timeline(a: Args) -> None:
 
 OPS = {"moe_w4_timeline": bench_moe_w4_timeline, "gemm_chain_timeline": bench_gemm_chain_timeline, "gemm": bench_gemm, "decode_attention": bench_decode_attention, "prefill_attention": bench_prefill_attention,
        "moe": bench_moe, "gated_delta_scan": bench_gated_delta_scan, "decode_layers": bench_decode_layers,
-       "latent_prefill": bench_latent_prefill, "latent_decode": bench_latent_decode, "wkv_scan": bench_wkv_scan, "stream": bench_stream}
+       "latent_prefill": bench_latent_prefill, "latent_decode": bench_latent_decode, "wkv_scan": bench_wkv_scan, "stream": bench_stream,
+       "gqa_prefill": bench_gqa_prefill, "gqa_decode": bench_gqa_decode, "channel_delta": bench_channel_delta, "mixture": bench_mixture}
 
 
 def main(argv=None) -> int:

@@ -141,6 +141,7 @@ ATTN = {
     "tensor cores": (4, 1, 128, 128, 100, 5, 30.0, True),
     "tensor cores, narrower": (2, 1, 100, 72, 70, 64, 50.0, True),
     "tensor cores, no sink, no window": (4, 2, 128, 128, 0, 0, 20.0, False),
+    "tensor cores, low cap": (4, 2, 128, 128, 100, 3, 7.0, True),
     "64": (3, 3, 64, 64, 64, 65, 8.0, True),
     "256": (2, 2, 256, 200, 130, 1, 30.0, True),
     "no cap": (2, 1, 128, 128, 90, 4, 0.0, True),

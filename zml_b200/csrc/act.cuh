@@ -30,3 +30,46 @@ ZB_DEVICE bool zb_find_block(const ZbVarlen& b, int rows, int idx, int& seq, int
   }
   return false;
 }
+
+// The same by all 32 lanes of a warp together, 32 sequences at a time.
+ZB_DEVICE bool zb_find_block_warp(const ZbVarlen& b, int rows, int idx, int& seq, int& block) {
+  const int lane = threadIdx.x & 31;
+  for (int base = 0; base < b.num_seqs; base += 32) {
+    const int s = base + lane;
+    const int nb = s < b.num_seqs ? (b.q_start[s + 1] - b.q_start[s] + rows - 1) / rows : 0;
+    int incl = nb;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += v;
+    }
+    const unsigned hit = __ballot_sync(0xffffffffu, idx < incl);
+    if (hit != 0u) {
+      const int l = __ffs(hit) - 1;
+      seq = base + l;
+      block = idx - __shfl_sync(0xffffffffu, incl - nb, l);
+      return true;
+    }
+    idx -= __shfl_sync(0xffffffffu, incl, 31);
+  }
+  return false;
+}
+
+// Blocks in front of sequence `seq`, by a warp.
+ZB_DEVICE int zb_blocks_before(const ZbVarlen& b, int rows, int seq) {
+  int n = 0;
+  for (int s = threadIdx.x & 31; s < seq; s += 32) n += (b.q_start[s + 1] - b.q_start[s] + rows - 1) / rows;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) n += __shfl_xor_sync(0xffffffffu, n, o);
+  return n;
+}
+
+// The sequence of token t, by a warp.
+ZB_DEVICE int zb_sequence_of(const ZbVarlen& b, int t) {
+  int n = 0;
+  for (int base = 1; base < b.num_seqs; base += 32) {
+    const int s = base + (threadIdx.x & 31);
+    n += __popc(__ballot_sync(0xffffffffu, s < b.num_seqs && b.q_start[s] <= t));
+  }
+  return n;
+}

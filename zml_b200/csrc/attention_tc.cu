@@ -43,6 +43,9 @@ constexpr int kThreads = 320;
 constexpr uint32_t kKernelId = 13;
 constexpr uint32_t kTmemCols = 512;
 constexpr float kMaxCap = 60.f;                    // exp(cap) times the number of keys stays far inside fp32
+// tanh(x) / x in powers of x^2, interpolated at Chebyshev nodes on |x| <= kPolyMax (error 3e-9)
+constexpr float kPolyMax = 0.6f;
+__device__ constexpr float kTanh[6] = {1.0f, -0.333332837f, 0.1333168f, -0.0537679829f, 0.0207513496f, -0.00584964408f};
 constexpr uint32_t kColS = 0, kColP = 128, kColO = 192;
 
 struct PrefillTcParams {
@@ -63,6 +66,7 @@ struct PrefillTcParams {
   int keep;
   float cap_log2;               // cap * log2(e)
   float cap_in;                 // 2 * scale * log2(e) / cap
+  float cap_x;                  // scale / cap
   int sink;
   int vdim;                     // output [tokens, num_q_heads, vdim]
   const __nv_bfloat16* gate;    // [tokens, ldg] or null
@@ -330,30 +334,46 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       uint32_t pw[32];
       float sum0 = 0.f, sum1 = 0.f;
       if constexpr (EXT) {
-        // c * tanh(x) = c - 2 c / (1 + e^(2x)) in units of log2
-        const float c2 = -2.f * p.cap_log2;
+        // The capped score in units of log2, over sr: with x = s * scale / c, where a warp's scores are small tanh(x) / x as a
+        // polynomial in x^2, else c - 2 c / (1 + e^(2x)).
+        float mx = 0.f;
+#pragma unroll
+        for (int i = 0; i < 64; ++i) mx = fmaxf(mx, fabsf(__uint_as_float(sr[i])));
+        if (__all_sync(0xffffffffu, mx * p.cap_x <= kPolyMax)) {
+          const ZbF2 cx = zb_pack2(p.cap_x, p.cap_x), cs = zb_pack2(p.scale_log2, p.scale_log2);
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const ZbF2 s2 = zb_pack2(__uint_as_float(sr[2 * i]), __uint_as_float(sr[2 * i + 1])), x = zb_mul2(s2, cx), t = zb_mul2(x, x);
+            ZbF2 q = zb_pack2(kTanh[5], kTanh[5]);
+#pragma unroll
+            for (int k = 4; k >= 0; --k) q = zb_fma2(q, t, zb_pack2(kTanh[k], kTanh[k]));
+            float a0, a1;
+            zb_unpack2(zb_mul2(zb_mul2(s2, cs), q), a0, a1);
+            sr[2 * i] = __float_as_uint(a0);
+            sr[2 * i + 1] = __float_as_uint(a1);
+          }
+        } else {
+          const float c2 = -2.f * p.cap_log2;
+#pragma unroll
+          for (int i = 0; i < 64; ++i)
+            sr[i] = __float_as_uint(fmaf(c2, zb_rcp(1.f + zb_ex2(__uint_as_float(sr[i]) * p.cap_in)), p.cap_log2));
+        }
         if (!full) {
 #pragma unroll
           for (int i = 0; i < 64; ++i) {
             const int kidx = key0 + i;
             const bool vis = kidx <= qpos && kidx < len && (p.window <= 0 || kidx > qpos - p.window || kidx < p.keep);
-            if (!vis) sr[i] = 0x7fc00000u;           // marks a masked score
+            if (!vis) sr[i] = 0xff800000u;           // -inf
           }
         }
+        ZbF2 sum = 0ull;
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          float pv[2];
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            const float s = __uint_as_float(sr[2 * i + e]);
-            const float r = zb_rcp(1.f + zb_ex2(s * p.cap_in));
-            pv[e] = zb_ex2(fmaf(c2, r, p.cap_log2));
-            if (!full && sr[2 * i + e] == 0x7fc00000u) pv[e] = 0.f;
-          }
-          pw[i] = zb_pack_bf16x2(pv[0], pv[1]);
-          sum0 += pv[0];
-          sum1 += pv[1];
+          const float p0 = zb_ex2(__uint_as_float(sr[2 * i])), p1 = zb_ex2(__uint_as_float(sr[2 * i + 1]));
+          pw[i] = zb_pack_bf16x2(p0, p1);
+          sum = zb_add2(sum, zb_pack2(p0, p1));
         }
+        zb_unpack2(sum, sum0, sum1);
       } else {
         float mx_raw = -INFINITY;                      // maximum of the raw (unscaled) scores of this page
         if (full) {
@@ -526,6 +546,7 @@ int zb_paged_prefill_tc(const void* q, const void* k_cache, const void* v_cache,
     p.keep = ext->keep;
     p.cap_log2 = ext->cap * 1.4426950408889634f;
     p.cap_in = 2.f * scale * 1.4426950408889634f / ext->cap;
+    p.cap_x = scale / ext->cap;
     p.sink = ext->sink;
     p.vdim = ext->vdim;
     p.gate = reinterpret_cast<const __nv_bfloat16*>(ext->gate);

@@ -71,182 +71,30 @@ struct BlockLayout {
   __host__ __device__ int total() const { return vals(groups); }
 };
 
-ZB_DEVICE float silu(float z) { return z / (1.f + expf(-z)); }
-ZB_DEVICE float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
-// exp(-exp(a_log) softplus(z)).  Decays close to one act over many tokens, so their last bit counts: 1 + expm1 is correctly
-// rounded there, expf is not.
-ZB_DEVICE float decay_of(float a_log, float z) {
-  const float x = -expf(a_log) * (z > 20.f ? z : log1pf(expf(z)));
-  return x > -0.5f ? 1.f + expm1f(x) : expf(x);
+// A: the activation type.  fp32 models take CUDA's accurate functions; with bf16 inputs a few units in the last place of the
+// fast ones do not count, except where a decay close to one acts over many tokens: there the exponential and the logarithm
+// are short series (arguments below 2^-6, fourth order: 2^-26 relative).
+template <typename A>
+ZB_DEVICE float sigmoid(float z) {
+  if constexpr (sizeof(A) == 2) return __fdividef(1.f, 1.f + __expf(-z));
+  return 1.f / (1.f + expf(-z));
 }
-
-// ------------------------------------------------------------------------------------------ portions: blocks
-template <typename A, int KI>      // KI = DK / 32
-__global__ void __launch_bounds__(128) zb_delta_prep_kernel(const DeltaArgs p, const BlockLayout bl, const ZbVarlen b) {
-  constexpr int DK = KI * 32;
-  constexpr int RC = (DK + 127) / 128;
-  __shared__ float sk[kB][DK], sq[kB][DK], sg[kB][DK];
-  __shared__ float red[4][2 * kB], sbeta[kB];
-  zb_pdl_launch();
-  zb_pdl_wait();
-  const int h = blockIdx.y, g = h / (p.H / p.G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  int s, blk;
-  if (!zb_find_block(b, kB, blockIdx.x, s, blk)) return;
-  const int t0 = b.q_start[s], n = b.q_start[s + 1] - t0, i0 = blk * kB, cn = min(kB, n - i0);
-  const int pos0 = b.seq_lens[s] - n;
-  const int slot = p.slots[s];
-  if (!ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelDelta, 1)) return;
-  const int C = 2 * p.G * p.dk + p.H * p.dv;
-  const A* in = reinterpret_cast<const A*>(p.in) + t0 * p.ld_in;
-  const A* ring = reinterpret_cast<const A*>(p.ring) + static_cast<long long>(slot) * p.taps * C;
-  float* blob = p.blocks + (static_cast<long long>(blockIdx.x) * p.H + h) * bl.total();
-
-  // convolution and silu of one channel for the block's tokens (zero past the last one)
-  auto conv = [&](int col, float (&y)[kB]) {
-    float x[kMaxTaps - 1 + kB], w[kMaxTaps];               // w[d]: the tap on the input d tokens back
-#pragma unroll
-    for (int d = 0; d < kMaxTaps; ++d) w[d] = d < p.taps ? p.conv_w[static_cast<long long>(p.taps - 1 - d) * C + col] : 0.f;
-#pragma unroll
-    for (int e = 0; e < kMaxTaps - 1 + kB; ++e) {
-      const int i = i0 + e - (kMaxTaps - 1);
-      x[e] = 0.f;
-      if (e < kMaxTaps - 1 && kMaxTaps - 1 - e >= p.taps) continue;      // further back than the taps reach
-      if (i >= n) continue;
-      if (i >= 0) x[e] = zb_ld_act(in + i * p.ld_in + col);
-      else if (pos0 + i >= 0) x[e] = zb_ld_act(ring + static_cast<long long>((pos0 + i) % p.taps) * C + col);
-    }
-#pragma unroll
-    for (int t = 0; t < kB; ++t) {
-      float acc = 0.f;
-#pragma unroll
-      for (int d = 0; d < kMaxTaps; ++d) acc = fmaf(w[d], x[kMaxTaps - 1 + t - d], acc);
-      y[t] = t < cn ? silu(acc) : 0.f;
-    }
-  };
-
-  if (tid < kB) sbeta[tid] = tid < cn ? sigmoid(zb_ld_act(in + (i0 + tid) * p.ld_in + p.beta_off + h)) : 0.f;
-  float q[RC][kB], k[RC][kB], ss[2 * kB];
-#pragma unroll
-  for (int j = 0; j < 2 * kB; ++j) ss[j] = 0.f;
-#pragma unroll
-  for (int r = 0; r < RC; ++r) {
-    const int c = tid + 128 * r;
-#pragma unroll
-    for (int t = 0; t < kB; ++t) q[r][t] = k[r][t] = 0.f;
-    if (c < p.dk) {
-      conv(g * p.dk + c, q[r]);
-      conv((p.G + g) * p.dk + c, k[r]);
-    }
-#pragma unroll
-    for (int t = 0; t < kB; ++t) {
-      ss[t] = fmaf(q[r][t], q[r][t], ss[t]);
-      ss[kB + t] = fmaf(k[r][t], k[r][t], ss[kB + t]);
-    }
-  }
-#pragma unroll
-  for (int j = 0; j < 2 * kB; ++j) {
-    ss[j] = zb_warp_sum(ss[j]);
-    if (lane == 0) red[warp][j] = ss[j];
-  }
-  __syncthreads();
-  const float q_scale = 1.f / sqrtf(static_cast<float>(p.dk));
-#pragma unroll
-  for (int j = 0; j < 2 * kB; ++j) {
-    const float tot = red[0][j] + red[1][j] + red[2][j] + red[3][j];
-    ss[j] = (j < kB ? q_scale : 1.f) / sqrtf(tot + 1e-6f);
-  }
-  const float a_log = p.a_log[h];
-#pragma unroll
-  for (int r = 0; r < RC; ++r) {
-    const int c = tid + 128 * r;
-    if (c >= DK) continue;
-    float dec[kB];
-    const float bias = c < p.dk ? p.dt_bias[h * p.dk + c] : 0.f;
-#pragma unroll
-    for (int t = 0; t < kB; ++t) {
-      q[r][t] *= ss[t];
-      k[r][t] *= ss[kB + t];
-      dec[t] = 1.f;                                       // a token past the end leaves the state as it is
-      if (t < cn && c < p.dk) dec[t] = decay_of(a_log, p.low[(t0 + i0 + t) * p.ld_low + h * p.dk + c] + bias);
-      sq[t][c] = q[r][t];
-      sk[t][c] = k[r][t];
-      sg[t][c] = dec[t];
-    }
-    float prod = 1.f;
-#pragma unroll
-    for (int t = 0; t < kB; ++t) {
-      prod *= dec[t];
-      blob[bl.pk() + t * DK + c] = prod * k[r][t];
-      blob[bl.pq() + t * DK + c] = prod * q[r][t];
-    }
-    blob[bl.p7() + c] = prod;
-    prod = 1.f;
-#pragma unroll
-    for (int t = kB - 1; t >= 0; --t) {
-      blob[bl.rk() + t * DK + c] = prod * k[r][t];
-      prod *= dec[t];
-    }
-  }
-  for (int c = tid; c < bl.groups * kColsPerCta; c += 128) {
-    float v[kB];
-#pragma unroll
-    for (int t = 0; t < kB; ++t) v[t] = 0.f;
-    if (c < p.dv) conv(2 * p.G * p.dk + h * p.dv + c, v);
-    float* dst = blob + bl.vals(c / kColsPerCta) + c % kColsPerCta;
-#pragma unroll
-    for (int t = 0; t < kB; ++t) dst[t * kColsPerCta] = v[t];
-  }
-  __syncthreads();
-  // L and Q, a warp per column j (two of them, so that all warps have nine pairs)
-#pragma unroll
-  for (int half = 0; half < 2; ++half) {
-    const int j = half == 0 ? warp : kB - 1 - warp;
-    float kp[KI];
-#pragma unroll
-    for (int i = 0; i < KI; ++i) kp[i] = sk[j][lane + 32 * i];
-    for (int t = 0; t < kB; ++t) {
-      float l = 0.f, qq = 0.f;
-      if (t >= j) {
-#pragma unroll
-        for (int i = 0; i < KI; ++i) {
-          const int c = lane + 32 * i;
-          if (t > j) kp[i] *= sg[t][c];
-          l = fmaf(kp[i], sk[t][c], l);
-          qq = fmaf(kp[i], sq[t][c], qq);
-        }
-        l = zb_warp_sum(l);
-        qq = zb_warp_sum(qq);
-      }
-      if (lane == 0) {
-        blob[bl.bl() + t * kB + j] = t > j ? sbeta[t] * l : 0.f;
-        blob[bl.ql() + t * kB + j] = t >= j ? qq : 0.f;
-      }
-    }
-  }
-  if (tid < kB) blob[bl.beta() + tid] = sbeta[tid];
+template <typename A>
+ZB_DEVICE float silu(float z) {
+  if constexpr (sizeof(A) == 2) return __fdividef(z, 1.f + __expf(-z));
+  return z / (1.f + expf(-z));
 }
-
-// ------------------------------------------------------------------------------------------ portions: scan
-using F2 = unsigned long long;              // two packed fp32
-ZB_DEVICE F2 fma2(F2 a, F2 b, F2 c) {
-  F2 d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-ZB_DEVICE F2 mul2(F2 a, F2 b) {
-  F2 d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-ZB_DEVICE F2 pack2(float a, float b) {
-  F2 d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(a), "f"(b));
-  return d;
-}
-ZB_DEVICE float sum2(F2 a) {
-  float x, y;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a));
-  return x + y;
+// exp(-rate * softplus(z)), rate = exp(a_log).
+template <typename A>
+ZB_DEVICE float decay_of(float rate, float z) {
+  if constexpr (sizeof(A) == 2) {
+    const float e = __expf(z);
+    const float sp = z > 20.f ? z : e < 0.015625f ? e * (1.f + e * (-0.5f + e * (1.f / 3.f - 0.25f * e))) : __logf(1.f + e);
+    const float x = -rate * sp;
+    return x > -0.015625f ? 1.f + x * (1.f + x * (0.5f + x * (1.f / 6.f + x * (1.f / 24.f)))) : __expf(x);
+  }
+  const float x = -rate * (z > 20.f ? z : log1pf(expf(z)));
+  return x > -0.5f ? 1.f + expm1f(x) : expf(x);             // 1 + expm1 is correctly rounded near one, expf is not
 }
 
 // Sums N values over the G lanes of a group; lane kl of the group ends up with values kl * N / G .. in v[0 .. N / G - 1].
@@ -266,6 +114,146 @@ ZB_DEVICE void reduce_scatter(float (&v)[N], int kl) {
   }
 }
 
+// ------------------------------------------------------------------------------------------ portions: blocks
+// One CTA per (block of tokens, head).  The head's query, key and value channels and its decays are dealt over the threads,
+// one channel's eight tokens each; T bounds the taps, KI = DK / 32.
+template <typename A, int KI, int T>
+__global__ void __launch_bounds__(512, 2) zb_delta_prep_kernel(const DeltaArgs p, const BlockLayout bl, const ZbVarlen b) {
+  constexpr int DK = KI * 32;
+  __shared__ float sk[kB][DK], sq[kB][DK], sg[kB][DK];
+  __shared__ float sinv[2 * kB], sbeta[kB];
+  zb_pdl_launch();
+  zb_pdl_wait();
+  const int h = blockIdx.y, g = h / (p.H / p.G), tid = threadIdx.x, NT = blockDim.x, warps = NT / 32, warp = tid >> 5, lane = tid & 31;
+  int s, blk;
+  if (!zb_find_block_warp(b, kB, blockIdx.x, s, blk)) return;
+  const int t0 = b.q_start[s], n = b.q_start[s + 1] - t0, i0 = blk * kB, cn = min(kB, n - i0);
+  const int pos0 = b.seq_lens[s] - n;
+  const int slot = p.slots[s];
+  if (!ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelDelta, 1)) return;
+  const int C = 2 * p.G * p.dk + p.H * p.dv, vals = bl.groups * kColsPerCta;
+  const A* in = reinterpret_cast<const A*>(p.in) + (t0 + i0) * p.ld_in;
+  float* blob = p.blocks + (static_cast<long long>(blockIdx.x) * p.H + h) * bl.total();
+  const float rate = expf(p.a_log[h]);
+  if (tid < kB) {
+    const float beta = tid < cn ? sigmoid<A>(zb_ld_act(in + tid * p.ld_in + p.beta_off + h)) : 0.f;
+    sbeta[tid] = beta;
+    blob[bl.beta() + tid] = beta;
+  }
+  for (int item = tid; item < 3 * DK + vals; item += NT) {
+    if (item < DK) {                                         // decays; a token past the end leaves the state as it is
+      float z[kB];
+      const int c = min(item, p.dk - 1);
+#pragma unroll
+      for (int t = 0; t < kB; ++t) z[t] = p.low[(t0 + i0 + min(t, cn - 1)) * p.ld_low + h * p.dk + c];
+      const float bias = p.dt_bias[h * p.dk + c];
+#pragma unroll
+      for (int t = 0; t < kB; ++t) sg[t][item] = t < cn && item < p.dk ? decay_of<A>(rate, z[t] + bias) : 1.f;
+      continue;
+    }
+    const int part = item < 2 * DK ? 0 : item < 3 * DK ? 1 : 2;           // q, k, v
+    const int c = item - (part + 1) * DK, width = part < 2 ? p.dk : p.dv;
+    const bool live = c < width;
+    const int col = (part < 2 ? (part * p.G + g) * p.dk : 2 * p.G * p.dk + h * p.dv) + min(c, width - 1);
+    A x[T - 1 + kB];                                         // raw inputs; all requested at once
+    if (i0 > 0) {
+#pragma unroll
+      for (int e = 0; e < T - 1; ++e) x[e] = in[(e - (T - 1)) * p.ld_in + col];
+    } else {
+      const A* ring = reinterpret_cast<const A*>(p.ring) + static_cast<long long>(slot) * p.taps * C + col;
+#pragma unroll
+      for (int e = 0; e < T - 1; ++e) x[e] = ring[static_cast<long long>(max(pos0 + e - (T - 1), 0) % p.taps) * C];
+    }
+#pragma unroll
+    for (int t = 0; t < kB; ++t) x[T - 1 + t] = in[min(t, cn - 1) * p.ld_in + col];
+    float w[T], y[kB];                                       // w[d]: the tap on the input d tokens back
+#pragma unroll
+    for (int d = 0; d < T; ++d) w[d] = d < p.taps ? p.conv_w[static_cast<long long>(p.taps - 1 - d) * C + col] : 0.f;
+    float f[T - 1 + kB];
+#pragma unroll
+    for (int e = 0; e < T - 1 + kB; ++e) {
+      const int back = T - 1 - e;                            // what lies before the start, or further back than the taps, counts nothing
+      f[e] = back > 0 && (back >= p.taps || pos0 + i0 < back) ? 0.f : zb_ld_act(&x[e]);
+    }
+#pragma unroll
+    for (int t = 0; t < kB; ++t) {
+      float acc = 0.f;
+#pragma unroll
+      for (int d = 0; d < T; ++d) acc = fmaf(w[d], f[T - 1 + t - d], acc);
+      y[t] = live && t < cn ? silu<A>(acc) : 0.f;
+    }
+    if (part < 2) {
+#pragma unroll
+      for (int t = 0; t < kB; ++t) (part == 0 ? sq : sk)[t][c] = y[t];
+    } else {
+      float* dst = blob + bl.vals(c / kColsPerCta) + c % kColsPerCta;
+#pragma unroll
+      for (int t = 0; t < kB; ++t) dst[t * kColsPerCta] = y[t];
+    }
+  }
+  __syncthreads();
+  for (int j = warp; j < 2 * kB; j += warps) {               // unit norms
+    const float* v = j < kB ? sq[j] : sk[j - kB];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < KI; ++i) ss = fmaf(v[lane + 32 * i], v[lane + 32 * i], ss);
+    ss = zb_warp_sum(ss);
+    if (lane == 0) sinv[j] = (j < kB ? 1.f / sqrtf(static_cast<float>(p.dk)) : 1.f) / sqrtf(ss + 1e-6f);
+  }
+  __syncthreads();
+  for (int item = tid; item < 3 * DK; item += NT) {
+    const int part = item / DK, c = item % DK;
+    float prod = 1.f;
+    if (part < 2) {
+      const float (*v)[DK] = part == 0 ? sk : sq;
+      float* dst = blob + (part == 0 ? bl.pk() : bl.pq()) + c;
+#pragma unroll
+      for (int t = 0; t < kB; ++t) {
+        prod *= sg[t][c];
+        dst[t * DK] = prod * v[t][c] * sinv[part == 0 ? kB + t : t];
+      }
+      if (part == 0) blob[bl.p7() + c] = prod;
+    } else {
+#pragma unroll
+      for (int t = kB - 1; t >= 0; --t) {
+        blob[bl.rk() + t * DK + c] = prod * sk[t][c] * sinv[kB + t];
+        prod *= sg[t][c];
+      }
+    }
+  }
+  // L and Q: a warp per column j of one of them
+  for (int jj = warp; jj < 2 * kB; jj += warps) {
+    const int j = jj % kB;
+    const bool is_q = jj >= kB;
+    const float (*other)[DK] = is_q ? sq : sk;
+    float kp[KI], sum[kB];
+#pragma unroll
+    for (int i = 0; i < KI; ++i) kp[i] = sk[j][lane + 32 * i];
+#pragma unroll
+    for (int t = 0; t < kB; ++t) {
+      sum[t] = 0.f;
+      if (t < j) continue;
+#pragma unroll
+      for (int i = 0; i < KI; ++i) {
+        const int c = lane + 32 * i;
+        if (t > j) kp[i] *= sg[t][c];
+        sum[t] = fmaf(kp[i], other[t][c], sum[t]);
+      }
+    }
+    reduce_scatter<kB, 8>(sum, lane & 7);                    // lane l: token l % 8, over the eight lanes that share l / 8
+    float v = sum[0];
+    v += __shfl_xor_sync(0xffffffffu, v, 8);
+    v += __shfl_xor_sync(0xffffffffu, v, 16);
+    if (lane < kB) {
+      const int t = lane;
+      v *= sinv[kB + j] * sinv[is_q ? t : kB + t];
+      if (is_q) blob[bl.ql() + t * kB + j] = t >= j ? v : 0.f;
+      else blob[bl.bl() + t * kB + j] = t > j ? sbeta[t] * v : 0.f;
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------ portions: scan
 // G lanes share a column, each with KT key channels (float4 number i at channel (i G + lane) 4); C columns per lane, TB
 // tokens summed over the lanes at a time.
 template <int G, int KT, int C, int TB>
@@ -296,8 +284,7 @@ __global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(co
   const int t0 = b.q_start[s], n = b.q_start[s + 1] - t0;
   const int slot = p.slots[s];
   if (n <= 0 || !ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelDelta, 2)) return;          // uniform over the block
-  int first = 0;
-  for (int i = 0; i < s; ++i) first += (b.q_start[i + 1] - b.q_start[i] + kB - 1) / kB;
+  const int first = zb_blocks_before(b, kB, s);
   const int nblk = (n + kB - 1) / kB;
   if (warp == kScanWarps) {
     if (lane == 0) {
@@ -321,7 +308,7 @@ __global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(co
     const int col_w = group * kColsPerCta + warp * CW;              // the warp's first column
     const bool fresh = b.seq_lens[s] - n <= 0;
     float* st = p.state + ((static_cast<long long>(slot) * p.H + h) * p.dv + col_w + grp * C) * p.dk4;
-    F2 S[C][KT / 2];
+    ZbF2 S[C][KT / 2];
 #pragma unroll
     for (int c = 0; c < C; ++c)
 #pragma unroll
@@ -329,14 +316,14 @@ __global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(co
         const int key = (i * G + kl) * 4;
         float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
         if (!fresh && key < p.dk4 && col_w + grp * C + c < p.dv) f = *reinterpret_cast<const float4*>(st + c * p.dk4 + key);
-        S[c][2 * i] = pack2(f.x, f.y);
-        S[c][2 * i + 1] = pack2(f.z, f.w);
+        S[c][2 * i] = zb_pack2(f.x, f.y);
+        S[c][2 * i + 1] = zb_pack2(f.z, f.w);
       }
     uint32_t stage = 0, phase = 0;
     for (int blk = 0; blk < nblk; ++blk) {
       if (!__all_sync(0xffffffffu, zb_mbar_wait(&full_bar[stage], phase, abort_flag))) break;
       const float* d = delta_smem + stage * stage_floats;
-      auto keys = [&](const float* row, F2 (&v)[KT / 2]) {
+      auto keys = [&](const float* row, ZbF2 (&v)[KT / 2]) {
 #pragma unroll
         for (int i = 0; i < KT / 4; ++i) {
           const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(row + (i * G + kl) * 4);
@@ -351,14 +338,14 @@ __global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(co
         for (int t = 0; t < TB; ++t)
 #pragma unroll
           for (int ab = 0; ab < 2; ++ab) {
-            F2 v[KT / 2];
+            ZbF2 v[KT / 2];
             keys(d + (ab == 0 ? bl.pk() : bl.pq()) + (tb + t) * DK, v);
 #pragma unroll
             for (int c = 0; c < C; ++c) {
-              F2 acc = mul2(v[0], S[c][0]);
+              ZbF2 acc = zb_mul2(v[0], S[c][0]);
 #pragma unroll
-              for (int i = 1; i < KT / 2; ++i) acc = fma2(v[i], S[c][i], acc);
-              part[(t * 2 + ab) * C + c] = sum2(acc);
+              for (int i = 1; i < KT / 2; ++i) acc = zb_fma2(v[i], S[c][i], acc);
+              part[(t * 2 + ab) * C + c] = zb_sum2(acc);
             }
           }
         reduce_scatter<2 * TB * C, G>(part, kl);
@@ -390,21 +377,21 @@ __global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(co
         if (i < n && col_w + c8 < p.dv) p.o[static_cast<long long>(t0 + i) * p.H * p.dv + h * p.dv + col_w + c8] = o;
       }
       __syncwarp();
-      F2 v[KT / 2];
+      ZbF2 v[KT / 2];
       keys(d + bl.p7(), v);
 #pragma unroll
       for (int c = 0; c < C; ++c)
 #pragma unroll
-        for (int i = 0; i < KT / 2; ++i) S[c][i] = mul2(S[c][i], v[i]);
+        for (int i = 0; i < KT / 2; ++i) S[c][i] = zb_mul2(S[c][i], v[i]);
 #pragma unroll
       for (int t = 0; t < kB; ++t) {
         keys(d + bl.rk() + t * DK, v);
 #pragma unroll
         for (int c = 0; c < C; ++c) {
           const float uc = su[warp][t][grp * C + c];
-          const F2 uu = pack2(uc, uc);
+          const ZbF2 uu = zb_pack2(uc, uc);
 #pragma unroll
-          for (int i = 0; i < KT / 2; ++i) S[c][i] = fma2(v[i], uu, S[c][i]);
+          for (int i = 0; i < KT / 2; ++i) S[c][i] = zb_fma2(v[i], uu, S[c][i]);
         }
       }
       __syncwarp();
@@ -447,11 +434,24 @@ __global__ void __launch_bounds__(256) zb_delta_finish_kernel(const DeltaArgs p,
   const float* gate = p.low + t * p.ld_low + p.H * p.dk + h * p.dv;
   A* out = reinterpret_cast<A*>(p.out) + t * p.ld_out + h * p.dv;
   float ss = 0.f;
-  for (int c = lane; c < p.dv; c += 32) ss = fmaf(o[c], o[c], ss);
+  constexpr int kHeld = 4;                                   // values per lane that stay in registers
+  float ov[kHeld], gv[kHeld];
+#pragma unroll
+  for (int i = 0; i < kHeld; ++i) {
+    const int c = lane + 32 * i;
+    ov[i] = c < p.dv ? o[c] : 0.f;
+    gv[i] = c < p.dv ? gate[c] : 0.f;
+    ss = fmaf(ov[i], ov[i], ss);
+  }
+  for (int c = lane + 32 * kHeld; c < p.dv; c += 32) ss = fmaf(o[c], o[c], ss);
   const float inv = 1.f / sqrtf(zb_warp_sum(ss) / static_cast<float>(p.dv) + p.eps);
-  for (int c = lane; c < p.dv; c += 32) zb_st_act(out + c, o[c] * inv * p.norm[c] * sigmoid(gate[c]));
-  int s = 0;
-  while (s + 1 < b.num_seqs && b.q_start[s + 1] <= t) ++s;
+#pragma unroll
+  for (int i = 0; i < kHeld; ++i) {
+    const int c = lane + 32 * i;
+    if (c < p.dv) zb_st_act(out + c, ov[i] * inv * p.norm[c] * sigmoid<A>(gv[i]));
+  }
+  for (int c = lane + 32 * kHeld; c < p.dv; c += 32) zb_st_act(out + c, o[c] * inv * p.norm[c] * sigmoid<A>(gate[c]));
+  const int s = zb_sequence_of(b, t);
   const int n = b.q_start[s + 1] - b.q_start[s], left = b.q_start[s + 1] - t;      // left: tokens from here to the portion's end
   if (left > p.taps || left <= 0) return;
   const int slot = p.slots[s], pos = b.seq_lens[s] - left;
@@ -468,26 +468,40 @@ __global__ void __launch_bounds__(256) zb_delta_finish_kernel(const DeltaArgs p,
 }
 
 // ------------------------------------------------------------------------------------------ one token
-// SG lanes share a column, KT key channels each; the columns of a head in passes of NT / SG.
-template <typename A, int KT, int SG>
-__global__ void __launch_bounds__(512) zb_delta_step_kernel(const DeltaArgs p, const ZbVarlen b) {
+// SG lanes share a column, KT key channels each; the columns of a head in passes of NT / SG.  The head's query, key and value
+// channels and its decays are dealt over the threads, a channel each; T bounds the taps.
+template <typename A, int KT, int SG, int T>
+__global__ void __launch_bounds__(512, 2) zb_delta_step_kernel(const DeltaArgs p, const ZbVarlen b) {
   constexpr int DP = KT * SG;
-  __shared__ __align__(16) float s_gk[DP], s_gq[DP], s_k[DP], s_g[DP];
-  extern __shared__ float step_smem[];                       // [dv] values, then outputs
+  __shared__ __align__(16) float s_q[DP], s_k[DP], s_g[DP], s_gk[DP];
+  extern __shared__ float sy[];                              // [dv] values, then outputs
   __shared__ float red[4][16];
   zb_pdl_launch();
   const int h = blockIdx.x, s = blockIdx.y, tid = threadIdx.x, NT = blockDim.x, warps = NT / 32;
   const int kg = tid % SG, rep = p.H / p.G, g = h / rep;
-  const int C = 2 * p.G * p.dk + p.H * p.dv;
-  const float a_log = p.a_log[h];
+  const int C = 2 * p.G * p.dk + p.H * p.dv, items = 3 * p.dk + p.dv;
+  // item: the head's query | key | value channels, then its decays; the first one's parameters do not wait for the input
+  auto column = [&](int item) {
+    return item < p.dk ? g * p.dk + item : item < 2 * p.dk ? p.G * p.dk + g * p.dk + item - p.dk : 2 * p.G * p.dk + h * p.dv + item - 2 * p.dk;
+  };
+  float w[T];                                                // w[d]: the tap on the input d tokens back
+  auto parameters = [&](int item) {
+    const bool decay = item >= 2 * p.dk + p.dv;
+    const int col = decay ? 0 : column(item);
+#pragma unroll
+    for (int d = 0; d < T; ++d) w[d] = !decay && d < p.taps ? p.conv_w[static_cast<long long>(p.taps - 1 - d) * C + col] : 0.f;
+    if (decay) w[0] = p.dt_bias[h * p.dk + item - 2 * p.dk - p.dv];
+  };
+  if (tid < items) parameters(tid);
+  const float rate = expf(p.a_log[h]);
   zb_pdl_wait();
   const int t = b.q_start[s];
   if (b.q_start[s + 1] <= t) return;
   const int slot = p.slots[s];
   if (!ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelDelta, 4)) return;
-  const int pos = max(0, b.seq_lens[s] - 1);
+  const int pos = max(0, b.seq_lens[s] - 1), row = pos % p.taps;
   float* st0 = p.state + (static_cast<long long>(slot) * p.H + h) * p.dv * p.dk4;
-  F2 S[KT / 2];
+  ZbF2 S[KT / 2];
   auto load = [&](int col) {
 #pragma unroll
     for (int i = 0; i < KT / 4; ++i) {
@@ -501,38 +515,43 @@ __global__ void __launch_bounds__(512) zb_delta_step_kernel(const DeltaArgs p, c
   load(tid / SG);
   const A* in = reinterpret_cast<const A*>(p.in) + t * p.ld_in;
   A* ring = reinterpret_cast<A*>(p.ring) + static_cast<long long>(slot) * p.taps * C;
-  auto conv = [&](int col, bool keep) {
-    float acc = 0.f;
-    const A cur = in[col];
-#pragma unroll
-    for (int d = 0; d < kMaxTaps; ++d) {
-      if (d >= p.taps) break;
-      float x = 0.f;
-      if (d == 0) x = zb_ld_act(&cur);
-      else if (pos - d >= 0) x = zb_ld_act(ring + static_cast<long long>((pos - d) % p.taps) * C + col);
-      acc = fmaf(p.conv_w[static_cast<long long>(p.taps - 1 - d) * C + col], x, acc);
+  const float beta_logit = zb_ld_act(in + p.beta_off + h);
+  for (int item = tid; item < items; item += NT) {
+    if (item >= NT) parameters(item);
+    if (item >= 2 * p.dk + p.dv) {
+      const int c = item - 2 * p.dk - p.dv;
+      s_g[c] = decay_of<A>(rate, p.low[t * p.ld_low + h * p.dk + c] + w[0]);
+      continue;
     }
-    if (keep) ring[static_cast<long long>(pos % p.taps) * C + col] = cur;
-    return silu(acc);
-  };
+    const int col = column(item);
+    A x[T];
+    x[0] = in[col];
+#pragma unroll
+    for (int d = 1; d < T; ++d) {                            // all requested at once; what lies before the start counts nothing
+      const int r = row - d < 0 ? row - d + p.taps : row - d;
+      x[d] = ring[static_cast<long long>(d < p.taps ? r : row) * C + col];
+    }
+    float acc = w[0] * zb_ld_act(&x[0]);
+#pragma unroll
+    for (int d = 1; d < T; ++d) acc = d < p.taps && d <= pos ? fmaf(w[d], zb_ld_act(&x[d]), acc) : acc;
+    if (item >= 2 * p.dk || h % rep == 0) ring[static_cast<long long>(row) * C + col] = x[0];
+    const float y = silu<A>(acc);
+    if (item < p.dk) s_q[item] = y;
+    else if (item < 2 * p.dk) s_k[item - p.dk] = y;
+    else sy[item - 2 * p.dk] = y;
+  }
+  for (int c = p.dk + tid; c < DP; c += NT) {
+    s_q[c] = s_k[c] = 0.f;
+    s_g[c] = 1.f;
+  }
+  __syncthreads();
   float qq = 0.f, kk = 0.f, qk = 0.f;
   for (int c = tid; c < DP; c += NT) {
-    float q = 0.f, k = 0.f, dec = 1.f;
-    if (c < p.dk) {
-      q = conv(g * p.dk + c, h % rep == 0);
-      k = conv((p.G + g) * p.dk + c, h % rep == 0);
-      dec = decay_of(a_log, p.low[t * p.ld_low + h * p.dk + c] + p.dt_bias[h * p.dk + c]);
-    }
+    const float q = s_q[c], k = s_k[c];
     qq = fmaf(q, q, qq);
     kk = fmaf(k, k, kk);
     qk = fmaf(q, k, qk);
-    s_gq[c] = q;
-    s_k[c] = k;
-    s_g[c] = dec;
   }
-  float* sy = step_smem;
-  for (int c = tid; c < p.dv; c += NT) sy[c] = conv(2 * p.G * p.dk + h * p.dv + c, true);
-  const float beta = sigmoid(zb_ld_act(in + p.beta_off + h));
   qq = zb_warp_sum(qq);
   kk = zb_warp_sum(kk);
   qk = zb_warp_sum(qk);
@@ -542,8 +561,9 @@ __global__ void __launch_bounds__(512) zb_delta_step_kernel(const DeltaArgs p, c
     red[2][tid >> 5] = qk;
   }
   __syncthreads();
+  const float beta = sigmoid<A>(beta_logit);
   qq = kk = qk = 0.f;
-  for (int i = 0; i < warps; ++i) {
+  for (int i = 0; i < min(warps, (DP + 31) / 32); ++i) {     // warps past the channels have nothing to add
     qq += red[0][i];
     kk += red[1][i];
     qk += red[2][i];
@@ -554,7 +574,7 @@ __global__ void __launch_bounds__(512) zb_delta_step_kernel(const DeltaArgs p, c
     const float k = s_k[c] * ki, dec = s_g[c];
     s_k[c] = k;
     s_gk[c] = dec * k;
-    s_gq[c] *= dec * qi;
+    s_q[c] *= dec * qi;
   }
   __syncthreads();
   float ss = 0.f;
@@ -562,16 +582,16 @@ __global__ void __launch_bounds__(512) zb_delta_step_kernel(const DeltaArgs p, c
     const int col = c0 + tid / SG;
     if (c0 > 0) load(col);
     const float v = col < p.dv ? sy[col] : 0.f;
-    F2 a2 = 0ull, b2 = 0ull;
+    ZbF2 a2 = 0ull, b2 = 0ull;
 #pragma unroll
     for (int i = 0; i < KT / 4; ++i) {
-      const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(s_gk + (i * SG + kg) * 4), y = *reinterpret_cast<const ulonglong2*>(s_gq + (i * SG + kg) * 4);
-      a2 = fma2(S[2 * i], x.x, a2);
-      b2 = fma2(S[2 * i], y.x, b2);
-      a2 = fma2(S[2 * i + 1], x.y, a2);
-      b2 = fma2(S[2 * i + 1], y.y, b2);
+      const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(s_gk + (i * SG + kg) * 4), y = *reinterpret_cast<const ulonglong2*>(s_q + (i * SG + kg) * 4);
+      a2 = zb_fma2(S[2 * i], x.x, a2);
+      b2 = zb_fma2(S[2 * i], y.x, b2);
+      a2 = zb_fma2(S[2 * i + 1], x.y, a2);
+      b2 = zb_fma2(S[2 * i + 1], y.y, b2);
     }
-    float a = sum2(a2), o = sum2(b2);
+    float a = zb_sum2(a2), o = zb_sum2(b2);
 #pragma unroll
     for (int m = 1; m < SG; m <<= 1) {
       a += __shfl_xor_sync(0xffffffffu, a, m);
@@ -579,14 +599,14 @@ __global__ void __launch_bounds__(512) zb_delta_step_kernel(const DeltaArgs p, c
     }
     const float u = beta * (v - a);
     o = fmaf(qk, u, o);
-    const F2 uu = pack2(u, u);
+    const ZbF2 uu = zb_pack2(u, u);
     if (col < p.dv) {
 #pragma unroll
       for (int i = 0; i < KT / 4; ++i) {
         const int key = (i * SG + kg) * 4;
         const ulonglong2 gg = *reinterpret_cast<const ulonglong2*>(s_g + key), k = *reinterpret_cast<const ulonglong2*>(s_k + key);
-        S[2 * i] = fma2(S[2 * i], gg.x, mul2(k.x, uu));
-        S[2 * i + 1] = fma2(S[2 * i + 1], gg.y, mul2(k.y, uu));
+        S[2 * i] = zb_fma2(S[2 * i], gg.x, zb_mul2(k.x, uu));
+        S[2 * i + 1] = zb_fma2(S[2 * i + 1], gg.y, zb_mul2(k.y, uu));
         if (key < p.dk4) *reinterpret_cast<ulonglong2*>(st0 + static_cast<long long>(col) * p.dk4 + key) = make_ulonglong2(S[2 * i], S[2 * i + 1]);
       }
       if (kg == 0) {
@@ -603,13 +623,17 @@ __global__ void __launch_bounds__(512) zb_delta_step_kernel(const DeltaArgs p, c
   const float inv = 1.f / sqrtf(ss / static_cast<float>(p.dv) + p.eps);
   const float* gate = p.low + t * p.ld_low + p.H * p.dk + h * p.dv;
   A* out = reinterpret_cast<A*>(p.out) + t * p.ld_out + h * p.dv;
-  for (int c = tid; c < p.dv; c += NT) zb_st_act(out + c, sy[c] * inv * p.norm[c] * sigmoid(gate[c]));
+  for (int c = tid; c < p.dv; c += NT) zb_st_act(out + c, sy[c] * inv * p.norm[c] * sigmoid<A>(gate[c]));
 }
 
 // ------------------------------------------------------------------------------------------ launches
 template <typename A, int KI>
 cudaError_t launch_prep(const DeltaArgs& p, const BlockLayout& bl, const ZbVarlen& b, int num_blocks, cudaStream_t s) {
-  return zb_launch(zb_delta_prep_kernel<A, KI>, dim3(num_blocks, p.H), dim3(128), 0, s, p, bl, b);
+  int threads = (3 * bl.DK + bl.groups * kColsPerCta + 127) / 128 * 128;
+  if (threads > 512) threads = 512;
+  const dim3 grid(num_blocks, p.H);
+  if (p.taps <= 4) return zb_launch(zb_delta_prep_kernel<A, KI, 4>, grid, dim3(threads), 0, s, p, bl, b);
+  return zb_launch(zb_delta_prep_kernel<A, KI, kMaxTaps>, grid, dim3(threads), 0, s, p, bl, b);
 }
 template <typename A>
 cudaError_t launch_prep(const DeltaArgs& p, const BlockLayout& bl, const ZbVarlen& b, int num_blocks, cudaStream_t s) {
@@ -636,7 +660,9 @@ template <typename A, int KT, int SG>
 cudaError_t launch_step(const DeltaArgs& p, const ZbVarlen& b, cudaStream_t s) {
   int threads = (p.dv * SG + 31) / 32 * 32;
   if (threads > 512) threads = 512;
-  return zb_launch(zb_delta_step_kernel<A, KT, SG>, dim3(p.H, b.num_seqs), dim3(threads), p.dv * sizeof(float), s, p, b);
+  const dim3 grid(p.H, b.num_seqs);
+  if (p.taps <= 4) return zb_launch(zb_delta_step_kernel<A, KT, SG, 4>, grid, dim3(threads), p.dv * sizeof(float), s, p, b);
+  return zb_launch(zb_delta_step_kernel<A, KT, SG, kMaxTaps>, grid, dim3(threads), p.dv * sizeof(float), s, p, b);
 }
 template <typename A>
 cudaError_t launch_step(const DeltaArgs& p, const ZbVarlen& b, cudaStream_t s) {

@@ -506,6 +506,35 @@ ZB_DEVICE float zb_rcp(float x) {
   return y;
 }
 
+// Two packed fp32 (one register pair), and the instructions that work on both at once.
+using ZbF2 = unsigned long long;
+ZB_DEVICE ZbF2 zb_pack2(float a, float b) {
+  ZbF2 d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(a), "f"(b));
+  return d;
+}
+ZB_DEVICE void zb_unpack2(ZbF2 a, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a)); }
+ZB_DEVICE ZbF2 zb_fma2(ZbF2 a, ZbF2 b, ZbF2 c) {
+  ZbF2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+ZB_DEVICE ZbF2 zb_mul2(ZbF2 a, ZbF2 b) {
+  ZbF2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+ZB_DEVICE ZbF2 zb_add2(ZbF2 a, ZbF2 b) {
+  ZbF2 d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+ZB_DEVICE float zb_sum2(ZbF2 a) {
+  float x, y;
+  zb_unpack2(a, x, y);
+  return x + y;
+}
+
 ZB_DEVICE float zb_warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
