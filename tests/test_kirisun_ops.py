@@ -330,6 +330,23 @@ def test_delta_rule_of_unequal_sequences_in_one_batch(target, name):
         close(torch.cat(got[i]), delta_want(name, t), TOL[dt], i)
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("dt", [F32, BF16])
+@pytest.mark.parametrize("name", ["32", "shared", "64", "square", "largest keys"])
+def test_delta_rule_of_many_sequences(name, dt):
+    """Batches large enough for the scan's wide form, more sequences than a warp has lanes."""
+    t = delta_case(name, 30, 81)
+    want = delta_want(name, t)
+    H, _, _, dv, _ = DELTA[name]
+    m = 300 // (H * ((dv + 31) // 32)) + 2
+    lens = [1 + (7 * i) % 23 for i in range(m)]
+    L = DeltaLayer(name, t, "cuda", dt, slots=m)
+    first = L.run([(t, 0, n) for n in lens], [0] * m, list(range(m))[::-1])
+    second = L.run([(t, n, n + 7) for n in lens], lens, list(range(m))[::-1])
+    close(first, np.concatenate([want[:n] for n in lens]), TOL[dt])
+    close(second, np.concatenate([want[n:n + 7] for n in lens]), TOL[dt])
+
+
 @pytest.mark.parametrize("target", TARGETS[:2])
 @pytest.mark.parametrize("decay", ["fast", "slow"])
 def test_extreme_decays(target, decay):

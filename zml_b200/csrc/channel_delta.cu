@@ -13,8 +13,8 @@
 //                             S <- diag(P_7) S + sum_t (R_t k_t) u_t^T
 //                           with L_tj = k_t^T diag(decays of j+1..t) k_j and Q_tj the same with q_t.  All factors are products
 //                           of decays, none a quotient, so nothing overflows however fast a channel forgets
-//   zb_delta_scan_kernel    walks the blocks of a (sequence, head): a warp owns eight columns of S (value channels), bulk
-//                           copies bring the blocks in through a ring of stages
+//   zb_delta_scan_kernel    walks the blocks of a (sequence, head): a warp owns four or eight columns of S (value channels),
+//                           bulk copies bring the blocks in through a ring of stages
 //   zb_delta_finish_kernel  norm and gate, and the convolution inputs that later tokens need
 //   zb_delta_step_kernel    one token per sequence: everything above in one launch, the whole state of the head requested
 //                           before anything else
@@ -30,7 +30,6 @@ constexpr uint32_t kKernelDelta = 36;
 constexpr int kB = 8;                       // tokens per block
 constexpr int kMaxTaps = 8;                 // at most kB: only a sequence's first block reaches back into the ring
 constexpr int kColsPerCta = 32;
-constexpr int kScanWarps = 4;               // eight columns each
 constexpr int kScanStages = 3;
 
 struct DeltaArgs {
@@ -254,18 +253,42 @@ __global__ void __launch_bounds__(512, 2) zb_delta_prep_kernel(const DeltaArgs p
 }
 
 // ------------------------------------------------------------------------------------------ portions: scan
-// G lanes share a column, each with KT key channels (float4 number i at channel (i G + lane) 4); C columns per lane, TB
-// tokens summed over the lanes at a time.
+// N consecutive floats of shared memory that start on a multiple of N.
+template <int N>
+ZB_DEVICE void ld_floats(float (&v)[N], const float* p) {
+  if constexpr (N % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+      const float4 f = *reinterpret_cast<const float4*>(p + i);
+      v[i] = f.x; v[i + 1] = f.y; v[i + 2] = f.z; v[i + 3] = f.w;
+    }
+  } else if constexpr (N == 2) {
+    const float2 f = *reinterpret_cast<const float2*>(p);
+    v[0] = f.x; v[1] = f.y;
+  } else {
+    v[0] = *p;
+  }
+}
+
+// G lanes share a column, each with KT key channels (float4 number i at channel (i G + lane) 4); C columns per lane, so
+// CW = 32 / G * C per warp; TB tokens are summed over the lanes at a time.
+template <int G, int C>
+constexpr int scan_columns() { return 32 / G * C; }
+template <int G, int C>
+constexpr int scan_warps() { return kColsPerCta / scan_columns<G, C>(); }
+
 template <int G, int KT, int C, int TB>
-__global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(const DeltaArgs p, const BlockLayout bl, const ZbVarlen b,
-                                                                              ZbStatus* status) {
+__global__ void __launch_bounds__(32 * (scan_warps<G, C>() + 1)) zb_delta_scan_kernel(const DeltaArgs p, const BlockLayout bl, const ZbVarlen b,
+                                                                                    ZbStatus* status) {
   constexpr int DK = G * KT;
-  constexpr int CW = 32 / G * C;
-  static_assert(CW == 8 && CW * kScanWarps == kColsPerCta && kB % TB == 0, "");
+  constexpr int CW = scan_columns<G, C>();
+  constexpr int kWarps = scan_warps<G, C>();
+  constexpr int R = 32 / CW;                                 // lanes that solve for the same column
+  static_assert((CW == 8 || CW == 4) && kB % TB == 0 && kB % R == 0, "");
   extern __shared__ __align__(128) float delta_smem[];
   __shared__ uint64_t full_bar[kScanStages], empty_bar[kScanStages];
   __shared__ uint32_t abort_word;
-  __shared__ __align__(16) float sa[kScanWarps][kB][8], sb[kScanWarps][kB][8], su[kScanWarps][kB][8];
+  __shared__ __align__(16) float sa[kWarps][kB][CW], sb[kWarps][kB][CW], su[kWarps][kB][CW];
   volatile uint32_t* abort_flag = &abort_word;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.x, s = blockIdx.y, group = blockIdx.z;
@@ -273,7 +296,7 @@ __global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(co
   if (threadIdx.x == 0) {
     for (int i = 0; i < kScanStages; ++i) {
       zb_mbar_init(&full_bar[i], 1);
-      zb_mbar_init(&empty_bar[i], kScanWarps);
+      zb_mbar_init(&empty_bar[i], kWarps);
     }
     abort_word = 0u;
     zb_mbar_fence_init();
@@ -286,7 +309,7 @@ __global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(co
   if (n <= 0 || !ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelDelta, 2)) return;          // uniform over the block
   const int first = zb_blocks_before(b, kB, s);
   const int nblk = (n + kB - 1) / kB;
-  if (warp == kScanWarps) {
+  if (warp == kWarps) {
     if (lane == 0) {
       uint32_t stage = 0, phase = 0;
       const uint32_t head_bytes = bl.head() * 4, val_bytes = kB * kColsPerCta * 4;
@@ -304,7 +327,7 @@ __global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(co
       }
     }
   } else {
-    const int kl = lane % G, grp = lane / G, c8 = lane & 7, r = lane >> 3;
+    const int kl = lane % G, grp = lane / G, cw = lane % CW, r = lane / CW;
     const int col_w = group * kColsPerCta + warp * CW;              // the warp's first column
     const bool fresh = b.seq_lens[s] - n <= 0;
     float* st = p.state + ((static_cast<long long>(slot) * p.H + h) * p.dv + col_w + grp * C) * p.dk4;
@@ -356,25 +379,30 @@ __global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(co
         }
       }
       __syncwarp();
-      // every lane solves for the block's u of column c8; lanes r = 0 .. 3 of a column then take outputs r and r + 4
-      float u[kB];
-      const float* vals = d + bl.head() + warp * CW + c8;
+      // every lane solves for the block's u of column cw; the R lanes of a column then take every R-th output
+      float u[kB], lo[kB][kB], beta[kB];
+      const float* vals = d + bl.head() + warp * CW + cw;
+      ld_floats<kB>(beta, d + bl.beta());
 #pragma unroll
       for (int t = 0; t < kB; ++t) {
-        float acc = d[bl.beta() + t] * (vals[t * kColsPerCta] - sa[warp][t][c8]);
-#pragma unroll
-        for (int j = 0; j < t; ++j) acc = fmaf(-d[bl.bl() + t * kB + j], u[j], acc);
-        u[t] = acc;
-        if ((t & 3) == r) su[warp][t][c8] = acc;
+        if (t > 0) ld_floats<4>(reinterpret_cast<float (&)[4]>(lo[t][0]), d + bl.bl() + t * kB);
+        if (t > 4) ld_floats<4>(reinterpret_cast<float (&)[4]>(lo[t][4]), d + bl.bl() + t * kB + 4);
+        u[t] = beta[t] * (vals[t * kColsPerCta] - sa[warp][t][cw]);
       }
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int t = r + 4 * e;
-        float o = sb[warp][t][c8];
+      for (int j = 0; j < kB; ++j) {
 #pragma unroll
-        for (int j = 0; j < kB; ++j) o = fmaf(d[bl.ql() + t * kB + j], u[j], o);
-        const int i = blk * kB + t;
-        if (i < n && col_w + c8 < p.dv) p.o[static_cast<long long>(t0 + i) * p.H * p.dv + h * p.dv + col_w + c8] = o;
+        for (int t = j + 1; t < kB; ++t) u[t] = fmaf(-lo[t][j], u[j], u[t]);
+        if (j % R == r) su[warp][j][cw] = u[j];
+      }
+#pragma unroll
+      for (int e = 0; e < kB / R; ++e) {
+        const int t = r + R * e, i = blk * kB + t;
+        float ql[kB], o = sb[warp][t][cw];
+        ld_floats<kB>(ql, d + bl.ql() + t * kB);
+#pragma unroll
+        for (int j = 0; j < kB; ++j) o = fmaf(ql[j], u[j], o);
+        if (i < n && col_w + cw < p.dv) p.o[static_cast<long long>(t0 + i) * p.H * p.dv + h * p.dv + col_w + cw] = o;
       }
       __syncwarp();
       ZbF2 v[KT / 2];
@@ -385,11 +413,12 @@ __global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(co
         for (int i = 0; i < KT / 2; ++i) S[c][i] = zb_mul2(S[c][i], v[i]);
 #pragma unroll
       for (int t = 0; t < kB; ++t) {
+        float uc[C];
+        ld_floats<C>(uc, &su[warp][t][grp * C]);
         keys(d + bl.rk() + t * DK, v);
 #pragma unroll
         for (int c = 0; c < C; ++c) {
-          const float uc = su[warp][t][grp * C + c];
-          const ZbF2 uu = zb_pack2(uc, uc);
+          const ZbF2 uu = zb_pack2(uc[c], uc[c]);
 #pragma unroll
           for (int i = 0; i < KT / 2; ++i) S[c][i] = zb_fma2(v[i], uu, S[c][i]);
         }
@@ -647,14 +676,16 @@ int launch_scan(const DeltaArgs& p, const BlockLayout& bl, const ZbVarlen& b, Zb
   const int smem = kScanStages * (bl.head() + kB * kColsPerCta) * 4;
   static bool configured[16] = {};
   if (const int rc = zb_config_smem_once(zb_delta_scan_kernel<G, KT, C, TB>, smem, configured)) return rc;
-  const cudaError_t e = zb_launch(zb_delta_scan_kernel<G, KT, C, TB>, dim3(p.H, b.num_seqs, bl.groups), dim3(32 * (kScanWarps + 1)), smem, s, p, bl, b, status);
+  const cudaError_t e = zb_launch(zb_delta_scan_kernel<G, KT, C, TB>, dim3(p.H, b.num_seqs, bl.groups), dim3(32 * (scan_warps<G, C>() + 1)), smem, s, p, bl, b, status);
   return static_cast<int>(e);
 }
 int launch_scan(const DeltaArgs& p, const BlockLayout& bl, const ZbVarlen& b, ZbStatus* status, cudaStream_t s) {
-  if (bl.DK == 32) return launch_scan<8, 4, 2, 8>(p, bl, b, status, s);
-  if (bl.DK == 64) return launch_scan<16, 4, 4, 8>(p, bl, b, status, s);
-  if (bl.DK == 128) return launch_scan<16, 8, 4, 8>(p, bl, b, status, s);
-  return launch_scan<32, 8, 8, 4>(p, bl, b, status, s);
+  // few (sequence, head) pairs: four columns per warp, twice the warps; many: eight, half the shared-memory reads
+  const bool narrow = static_cast<long long>(p.H) * b.num_seqs * bl.groups <= 2 * 148;
+  if (bl.DK == 32) return narrow ? launch_scan<8, 4, 1, 8>(p, bl, b, status, s) : launch_scan<8, 4, 2, 8>(p, bl, b, status, s);
+  if (bl.DK == 64) return narrow ? launch_scan<16, 4, 2, 8>(p, bl, b, status, s) : launch_scan<16, 4, 4, 8>(p, bl, b, status, s);
+  if (bl.DK == 128) return narrow ? launch_scan<16, 8, 2, 8>(p, bl, b, status, s) : launch_scan<16, 8, 4, 8>(p, bl, b, status, s);
+  return narrow ? launch_scan<32, 8, 4, 8>(p, bl, b, status, s) : launch_scan<32, 8, 8, 4>(p, bl, b, status, s);
 }
 template <typename A, int KT, int SG>
 cudaError_t launch_step(const DeltaArgs& p, const ZbVarlen& b, cudaStream_t s) {
