@@ -334,7 +334,7 @@ def test_delta_rule_of_unequal_sequences_in_one_batch(target, name):
 @pytest.mark.parametrize("dt", [F32, BF16])
 @pytest.mark.parametrize("name", ["32", "shared", "64", "square", "largest keys"])
 def test_delta_rule_of_many_sequences(name, dt):
-    """Batches large enough for the scan's wide form, more sequences than a warp has lanes."""
+    """More sequences than a warp has lanes, every padded key size."""
     t = delta_case(name, 30, 81)
     want = delta_want(name, t)
     H, _, _, dv, _ = DELTA[name]

@@ -13,8 +13,8 @@
 //                             S <- diag(P_7) S + sum_t (R_t k_t) u_t^T
 //                           with L_tj = k_t^T diag(decays of j+1..t) k_j and Q_tj the same with q_t.  All factors are products
 //                           of decays, none a quotient, so nothing overflows however fast a channel forgets
-//   zb_delta_scan_kernel    walks the blocks of a (sequence, head): a warp owns four or eight columns of S (value channels),
-//                           bulk copies bring the blocks in through a ring of stages
+//   zb_delta_scan_kernel    walks the blocks of a (sequence, head): a warp owns eight columns of S (value channels), bulk
+//                           copies bring the blocks in through a ring of stages
 //   zb_delta_finish_kernel  norm and gate, and the convolution inputs that later tokens need
 //   zb_delta_step_kernel    one token per sequence: everything above in one launch, the whole state of the head requested
 //                           before anything else
@@ -270,25 +270,22 @@ ZB_DEVICE void ld_floats(float (&v)[N], const float* p) {
   }
 }
 
-// G lanes share a column, each with KT key channels (float4 number i at channel (i G + lane) 4); C columns per lane, so
-// CW = 32 / G * C per warp; TB tokens are summed over the lanes at a time.
-template <int G, int C>
-constexpr int scan_columns() { return 32 / G * C; }
-template <int G, int C>
-constexpr int scan_warps() { return kColsPerCta / scan_columns<G, C>(); }
+constexpr int kScanColumns = 8;              // per warp
+constexpr int kScanWarps = kColsPerCta / kScanColumns;
 
+// G lanes share a column, each with KT key channels (float4 number i at channel (i G + lane) 4); C columns per lane; TB
+// tokens are summed over the lanes at a time.
 template <int G, int KT, int C, int TB>
-__global__ void __launch_bounds__(32 * (scan_warps<G, C>() + 1)) zb_delta_scan_kernel(const DeltaArgs p, const BlockLayout bl, const ZbVarlen b,
-                                                                                    ZbStatus* status) {
+__global__ void __launch_bounds__(32 * (kScanWarps + 1)) zb_delta_scan_kernel(const DeltaArgs p, const BlockLayout bl, const ZbVarlen b,
+                                                                              ZbStatus* status) {
   constexpr int DK = G * KT;
-  constexpr int CW = scan_columns<G, C>();
-  constexpr int kWarps = scan_warps<G, C>();
+  constexpr int CW = kScanColumns;
   constexpr int R = 32 / CW;                                 // lanes that solve for the same column
-  static_assert((CW == 8 || CW == 4) && kB % TB == 0 && kB % R == 0, "");
+  static_assert(32 / G * C == CW && kB % TB == 0 && kB % R == 0, "");
   extern __shared__ __align__(128) float delta_smem[];
   __shared__ uint64_t full_bar[kScanStages], empty_bar[kScanStages];
   __shared__ uint32_t abort_word;
-  __shared__ __align__(16) float sa[kWarps][kB][CW], sb[kWarps][kB][CW], su[kWarps][kB][CW];
+  __shared__ __align__(16) float sa[kScanWarps][kB][CW], sb[kScanWarps][kB][CW], su[kScanWarps][kB][CW];
   volatile uint32_t* abort_flag = &abort_word;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.x, s = blockIdx.y, group = blockIdx.z;
@@ -296,7 +293,7 @@ __global__ void __launch_bounds__(32 * (scan_warps<G, C>() + 1)) zb_delta_scan_k
   if (threadIdx.x == 0) {
     for (int i = 0; i < kScanStages; ++i) {
       zb_mbar_init(&full_bar[i], 1);
-      zb_mbar_init(&empty_bar[i], kWarps);
+      zb_mbar_init(&empty_bar[i], kScanWarps);
     }
     abort_word = 0u;
     zb_mbar_fence_init();
@@ -309,7 +306,7 @@ __global__ void __launch_bounds__(32 * (scan_warps<G, C>() + 1)) zb_delta_scan_k
   if (n <= 0 || !ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelDelta, 2)) return;          // uniform over the block
   const int first = zb_blocks_before(b, kB, s);
   const int nblk = (n + kB - 1) / kB;
-  if (warp == kWarps) {
+  if (warp == kScanWarps) {
     if (lane == 0) {
       uint32_t stage = 0, phase = 0;
       const uint32_t head_bytes = bl.head() * 4, val_bytes = kB * kColsPerCta * 4;
@@ -676,16 +673,14 @@ int launch_scan(const DeltaArgs& p, const BlockLayout& bl, const ZbVarlen& b, Zb
   const int smem = kScanStages * (bl.head() + kB * kColsPerCta) * 4;
   static bool configured[16] = {};
   if (const int rc = zb_config_smem_once(zb_delta_scan_kernel<G, KT, C, TB>, smem, configured)) return rc;
-  const cudaError_t e = zb_launch(zb_delta_scan_kernel<G, KT, C, TB>, dim3(p.H, b.num_seqs, bl.groups), dim3(32 * (scan_warps<G, C>() + 1)), smem, s, p, bl, b, status);
+  const cudaError_t e = zb_launch(zb_delta_scan_kernel<G, KT, C, TB>, dim3(p.H, b.num_seqs, bl.groups), dim3(32 * (kScanWarps + 1)), smem, s, p, bl, b, status);
   return static_cast<int>(e);
 }
 int launch_scan(const DeltaArgs& p, const BlockLayout& bl, const ZbVarlen& b, ZbStatus* status, cudaStream_t s) {
-  // few (sequence, head) pairs: four columns per warp, twice the warps; many: eight, half the shared-memory reads
-  const bool narrow = static_cast<long long>(p.H) * b.num_seqs * bl.groups <= 2 * 148;
-  if (bl.DK == 32) return narrow ? launch_scan<8, 4, 1, 8>(p, bl, b, status, s) : launch_scan<8, 4, 2, 8>(p, bl, b, status, s);
-  if (bl.DK == 64) return narrow ? launch_scan<16, 4, 2, 8>(p, bl, b, status, s) : launch_scan<16, 4, 4, 8>(p, bl, b, status, s);
-  if (bl.DK == 128) return narrow ? launch_scan<16, 8, 2, 8>(p, bl, b, status, s) : launch_scan<16, 8, 4, 8>(p, bl, b, status, s);
-  return narrow ? launch_scan<32, 8, 4, 8>(p, bl, b, status, s) : launch_scan<32, 8, 8, 4>(p, bl, b, status, s);
+  if (bl.DK == 32) return launch_scan<8, 4, 2, 8>(p, bl, b, status, s);
+  if (bl.DK == 64) return launch_scan<16, 4, 4, 8>(p, bl, b, status, s);
+  if (bl.DK == 128) return launch_scan<16, 8, 4, 8>(p, bl, b, status, s);
+  return launch_scan<32, 8, 8, 4>(p, bl, b, status, s);
 }
 template <typename A, int KT, int SG>
 cudaError_t launch_step(const DeltaArgs& p, const ZbVarlen& b, cudaStream_t s) {
