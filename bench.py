@@ -48,6 +48,9 @@ WORKLOADS = {
     "kirisun-3b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
     "kirisun-10b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
     "tiny-kirisun-test": dict(batch=4, prompt=(16, 64), new_tokens=8),
+    "sodotar-3b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
+    "sodotar-10b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
+    "tiny-sodotar-test": dict(batch=4, prompt=(16, 64), new_tokens=8),
 }
 
 
@@ -217,7 +220,9 @@ def run_workload(name: str, comm, args, steps: int, warmup: int, sample_clocks: 
 # Designs whose prefill and decode throughput `--compare` sets beside the closest other family at equal size: a hybrid of
 # gated full attention (where the design has attention) and gated delta net (where it has a recurrence) with the same width,
 # depth, vocabulary, head sizes of the recurrent layers and feed-forward parameters (Dopurax: three matrices of 2/3 the
-# units; Kirisun: the same experts, and the shared expert that the family always has at its smallest size).
+# units; Kirisun: the same experts, and the shared expert that the family always has at its smallest size).  Sodotar, which
+# has no recurrence, stands beside the same family with gated full attention in every layer and the same routed and shared
+# experts.
 COMPARE_SHAPES = [dict(batch=1, prompt=4096), dict(batch=8, prompt=1024), dict(batch=32, prompt=1024), dict(batch=64, prompt=2048)]
 
 
@@ -231,6 +236,18 @@ def moe_hybrid_twin(cfg) -> dict:
                 linear_key_head_dim=rec.dim, linear_num_key_heads=rec.kv_heads, linear_value_head_dim=rec.vdim, linear_num_value_heads=rec.heads,
                 layer_types=["full_attention" if s.kind == ATTENTION else "linear_attention" for s in cfg.layers], num_experts=att.experts,
                 num_experts_per_tok=att.top, moe_intermediate_size=att.ff, shared_expert_intermediate_size=64, tie_word_embeddings=False)
+
+
+def moe_attention_twin(cfg) -> dict:
+    from zml_b200.models.sodotar import ATTENTION
+    att = next(s for s in cfg.layers if s.kind == ATTENTION)
+    e = att.moe
+    return dict(hidden_size=cfg.hidden_size, num_hidden_layers=len(cfg.layers), num_attention_heads=att.heads, num_key_value_heads=att.kv_heads,
+                head_dim=2 * att.dim, vocab_size=cfg.vocab_size, rms_norm_eps=cfg.norm_eps,
+                rope_parameters=dict(rope_theta=att.base, partial_rotary_factor=att.rot / (2 * att.dim)), linear_conv_kernel_dim=4,
+                linear_key_head_dim=128, linear_num_key_heads=att.heads, linear_value_head_dim=128, linear_num_value_heads=att.heads,
+                layer_types=["full_attention"] * len(cfg.layers), num_experts=e.experts, num_experts_per_tok=e.top, moe_intermediate_size=e.ff,
+                shared_expert_intermediate_size=e.shared_ff, tie_word_embeddings=False)
 
 
 def hybrid_twin(cfg) -> dict:
@@ -257,6 +274,10 @@ def compare(name: str, args) -> None:
         from zml_b200.models.kirisun import PRESETS, KirisunConfig as Config, KirisunModel as Model
         from zml_b200.models.qwen3_5_moe import Qwen35MoeConfig as TwinConfig, Qwen35MoeModel as TwinModel
         to_twin = moe_hybrid_twin
+    elif name.startswith("sodotar"):
+        from zml_b200.models.sodotar import PRESETS, SodotarConfig as Config, SodotarModel as Model
+        from zml_b200.models.qwen3_5_moe import Qwen35MoeConfig as TwinConfig, Qwen35MoeModel as TwinModel
+        to_twin = moe_attention_twin
     else:
         from zml_b200.models.dopurax import PRESETS, DopuraxConfig as Config, DopuraxModel as Model
         from zml_b200.models.qwen3_5 import Qwen35Config as TwinConfig, Qwen35Model as TwinModel
@@ -265,7 +286,7 @@ def compare(name: str, args) -> None:
     twin = TwinConfig.from_hf(to_twin(cfg))
     sampler = ClockSampler(True)
     new, out = args.new_tokens or 128, {}
-    for label, build in ((name, lambda: Model(cfg, device="cuda:0")), ("hybrid of equal size", lambda: TwinModel(twin, device="cuda:0"))):
+    for label, build in ((name, lambda: Model(cfg, device="cuda:0")), ("other family at equal size" if to_twin is moe_attention_twin else "hybrid of equal size", lambda: TwinModel(twin, device="cuda:0"))):
         model = build().init_random(args.seed)
         model.SERIAL_PREFILL = True                  # the same launch mode for both
         rows = []
@@ -315,7 +336,7 @@ def main() -> None:
     ap.add_argument("--headline", default="auto", choices=["auto", "none"],
                     help="auto: after the scaling configuration also measure the headline configurations that fit this "
                          "number of GPUs (Llama-3.1-70B and the NVFP4 MoE at 8, the MoE at 2 and 4), 3 timed jobs each")
-    ap.add_argument("--compare", default="", choices=["", "dopurax-1b", "dopurax-8b", "kirisun-3b", "kirisun-10b"],
+    ap.add_argument("--compare", default="", choices=["", "dopurax-1b", "dopurax-8b", "kirisun-3b", "kirisun-10b", "sodotar-3b", "sodotar-10b"],
                     help="instead of the benchmark: prefill and decode throughput of this design beside the closest other family at equal "
                          "size, at a few batch shapes (1 GPU)")
     args = ap.parse_args()

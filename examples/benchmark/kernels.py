@@ -60,7 +60,7 @@ class Args:
     warmup: int = 3
     splits: int = 0          # decode_attention: KV chunks per sequence (0: the planner's choice)
     w4: int = 0              # moe: 1 = NVFP4 expert weights de-quantised inside the grouped GEMM
-    window: int = 4096       # latent and gated attention: keys a position sees
+    window: int = 4096       # latent and gated attention: keys a position sees; differential attention: its chunk
     copies: int = 0          # operand copies to rotate through (0: enough to exceed the L2)
     help = __doc__
 
@@ -342,6 +342,46 @@ def bench_gqa_decode(a: Args) -> None:
     report(a, ms, kvb, 4.0 * a.batch * a.hq * a.seqlen * a.hd, {"batch": a.batch, "seqlen": a.seqlen, "part": "the plain kernel"})
 
 
+def _diff(a: Args, n: int):
+    """Differential heads (two maps of hd / 2 over values of hd) that see their chunk of `window` tokens, with filled caches: a
+    key / value head takes the bytes of a plain one of size hd."""
+    from types import SimpleNamespace
+    from zml_b200.ops import gqa
+    s = gqa.GqaSpec(a.hq, a.hkv, a.hd // 2, a.hd, a.hd // 4, scale=(a.hd // 2) ** -0.5, chunk=a.window, maps=2)
+    caches, bt = _kv(a, n_copies(a, a.batch * a.seqlen * a.hkv * a.hd * 4) if n == 1 else 2)
+    t = a.batch * n
+    qs = (torch.arange(a.batch + 1, dtype=torch.int32, device="cuda") * n).int()
+    sl = torch.full((a.batch,), a.seqlen, dtype=torch.int32, device="cuda")
+    meta = SimpleNamespace(is_prefill=n > 1, q_start=qs, seq_lens=sl, block_table=bt, total_q_blocks=a.batch * ((n + 63) // 64),
+                           num_splits=a.splits or ops.decode_plan_splits(a.batch, a.hkv, s.visible(a.seqlen)), max_seq_len=a.seqlen)
+    proj = torch.randn(t, s.columns(), device="cuda").bfloat16()
+    slots = (torch.arange(t, dtype=torch.int32, device="cuda") + 64).int()
+    pos = (torch.arange(t, device="cuda") % a.seqlen).int()
+    freq = s.inv_freq("cuda")
+    prep = lambda c: gqa.prep(proj, None, None, freq, pos, slots, c, 1e-6, s)
+    return gqa, s, caches, meta, prep, gqa.DiffMix(0.3, 0.5, 1e-6), t
+
+
+def bench_diff_prefill(a: Args) -> None:
+    gqa, s, caches, meta, prep, mix, t = _diff(a, a.seqlen)
+    q = prep(caches[0])
+    shape = {"batch": a.batch, "seqlen": a.seqlen, "hq": a.hq, "hkv": a.hkv, "map": s.dim, "vdim": s.vdim, "chunk": s.chunk}
+    pairs = a.batch * sum(i % s.chunk + 1 for i in range(a.seqlen))
+    ms = timed([lambda c=c: gqa.attention(q, None, c, meta, s, mix) for c in caches], a.iters, a.warmup)
+    report(a, ms, (t * a.hq * 2 * a.hd + 2 * t * a.hkv * a.hd) * 2, 2.0 * pairs * s.rows_q * (s.dim + s.vdim), dict(shape, part="attention"))
+    ms = timed([lambda c=c: prep(c) for c in caches], a.iters, a.warmup)
+    report(a, ms, t * 2 * s.columns() * 2, 0, dict(shape, part="rotation, cache write"))
+
+
+def bench_diff_decode(a: Args) -> None:
+    gqa, s, caches, meta, prep, mix, t = _diff(a, 1)
+    q = prep(caches[0])
+    seen = (a.seqlen - 1) % s.chunk + 1
+    ms = timed_graph([lambda c=c: gqa.attention(q, None, c, meta, s, mix) for c in caches], a.iters, a.warmup)
+    report(a, ms, a.batch * seen * a.hkv * a.hd * 4, 2.0 * a.batch * seen * s.rows_q * (s.dim + s.vdim),
+           {"batch": a.batch, "seqlen": a.seqlen, "seen": seen, "splits": meta.num_splits, "hq": a.hq, "hkv": a.hkv, "map": s.dim, "vdim": s.vdim})
+
+
 def bench_channel_delta(a: Args) -> None:
     from zml_b200.ops import linear_attn as la
     H, D, t = a.hq, a.hd, a.batch * a.seqlen
@@ -391,6 +431,61 @@ def bench_mixture(a: Args) -> None:
     for part, fn in (("mixture", mine), ("other families", theirs)):
         ms = timed_graph([lambda w=w, fn=fn: fn(w) for w in ws], a.iters, a.warmup)
         report(a, ms, active * 3 * f * d * 2, 6.0 * t * k * f * d, {"part": part, "tokens": t, "experts": e, "top": k, "ff": f, "d": d})
+
+
+def bench_shared_mixture(a: Args) -> None:
+    """Router, routed and shared experts with clipped units, and the streams' update that sums their rows; the same sizes with the
+    routed mixture alone, and with the mixture, shared expert and norm of the Qwen3.5-MoE family."""
+    from zml_b200 import moe
+    from zml_b200.moe import ops as mops
+    from zml_b200.ops import stream
+    e, k, f, d, t = a.experts, a.topk, a.n, a.k, a.tokens
+    c = max(2, min(8, math.ceil(300e6 / (e * f * d * 6)) + 1))
+    rand = lambda *s: torch.randn(*s, device="cuda").bfloat16() * 0.02
+    ws = [mops.pad_experts(rand(e + 1, f, d), rand(e + 1, f, d), rand(e + 1, d, f)) for _ in range(c)]
+    router, sg = rand(e + 1, d), rand(8, d)
+    corr, limits = torch.zeros(e, device="cuda"), torch.full((e + 1,), 7.0, device="cuda")
+    h, res = torch.randn(t, d, device="cuda").bfloat16(), torch.randn(t, d, device="cuda").bfloat16()
+    x = torch.randn(t, 4, d, device="cuda")
+    nw, nb = torch.ones(d, device="cuda"), torch.ones(d, device="cuda").bfloat16()
+    hm = stream.HyperMix(torch.full((4,), 0.25, device="cuda"), torch.eye(4, device="cuda"), torch.ones(4, device="cuda"))
+    dense = [(torch.cat([rand(f, d), rand(f, d)], 0), rand(d, f)) for _ in range(c)]
+
+    def mine(i, shared, update=True):
+        w1, w2 = ws[i]
+        z = ops.gemm(h, router, out_dtype=torch.float32, static_w=True)
+        ids, wt = mops.route(z, k, e, corr, shared, 0)
+        s = 1 - shared
+        rows, pos = mops.expert_rows(h, ids, w1[s:], w2[s:], 0, e + shared, "clipped_glu", limits[s:])
+        return stream.hyper_norm(x, stream.ExpertRows(rows, pos, wt), hm, hm.inp, nw, 1e-6, torch.bfloat16) if update else rows
+
+    def theirs(i):
+        w1, w2 = ws[i]
+        z = ops.gemm(h, router[:e], out_dtype=torch.float32, static_w=True)
+        ids, wt = mops.router_topk(z, k)
+        y = ops.gemm(ops.swiglu(ops.gemm(h, dense[i][0], static_w=True)), dense[i][1], static_w=True)
+        gate = torch.sigmoid(ops.gemm(h, sg, out_dtype=torch.float32, static_w=True)[:, :1])
+        y = (y.float() * gate).to(y.dtype)
+        return ops.rmsnorm(moe.forward_moe(h, ids, wt, w1[1:], w2[1:], None, e, residual=res, extra_partial=y), nb)
+
+    active = min(e, t * k) + 1
+    for part, fn in (("mixture with shared expert, streams", lambda i: mine(i, 1)), ("the same without the streams", lambda i: mine(i, 1, False)),
+                     ("without the shared expert", lambda i: mine(i, 0)), ("other family, one stream", theirs)):
+        ms = timed_graph([lambda i=i, fn=fn: fn(i) for i in range(c)], a.iters, a.warmup)
+        report(a, ms, active * 3 * f * d * 2, 6.0 * t * (k + 1) * f * d, {"part": part, "tokens": t, "experts": e, "top": k, "ff": f, "d": d})
+
+
+def bench_hyper(a: Args) -> None:
+    """The streams' update behind a sublayer with the norm in front of the next one, beside the norms of a single stream."""
+    from zml_b200.ops import stream
+    t, d = a.tokens, a.k
+    y, w = torch.randn(t, d, device="cuda"), torch.ones(d, device="cuda")
+    for s in (1, 2, 4, 8):
+        hm = stream.HyperMix(torch.full((s,), 1.0 / s, device="cuda"), torch.eye(s, device="cuda"), torch.ones(s, device="cuda"))
+        xs = [torch.randn(t, s, d, device="cuda") for _ in range(max(2, min(64, math.ceil(256e6 / (t * d * s * 8)) + 1)))]
+        ms = timed_graph([lambda x=x: stream.hyper_norm(x, y, hm, hm.inp, w, 1e-6, torch.bfloat16) for x in xs], a.iters, a.warmup)
+        report(a, ms, t * d * (8 * s + 6), 0, {"part": "hyper_norm", "streams": s, "tokens": t, "d": d})
+        del xs
 
 
 def bench_stream(a: Args) -> None:
@@ -578,6 +673,7 @@ def bench_moe_w4_timeline(a: Args) -> None:
 OPS = {"moe_w4_timeline": bench_moe_w4_timeline, "gemm_chain_timeline": bench_gemm_chain_timeline, "gemm": bench_gemm, "decode_attention": bench_decode_attention, "prefill_attention": bench_prefill_attention,
        "moe": bench_moe, "gated_delta_scan": bench_gated_delta_scan, "decode_layers": bench_decode_layers,
        "latent_prefill": bench_latent_prefill, "latent_decode": bench_latent_decode, "wkv_scan": bench_wkv_scan, "stream": bench_stream,
+       "diff_prefill": bench_diff_prefill, "diff_decode": bench_diff_decode, "hyper": bench_hyper, "shared_mixture": bench_shared_mixture,
        "gqa_prefill": bench_gqa_prefill, "gqa_decode": bench_gqa_decode, "channel_delta": bench_channel_delta, "mixture": bench_mixture}
 
 

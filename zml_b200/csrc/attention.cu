@@ -107,7 +107,20 @@ struct AttnParams {
   int vdim;                     // value columns written per head; the output is [tokens, num_q_heads, vdim]
   const __nv_bfloat16* gate;    // [tokens, ldg]: output *= sigmoid(gate), or null
   long long ldg;
+  int chunk;                    // keys of the position's own chunk only, 0: off
+  int out_f32;                  // out is fp32
+  int pair;                     // decode: heads 2 h and 2 h + 1 are combined (ZbAttnExt)
+  float pair_lambda, pair_scale, pair_eps;
 };
+
+// First key in a position's window or chunk.
+template <bool EXT>
+ZB_DEVICE int attn_first_key(const AttnParams& p, int pos) {
+  if constexpr (EXT) {
+    if (p.chunk > 0) return max(0, pos) / p.chunk * p.chunk;
+  }
+  return p.window > 0 ? max(0, pos - p.window + 1) : 0;
+}
 
 // Score of a raw dot product in units of log2: scaled, and with a cap c * tanh(s * scale / c) as c * (1 - 2 / (1 + e^(2x))).
 template <bool EXT>
@@ -127,9 +140,33 @@ ZB_DEVICE void attn_store(const AttnParams& p, size_t tok, int head, int c, floa
       const float g = __bfloat162float(p.gate[tok * p.ldg + static_cast<size_t>(head) * p.vdim + c]);
       v *= __fdividef(1.f, 1.f + __expf(-g));
     }
-    p.out[(tok * p.num_q_heads + head) * p.vdim + c] = __float2bfloat16(v);
+    const size_t at = (tok * p.num_q_heads + head) * p.vdim + c;
+    if (p.out_f32) reinterpret_cast<float*>(p.out)[at] = v;
+    else p.out[at] = __float2bfloat16(v);
   } else {
     p.out[(tok * p.num_q_heads + head) * HD + c] = __float2bfloat16(v);
+  }
+}
+
+// The differential heads of one KV head out of their maps' results res [group][HD] in shared memory: one warp per head.
+template <int HD>
+ZB_DEVICE void attn_store_pairs(const AttnParams& p, const float* res, int seq, int kvh, int group) {
+  const int lane = threadIdx.x & 31, heads = group / 2;
+  for (int i = threadIdx.x >> 5; i < heads; i += blockDim.x >> 5) {
+    const float* a1 = res + 2 * i * HD;
+    const float* a2 = a1 + HD;
+    float o[HD / 32], ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < HD / 32; ++j) {
+      const int c = lane + 32 * j;
+      o[j] = c < p.vdim ? a1[c] - p.pair_lambda * a2[c] : 0.f;
+      ss = fmaf(o[j], o[j], ss);
+    }
+    const float f = p.pair_scale / sqrtf(zb_warp_sum(ss) / static_cast<float>(p.vdim) + p.pair_eps);
+    __nv_bfloat16* dst = p.out + (static_cast<size_t>(seq) * (p.num_q_heads / 2) + kvh * heads + i) * p.vdim;
+#pragma unroll
+    for (int j = 0; j < HD / 32; ++j)
+      if (lane + 32 * j < p.vdim) dst[lane + 32 * j] = __float2bfloat16(o[j] * f);
   }
 }
 
@@ -266,7 +303,8 @@ ZB_DEVICE void decode_tail(const AttnParams& p, uint8_t* smem, const float (&o)[
     const int head = kvh * group + r;
     if (my_splits == 1) {
       const float inv = ll > 0.f ? 1.f / ll : 0.f;
-      attn_store<HD, EXT>(p, seq, head, c, acc * inv);
+      if (EXT && p.pair) sm_o[idx] = acc * inv;                 // nobody else reads this element (warp 0's) any more
+      else attn_store<HD, EXT>(p, seq, head, c, acc * inv);
     } else {
       const size_t pi = (static_cast<size_t>(seq) * p.num_q_heads + head) * p.num_splits + split;
       p.part_o[pi * HD + c] = acc;
@@ -276,7 +314,15 @@ ZB_DEVICE void decode_tail(const AttnParams& p, uint8_t* smem, const float (&o)[
       }
     }
   }
-  if (my_splits == 1) return;
+  if (my_splits == 1) {
+    if constexpr (EXT) {
+      if (p.pair) {
+        __syncthreads();
+        attn_store_pairs<HD>(p, sm_o, seq, kvh, group);
+      }
+    }
+    return;
+  }
   // the last chunk to finish merges all chunks of this (sequence, kv head)
   __shared__ uint32_t s_last;
   __threadfence();
@@ -294,6 +340,7 @@ ZB_DEVICE void decode_tail(const AttnParams& p, uint8_t* smem, const float (&o)[
   // batched eight at a time, so that the merge costs a few round trips, not one per chunk.
   float* s_m = reinterpret_cast<float*>(smem);          // [group][my_splits]
   float* s_l = s_m + 16 * 64;                           // [group][my_splits] (at most 16 rows x 64 chunks)
+  float* s_res = s_l + 16 * 64;                         // [group][HD] results of the maps to combine
   const int nsp = min(my_splits, 64);
   for (int i = threadIdx.x; i < group * nsp; i += blockDim.x) {
     const int r = i / nsp, sp = i - r * nsp;
@@ -324,7 +371,15 @@ ZB_DEVICE void decode_tail(const AttnParams& p, uint8_t* smem, const float (&o)[
         }
       }
     }
-    attn_store<HD, EXT>(p, seq, head, c, ll > 0.f ? acc / ll : 0.f);
+    const float v = ll > 0.f ? acc / ll : 0.f;
+    if (EXT && p.pair) s_res[idx] = v;
+    else attn_store<HD, EXT>(p, seq, head, c, v);
+  }
+  if constexpr (EXT) {
+    if (p.pair) {
+      __syncthreads();
+      attn_store_pairs<HD>(p, s_res, seq, kvh, group);
+    }
   }
 }
 
@@ -345,7 +400,7 @@ __global__ void __launch_bounds__(128) zb_paged_decode_kernel(const AttnParams p
   const int split = blockIdx.y;
   const int group = p.num_q_heads / p.num_kv_heads;
   const int len = p.seq_lens[seq];
-  const int first_visible = p.window > 0 ? max(0, len - p.window) : 0;
+  const int first_visible = attn_first_key<EXT>(p, len - 1);
   ZbTileList tiles = {0, 0, (len + 15) >> 4};
   if constexpr (EXT) tiles = zb_visible_tiles(first_visible, p.keep, tiles.count, 16);
   const int nblk = tiles.count;
@@ -478,7 +533,7 @@ __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_c
   const int split = blockIdx.y;
   const int group = p.num_q_heads / p.num_kv_heads;
   const int len = p.seq_lens[seq];
-  const int first_visible = p.window > 0 ? max(0, len - p.window) : 0;
+  const int first_visible = attn_first_key<EXT>(p, len - 1);
   ZbTileList tiles = {0, 0, (len + 63) >> 6};
   if constexpr (EXT) tiles = zb_visible_tiles(first_visible, p.keep, tiles.count, 64);
   const int nblk = EXT ? tiles.count * 4 : (len + 15) >> 4;
@@ -610,7 +665,7 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
   const int tok_base = p.q_start[seq] + row_base;     // its token index
   const int rows_valid = min(64, q_len - row_base);
   const int last_key = min(len, ctx + row_base + 64);  // exclusive
-  const int first_key = p.window > 0 ? max(0, ctx + row_base - p.window + 1) : 0;
+  const int first_key = attn_first_key<EXT>(p, ctx + row_base);
   const ZbTileList tiles = zb_visible_tiles(first_key, EXT ? p.keep : 0, (last_key + 63) >> 6, 64);
 
   const uint32_t q_s = zb_smem_u32(smem);
@@ -653,6 +708,7 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
   if (EXT && p.sink) m[0] = m[1] = 0.f, l[0] = l[1] = 1.f;
   const int g = lane >> 2;
   const int qpos0 = ctx + row_base + warp * 16 + g;   // key position limit of row g (row g+8: +8)
+  const int from[2] = {attn_first_key<EXT>(p, qpos0), attn_first_key<EXT>(p, qpos0 + 8)};
 
   for (int it = 0; it < tiles.count; ++it) {
     const int tile = tiles.at(it), stage = it & 1;
@@ -679,9 +735,8 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
       attn_block16<HD, 0>(qf, ks, vs, sub * 16, o, m, l, [&](float v) { return attn_score<EXT>(p, v); }, [&](int half, int col) {
         const int kidx = key0 + col;
         const int qp = qpos0 + half * 8;
-        bool vis = kidx <= qp && kidx < len;
-        if (p.window > 0) vis = vis && (kidx > qp - p.window || (EXT && kidx < p.keep));
-        return vis;
+        const bool vis = kidx <= qp && kidx < len;
+        return vis && (kidx >= from[half] || (EXT && kidx < p.keep));
       });
     }
   }
@@ -782,6 +837,12 @@ void set_ext(AttnParams& p, const ZbAttnExt& x, float scale) {
   p.vdim = x.vdim;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(x.gate);
   p.ldg = x.ldg;
+  p.chunk = x.chunk;
+  p.out_f32 = x.out_f32;
+  p.pair = x.pair;
+  p.pair_lambda = x.pair_lambda;
+  p.pair_scale = x.pair_scale;
+  p.pair_eps = x.pair_eps;
 }
 
 }  // namespace
@@ -853,9 +914,11 @@ int zb_paged_decode_ex(const void* q, const void* k_cache, const void* v_cache, 
     --num_splits;
   // chunk length that lets `num_splits` chunks cover the longest sequence the block table allows
   int max_blocks = (max_pages * page_size + 15) / 16;
-  if (ext != nullptr && window > 0) {          // the longest list of visible tiles: the kept ones and a window that starts inside a tile
+  if (ext != nullptr && ext->pair != 0 && ((num_q_heads / num_kv_heads) % 2 != 0 || ext->gate != nullptr || ext->out_f32 != 0)) return -35;
+  if (ext != nullptr && (window > 0 || ext->chunk > 0)) {      // the longest list of visible tiles: the kept ones and a window that starts inside a tile
     const int tile = page_size == 64 ? 64 : 16;
-    const int visible = ((ext->keep + tile - 1) / tile + (window + tile - 2) / tile + 1) * (tile / 16);
+    const int span = ext->chunk > 0 ? ext->chunk : window;
+    const int visible = ((ext->keep + tile - 1) / tile + (span + tile - 2) / tile + 1) * (tile / 16);
     if (visible < max_blocks) max_blocks = visible;
   }
   int chunk_blocks = (max_blocks + num_splits - 1) / num_splits;
@@ -934,6 +997,7 @@ int zb_paged_prefill(const void* q, const void* k_cache, const void* v_cache, vo
   p.status = st->status;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (ext == nullptr) return dispatch_prefill<false>(p, head_dim, total_q_blocks, s);
+  if (ext->pair != 0) return -35;                 // the caller combines the maps (zb_pair_combine)
   set_ext(p, *ext, scale);
   return dispatch_prefill<true>(p, head_dim, total_q_blocks, s);
 }

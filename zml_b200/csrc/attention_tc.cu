@@ -18,9 +18,13 @@
 // P = exp2(S - m) as bf16 straight back into tensor memory -> O += P V (A = P from tensor memory,
 // B = V from shared memory in its natural [key][head_dim] layout, i.e. MN-major).
 // Tensor memory columns: S_A 0-63 | S_B 64-127 | P_A 128-159 | P_B 160-191 | O_A 192-319 | O_B 320-447.
-// With a score cap c (EXT; at most kMaxCap) the running maximum goes: every score lies in [-c, c], so P = exp2(S') needs no
-// reference and O no rescaling.  Kept first keys join the window's tiles as one list, a sink is one more term of the sum,
-// and the output gate is applied as the rows are stored.
+// Three instantiations: kPlain; with what ZbAttnExt adds (kExt); and that with a score cap c of at most kMaxCap (kCapped),
+// where the running maximum goes: every score lies in [-c, c], so P = exp2(S') needs no reference and O no rescaling.  Kept
+// first keys join the window's tiles as one list, a chunk is a window whose start is the same for all its positions, a sink
+// is one more term of the sum, and the output gate is applied as the rows are stored.
+// Differential heads (ZbAttnExt.pair, kExt): the two pipelines are the two maps of one head.  A map's keys are one 64-column
+// sub-tile of the cached key, so its scores take half the products; at the end both warpgroups read both accumulators, the
+// upper and the lower 64 columns each, and exchange row sums and partial sums of squares through shared memory.
 // Every wait is bounded; a wait that runs out records a status and the CTA leaves through its normal exit.
 #include <cuda.h>
 
@@ -47,6 +51,7 @@ constexpr float kMaxCap = 60.f;                    // exp(cap) times the number 
 constexpr float kPolyMax = 0.6f;
 __device__ constexpr float kTanh[6] = {1.0f, -0.333332837f, 0.1333168f, -0.0537679829f, 0.0207513496f, -0.00584964408f};
 constexpr uint32_t kColS = 0, kColP = 128, kColO = 192;
+enum Mode { kPlain, kCapped, kExt };
 
 struct PrefillTcParams {
   __nv_bfloat16* out;           // [tokens, num_q_heads, 128]
@@ -62,8 +67,9 @@ struct PrefillTcParams {
   uint32_t v_lbo;               // byte offsets of the MN-major descriptor of V (between 64-column groups / 8-key groups)
   uint32_t v_sbo;
   ZbStatus* status;
-  // EXT only (ZbAttnExt)
+  // not kPlain (ZbAttnExt)
   int keep;
+  int chunk;
   float cap_log2;               // cap * log2(e)
   float cap_in;                 // 2 * scale * log2(e) / cap
   float cap_x;                  // scale / cap
@@ -71,11 +77,25 @@ struct PrefillTcParams {
   int vdim;                     // output [tokens, num_q_heads, vdim]
   const __nv_bfloat16* gate;    // [tokens, ldg] or null
   long long ldg;
+  int pair;                     // kExt
+  float pair_lambda, pair_scale, pair_eps;
 };
+
+// First key in a position's window or chunk.
+template <bool EXT>
+ZB_DEVICE int first_key_of(const PrefillTcParams& p, int pos) {
+  if constexpr (EXT) {
+    if (p.chunk > 0) return pos / p.chunk * p.chunk;
+  }
+  return p.window > 0 ? max(0, pos - p.window + 1) : 0;
+}
 
 ZB_DEVICE void wg_bar_sync(int wg) {
   asm volatile("bar.sync %0, 128;" ::"r"(1 + wg) : "memory");
 }
+
+// Both softmax warpgroups.
+ZB_DEVICE void pair_bar_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
 // Eight output values of one row at column c: gated, and cut at vdim.
 ZB_DEVICE void store_ext8(const PrefillTcParams& p, size_t tok, int head, int c, const uint32_t* o, float inv) {
@@ -117,10 +137,13 @@ ZB_DEVICE void store_ext8(const PrefillTcParams& p, size_t tok, int head, int c,
   }
 }
 
-template <bool EXT>
+template <Mode MODE>
 __global__ void __launch_bounds__(kThreads, 1)
 zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                            const __grid_constant__ CUtensorMap tmap_v, const PrefillTcParams p) {
+  constexpr bool EXT = MODE != kPlain;
+  const bool pair = MODE == kExt && p.pair != 0;
+  __shared__ float pair_x[4][kQRows];                // differential heads: 1 / row sum of either map, partial sums of squares
   zb_pdl_launch();
   zb_pdl_wait();                                     // q, the KV cache and the batch description come from preceding work
   extern __shared__ uint8_t smem_raw[];
@@ -169,7 +192,7 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
   const int tok_base = p.q_start[seq] + row_base;
   const int rows_valid = min(kQRows, q_len - row_base);
   const int last_key = min(len, ctx + row_base + kQRows);     // exclusive
-  const int first_key = p.window > 0 ? max(0, ctx + row_base - p.window + 1) : 0;
+  const int first_key = first_key_of<EXT>(p, ctx + row_base);
   const ZbTileList tiles = zb_visible_tiles(first_key, EXT ? p.keep : 0, (last_key + kKeys - 1) / kKeys, kKeys);
   const int n_tiles = tiles.count;
 
@@ -204,10 +227,11 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
   if (warp == 8) {
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
-      zb_mbar_expect_tx(q_full, 2 * kQBytes);
+      zb_mbar_expect_tx(q_full, pair ? kQBytes : 2 * kQBytes);
       for (int w = 0; w < 2; ++w)
         for (int c = 0; c < 2; ++c)
-          zb_tma_load_2d(q_s + w * kQBytes + c * (kQRows * 128), &tmap_q, q_full, (head0 + w) * kHD + c * 64, tok_base);
+          if (!pair || c == w)
+            zb_tma_load_2d(q_s + w * kQBytes + c * (kQRows * 128), &tmap_q, q_full, (head0 + w) * kHD + c * 64, tok_base);
       const int32_t* bt = p.block_table + static_cast<size_t>(seq) * p.max_pages;
       uint32_t stage = 0, phase = 0;
       for (int j = 0; j < n_tiles; ++j) {
@@ -241,10 +265,11 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
         const uint32_t qa = zb_smem_u32(q_s + w * kQBytes), ka = zb_smem_u32(k_s + st * kKvBytes);
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
+          if (pair && c != w) continue;
           const uint64_t dq = zb_make_desc_sw128(qa + c * (kQRows * 128)), dk = zb_make_desc_sw128(ka + c * (kKeys * 128));
 #pragma unroll
           for (int kk = 0; kk < 4; ++kk)
-            zb_umma_f16(tmem_base + kColS + w * kKeys, dq + 2 * kk, dk + 2 * kk, kIdescS, (c > 0 || kk > 0) ? 1u : 0u);
+            zb_umma_f16(tmem_base + kColS + w * kKeys, dq + 2 * kk, dk + 2 * kk, kIdescS, ((c > 0 && !pair) || kk > 0) ? 1u : 0u);
         }
         zb_umma_commit(&s_full[w]);
       };
@@ -312,7 +337,8 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
     const uint32_t t_s = tmem_base + kColS + w * kKeys + lane_off;
     const uint32_t t_p = tmem_base + kColP + w * 32 + lane_off;
     const uint32_t t_o = tmem_base + kColO + w * kHD + lane_off;
-    float m = -INFINITY, l = EXT && p.sink ? 1.f : 0.f;
+    float m = MODE == kExt && p.sink ? 0.f : -INFINITY, l = EXT && p.sink ? 1.f : 0.f;
+    const int from = first_key_of<EXT>(p, qpos), from_last = first_key_of<EXT>(p, ctx + row_base + kQRows - 1);
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
       const uint32_t jj = static_cast<uint32_t>(j);
@@ -329,11 +355,10 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       const int key0 = tiles.at(j) * kKeys;
       // pages below the block's first row and inside every row's window need no mask (a branch per page, not a
       // predicate per score: predicated-off instructions still take issue slots, and this loop is issue-bound)
-      const bool full = (key0 + kKeys - 1 <= ctx + row_base) && (key0 + kKeys <= len) &&
-                        (p.window <= 0 || key0 > ctx + row_base + kQRows - 1 - p.window);
+      const bool full = (key0 + kKeys - 1 <= ctx + row_base) && (key0 + kKeys <= len) && key0 >= from_last;
       uint32_t pw[32];
       float sum0 = 0.f, sum1 = 0.f;
-      if constexpr (EXT) {
+      if constexpr (MODE == kCapped) {
         // The capped score in units of log2, over sr: with x = s * scale / c, where a warp's scores are small tanh(x) / x as a
         // polynomial in x^2, else c - 2 c / (1 + e^(2x)).
         float mx = 0.f;
@@ -362,7 +387,7 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
 #pragma unroll
           for (int i = 0; i < 64; ++i) {
             const int kidx = key0 + i;
-            const bool vis = kidx <= qpos && kidx < len && (p.window <= 0 || kidx > qpos - p.window || kidx < p.keep);
+            const bool vis = kidx <= qpos && kidx < len && (kidx >= from || kidx < p.keep);
             if (!vis) sr[i] = 0xff800000u;           // -inf
           }
         }
@@ -383,19 +408,18 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
 #pragma unroll
           for (int i = 0; i < 64; ++i) {
             const int kidx = key0 + i;
-            bool vis = kidx <= qpos && kidx < len;
-            if (p.window > 0) vis = vis && (kidx > qpos - p.window);
+            const bool vis = kidx <= qpos && kidx < len && (kidx >= from || (EXT && kidx < p.keep));
             if (!vis) sr[i] = 0xff800000u;             // -inf
             mx_raw = fmaxf(mx_raw, __uint_as_float(sr[i]));
           }
         }
         const float mx = fmaxf(m, mx_raw * p.scale_log2);           // running maximum, in units of log2
         const float m_use = mx == -INFINITY ? 0.f : mx;             // a row without a visible key so far
-        if (jj > 0) {
+        {
           // the output accumulated so far is relative to the old maximum: rescale it where the maximum moved
           const float alpha = m == -INFINITY ? 1.f : zb_ex2(m - m_use);
           const bool moved = alpha != 1.f;
-          if (__any_sync(0xffffffffu, moved)) {
+          if (jj > 0 && __any_sync(0xffffffffu, moved)) {
             if (!zb_mbar_wait(&o_ready[w], (jj - 1u) & 1u, abort_flag)) {      // O += P V of the previous page is done
               *abort_where = 12u + w;
               ok = false;
@@ -435,7 +459,51 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       zb_tc_fence_before();
       zb_mbar_arrive(&p_full[w]);
     }
-    if (ok && n_tiles > 0) {
+    if (pair) {
+      // every thread of both warpgroups passes both barriers, whatever its waits said
+      const uint32_t last = static_cast<uint32_t>(n_tiles - 1);
+      ok = ok && n_tiles > 0;
+      if (ok && !(zb_mbar_wait(&o_ready[0], last & 1u, abort_flag) && zb_mbar_wait(&o_ready[1], last & 1u, abort_flag))) {
+        *abort_where = 14u + w;
+        ok = false;
+      }
+      zb_tc_fence_after();
+      pair_x[w][r] = l > 0.f ? 1.f / l : 0.f;
+      pair_bar_sync();
+      const float inv1 = pair_x[0][r], inv2 = p.pair_lambda * pair_x[1][r];
+      float v[64], ss = 0.f;
+      const uint32_t t_o1 = tmem_base + kColO + w * 64 + lane_off, t_o2 = t_o1 + kHD;
+#pragma unroll
+      for (int c0 = 0; c0 < 64; c0 += 32) {
+        uint32_t o1[32], o2[32];
+        zb_tmem_ld32(t_o1 + c0, o1);
+        zb_tmem_ld32(t_o2 + c0, o2);
+        zb_tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          v[c0 + i] = fmaf(-inv2, __uint_as_float(o2[i]), __uint_as_float(o1[i]) * inv1);
+          if (w * 64 + c0 + i < p.vdim) ss = fmaf(v[c0 + i], v[c0 + i], ss);
+        }
+      }
+      pair_x[2 + w][r] = ss;
+      pair_bar_sync();
+      const float f = p.pair_scale / sqrtf((pair_x[2][r] + pair_x[3][r]) / static_cast<float>(p.vdim) + p.pair_eps);
+      if (ok && r < rows_valid) {
+        const int c1 = w * 64;
+        __nv_bfloat16* dst = p.out + (static_cast<size_t>(tok_base + r) * (p.num_q_heads / 2) + head0 / 2) * p.vdim + c1;
+        if ((p.vdim & 7) == 0) {
+#pragma unroll
+          for (int i = 0; i < 64; i += 8)
+            if (c1 + i < p.vdim)
+              *reinterpret_cast<uint4*>(dst + i) = make_uint4(zb_pack_bf16x2(v[i] * f, v[i + 1] * f), zb_pack_bf16x2(v[i + 2] * f, v[i + 3] * f),
+                                                              zb_pack_bf16x2(v[i + 4] * f, v[i + 5] * f), zb_pack_bf16x2(v[i + 6] * f, v[i + 7] * f));
+        } else {
+#pragma unroll
+          for (int i = 0; i < 64; ++i)
+            if (c1 + i < p.vdim) dst[i] = __float2bfloat16(v[i] * f);
+        }
+      }
+    } else if (ok && n_tiles > 0) {
       const uint32_t last = static_cast<uint32_t>(n_tiles - 1);
       if (zb_mbar_wait(&o_ready[w], last & 1u, abort_flag)) {
         zb_tc_fence_after();
@@ -501,8 +569,8 @@ int zb_paged_prefill_tc_supported(int num_q_heads, int num_kv_heads, int head_di
   return ((num_q_heads / num_kv_heads) % 2) == 0 ? 1 : 0;
 }
 
-// 1 when the kernel takes a call with ZbAttnExt: it needs a cap whose exponential fp32 holds.
-int zb_paged_prefill_tc_ext_supported(float cap) { return cap > 0.f && cap <= kMaxCap ? 1 : 0; }
+// 1 when the kernel takes a call with ZbAttnExt: no cap, or one whose exponential fp32 holds; differential heads without a cap.
+int zb_paged_prefill_tc_ext_supported(float cap, int pair) { return cap == 0.f || (cap > 0.f && cap <= kMaxCap && pair == 0) ? 1 : 0; }
 
 // Same contract as zb_paged_prefill.  total_q_blocks128 >= sum over sequences of ceil(q_len / 128).
 // `v_lbo` / `v_sbo` = 0 select the defaults of the V descriptor (8192 / 1024 bytes).
@@ -514,11 +582,12 @@ int zb_paged_prefill_tc(const void* q, const void* k_cache, const void* v_cache,
   if (!zb_paged_prefill_tc_supported(num_q_heads, num_kv_heads, kHD, kKeys)) return -32;
   ZbDeviceState* st = zb_device_state();
   if (!st) return -20;
-  if (ext != nullptr && !zb_paged_prefill_tc_ext_supported(ext->cap)) return -34;
-  static bool configured[2][16] = {};
-  if (const int rc = ext != nullptr ? zb_config_smem_once(zb_paged_prefill_tc_kernel<true>, kSmemBytes, configured[1])
-                                    : zb_config_smem_once(zb_paged_prefill_tc_kernel<false>, kSmemBytes, configured[0]))
-    return rc;
+  if (ext != nullptr && (!zb_paged_prefill_tc_ext_supported(ext->cap, ext->pair) || ext->out_f32 != 0 || (ext->pair != 0 && ext->gate != nullptr)))
+    return -34;
+  static bool configured[3][16] = {};
+  const Mode mode = ext == nullptr ? kPlain : (ext->cap > 0.f ? kCapped : kExt);
+  const auto kernel = mode == kPlain ? zb_paged_prefill_tc_kernel<kPlain> : (mode == kCapped ? zb_paged_prefill_tc_kernel<kCapped> : zb_paged_prefill_tc_kernel<kExt>);
+  if (const int rc = zb_config_smem_once(kernel, kSmemBytes, configured[mode])) return rc;
   CUtensorMap tq, tk, tv;
   // q as a [tokens, heads * 128] matrix with leading dimension q_stride: boxes of 128 rows x 64 columns
   int rc = zb_make_tmap_bf16_2d(&tq, q, total_tokens, num_q_heads * kHD, static_cast<int>(q_stride), kQRows);
@@ -544,16 +613,22 @@ int zb_paged_prefill_tc(const void* q, const void* k_cache, const void* v_cache,
   p.status = st->status;
   if (ext != nullptr) {
     p.keep = ext->keep;
-    p.cap_log2 = ext->cap * 1.4426950408889634f;
-    p.cap_in = 2.f * scale * 1.4426950408889634f / ext->cap;
-    p.cap_x = scale / ext->cap;
+    p.chunk = ext->chunk;
+    if (ext->cap > 0.f) {
+      p.cap_log2 = ext->cap * 1.4426950408889634f;
+      p.cap_in = 2.f * scale * 1.4426950408889634f / ext->cap;
+      p.cap_x = scale / ext->cap;
+    }
+    p.pair = ext->pair;
+    p.pair_lambda = ext->pair_lambda;
+    p.pair_scale = ext->pair_scale;
+    p.pair_eps = ext->pair_eps;
     p.sink = ext->sink;
     p.vdim = ext->vdim;
     p.gate = reinterpret_cast<const __nv_bfloat16*>(ext->gate);
     p.ldg = ext->ldg;
   }
-  const cudaError_t le = zb_launch(ext != nullptr ? zb_paged_prefill_tc_kernel<true> : zb_paged_prefill_tc_kernel<false>,
-                                   dim3(total_q_blocks128, num_q_heads / 2), dim3(kThreads), kSmemBytes,
+  const cudaError_t le = zb_launch(kernel, dim3(total_q_blocks128, num_q_heads / 2), dim3(kThreads), kSmemBytes,
                                    reinterpret_cast<cudaStream_t>(stream), tq, tk, tv, p);
   zb_count_launch(1);
   return static_cast<int>(le != cudaSuccess ? le : cudaGetLastError());

@@ -468,8 +468,10 @@ __host__ __device__ constexpr uint32_t zb_make_idesc_bf16(uint32_t m, uint32_t n
 // Activations of the expert MLPs (the reference's zml/moe/cutlass_flashinfer.zig:24-28).  The grouped GEMMs take
 // the code in their `swiglu` argument: 0 none, 1 swiglu (silu(gate) * up), 2 geglu (erf GELU), 3 geglu_tanh,
 // 4 relu2 (not gated: relu(x)^2 on a plain projection).
-enum ZbMoeAct : int { ZB_ACT_NONE = 0, ZB_ACT_SWIGLU = 1, ZB_ACT_GEGLU = 2, ZB_ACT_GEGLU_TANH = 3, ZB_ACT_RELU2 = 4 };
-ZB_DEVICE bool zb_act_is_gated(int act) { return act >= ZB_ACT_SWIGLU && act <= ZB_ACT_GEGLU_TANH; }
+enum ZbMoeAct : int { ZB_ACT_NONE = 0, ZB_ACT_SWIGLU = 1, ZB_ACT_GEGLU = 2, ZB_ACT_GEGLU_TANH = 3, ZB_ACT_RELU2 = 4, ZB_ACT_CLIPPED_GLU = 5 };
+__host__ __device__ constexpr bool zb_act_is_gated(int act) {
+  return (act >= ZB_ACT_SWIGLU && act <= ZB_ACT_GEGLU_TANH) || act == ZB_ACT_CLIPPED_GLU;
+}
 ZB_DEVICE float zb_gate_act(float g, int act) {
   if (act == ZB_ACT_GEGLU) return 0.5f * g * (1.f + erff(g * 0.70710678118654752f));
   if (act == ZB_ACT_GEGLU_TANH) {
@@ -477,6 +479,18 @@ ZB_DEVICE float zb_gate_act(float g, int act) {
     return 0.5f * g * (1.f + tanhf(u));
   }
   return g / (1.f + __expf(-g));
+}
+// Clipped gated unit: with g = min(gate, limit) and u = up cut to [-limit, limit], g * sigmoid(1.702 g) * (u + 1).
+template <bool EXACT>
+ZB_DEVICE float zb_clipped_glu(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  const float e = EXACT ? expf(-1.702f * g) : __expf(-1.702f * g);
+  return g / (1.f + e) * (u + 1.f);
+}
+// Any gated activation; `limit` is read by ZB_ACT_CLIPPED_GLU only.
+ZB_DEVICE float zb_gated(float g, float u, int act, float limit) {
+  return act == ZB_ACT_CLIPPED_GLU ? zb_clipped_glu<false>(g, u, limit) : zb_gate_act(g, act) * u;
 }
 ZB_DEVICE float zb_plain_act(float x, int act) {
   if (act == ZB_ACT_RELU2) {

@@ -1,13 +1,16 @@
-// Grouped-query attention whose heads are normalised, partly rotated, soft-capped, windowed with kept first tokens, sunk and
-// gated (any of these may be off), with key and value sizes of their own, bf16 or fp32:
+// Grouped-query attention whose heads are normalised, partly rotated, soft-capped, windowed with kept first tokens or chunked,
+// sunk and gated (any of these may be off), with key and value sizes of their own and one or two maps per head, bf16 or fp32:
 //
 //   zb_gqa_prep     per head RMS norm of q and k, rotation of the first `rot` dimensions (pairs (i, i + rot / 2)), cache write
 //                   of k and v.  Heads are written with a padded stride (zeros behind their elements), so that the
-//                   tensor-core kernels of attention.cu / attention_tc.cu take any size up to theirs
+//                   tensor-core kernels of attention.cu / attention_tc.cu take any size up to theirs.  With two maps a cached
+//                   key is [map 1 | map 2], and a head has two query rows, each zero where the other map's keys are
 //   zb_gqa_attend   attention over the paged cache for any sizes: the fp32 path and the fall-back for sizes the tensor-core
 //                   kernels do not take
+//   zb_pair_combine differential attention: the two maps' results a1, a2 of every head -> a1 - lambda a2 at unit root mean
+//                   square, times a constant (the kernels of attention.cu and attention_tc.cu do it as they store)
 //
-// Position i sees j when j <= i and (i - j < window or j < keep).  score = q . k * scale, then cap * tanh(score / cap); with
+// Position i sees j when j <= i and (i - j < window or j < keep), or with chunks when floor(i / chunk) = floor(j / chunk).  score = q . k * scale, then cap * tanh(score / cap); with
 // a sink the softmax denominator has an additional exp(0).  Norms, angles, scores and softmax are fp32.
 #include "act.cuh"
 #include "host_api.h"
@@ -19,8 +22,8 @@ constexpr uint32_t kKernelGqaAttend = 35;
 struct GqaPrepArgs {
   const void* in;            // [T, ld_in]: q heads | k heads | v heads
   long long ld_in;
-  const float* q_norm;       // [dk]
-  const float* k_norm;       // [dk]
+  const float* q_norm;       // [dk], or null: no norm
+  const float* k_norm;
   const float* inv_freq;     // [rot / 2]
   const int32_t* positions;
   const int32_t* slots;      // cache row of every token, negative: no write
@@ -29,8 +32,9 @@ struct GqaPrepArgs {
   void* v_cache;             // [rows, hkv, ldv]
   long long num_rows;
   float eps;
-  int hq, hkv, dk, dv, rot;
-  int ldq, ldk, ldv;         // elements per head where it is written
+  int hq, hkv, dk, dv, rot;  // hq: query rows, maps of a head counted one by one; hkv 0: queries only
+  int maps;
+  int ldq, ldk, ldv;         // elements per row where it is written
 };
 
 template <int V>
@@ -85,15 +89,17 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
   if (slot >= p.num_rows) (void)ZB_BC_OK(slot, p.num_rows, kKernelGqaPrep, 1);
   const bool slot_ok = slot >= 0 && slot < p.num_rows;
   const A* in = reinterpret_cast<const A*>(p.in) + t * p.ld_in;
-  const int heads = p.hq + 2 * p.hkv;
+  const int keys = p.hkv * p.maps, heads = p.hq + keys + p.hkv;
   for (int h = warp; h < heads; h += kPrepThreads / 32) {
-    const bool is_q = h < p.hq, is_v = h >= p.hq + p.hkv;
+    const bool is_q = h < p.hq, is_v = h >= p.hq + keys;
     if (!is_q && !slot_ok) continue;
-    const int g = is_q ? h : (is_v ? h - p.hq - p.hkv : h - p.hq);
-    const int n = is_v ? p.dv : p.dk, ld = is_q ? p.ldq : (is_v ? p.ldv : p.ldk);
-    const A* src = in + (is_v ? (p.hq + p.hkv) * p.dk + g * p.dv : h * p.dk);
-    A* dst = is_q ? reinterpret_cast<A*>(p.q) + (static_cast<long long>(t) * p.hq + g) * ld
-                  : reinterpret_cast<A*>(is_v ? p.v_cache : p.k_cache) + (slot * p.hkv + g) * ld;
+    const int u = is_q ? h : (is_v ? h - p.hq - keys : h - p.hq);        // row among its kind
+    const int map = is_v ? 0 : u % p.maps;
+    const int n = is_v ? p.dv : p.dk, ld = is_v ? p.ldv : (is_q ? p.ldq : p.ldk) / p.maps;
+    const A* src = in + (is_v ? (p.hq + keys) * p.dk + u * p.dv : h * p.dk);
+    A* dst = is_q ? reinterpret_cast<A*>(p.q) + (static_cast<long long>(t) * p.hq + u) * p.ldq + map * ld
+                  : (is_v ? reinterpret_cast<A*>(p.v_cache) + (slot * p.hkv + u) * p.ldv
+                          : reinterpret_cast<A*>(p.k_cache) + (slot * p.hkv + u / p.maps) * p.ldk + map * ld);
     float v[NR][V];
     float ss = 0.f;
 #pragma unroll
@@ -106,8 +112,8 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
       for (int e = 0; e < V; ++e) ss = fmaf(v[r][e], v[r][e], ss);
     }
     if (!is_v) {
-      const float inv = 1.f / sqrtf(zb_warp_sum(ss) / static_cast<float>(n) + p.eps);
       const float* nw = is_q ? p.q_norm : p.k_norm;
+      const float inv = nw != nullptr ? 1.f / sqrtf(zb_warp_sum(ss) / static_cast<float>(n) + p.eps) : 1.f;
       __syncwarp();
 #pragma unroll
       for (int r = 0; r < NR; ++r) {
@@ -115,7 +121,7 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
         if (i >= n) continue;
 #pragma unroll
         for (int e = 0; e < V; ++e) {
-          v[r][e] *= inv * nw[i + e];
+          if (nw != nullptr) v[r][e] *= inv * nw[i + e];
           if (i + e < p.rot) row[i + e] = v[r][e];
         }
       }
@@ -137,14 +143,19 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
 #pragma unroll
     for (int r = 0; r < NR; ++r) {
       const int i = (lane + 32 * r) * V;
-      if (i < ld) st_elems<V>(dst + i, v[r]);             // elements n .. ld are zero
+      if (i >= ld) continue;
+      st_elems<V>(dst + i, v[r]);                          // elements n .. ld are zero
+      if (is_q && p.maps == 2) {
+        const float zero[V] = {};
+        st_elems<V>(dst + i + (map == 0 ? ld : -ld), zero);
+      }
     }
   }
 }
 
 template <typename A, int V>
 cudaError_t launch_prep(const GqaPrepArgs& p, int tokens, cudaStream_t s) {
-  const int widest = max(max(p.ldq, p.ldk), p.ldv);
+  const int widest = max(max(p.ldq, p.hkv > 0 ? p.ldk : 0) / p.maps, p.hkv > 0 ? p.ldv : 0);
   const size_t smem = static_cast<size_t>(p.rot) * (1 + kPrepThreads / 32) * sizeof(float);
   if (smem > 48 * 1024) return cudaErrorInvalidValue;
   const int nr = (widest + 32 * V - 1) / (32 * V);
@@ -156,7 +167,7 @@ cudaError_t launch_prep(const GqaPrepArgs& p, int tokens, cudaStream_t s) {
 }
 template <typename A>
 cudaError_t launch_prep(const GqaPrepArgs& p, int tokens, cudaStream_t s) {
-  const bool vec = p.dk % 4 == 0 && p.dv % 4 == 0 && p.ld_in % 4 == 0 && p.ldq % 4 == 0 && p.ldk % 4 == 0 && p.ldv % 4 == 0 &&
+  const bool vec = p.dk % 4 == 0 && p.dv % 4 == 0 && p.ld_in % 4 == 0 && p.ldq / p.maps % 4 == 0 && p.ldk / p.maps % 4 == 0 && p.ldv % 4 == 0 &&
                    (reinterpret_cast<uintptr_t>(p.in) & (4 * sizeof(A) - 1)) == 0;
   return vec ? launch_prep<A, 4>(p, tokens, s) : launch_prep<A, 1>(p, tokens, s);
 }
@@ -171,10 +182,11 @@ struct GqaArgs {
   long long ld_gate;
   void* out;                 // [T, ld_out]: hq * dv columns
   long long ld_out;
+  int out_f32;
   const int32_t* block_table;
   int max_pages, page_size;
   int hq, hkv, dk, dv;
-  int window, keep;
+  int window, keep, chunk;
   float scale, cap;          // cap 0: none
   int sink;
 };
@@ -193,12 +205,17 @@ __global__ void __launch_bounds__(128) zb_gqa_attend_kernel(const GqaArgs p, con
   while (s + 1 < b.num_seqs && b.q_start[s + 1] <= t) ++s;
   const int n = b.q_start[s + 1] - b.q_start[s];
   const int pos = b.seq_lens[s] - n + (t - b.q_start[s]);
-  A* out = reinterpret_cast<A*>(p.out) + t * p.ld_out + static_cast<long long>(h) * p.dv;
+  const long long out_at = t * p.ld_out + static_cast<long long>(h) * p.dv;
+  auto store = [&](int c, float v) {
+    if (p.out_f32) reinterpret_cast<float*>(p.out)[out_at + c] = v;
+    else zb_st_act(reinterpret_cast<A*>(p.out) + out_at + c, v);
+  };
   if (pos < 0) {                                     // a padding row of a decode batch: no key
-    for (int c = threadIdx.x; c < p.dv; c += 128) zb_st_act(out + c, 0.f);
+    for (int c = threadIdx.x; c < p.dv; c += 128) store(c, 0.f);
     return;
   }
-  const int first = p.window > 0 ? max(0, pos - p.window + 1) : 0;      // seen: [0, kept) and [first, pos]
+  // seen: [0, kept) and [first, pos]
+  const int first = p.chunk > 0 ? pos / p.chunk * p.chunk : (p.window > 0 ? max(0, pos - p.window + 1) : 0);
   const int kept = min(p.keep, first);
   const A* q = reinterpret_cast<const A*>(p.q) + (static_cast<long long>(t) * p.hq + h) * p.ldq;
   for (int i = threadIdx.x; i < p.dk; i += 128) gqa_smem[i] = zb_ld_act(q + i);
@@ -255,8 +272,27 @@ __global__ void __launch_bounds__(128) zb_gqa_attend_kernel(const GqaArgs p, con
     if (c >= p.dv) continue;
     float o = acc[i] * inv;
     if (gate != nullptr) o *= 1.f / (1.f + expf(-zb_ld_act(gate + c)));
-    zb_st_act(out + c, o);
+    store(c, o);
   }
+}
+
+// One warp per (token, head); a [T, 2 heads, dv].
+template <typename A>
+__global__ void __launch_bounds__(256) zb_pair_combine_kernel(const float* __restrict__ a, A* __restrict__ out, long long ld_out, int rows, int heads,
+                                                              int dv, float lambda, float scale, float eps) {
+  zb_pdl_launch();
+  zb_pdl_wait();
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  const float* a1 = a + static_cast<long long>(row) * 2 * dv;
+  float ss = 0.f;
+  for (int c = lane; c < dv; c += 32) {
+    const float o = a1[c] - lambda * a1[dv + c];
+    ss = fmaf(o, o, ss);
+  }
+  const float f = scale / sqrtf(zb_warp_sum(ss) / static_cast<float>(dv) + eps);
+  A* dst = out + row / heads * ld_out + static_cast<long long>(row % heads) * dv;
+  for (int c = lane; c < dv; c += 32) zb_st_act(dst + c, (a1[c] - lambda * a1[dv + c]) * f);
 }
 
 template <typename A>
@@ -275,10 +311,12 @@ extern "C" {
 
 int zb_gqa_prep(const void* in, long long ld_in, const float* q_norm, const float* k_norm, const float* inv_freq, const int32_t* positions,
                 const int32_t* slots, void* q, void* k_cache, void* v_cache, long long num_rows, float eps, int hq, int hkv, int dk, int dv,
-                int rot, int ldq, int ldk, int ldv, int act_f32, int tokens, void* stream) {
+                int rot, int maps, int ldq, int ldk, int ldv, int act_f32, int tokens, void* stream) {
   if (tokens <= 0) return 0;
-  if (rot % 2 != 0 || rot > dk || ldq < dk || ldk < dk || ldv < dv) return -70;
-  const GqaPrepArgs p = {in, ld_in, q_norm, k_norm, inv_freq, positions, slots, q, k_cache, v_cache, num_rows, eps, hq, hkv, dk, dv, rot, ldq, ldk, ldv};
+  if ((maps != 1 && maps != 2) || hq % maps != 0 || ldq % maps != 0 || ldk % maps != 0) return -70;
+  if (rot % 2 != 0 || rot > dk || ldq < maps * dk || (hkv > 0 && (ldk < maps * dk || ldv < dv))) return -70;
+  const GqaPrepArgs p = {in, ld_in, q_norm, k_norm, inv_freq, positions, slots, q, k_cache, v_cache, num_rows, eps,
+                         hq, hkv, dk, dv, rot, maps, ldq, ldk, ldv};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const cudaError_t e = act_f32 ? launch_prep<float>(p, tokens, s) : launch_prep<__nv_bfloat16>(p, tokens, s);
   zb_count_launch(1);
@@ -286,16 +324,31 @@ int zb_gqa_prep(const void* in, long long ld_in, const float* q_norm, const floa
 }
 
 int zb_gqa_attend(const void* q, int ldq, const void* k_cache, int ldk, const void* v_cache, int ldv, const void* gate, long long ld_gate, void* out,
-                  long long ld_out, const int32_t* block_table, int max_pages, int page_size, int hq, int hkv, int dk, int dv, int window, int keep,
-                  float scale, float cap, int sink, const int32_t* q_start, const int32_t* seq_lens, int num_seqs, int tokens, int act_f32,
+                  long long ld_out, int out_f32, const int32_t* block_table, int max_pages, int page_size, int hq, int hkv, int dk, int dv,
+                  int window, int keep, int chunk, float scale, float cap, int sink, const int32_t* q_start, const int32_t* seq_lens, int num_seqs, int tokens, int act_f32,
                   void* stream) {
   if (tokens <= 0) return 0;
   if (hkv <= 0 || hq % hkv != 0) return -30;
-  const GqaArgs p = {q, k_cache, v_cache, ldq, ldk, ldv, gate, ld_gate, out, ld_out, block_table, max_pages, page_size,
-                     hq, hkv, dk, dv, window, keep, scale, cap, sink};
+  const GqaArgs p = {q, k_cache, v_cache, ldq, ldk, ldv, gate, ld_gate, out, ld_out, out_f32, block_table, max_pages, page_size,
+                     hq, hkv, dk, dv, window, keep, chunk, scale, cap, sink};
   const ZbVarlen b = {q_start, seq_lens, num_seqs};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const cudaError_t e = act_f32 ? launch_attend<float>(p, b, tokens, s) : launch_attend<__nv_bfloat16>(p, b, tokens, s);
+  zb_count_launch(1);
+  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+}
+
+// a fp32 [tokens, 2 heads, dv] -> out [tokens, ld_out] with heads * dv columns (fp32 or bf16).
+int zb_pair_combine(const float* a, void* out, long long ld_out, int tokens, int heads, int dv, float lambda, float scale, float eps, int act_f32,
+                    void* stream) {
+  if (tokens <= 0) return 0;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const int rows = tokens * heads;
+  const dim3 grid((rows + 7) / 8);
+  const cudaError_t e =
+      act_f32 ? zb_launch(zb_pair_combine_kernel<float>, grid, dim3(256), 0, s, a, reinterpret_cast<float*>(out), ld_out, rows, heads, dv, lambda, scale, eps)
+              : zb_launch(zb_pair_combine_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, a, reinterpret_cast<__nv_bfloat16*>(out), ld_out, rows, heads, dv,
+                          lambda, scale, eps);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }

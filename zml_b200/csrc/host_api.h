@@ -106,6 +106,13 @@ struct ZbAttnExt {
   int vdim;                    // value columns of a head that are written (heads are stored padded to the kernel's size)
   const void* gate;            // bf16 [tokens, ldg]: the output times sigmoid(gate), or null
   long long ldg;
+  int chunk;                   // position i sees the keys of its own chunk floor(i / chunk) only (instead of a window); 0: off
+  int out_f32;                 // the output is fp32 (prefill of attention.cu)
+  // Query heads 2 h and 2 h + 1 are the two maps of a differential head: their keys are the two halves of a cached key (the
+  // query is zero in the other half), the values are common, and the output [tokens, heads / 2, vdim] is
+  // a1 - pair_lambda * a2 at unit root mean square (pair_eps inside the root) times pair_scale.
+  int pair;
+  float pair_lambda, pair_scale, pair_eps;
 };
 
 ZbDeviceState* zb_device_state();       // state of the current device, or nullptr before zb_init

@@ -1,18 +1,20 @@
 // Latent attention (multi-head attention whose keys and values are projections of one low-rank latent per token), as
-// Dopurax layers use it: the paged cache holds, per token, the normalised latent c [rank] and one rotated key part
+// Dopurax and Sodotar layers use it: the paged cache holds, per token, the normalised latent c [rank] and one rotated key part
 // [rot] for every head.  A cache row is [c | pad | rotated part | pad] with both parts padded to 16 elements.
 //
-//   zb_latent_prep     one token per CTA: RMS norm of the query latent, RMS norm of c, rotation of the shared key
-//                      part, cache write
+//   zb_latent_prep     one token per CTA: RMS norm of the query latent (where there is one), RMS norm of c, rotation of the
+//                      shared key part, cache write
 //   zb_latent_absorb   per head out[t, h] = a[t, h] * W[h]^T for the small per-head matrices: queries into the latent
 //                      space (together with the rotation of their rotated part) and attention results out of it
-//                      (together with the sigmoid output gate)
+//                      (together with the sigmoid output gate, where there is one)
 //   zb_latent_attend   attention in the latent space (one key vector per token for all heads), any sizes, bf16 or fp32:
 //                      the fp32 path and the fall-back for sizes the tensor-core kernels do not take
 //   zb_latent_gather   visible cache rows of a batch -> contiguous rows, for the prefill path that expands keys and values
 //   zb_latent_q_pack   queries [T, H, dim + rot] -> zero-padded rows with the rotated part rotated, for the prefill kernel
 //
-// Scores, softmax, norms and angles are fp32.
+// Rotated parts are turned in neighbouring pairs; a design that pairs i with i + rot / 2 has its projections' rows permuted at
+// load.  A sink (one number per head, or none) is a term exp(sink) of the softmax denominator: a running maximum of `sink` and a
+// running sum of 1 before the first key.  Scores, softmax, norms and angles are fp32.
 #include "act.cuh"
 #include "host_api.h"
 
@@ -82,7 +84,7 @@ __global__ void __launch_bounds__(256) zb_latent_prep_kernel(const PrepArgs p) {
     sq += red[0][i];
     sc += red[1][i];
   }
-  const float iq = 1.f / sqrtf(sq / static_cast<float>(p.q_rank) + p.eps), ic = 1.f / sqrtf(sc / static_cast<float>(p.rank) + p.eps);
+  const float iq = 1.f / sqrtf(sq / static_cast<float>(max(p.q_rank, 1)) + p.eps), ic = 1.f / sqrtf(sc / static_cast<float>(p.rank) + p.eps);
   if (slot >= p.num_rows) (void)ZB_BC_OK(slot, p.num_rows, kKernelPrep, 1);
   const bool write = slot >= 0 && slot < p.num_rows;
   A* cq = reinterpret_cast<A*>(p.cq) + t * p.ld_cq;
@@ -253,6 +255,7 @@ struct AttendArgs {
   int heads, rank, rot, rot_off;
   int window;
   float scale;
+  const float* sink;         // [heads] or null
 };
 
 constexpr int kAttendKeys = 64;
@@ -282,7 +285,7 @@ __global__ void __launch_bounds__(128) zb_latent_attend_kernel(const AttendArgs 
   const int32_t* bt = p.block_table + static_cast<long long>(s) * p.max_pages;
   const A* cache = reinterpret_cast<const A*>(p.cache);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  float m = -INFINITY, l = 0.f, acc[RC];
+  float m = p.sink != nullptr ? p.sink[h] : -INFINITY, l = p.sink != nullptr ? 1.f : 0.f, acc[RC];
 #pragma unroll
   for (int i = 0; i < RC; ++i) acc[i] = 0.f;
   for (int k0 = first; k0 <= pos; k0 += kAttendKeys) {
@@ -445,10 +448,10 @@ int zb_latent_absorb(const void* a, long long lda, long long ha, const void* w, 
 }
 
 int zb_latent_attend(const void* q, const void* cache, long long ld_cache, void* out, long long ld_out, const int32_t* block_table,
-                     int max_pages, int page_size, int heads, int rank, int rot, int rot_off, int window, float scale,
+                     int max_pages, int page_size, int heads, int rank, int rot, int rot_off, int window, float scale, const float* sink,
                      const int32_t* q_start, const int32_t* seq_lens, int num_seqs, int tokens, int act_f32, void* stream) {
   if (tokens <= 0) return 0;
-  const AttendArgs p = {q, cache, ld_cache, out, ld_out, block_table, max_pages, page_size, heads, rank, rot, rot_off, window, scale};
+  const AttendArgs p = {q, cache, ld_cache, out, ld_out, block_table, max_pages, page_size, heads, rank, rot, rot_off, window, scale, sink};
   const ZbVarlen b = {q_start, seq_lens, num_seqs};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return act_f32 ? launch_attend<float>(p, b, tokens, s) : launch_attend<__nv_bfloat16>(p, b, tokens, s);

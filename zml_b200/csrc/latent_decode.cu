@@ -34,6 +34,7 @@ struct DecodeParams {
   float* part_ml;               // [B, groups, splits, 16 * MT, 2]
   int max_pages, page_size, heads, row, rank_p, window, num_splits, stages;
   float scale_log2;
+  const float* sink;            // [heads] or null: the first chunk of a sequence starts with it as its running maximum
   ZbStatus* status;
 };
 
@@ -149,6 +150,10 @@ __global__ void __launch_bounds__(kThreads, 1) zb_latent_decode_kernel(const Dec
     const uint32_t qa = zb_smem_u32(q_s), ka = zb_smem_u32(kv_s), pa = zb_smem_u32(p_s);
     const int col0 = warp * 8 * NT;
     float m_run = -INFINITY, l_run = 0.f;
+    if (p.sink != nullptr && split == 0 && srow < nh) {
+      m_run = p.sink[h0 + srow] * 1.4426950408889634f;
+      l_run = 1.f;
+    }
     bool fine = true;
     uint32_t stage = 0, phase = 0;
     for (int t = tile0; t < tile1; ++t) {
@@ -380,8 +385,8 @@ int zb_latent_decode_supported(int row, int rank_p) {
 int zb_latent_decode_groups(int heads) { return (heads + rows_for(heads) - 1) / rows_for(heads); }
 
 int zb_latent_decode(const void* q, const void* cache, int row, void* out, long long ld_out, const int32_t* block_table, int max_pages,
-                     int page_size, const int32_t* seq_lens, int batch, int heads, int rank_p, int window, float scale, int num_splits,
-                     void* stream) {
+                     int page_size, const int32_t* seq_lens, int batch, int heads, int rank_p, int window, float scale, const float* sink,
+                     int num_splits, void* stream) {
   if (batch <= 0) return 0;
   if (!zb_latent_decode_supported(row, rank_p) || ld_out % 4 != 0) return -32;
   ZbDeviceState* st = zb_device_state();
@@ -410,6 +415,7 @@ int zb_latent_decode(const void* q, const void* cache, int row, void* out, long 
   p.num_splits = num_splits;
   p.stages = pick_stages(rows, row);
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.sink = sink;
   p.status = st->status;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int nt = rank_p <= 128 ? 2 : (rank_p <= 256 ? 4 : 8);

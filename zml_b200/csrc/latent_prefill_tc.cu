@@ -13,8 +13,9 @@
 //   warp  9         : MMA issuer (one thread)
 // Each pipeline only touches the tiles between its own window edge and diagonal.  S, P and O live in tensor memory:
 // S_0 0-63 | S_1 64-127 | P_0 128-159 | P_1 160-191 | O_0 192.. | O_1 behind it.  The structure of a step (scores -> running
-// maximum -> lazy rescale of O -> P back into tensor memory -> O += P V) is that of attention_tc.cu.  The epilogue
-// normalises and applies the sigmoid output gate.  Every wait is bounded.
+// maximum -> lazy rescale of O -> P back into tensor memory -> O += P V) is that of attention_tc.cu.  A sink is the running
+// maximum, with a running sum of 1, in front of the first tile.  The epilogue normalises and applies the sigmoid output gate
+// (either may be absent).  Every wait is bounded.
 #include <cuda.h>
 
 #include "act.cuh"
@@ -35,7 +36,7 @@ constexpr int kKvSub = kKeys * 128;              // one 64-column sub-tile of 64
 
 struct LatentPrefillParams {
   __nv_bfloat16* out;           // [T, ld_out]
-  const __nv_bfloat16* gate;    // [T, ld_gate]
+  const __nv_bfloat16* gate;    // [T, ld_gate] or null
   long long ld_out, ld_gate;
   ZbVarlen b;
   const int32_t* key_start;     // [num_seqs + 1] first gathered row of every sequence
@@ -45,6 +46,7 @@ struct LatentPrefillParams {
   int rot_out;                  // its first column in the gathered rows
   int window;
   float scale_log2;
+  const float* sink;            // [heads] or null
   ZbStatus* status;
 };
 
@@ -244,7 +246,7 @@ zb_latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
     const uint32_t t_p = tmem_base + kColP + w * 32 + lane_off;
     const uint32_t t_o = tmem_base + kColO + w * kOCols + lane_off;
     const int jb = t_begin[w], je = t_end[w];
-    float m = -INFINITY, l = 0.f;
+    float m = p.sink != nullptr ? p.sink[head] * 1.4426950408889634f : -INFINITY, l = p.sink != nullptr ? 1.f : 0.f;
     bool ok = true;
     for (int j = jb; j < je; ++j) {
       const uint32_t jj = static_cast<uint32_t>(j - jb);
@@ -274,10 +276,10 @@ zb_latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
       }
       const float mx = fmaxf(m, mx_raw * p.scale_log2);
       const float m_use = mx == -INFINITY ? 0.f : mx;
-      if (jj > 0) {
+      {
         const float alpha = m == -INFINITY ? 1.f : zb_ex2(m - m_use);
         const bool moved = alpha != 1.f;
-        if (__any_sync(0xffffffffu, moved)) {
+        if (jj > 0 && __any_sync(0xffffffffu, moved)) {
           if (!zb_mbar_wait(&o_ready[w], (jj - 1u) & 1u, abort_flag)) {
             *abort_where = 12u + w;
             ok = false;
@@ -325,7 +327,7 @@ zb_latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
         const int row = w * kQRows + r;
         const long long t = tok_base + row;
         __nv_bfloat16* orow = p.out + t * p.ld_out + static_cast<long long>(head) * p.vdim;
-        const __nv_bfloat16* grow = p.gate + t * p.ld_gate + static_cast<long long>(head) * p.vdim;
+        const __nv_bfloat16* grow = p.gate != nullptr ? p.gate + t * p.ld_gate + static_cast<long long>(head) * p.vdim : nullptr;
 #pragma unroll 1
         for (int c0 = 0; c0 < kOCols; c0 += 32) {
           uint32_t o[32];
@@ -336,14 +338,20 @@ zb_latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
           for (int i = 0; i < 4; ++i) {
             const int c = c0 + 8 * i;
             if (c >= p.vdim) continue;
-            const uint4 gv = *reinterpret_cast<const uint4*>(grow + c);
-            const uint32_t gu[4] = {gv.x, gv.y, gv.z, gv.w};
             uint32_t wd[4];
+            if (grow == nullptr) {
 #pragma unroll
-            for (int q = 0; q < 4; ++q) {
-              const float2 g = zb_unpack_bf16x2(gu[q]);
-              wd[q] = zb_pack_bf16x2(__uint_as_float(o[8 * i + 2 * q]) * inv / (1.f + __expf(-g.x)),
-                                     __uint_as_float(o[8 * i + 2 * q + 1]) * inv / (1.f + __expf(-g.y)));
+              for (int q = 0; q < 4; ++q)
+                wd[q] = zb_pack_bf16x2(__uint_as_float(o[8 * i + 2 * q]) * inv, __uint_as_float(o[8 * i + 2 * q + 1]) * inv);
+            } else {
+              const uint4 gv = *reinterpret_cast<const uint4*>(grow + c);
+              const uint32_t gu[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+              for (int q = 0; q < 4; ++q) {
+                const float2 g = zb_unpack_bf16x2(gu[q]);
+                wd[q] = zb_pack_bf16x2(__uint_as_float(o[8 * i + 2 * q]) * inv / (1.f + __expf(-g.x)),
+                                       __uint_as_float(o[8 * i + 2 * q + 1]) * inv / (1.f + __expf(-g.y)));
+              }
             }
             *reinterpret_cast<uint4*>(orow + c) = make_uint4(wd[0], wd[1], wd[2], wd[3]);
           }
@@ -398,7 +406,7 @@ int zb_latent_prefill_tc_supported(int dim, int rot, int vdim, int rank) {
 int zb_latent_prefill_tc(const void* q, const void* kv, long long ld_kv, const void* shared, long long ld_shared, int rot_out, void* out,
                          long long ld_out, const void* gate, long long ld_gate, const int32_t* q_start, const int32_t* seq_lens,
                          int num_seqs, const int32_t* key_start, const int32_t* first_key, int tokens, int rows, int blocks, int heads,
-                         int dim, int rot, int vdim, int window, float scale, void* stream) {
+                         int dim, int rot, int vdim, int window, float scale, const float* sink, void* stream) {
   if (tokens <= 0 || blocks <= 0) return 0;
   if (!zb_latent_prefill_tc_supported(dim, rot, vdim, 8)) return -32;
   if (ld_kv % 8 != 0 || ld_shared % 8 != 0 || ld_out % 8 != 0 || ld_gate % 8 != 0 || rot_out % 8 != 0 ||
@@ -429,6 +437,7 @@ int zb_latent_prefill_tc(const void* q, const void* kv, long long ld_kv, const v
   p.rot_out = rot_out;
   p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.sink = sink;
   p.status = st->status;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   switch (nq * 2 + nv) {

@@ -90,6 +90,89 @@ __global__ void __launch_bounds__(128) zb_moe_router_topk_kernel(const float* __
   }
 }
 
+// One warp per token: scores s = softmax of the first `experts` logits; the k largest s + correction are chosen and weighted by
+// their s, divided by the sum.  Behind the routed choices come `shared` always-on experts (ids 0 .. shared - 1), weighted by the
+// sigmoid of the logit in column `experts`; routed expert e has id shared + (e - e0) mod experts, so that the experts of the
+// rank that starts at e0 directly follow its shared ones.
+template <int MAX_PER_LANE>
+__global__ void __launch_bounds__(128) zb_moe_route_kernel(const float* __restrict__ logits, long long stride,
+                                                           const float* __restrict__ correction, int32_t* __restrict__ ids,
+                                                           float* __restrict__ weights, int tokens, int experts, int k, int shared,
+                                                           int e0) {
+  const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+  const int lane = threadIdx.x & 31;
+  float corr[MAX_PER_LANE];
+  zb_pdl_launch();
+#pragma unroll
+  for (int i = 0; i < MAX_PER_LANE; ++i) corr[i] = correction != nullptr && lane + 32 * i < experts ? correction[lane + 32 * i] : 0.f;
+  zb_pdl_wait();
+  if (warp >= tokens) return;
+  const float* row = logits + static_cast<size_t>(warp) * stride;
+  const float gate = shared > 0 ? row[experts] : 0.f;
+  float s[MAX_PER_LANE], v[MAX_PER_LANE], mx = -INFINITY, sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < MAX_PER_LANE; ++i) {
+    s[i] = lane + 32 * i < experts ? row[lane + 32 * i] : -INFINITY;
+    mx = fmaxf(mx, s[i]);
+  }
+  mx = zb_warp_max(mx);
+#pragma unroll
+  for (int i = 0; i < MAX_PER_LANE; ++i) {
+    s[i] = lane + 32 * i < experts ? expf(s[i] - mx) : 0.f;
+    sum += s[i];
+  }
+  sum = zb_warp_sum(sum);
+#pragma unroll
+  for (int i = 0; i < MAX_PER_LANE; ++i) {
+    s[i] /= sum;
+    v[i] = lane + 32 * i < experts ? s[i] + corr[i] : -INFINITY;
+  }
+  float my_s = 0.f, total = 0.f;
+  int my_e = 0;
+  for (int j = 0; j < k; ++j) {
+    float best = -INFINITY, best_s = 0.f;
+    int bi = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i) {
+      const int e = lane + 32 * i;
+      if (e < experts && (v[i] > best || (v[i] == best && e < bi))) {
+        best = v[i];
+        best_s = s[i];
+        bi = e;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o), os = __shfl_xor_sync(0xffffffffu, best_s, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ov > best || (ov == best && oi < bi)) {
+        best = ov;
+        best_s = os;
+        bi = oi;
+      }
+    }
+    if (bi == 0x7fffffff) bi = 0;                  // only NaN logits come here
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i)
+      if (lane + 32 * i == bi) v[i] = -INFINITY;
+    total += best_s;
+    if (lane == j) {
+      my_s = best_s;
+      my_e = bi;
+    }
+  }
+  const size_t at = static_cast<size_t>(warp) * (k + shared);
+  if (lane < k) {
+    ids[at + lane] = shared + (my_e >= e0 ? my_e - e0 : my_e - e0 + experts);
+    weights[at + lane] = my_s / (total + 1e-20f);
+  }
+  const float on = 1.f / (1.f + expf(-gate));
+  for (int j = lane; j < shared; j += 32) {
+    ids[at + k + j] = j;
+    weights[at + k + j] = on;
+  }
+}
+
 // ------------------------------------------------------------------ permutation by expert
 // meta layout (int32): [0, E]      offsets (exclusive prefix of counts, E + 1 entries)
 //                      [E+1, 2E]   cursors (scratch)
@@ -444,7 +527,8 @@ struct GroupedParams {
   int ldo;                  // leading dimension of out
   __nv_bfloat16* out;
   int cap;                  // rows allocated in xs / out
-  int act;                  // ZbMoeAct: which gate activation the gated epilogue applies, or relu2 on a plain projection
+  int act;                  // ZbMoeAct: which gated unit the gated epilogue applies, or relu2 on a plain projection
+  const float* limits;      // [e_local] of ZB_ACT_CLIPPED_GLU, else null
   ZbStatus* status;
 };
 
@@ -605,6 +689,7 @@ zb_moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __g
       const uint32_t taddr = tmem_base + acc * BN + (static_cast<uint32_t>(quad * 32) << 16);
       const int off_e = prm.offsets[c.e];
       const int end_e = min(prm.offsets[c.e + 1], prm.cap);
+      const float limit = SWIGLU && prm.limits != nullptr ? prm.limits[c.e] : 0.f;
       if constexpr (SWAP) {
         // thread row = weight row (output feature), columns = tokens of this tile
         const int tok0 = off_e + tt * BN;
@@ -645,7 +730,7 @@ zb_moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __g
                 if (tok < end_e) {
                   const float gt = __uint_as_float(r[j]);
                   const float up = xch[(c0 + j) * 64 + row_in_tile];
-                  prm.out[static_cast<size_t>(tok) * prm.ldo + feat] = __float2bfloat16(zb_gate_act(gt, prm.act) * up);
+                  prm.out[static_cast<size_t>(tok) * prm.ldo + feat] = __float2bfloat16(zb_gated(gt, up, prm.act, limit));
                 }
               }
             }
@@ -694,7 +779,7 @@ zb_moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __g
 #pragma unroll
                 for (int j = 0; j < 16; ++j) {
                   const float gt = __uint_as_float(gr[j]);
-                  h[j] = zb_gate_act(gt, prm.act) * __uint_as_float(ur[j]);
+                  h[j] = zb_gated(gt, __uint_as_float(ur[j]), prm.act, limit);
                 }
                 uint4* op = reinterpret_cast<uint4*>(prm.out + static_cast<size_t>(tok) * prm.ldo + wt * (BN / 2) +
                                                      blk * 64 + c0);
@@ -754,6 +839,21 @@ int zb_moe_router_topk(const float* logits, int32_t* ids, float* weights, int to
   else zb_launch(zb_moe_router_topk_kernel<16>, dim3(blocks), dim3(128), 0, s, logits, ids, weights, tokens, experts, k, stride, renormalize);
   zb_count_launch(1);
   return static_cast<int>(cudaGetLastError());
+}
+
+// ids, weights [tokens, k + shared]; logits [tokens, >= experts (+ 1 with shared experts)]; see the kernel.
+int zb_moe_route(const float* logits, long long stride, const float* correction, int32_t* ids, float* weights, int tokens, int experts,
+                 int k, int shared, int e0, void* stream) {
+  if (tokens <= 0) return 0;
+  if (k < 1 || k > 32 || experts < k || experts > 512 || shared < 0 || e0 < 0 || e0 >= experts) return -60;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid((tokens + 3) / 4), block(128);
+  cudaError_t e;
+  if (experts <= 32) e = zb_launch(zb_moe_route_kernel<1>, grid, block, 0, s, logits, stride, correction, ids, weights, tokens, experts, k, shared, e0);
+  else if (experts <= 128) e = zb_launch(zb_moe_route_kernel<4>, grid, block, 0, s, logits, stride, correction, ids, weights, tokens, experts, k, shared, e0);
+  else e = zb_launch(zb_moe_route_kernel<16>, grid, block, 0, s, logits, stride, correction, ids, weights, tokens, experts, k, shared, e0);
+  zb_count_launch(1);
+  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }
 
 // Permutation of the (token, expert) pairs whose expert is in [e0, e0 + e_local): fills
@@ -854,10 +954,11 @@ int zb_moe_combine(const void* o, const int32_t* pair_pos, const float* weights,
 
 // out[rows of expert e, :] = xs[rows of expert e, :K] * w[e][N, K]^T for all local experts.
 // swiglu = 1 / 2 / 3 (swiglu / geglu / geglu_tanh, see ZbMoeAct): w holds the interleaved gate/up weight (N = 2F, see
-// above) and out is [cap, F]; swiglu = 4 (relu2): a plain projection followed by relu(x)^2; 0: a plain projection.
+// above) and out is [cap, F]; swiglu = 5 (clipped): likewise, with one limit per expert in `limits`; swiglu = 4 (relu2): a
+// plain projection followed by relu(x)^2; 0: a plain projection.
 // avg_tokens (expected tokens per expert) picks the tile orientation.
 int zb_moe_grouped_gemm(const void* xs, const void* w, void* out, const int32_t* offsets, int e_local, int n, int k,
-                        int cap, int ldo, int swiglu, int avg_tokens, void* stream) {
+                        int cap, int ldo, int swiglu, const float* limits, int avg_tokens, void* stream) {
   if (cap <= 0 || e_local <= 0) return 0;
   if (k % 8 != 0 || ldo % 8 != 0) return -63;
   if (e_local > kZbMaxExperts) return -61;
@@ -884,8 +985,9 @@ int zb_moe_grouped_gemm(const void* xs, const void* w, void* out, const int32_t*
   prm.cap = cap;
   prm.act = swiglu;
   prm.status = st->status;
-  if (swiglu < 0 || swiglu > ZB_ACT_RELU2) return -67;
-  const bool gated = swiglu >= ZB_ACT_SWIGLU && swiglu <= ZB_ACT_GEGLU_TANH;
+  prm.limits = limits;
+  if (swiglu < 0 || swiglu > ZB_ACT_CLIPPED_GLU || (swiglu == ZB_ACT_CLIPPED_GLU && limits == nullptr)) return -67;
+  const bool gated = zb_act_is_gated(swiglu);
   CUtensorMap tx, tw;
   int rc = zb_make_tmap_bf16_2d(&tx, xs, cap, k, k, swap ? bn : kBlockP);
   if (rc != 0) return rc;

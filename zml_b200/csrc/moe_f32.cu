@@ -1,7 +1,7 @@
 // fp32 grouped GEMM over the experts on the FMA pipes, with the token gather in its loads and the gate in its epilogue: the
 // counterpart of the bf16 grouped GEMM of moe.cu for models that run in fp32.
 //
-//   out[rows of expert e, :] = x[source of the row, :K] * w[e][N, K]^T,  or act(gate) * up on interleaved gate / up rows
+//   out[rows of expert e, :] = x[source of the row, :K] * w[e][N, K]^T,  or the gated unit of interleaved gate / up rows
 #include "act.cuh"
 #include "host_api.h"
 
@@ -19,6 +19,7 @@ struct GroupedF32 {
   const int32_t* offsets;   // [E + 1]
   int n, k;
   int act;                  // ZbMoeAct; gated: rows of w in blocks of [64 gate | 64 up]
+  const float* limits;      // [E] of ZB_ACT_CLIPPED_GLU
 };
 
 template <bool GATED>
@@ -75,9 +76,11 @@ __global__ void __launch_bounds__(256) zb_moe_grouped_f32_kernel(const GroupedF3
     for (int j = 0; j < 4; ++j) {
       const int c = tx * 4 + j;
       if constexpr (GATED) {
-        const float g = acc[0][i][j];
-        const float a = p.act == ZB_ACT_SWIGLU ? g / (1.f + expf(-g)) : zb_gate_act(g, p.act);
-        p.out[row * p.ldo + blockIdx.x * kT + c] = a * acc[1][i][j];
+        const float g = acc[0][i][j], u = acc[1][i][j];
+        float v;
+        if (p.act == ZB_ACT_CLIPPED_GLU) v = zb_clipped_glu<true>(g, u, p.limits[e]);
+        else v = (p.act == ZB_ACT_SWIGLU ? g / (1.f + expf(-g)) : zb_gate_act(g, p.act)) * u;
+        p.out[row * p.ldo + blockIdx.x * kT + c] = v;
       } else if (n0 + c < p.n) {
         p.out[row * p.ldo + n0 + c] = zb_plain_act(acc[0][i][j], p.act);
       }
@@ -86,16 +89,17 @@ __global__ void __launch_bounds__(256) zb_moe_grouped_f32_kernel(const GroupedF3
 }
 }  // namespace
 
-// max_rows: an upper bound of the rows of one expert.  act as zb_moe_grouped_gemm's (gated: n a multiple of 128).
+// max_rows: an upper bound of the rows of one expert.  act and limits as zb_moe_grouped_gemm's (gated: n a multiple of 128).
 extern "C" int zb_moe_grouped_f32(const float* x, long long ldx, const int32_t* pair, int per, const float* w, float* out, long long ldo,
-                                  const int32_t* offsets, int experts, int n, int k, int max_rows, int act, void* stream) {
+                                  const int32_t* offsets, int experts, int n, int k, int max_rows, int act, const float* limits,
+                                  void* stream) {
   if (max_rows <= 0 || experts <= 0) return 0;
-  if (act < 0 || act > ZB_ACT_RELU2) return -67;
-  const bool gated = act >= ZB_ACT_SWIGLU && act <= ZB_ACT_GEGLU_TANH;
+  if (act < 0 || act > ZB_ACT_CLIPPED_GLU || (act == ZB_ACT_CLIPPED_GLU && limits == nullptr)) return -67;
+  const bool gated = zb_act_is_gated(act);
   if (gated && n % (2 * kT) != 0) return -64;
   const int rows = (max_rows + kT - 1) / kT;
   if (rows > 65535 || experts > 65535) return -61;
-  const GroupedF32 p = {x, ldx, pair, per, w, out, ldo, offsets, n, k, act};
+  const GroupedF32 p = {x, ldx, pair, per, w, out, ldo, offsets, n, k, act, limits};
   const dim3 grid(gated ? n / (2 * kT) : (n + kT - 1) / kT, rows, experts);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const cudaError_t e = gated ? zb_launch(zb_moe_grouped_f32_kernel<true>, grid, dim3(256), 0, s, p)

@@ -1,6 +1,6 @@
 // Layer glue of decoders that keep the residual stream in fp32:
 //
-//   zb_embedding_f32   gathers table rows (bf16 or fp32), times a constant, into the fp32 stream
+//   zb_embedding_f32   gathers table rows (bf16 or fp32), times a constant, into the fp32 stream (or several copies of it)
 //   zb_post_norm       x <- layernorm(alpha * x + y) * w, the normalisation behind a sublayer;
 //                      without y a plain layer norm.  For decode steps the same launch continues with the input
 //                      convolution of the next layer (one token per sequence: everything it needs is in the row and
@@ -8,6 +8,8 @@
 //   zb_sandwich_norm   x <- x + m * rmsnorm(y) * w, the residual sum of a sublayer with a norm behind it, and in the same
 //                      launch rmsnorm(x) * w_next, what the next sublayer reads.  y is a row, or the weighted sum of a
 //                      token's expert rows
+//   zb_hyper_norm      hyper-connections: S streams per token instead of one.  x_t <- sum_s mix[s, t] x_s + out[t] y behind a
+//                      sublayer (y as above), and in the same launch rmsnorm(sum_s in[s] x_s) * w, what the next one reads
 //   zb_stream_conv     that input convolution over a varlen batch: h = x + conv(x), causal and per channel, and for
 //                      token-shift mixers the interpolations h + (h_prev - h) * mu of h with the previous token's h
 //
@@ -25,7 +27,7 @@ constexpr int kMaxTaps = 8;
 
 template <typename W>
 __global__ void __launch_bounds__(256) zb_embedding_f32_kernel(const int32_t* __restrict__ ids, const W* __restrict__ table,
-                                                               float* __restrict__ out, int d, int vocab, float scale) {
+                                                               float* __restrict__ out, int d, int vocab, float scale, int copies) {
   zb_pdl_launch();
   zb_pdl_wait();
   const int t = blockIdx.x;
@@ -35,8 +37,11 @@ __global__ void __launch_bounds__(256) zb_embedding_f32_kernel(const int32_t* __
     id = 0;
   }
   const W* src = table + static_cast<size_t>(id) * d;
-  float* dst = out + static_cast<size_t>(t) * d;
-  for (int i = threadIdx.x; i < d; i += 256) dst[i] = scale * zb_ld_act(src + i);
+  float* dst = out + static_cast<size_t>(t) * copies * d;
+  for (int i = threadIdx.x; i < d; i += 256) {
+    const float v = scale * zb_ld_act(src + i);
+    for (int c = 0; c < copies; ++c) dst[static_cast<size_t>(c) * d + i] = v;
+  }
 }
 
 // ------------------------------------------------------------------------------------------ convolution
@@ -592,6 +597,171 @@ cudaError_t launch_sandwich(const SandwichArgs& p, int act_f32, int tokens, cuda
   return vec ? launch_sandwich<Y, __nv_bfloat16, 4>(p, tokens, s) : launch_sandwich<Y, __nv_bfloat16, 1>(p, tokens, s);
 }
 
+// ------------------------------------------------------------------------------------------ hyper-connections
+constexpr int kMaxStreams = 8;
+
+struct HyperArgs {
+  const void* y;               // sublayer output [T, ldy], or expert rows [*, ldy] with pair_pos, or null: nothing to add
+  long long ldy;
+  int y_f32;
+  const int32_t* pair_pos;     // [T, k], as SandwichArgs
+  const float* pair_w;
+  int k;
+  const float* x;              // [T, streams, d]
+  int streams;
+  const float* mix;            // [streams, streams]: from, to
+  const float* out;            // [streams]
+  const float* in;             // [streams] of what comes next, or null: no norm
+  const float* w;              // [d]
+  float eps;
+  float* x_out;                // [T, streams, d] (may be x) or null
+  void* act;                   // [T, ld_act]: columns d .. ld_act are zero
+  long long ld_act;
+  int act_f32;
+  int d;
+};
+
+// S >= streams; NT threads, NG groups of V neighbouring channels per thread, all streams of a channel in one thread.
+template <int S, int NT, int NG, int V>
+__global__ void __launch_bounds__(NT) zb_hyper_norm_kernel(const HyperArgs p) {
+  constexpr int kSlots = 32;                             // expert slots read through shared memory at a time
+  __shared__ float red[NT / 32];
+  __shared__ float sw[kSlots];
+  __shared__ int spos[kSlots];
+  __shared__ float s_mix[S][S], s_out[S], s_in[S];
+  zb_pdl_launch();
+  const int d = p.d, ns = p.streams;
+  for (int i = threadIdx.x; i < S * S; i += NT) {        // coefficients of streams that do not exist are zero
+    const int from = i / S, to = i % S;
+    s_mix[from][to] = p.y != nullptr && from < ns && to < ns ? p.mix[from * ns + to] : 0.f;
+    if (i < S) {
+      s_out[i] = p.y != nullptr && i < ns ? p.out[i] : 0.f;
+      s_in[i] = p.in != nullptr && i < ns ? p.in[i] : 0.f;
+    }
+  }
+  float w[NG][V];
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + NT * i) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) w[i][e] = 0.f;
+    if (c < d && p.in != nullptr) ld_vec<V>(w[i], p.w + c);
+  }
+  __syncthreads();
+  zb_pdl_wait();
+  const long long t = blockIdx.x;
+  float x[NG][S][V], y[NG][V];
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + NT * i) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) y[i][e] = 0.f;
+#pragma unroll
+    for (int s = 0; s < S; ++s) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[i][s][e] = 0.f;
+      if (c < d && s < ns) ld_vec<V>(x[i][s], p.x + (t * ns + s) * d + c);
+    }
+  }
+  if (p.y != nullptr) {
+    auto add = [&](long long row, float wt) {
+#pragma unroll
+      for (int i = 0; i < NG; ++i) {
+        const int c = (threadIdx.x + NT * i) * V;
+        if (c >= d) continue;
+        float v[V];
+        if (p.y_f32) {
+          ld_vec<V>(v, reinterpret_cast<const float*>(p.y) + row * p.ldy + c);
+        } else {
+          const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.y) + row * p.ldy + c;
+          if constexpr (V == 4) ld_row4(v, src);
+          else v[0] = zb_ld_act(src);
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[i][e] = fmaf(wt, v[e], y[i][e]);
+      }
+    };
+    if (p.pair_pos == nullptr) {
+      add(t, 1.f);
+    } else {
+      for (int j0 = 0; j0 < p.k; j0 += kSlots) {
+        const int n = min(kSlots, p.k - j0);
+        __syncthreads();
+        if (threadIdx.x < n) {
+          spos[threadIdx.x] = p.pair_pos[t * p.k + j0 + threadIdx.x];
+          sw[threadIdx.x] = p.pair_w[t * p.k + j0 + threadIdx.x];
+        }
+        __syncthreads();
+#pragma unroll 4
+        for (int j = 0; j < n; ++j)
+          if (spos[j] >= 0) add(spos[j], sw[j]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NG; ++i) {
+      const int c = (threadIdx.x + NT * i) * V;
+      float n[S][V];
+#pragma unroll
+      for (int to = 0; to < S; ++to) {
+        const float o = s_out[to];
+#pragma unroll
+        for (int e = 0; e < V; ++e) n[to][e] = o * y[i][e];
+#pragma unroll
+        for (int from = 0; from < S; ++from) {
+          const float f = s_mix[from][to];
+#pragma unroll
+          for (int e = 0; e < V; ++e) n[to][e] = fmaf(f, x[i][from][e], n[to][e]);
+        }
+      }
+#pragma unroll
+      for (int s = 0; s < S; ++s) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[i][s][e] = n[s][e];
+        if (p.x_out != nullptr && c < d && s < ns) st_vec<float, V>(p.x_out + (t * ns + s) * d + c, x[i][s]);
+      }
+    }
+  }
+  if (p.act == nullptr) return;
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < NG; ++i)
+#pragma unroll
+    for (int e = 0; e < V; ++e) {                        // the mix that the next sublayer reads, over y
+      float u = 0.f;
+#pragma unroll
+      for (int s = 0; s < S; ++s) u = fmaf(s_in[s], x[i][s][e], u);
+      y[i][e] = u;
+      sq = fmaf(u, u, sq);
+    }
+  const float inv = 1.f / sqrtf(block_sum_warps<NT / 32>(sq, red) / static_cast<float>(d) + p.eps);
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + NT * i) * V;
+    if (c >= p.ld_act) continue;
+    float v[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = inv * y[i][e] * w[i][e];        // columns past d: zero
+    if (p.act_f32) st_vec<float, V>(reinterpret_cast<float*>(p.act) + t * p.ld_act + c, v);
+    else st_vec<__nv_bfloat16, V>(reinterpret_cast<__nv_bfloat16*>(p.act) + t * p.ld_act + c, v);
+  }
+}
+
+template <int S, int V>
+cudaError_t launch_hyper(const HyperArgs& p, int tokens, cudaStream_t s) {
+  const long long groups = ((p.act != nullptr && p.ld_act > p.d ? p.ld_act : p.d) + V - 1) / V;
+  if (groups <= 128) return zb_launch(zb_hyper_norm_kernel<S, 128, 1, V>, dim3(tokens), dim3(128), 0, s, p);
+  if (groups <= 512) return zb_launch(zb_hyper_norm_kernel<S, 512, 1, V>, dim3(tokens), dim3(512), 0, s, p);
+  if (groups <= 1024) return zb_launch(zb_hyper_norm_kernel<S, 512, 2, V>, dim3(tokens), dim3(512), 0, s, p);
+  if (groups <= 4096) return zb_launch(zb_hyper_norm_kernel<S, 512, 8, V>, dim3(tokens), dim3(512), 0, s, p);
+  return cudaErrorInvalidValue;
+}
+template <int V>
+cudaError_t launch_hyper(const HyperArgs& p, int tokens, cudaStream_t s) {
+  if (p.streams <= 2) return launch_hyper<2, V>(p, tokens, s);
+  if (p.streams <= 4) return launch_hyper<4, V>(p, tokens, s);
+  return launch_hyper<kMaxStreams, V>(p, tokens, s);
+}
+
 template <typename A, int NG, bool MIX>
 cudaError_t launch_post_norm_conv(const PostNormArgs& p, const ConvArgs& a, const ZbVarlen& b, int tokens, cudaStream_t s) {
   if (a.taps <= 4) return zb_launch(zb_post_norm_conv_kernel<A, NG, 4, MIX>, dim3(tokens), dim3(512), 0, s, p, a, b);
@@ -629,14 +799,17 @@ bool conv_ok(int taps, int rows, int nmix) {
 
 extern "C" {
 
+// out [tokens, copies, d].
 int zb_embedding_f32(const int32_t* ids, const void* table, int table_f32, float* out, int tokens, int d, int vocab, float scale,
-                     void* stream) {
+                     int copies, void* stream) {
   if (tokens <= 0) return 0;
+  if (copies < 1) return -70;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const cudaError_t e =
-      table_f32 ? zb_launch(zb_embedding_f32_kernel<float>, dim3(tokens), dim3(256), 0, s, ids, reinterpret_cast<const float*>(table), out, d, vocab, scale)
+      table_f32 ? zb_launch(zb_embedding_f32_kernel<float>, dim3(tokens), dim3(256), 0, s, ids, reinterpret_cast<const float*>(table), out, d, vocab, scale,
+                            copies)
                 : zb_launch(zb_embedding_f32_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, s, ids,
-                            reinterpret_cast<const __nv_bfloat16*>(table), out, d, vocab, scale);
+                            reinterpret_cast<const __nv_bfloat16*>(table), out, d, vocab, scale, copies);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }
@@ -691,6 +864,22 @@ int zb_sandwich_norm(const void* y, long long ldy, int y_f32, const int32_t* pai
   const SandwichArgs p = {y, ldy, pair_pos, pair_w, k, x, mult, w, w_next, eps, x_out, act, ld_act, d};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const cudaError_t e = y_f32 ? launch_sandwich<float>(p, act_f32, tokens, s) : launch_sandwich<__nv_bfloat16>(p, act_f32, tokens, s);
+  zb_count_launch(1);
+  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+}
+
+// x [tokens, streams, d]: x_out[t] = sum_s mix[s, t] x[s] + out[t] * y, act = rmsnorm(sum_s in[s] x_out[s]) * w.  y as in
+// zb_sandwich_norm; null: act alone, of x.  At most 8 streams; d as in zb_sandwich_norm.
+int zb_hyper_norm(const void* y, long long ldy, int y_f32, const int32_t* pair_pos, const float* pair_w, int k, const float* x, int streams,
+                  const float* mix, const float* out, const float* in, const float* w, float eps, float* x_out, void* act, long long ld_act,
+                  int act_f32, int tokens, int d, void* stream) {
+  if (tokens <= 0) return 0;
+  if (streams < 1 || streams > kMaxStreams || (act != nullptr && (w == nullptr || in == nullptr || ld_act < d))) return -70;
+  if (y != nullptr && (mix == nullptr || out == nullptr)) return -70;
+  const HyperArgs p = {y, ldy, y_f32, pair_pos, pair_w, k, x, streams, mix, out, in, w, eps, x_out, act, ld_act, act_f32, d};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const bool vec = d % 4 == 0 && (act == nullptr || ld_act % 4 == 0) && (y == nullptr || (ldy % 4 == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0));
+  const cudaError_t e = vec ? launch_hyper<4>(p, tokens, s) : launch_hyper<1>(p, tokens, s);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }

@@ -21,10 +21,11 @@ def _families():
     from .qwen3_5 import PRESETS as P_Q35, Qwen35Config, Qwen35Model
     from .qwen3_5_moe import PRESETS as P_Q35M, Qwen35MoeConfig, Qwen35MoeModel
     from .qwen3_moe import PRESETS as P_MOE, Qwen3MoeConfig, Qwen3MoeModel
+    from .sodotar import PRESETS as P_SOD, SodotarConfig, SodotarModel
     return [(LLAMA_PRESETS, LlamaConfig, LlamaModel), (P_MOE, Qwen3MoeConfig, Qwen3MoeModel),
             (P_Q35, Qwen35Config, Qwen35Model), (P_Q35M, Qwen35MoeConfig, Qwen35MoeModel),
             (P_LFM2, Lfm2Config, Lfm2Model), (P_DOP, DopuraxConfig, DopuraxModel),
-            (P_KIR, KirisunConfig, KirisunModel)]
+            (P_KIR, KirisunConfig, KirisunModel), (P_SOD, SodotarConfig, SodotarModel)]
 
 
 def preset_names() -> list[str]:
@@ -76,4 +77,7 @@ def model_class_for(config: dict):
     if kind == "kirisun":
         from .kirisun import KirisunConfig, KirisunModel
         return KirisunConfig, KirisunModel
+    if kind == "sodotar":
+        from .sodotar import SodotarConfig, SodotarModel
+        return SodotarConfig, SodotarModel
     raise ValueError(kind)

@@ -17,10 +17,12 @@ _lib.register_signature("zb_moe_gather", C.c_int, [C.c_void_p, C.c_void_p, C.c_v
 _lib.register_signature("zb_moe_finalize", C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int,
                                                       C.c_int, C.c_void_p], optional=False)
 _lib.register_signature("zb_moe_grouped_gemm", C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int,
-                                                          C.c_int, C.c_int, C.c_int, C.c_int, C.c_int, C.c_void_p],
+                                                          C.c_int, C.c_int, C.c_int, C.c_int, C.c_void_p, C.c_int, C.c_void_p],
                         optional=False)
 _lib.register_signature("zb_moe_grouped_f32", C.c_int, [C.c_void_p, C.c_longlong, C.c_void_p, C.c_int, C.c_void_p, C.c_void_p, C.c_longlong,
-                                                         C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_int, C.c_int, C.c_void_p])
+                                                         C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_int, C.c_int, C.c_void_p, C.c_void_p])
+_lib.register_signature("zb_moe_route", C.c_int, [C.c_void_p, C.c_longlong, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_int,
+                                                  C.c_int, C.c_void_p])
 
 
 class Backend(enum.Enum):
@@ -53,6 +55,32 @@ def router_topk(logits: torch.Tensor, k: int, renormalize: bool = True):
     w = torch.empty((t, k), dtype=torch.float32, device=logits.device)
     _lib.check(_lib.lib().zb_moe_router_topk(logits.data_ptr(), ids.data_ptr(), w.data_ptr(), t, e, k,
                                              logits.stride(0), int(renormalize), _lib.stream_ptr()), "zb_moe_router_topk")
+    return ids, w
+
+
+def route(logits: torch.Tensor, k: int, experts: int, correction: Optional[torch.Tensor] = None, shared: int = 0, e0: int = 0):
+    """Routing by softmax scores: s = softmax(logits[:, :experts]); the k experts with the largest s + correction, weighted by
+    their s divided by the sum (+ 1e-20).  `shared` experts run for every token, weighted by sigmoid(logits[:, experts]).
+    Returns (ids int32 [T, k + shared], weights float32): the choices first, then the shared ones.  Shared experts have the ids
+    0 .. shared - 1, expert e has shared + (e - e0) mod experts: the local experts of the rank that starts at e0 follow its
+    shared ones, so `moe_align(ids, 0, shared + local)` takes both."""
+    t = logits.shape[0]
+    assert logits.shape[1] >= experts + (1 if shared else 0)
+    if not logits.is_cuda:
+        s = torch.softmax(logits[:, :experts].float(), -1)
+        i = torch.topk(s if correction is None else s + correction.float(), k, dim=-1).indices
+        w = s.gather(1, i)
+        ids, w = shared + (i - e0) % experts, w / (w.sum(-1, keepdim=True) + 1e-20)
+        if shared:
+            ids = torch.cat([ids, torch.arange(shared).expand(t, shared)], 1)
+            w = torch.cat([w, torch.sigmoid(logits[:, experts:experts + 1].float()).expand(t, shared)], 1)
+        return ids.to(torch.int32).contiguous(), w.contiguous()
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == experts)
+    ids = torch.empty((t, k + shared), dtype=torch.int32, device=logits.device)
+    w = torch.empty((t, k + shared), dtype=torch.float32, device=logits.device)
+    _lib.check(_lib.lib().zb_moe_route(logits.data_ptr(), logits.stride(0), correction.data_ptr() if correction is not None else None, ids.data_ptr(),
+                                       w.data_ptr(), t, experts, k, shared, e0, _lib.stream_ptr()), "zb_moe_route")
     return ids, w
 
 
@@ -131,7 +159,9 @@ def deinterleave_gate_up(w: torch.Tensor):
 
 # Activations of the expert MLP (zml/moe/cutlass_flashinfer.zig:24-28 of the reference): the gated ones take an
 # interleaved gate|up weight, `relu2` a plain up projection.  The code is what the kernels' `swiglu` argument carries.
-ACTIVATIONS = {"none": 0, "swiglu": 1, "geglu": 2, "geglu_tanh": 3, "relu2": 4}
+# `clipped_glu`, with a limit per expert: g = min(gate, limit), u = up cut to +-limit, g * sigmoid(1.702 g) * (u + 1).
+ACTIVATIONS = {"none": 0, "swiglu": 1, "geglu": 2, "geglu_tanh": 3, "relu2": 4, "clipped_glu": 5}
+GATED = (1, 2, 3, 5)
 
 
 def activation_code(swiglu) -> int:
@@ -149,13 +179,23 @@ def _gate_act(g: torch.Tensor, code: int) -> torch.Tensor:
     return torch.nn.functional.silu(g)
 
 
-def grouped_gemm(xs: torch.Tensor, w: torch.Tensor, meta: torch.Tensor, swiglu=False, avg_tokens: int = 8):
-    """Per local expert e: out[rows_e] = xs[rows_e] @ w[e]^T.  `swiglu` True or "swiglu" / "geglu" / "geglu_tanh": w is
-    the interleaved gate/up weight [E, 2F, K] and out is act(gate) * up, [cap, F]; "relu2": relu(x w^T)^2."""
+def _gated_unit(g: torch.Tensor, u: torch.Tensor, code: int, limit: float) -> torch.Tensor:
+    if code == 5:
+        g, u = g.clamp_max(limit), u.clamp(-limit, limit)
+        return g * torch.sigmoid(1.702 * g) * (u + 1)
+    return _gate_act(g, code) * u
+
+
+def grouped_gemm(xs: torch.Tensor, w: torch.Tensor, meta: torch.Tensor, swiglu=False, avg_tokens: int = 8,
+                 limits: Optional[torch.Tensor] = None):
+    """Per local expert e: out[rows_e] = xs[rows_e] @ w[e]^T.  `swiglu` True or "swiglu" / "geglu" / "geglu_tanh" / "clipped_glu":
+    w is the interleaved gate/up weight [E, 2F, K] and out is the gated unit of the two, [cap, F]; "relu2": relu(x w^T)^2.
+    `limits` float32 [E]: of "clipped_glu"."""
     e_local, n, k = w.shape
     cap = xs.shape[0]
     code = activation_code(swiglu)
-    gated = 1 <= code <= 3
+    gated = code in GATED
+    assert (limits is not None) == (code == 5) and (limits is None or (limits.dtype == torch.float32 and limits.numel() == e_local))
     n_out = n // 2 if gated else n
     if not xs.is_cuda:
         out = torch.zeros((cap, n_out), dtype=xs.dtype)
@@ -167,29 +207,30 @@ def grouped_gemm(xs: torch.Tensor, w: torch.Tensor, meta: torch.Tensor, swiglu=F
             x = xs[a:b].float()
             if gated:
                 g, u = gate_up
-                out[a:b] = (_gate_act(x @ g[e].float().t(), code) * (x @ u[e].float().t())).to(xs.dtype)
+                out[a:b] = _gated_unit(x @ g[e].float().t(), x @ u[e].float().t(), code, float(limits[e]) if limits is not None else 0.0).to(xs.dtype)
             elif code == 4:
                 out[a:b] = torch.relu(x @ w[e].float().t()).square().to(xs.dtype)
             else:
                 out[a:b] = (x @ w[e].float().t()).to(xs.dtype)
         return out
     if xs.dtype == torch.float32:
-        return _grouped_f32(xs, None, 1, w, meta, cap, cap, code)
+        return _grouped_f32(xs, None, 1, w, meta, cap, cap, code, limits)
     assert xs.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and xs.is_contiguous() and w.is_contiguous()
     out = torch.empty((cap, n_out), dtype=xs.dtype, device=xs.device)
     _lib.check(_lib.lib().zb_moe_grouped_gemm(xs.data_ptr(), w.data_ptr(), out.data_ptr(), meta.data_ptr(), e_local, n, k,
-                                              cap, n_out, code, int(avg_tokens), _lib.stream_ptr()),
-               "zb_moe_grouped_gemm")
+                                              cap, n_out, code, limits.data_ptr() if limits is not None else None, int(avg_tokens),
+                                              _lib.stream_ptr()), "zb_moe_grouped_gemm")
     return out
 
 
-def _grouped_f32(x, pair, per: int, w, meta, cap: int, max_rows: int, code: int):
+def _grouped_f32(x, pair, per: int, w, meta, cap: int, max_rows: int, code: int, limits=None):
     """The fp32 grouped GEMM (libzb_cuda.so: moe_f32.cu); with `pair` the rows are gathered by its loads."""
     e, n, k = w.shape
     assert x.dtype == torch.float32 and w.dtype == torch.float32 and w.is_contiguous() and x.stride(1) == 1 and x.shape[1] == k
-    out = torch.empty((cap, n // 2 if 1 <= code <= 3 else n), dtype=torch.float32, device=x.device)
+    out = torch.empty((cap, n // 2 if code in GATED else n), dtype=torch.float32, device=x.device)
     _lib.check(_lib.lib().zb_moe_grouped_f32(x.data_ptr(), x.stride(0), pair.data_ptr() if pair is not None else None, per, w.data_ptr(),
-                                             out.data_ptr(), out.stride(0), meta.data_ptr(), e, n, k, max_rows, code, _lib.stream_ptr()),
+                                             out.data_ptr(), out.stride(0), meta.data_ptr(), e, n, k, max_rows, code,
+                                              limits.data_ptr() if limits is not None else None, _lib.stream_ptr()),
                "zb_moe_grouped_f32")
     return out
 
@@ -479,7 +520,7 @@ def pad_experts(gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor):
 
 
 def expert_rows(x: torch.Tensor, topk_ids: torch.Tensor, w_gate_up_il: torch.Tensor, w_down: torch.Tensor, e0: int = 0,
-                num_experts_total: Optional[int] = None, activation: str = "swiglu"):
+                num_experts_total: Optional[int] = None, activation: str = "swiglu", limits: Optional[torch.Tensor] = None):
     """The LOCAL experts' outputs before they are summed: (rows [T * k, D'], pair_pos [T * k]), bf16 or fp32 as x is.  Pair
     t * k + j has its row at pair_pos (-1: another rank's expert); routing weights are applied by whoever sums them."""
     t = x.shape[0]
@@ -488,10 +529,10 @@ def expert_rows(x: torch.Tensor, topk_ids: torch.Tensor, w_gate_up_il: torch.Ten
     avg = max(1, (t * k) // max(num_experts_total or e_local, 1))
     meta, sorted_pair, pair_pos = moe_align(topk_ids, e0, e_local)
     if x.is_cuda and x.dtype == torch.float32:
-        h = _grouped_f32(x, sorted_pair, k, w_gate_up_il, meta, t * k, t, activation_code(activation))
+        h = _grouped_f32(x, sorted_pair, k, w_gate_up_il, meta, t * k, t, activation_code(activation), limits)
         return _grouped_f32(h, None, 1, w_down, meta, t * k, t, 0), pair_pos
     xs = gather(x, sorted_pair, meta, e_local, k, t * k)
-    h = grouped_gemm(xs, w_gate_up_il, meta, swiglu=activation, avg_tokens=avg)
+    h = grouped_gemm(xs, w_gate_up_il, meta, swiglu=activation, avg_tokens=avg, limits=limits)
     return grouped_gemm(h, w_down, meta, swiglu=False, avg_tokens=avg), pair_pos
 
 

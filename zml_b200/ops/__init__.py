@@ -395,6 +395,17 @@ import os as _os
 _ATTN_TC = _os.environ.get("ZB_ATTN_TC", "1") != "0"
 
 
+def _tc_takes(q, k_cache, ext) -> bool:
+    l = _lib.lib()
+    ok = bool(l.zb_paged_prefill_tc_supported(q.shape[1], k_cache.shape[2], q.shape[2], k_cache.shape[1])) and q.stride(0) % 8 == 0
+    return ok and (ext is None or bool(l.zb_paged_prefill_tc_ext_supported(ext.cap, ext.pair)))
+
+
+def prefill_on_tc(q, k_cache, ext=None) -> bool:
+    """Whether `paged_prefill` (impl "auto") runs the tcgen05 kernel."""
+    return _ATTN_TC and _tc_takes(q, k_cache, ext)
+
+
 def paged_prefill(q, k_cache, v_cache, block_table, seq_lens, q_start, scale: float | None = None,
                   window: int = 0, out=None, total_q_blocks: int | None = None, impl: str = "auto", ext=None):
     """Varlen causal attention of new tokens against the paged KV (which already holds them).
@@ -417,8 +428,7 @@ def paged_prefill(q, k_cache, v_cache, block_table, seq_lens, q_start, scale: fl
         out = torch.empty((t, hq, hd), dtype=q.dtype, device=q.device)
     nqb = total_q_blocks if total_q_blocks is not None else t // 64 + b
     l = _lib.lib()
-    tc_ok = bool(l.zb_paged_prefill_tc_supported(hq, hkv, hd, page)) and q.stride(0) % 8 == 0
-    tc_ok = tc_ok and (ext is None or bool(l.zb_paged_prefill_tc_ext_supported(ext.cap)))
+    tc_ok = _tc_takes(q, k_cache, ext)
     if impl == "tc" and not tc_ok:
         raise ValueError(f"the tensor-core prefill kernel does not take hq={hq} hkv={hkv} hd={hd} page={page}")
     if tc_ok and (impl == "tc" or (impl == "auto" and _ATTN_TC)):

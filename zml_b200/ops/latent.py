@@ -9,6 +9,10 @@ Two formulations of the same attention, chosen by `latent_attention`:
 * expanded (`prefill`): the visible latents of the batch are gathered from the pages and projected to keys and
   values of every head, which costs a third of the products in the latent space when a chunk has many queries per key.
 
+The output gate and the sink (one learned number per head, a term exp(sink) of the softmax denominator) are optional, and so
+is the low-rank latent of the queries.  Rotated parts are turned in neighbouring pairs (2i, 2i + 1); `halves_to_pairs` gives
+the order of rows that brings projections of a design with pairs (i, i + rot / 2) into that layout.
+
 bf16 runs on the tensor cores, fp32 on the FMA pipes; CPU tensors take the plain torch branch.
 """
 from __future__ import annotations
@@ -24,19 +28,23 @@ from . import _lib
 _p, _i, _ll, _f = C.c_void_p, C.c_int, C.c_longlong, C.c_float
 _lib.register_signature("zb_latent_prep", _i, [_p, _ll, _p, _p, _p, _p, _p, _p, _ll, _p, _ll, _ll, _f, _i, _i, _i, _i, _i, _i, _p])
 _lib.register_signature("zb_latent_absorb", _i, [_p, _ll, _ll, _p, _ll, _p, _ll, _ll, _p, _ll, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _p])
-_lib.register_signature("zb_latent_attend", _i, [_p, _p, _ll, _p, _ll, _p, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _i, _i, _p])
+_lib.register_signature("zb_latent_attend", _i, [_p, _p, _ll, _p, _ll, _p, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p, _p, _i, _i, _i, _p])
 _lib.register_signature("zb_latent_gather", _i, [_p, _ll, _p, _i, _i, _p, _p, _i, _p, _ll, _i, _i, _i, _i, _i, _p])
 _lib.register_signature("zb_latent_q_pack", _i, [_p, _ll, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p])
 _lib.register_signature("zb_latent_prefill_tc_supported", _i, [_i, _i, _i, _i])
 _lib.register_signature("zb_latent_prefill_tc", _i, [_p, _p, _ll, _p, _ll, _i, _p, _ll, _p, _ll, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _i,
-                                                     _i, _i, _f, _p])
+                                                     _i, _i, _f, _p, _p])
 _lib.register_signature("zb_latent_decode_supported", _i, [_i, _i])
 _lib.register_signature("zb_latent_decode_groups", _i, [_i])
-_lib.register_signature("zb_latent_decode", _i, [_p, _p, _i, _p, _ll, _p, _i, _i, _p, _i, _i, _i, _i, _f, _i, _p])
+_lib.register_signature("zb_latent_decode", _i, [_p, _p, _i, _p, _ll, _p, _i, _i, _p, _i, _i, _i, _i, _f, _p, _i, _p])
 
 
 def _ptr(t: Optional[torch.Tensor]):
     return None if t is None else t.data_ptr()
+
+
+def _ld(t: Optional[torch.Tensor]) -> int:
+    return 0 if t is None else t.stride(0)
 
 
 def _up(n: int, m: int) -> int:
@@ -51,7 +59,7 @@ class LatentDims:
     rot: int            # rotated ones (keys: one such part for every head)
     vdim: int
     rank: int           # latent size
-    q_rank: int
+    q_rank: int         # of the queries' latent, 0: none
     window: int         # keys a position sees, itself included; <= 0: all
     scale: float
     base: float         # of the rotation frequencies
@@ -70,6 +78,11 @@ class LatentDims:
         return (float(self.base) ** (-i / self.rot)).to(torch.float32).to(device)
 
 
+def halves_to_pairs(rot: int) -> torch.Tensor:
+    """Row order that turns a rotated part with pairs (i, i + rot / 2) into one with pairs (2i, 2i + 1)."""
+    return torch.arange(rot).reshape(2, rot // 2).t().reshape(-1)
+
+
 def rotate_reference(x, positions, inv_freq):
     """Adjacent pairs of x [..., T, rot] (T second from the right or with heads between) turned by position * frequency."""
     a = positions.float()[:, None] * inv_freq[None]
@@ -86,10 +99,11 @@ def _rms(x, w, eps):
 # ---------------------------------------------------------------------------- norms, rotation, cache write
 def prep(proj, q_norm, c_norm, inv_freq, positions, slots, cache, eps: float, d: LatentDims):
     """proj [T, >= q_rank + rank + rot] (query latent | latent | shared key part): returns the normed query latent
-    [T, q_rank] and writes the normed latent and the rotated key part into cache [pages, page, row] at `slots`."""
+    [T, q_rank] (None without one) and writes the normed latent and the rotated key part into cache [pages, page, row] at
+    `slots`."""
     t = proj.shape[0]
     if not proj.is_cuda:
-        cq = _rms(proj[:, :d.q_rank].float(), q_norm, eps).to(proj.dtype)
+        cq = _rms(proj[:, :d.q_rank].float(), q_norm, eps).to(proj.dtype) if d.q_rank else None
         c = _rms(proj[:, d.q_rank:d.q_rank + d.rank].float(), c_norm, eps)
         kr = rotate_reference(proj[:, d.q_rank + d.rank:d.q_rank + d.rank + d.rot], positions, inv_freq)
         flat = cache.view(-1, cache.shape[-1])
@@ -99,9 +113,9 @@ def prep(proj, q_norm, c_norm, inv_freq, positions, slots, cache, eps: float, d:
         flat[idx, d.rot_off:d.rot_off + d.rot] = kr[ok].to(cache.dtype)
         return cq
     assert proj.stride(1) == 1 and cache.is_contiguous() and cache.dtype == proj.dtype and cache.shape[-1] == d.row
-    cq = torch.empty((t, d.q_rank), dtype=proj.dtype, device=proj.device)
+    cq = torch.empty((t, d.q_rank), dtype=proj.dtype, device=proj.device) if d.q_rank else None
     _lib.check(_lib.lib().zb_latent_prep(
-        _ptr(proj), proj.stride(0), _ptr(q_norm), _ptr(c_norm), _ptr(inv_freq), _ptr(positions), _ptr(slots), _ptr(cq), cq.stride(0),
+        _ptr(proj), proj.stride(0), _ptr(q_norm), _ptr(c_norm), _ptr(inv_freq), _ptr(positions), _ptr(slots), _ptr(cq), d.q_rank,
         _ptr(cache), d.row, cache.shape[0] * cache.shape[1], float(eps), d.q_rank, d.rank, d.rot, d.rot_off,
         int(proj.dtype == torch.float32), t, _lib.stream_ptr()), "zb_latent_prep")
     return cq
@@ -127,20 +141,20 @@ def absorb_q(q, w_uk_t, inv_freq, positions, d: LatentDims):
 
 def absorb_out(o, w_uv, gate, d: LatentDims):
     """o [T, H, rot_off] (latent-space results) -> sigmoid(gate) * (o w_uv^T) [T, H * vdim]; w_uv [H, vdim, rank],
-    gate [T, H * vdim] (row stride free)."""
+    gate [T, H * vdim] (row stride free) or None."""
     t = o.shape[0]
     if not o.is_cuda:
         y = torch.einsum("thk,hnk->thn", o[..., :d.rank].float(), w_uv.float()).reshape(t, -1)
-        return (y * torch.sigmoid(gate.float())).to(o.dtype)
+        return (y if gate is None else y * torch.sigmoid(gate.float())).to(o.dtype)
     out = torch.empty((t, d.heads * d.vdim), dtype=o.dtype, device=o.device)
-    assert gate.stride(1) == 1 and w_uv.is_contiguous() and gate.dtype == o.dtype
+    assert w_uv.is_contiguous() and (gate is None or (gate.stride(1) == 1 and gate.dtype == o.dtype))
     _lib.check(_lib.lib().zb_latent_absorb(
-        _ptr(o), o.stride(0), o.stride(1), _ptr(w_uv), d.rank, _ptr(out), out.stride(0), d.vdim, _ptr(gate), gate.stride(0), None, None, 0,
+        _ptr(o), o.stride(0), o.stride(1), _ptr(w_uv), d.rank, _ptr(out), out.stride(0), d.vdim, _ptr(gate), _ld(gate), None, None, 0,
         0, 0, t, d.heads, d.vdim, d.rank, int(o.dtype == torch.float32), _lib.stream_ptr()), "zb_latent_absorb")
     return out
 
 
-def attend_reference(q, cache, block_table, q_start, seq_lens, d: LatentDims):
+def attend_reference(q, cache, block_table, q_start, seq_lens, d: LatentDims, sink=None):
     out = torch.zeros((q.shape[0], d.heads, d.rot_off), dtype=q.dtype, device=q.device)
     flat = cache.view(-1, cache.shape[-1])
     page = cache.shape[1]
@@ -156,16 +170,19 @@ def attend_reference(q, cache, block_table, q_start, seq_lens, d: LatentDims):
         if d.window > 0:
             vis &= key[None] > pos[:, None] - d.window
         sc = torch.einsum("thc,kc->htk", q[a:b].float(), rows) * d.scale
-        pr = torch.softmax(sc.masked_fill(~vis[None], float("-inf")), -1)
+        sc = sc.masked_fill(~vis[None], float("-inf"))
+        if sink is not None:
+            sc = torch.cat([sc, sink.float()[:, None, None].expand(-1, sc.shape[1], 1)], -1)
+        pr = torch.softmax(sc, -1)[..., :n]
         out[a:b, :, :d.rank] = torch.einsum("htk,kc->thc", pr, rows[:, :d.rank]).to(q.dtype)
     return out
 
 
-def attend(q, cache, block_table, q_start, seq_lens, d: LatentDims, decode: bool = False, num_splits: int = 1):
+def attend(q, cache, block_table, q_start, seq_lens, d: LatentDims, decode: bool = False, num_splits: int = 1, sink=None):
     """Windowed causal attention of q [T, H, row] (`absorb_q`) against the cached rows; a sequence's queries are its last
-    tokens.  Returns [T, H, rot_off]."""
+    tokens; sink fp32 [H] or None.  Returns [T, H, rot_off]."""
     if not q.is_cuda:
-        return attend_reference(q, cache, block_table, q_start, seq_lens, d)
+        return attend_reference(q, cache, block_table, q_start, seq_lens, d, sink)
     t = q.shape[0]
     out = torch.empty((t, d.heads, d.rot_off), dtype=q.dtype, device=q.device)
     assert block_table.is_contiguous() and cache.dtype == q.dtype and q.is_contiguous()
@@ -173,11 +190,11 @@ def attend(q, cache, block_table, q_start, seq_lens, d: LatentDims, decode: bool
     if decode and q.dtype == torch.bfloat16 and l.zb_latent_decode_supported(d.row, d.rot_off):
         _lib.check(l.zb_latent_decode(
             _ptr(q), _ptr(cache), d.row, _ptr(out), d.rot_off, _ptr(block_table), block_table.shape[1], cache.shape[1], _ptr(seq_lens), t,
-            d.heads, d.rot_off, d.window, float(d.scale), int(num_splits), _lib.stream_ptr()), "zb_latent_decode")
+            d.heads, d.rot_off, d.window, float(d.scale), _ptr(sink), int(num_splits), _lib.stream_ptr()), "zb_latent_decode")
         return out
     _lib.check(l.zb_latent_attend(
         _ptr(q), _ptr(cache), d.row, _ptr(out), d.rot_off, _ptr(block_table), block_table.shape[1], cache.shape[1], d.heads, d.rank, d.rot,
-        d.rot_off, d.window, float(d.scale), _ptr(q_start), _ptr(seq_lens), seq_lens.shape[0], t, int(q.dtype == torch.float32),
+        d.rot_off, d.window, float(d.scale), _ptr(sink), _ptr(q_start), _ptr(seq_lens), seq_lens.shape[0], t, int(q.dtype == torch.float32),
         _lib.stream_ptr()), "zb_latent_attend")
     return out
 
@@ -234,40 +251,41 @@ def pack_q(q, inv_freq, positions, d: LatentDims):
     return out
 
 
-def attend_expanded(qp, gate, lat, kv, rot_out: int, plan, meta, d: LatentDims):
+def attend_expanded(qp, gate, lat, kv, rot_out: int, plan, meta, d: LatentDims, sink=None):
     """sigmoid(gate) * windowed causal attention of packed queries over expanded keys and values: [T, H * vdim]."""
     key_start, first_key, rows = plan
     t = qp.shape[0]
     out = torch.empty((t, d.heads * d.vdim), dtype=qp.dtype, device=qp.device)
     blocks = sum((b - a + 255) // 256 for a, b in zip(meta.q_start_host, meta.q_start_host[1:]))
     _lib.check(_lib.lib().zb_latent_prefill_tc(
-        _ptr(qp), _ptr(kv), kv.stride(0), _ptr(lat), lat.stride(0), rot_out, _ptr(out), out.stride(0), _ptr(gate), gate.stride(0),
+        _ptr(qp), _ptr(kv), kv.stride(0), _ptr(lat), lat.stride(0), rot_out, _ptr(out), out.stride(0), _ptr(gate), _ld(gate),
         _ptr(meta.q_start), _ptr(meta.seq_lens), meta.seq_lens.shape[0], _ptr(key_start), _ptr(first_key), t, rows, blocks, d.heads, d.dim,
-        d.rot, d.vdim, d.window, float(d.scale), _lib.stream_ptr()), "zb_latent_prefill_tc")
+        d.rot, d.vdim, d.window, float(d.scale), _ptr(sink), _lib.stream_ptr()), "zb_latent_prefill_tc")
     return out
 
 
-def prefill(q, gate, w_ukv, inv_freq, cache, meta, d: LatentDims):
+def prefill(q, gate, w_ukv, inv_freq, cache, meta, d: LatentDims, sink=None):
     """The expanded formulation on the tensor cores (bf16)."""
     lat, kv, rot_out, plan = expand(cache, w_ukv, meta, d)
-    return attend_expanded(pack_q(q, inv_freq, meta.positions, d), gate, lat, kv, rot_out, plan, meta, d)
+    return attend_expanded(pack_q(q, inv_freq, meta.positions, d), gate, lat, kv, rot_out, plan, meta, d, sink)
 
 
 def _expands(q, gate, meta, d: LatentDims) -> bool:
     return (q.is_cuda and q.dtype == torch.bfloat16 and meta.is_prefill and meta.q_start_host is not None and meta.seq_lens_host is not None
             and bool(_lib.lib().zb_latent_prefill_tc_supported(d.dim, d.rot, d.vdim, d.rank)) and q.stride(0) % 8 == 0
-            and gate.stride(0) % 8 == 0)
+            and _ld(gate) % 8 == 0)
 
 
 # ---------------------------------------------------------------------------- the layer's attention
-def latent_attention(q, gate, w_uk_t, w_ukv, inv_freq, cache, meta, d: LatentDims):
-    """sigmoid(gate) * attention of one step: q [T, H * (dim + rot)] unrotated, gate [T, H * vdim], w_uk_t [H, rank, dim],
-    w_ukv [H dim + H vdim, rank]; `meta` is the step's AttnMeta, the new tokens' cache rows are already written."""
+def latent_attention(q, gate, w_uk_t, w_ukv, inv_freq, cache, meta, d: LatentDims, sink=None):
+    """sigmoid(gate) * attention of one step: q [T, H * (dim + rot)] unrotated, gate [T, H * vdim] or None, w_uk_t [H, rank, dim],
+    w_ukv [H dim + H vdim, rank], sink fp32 [H] or None; `meta` is the step's AttnMeta, the new tokens' cache rows are already
+    written."""
     if _expands(q, gate, meta, d):
-        return prefill(q, gate, w_ukv, inv_freq, cache, meta, d)
+        return prefill(q, gate, w_ukv, inv_freq, cache, meta, d, sink)
     q_start = meta.q_start
     if q_start is None:
         q_start = torch.arange(q.shape[0] + 1, dtype=torch.int32, device=q.device)
     ql = absorb_q(q, w_uk_t, inv_freq, meta.positions, d)
-    o = attend(ql, cache, meta.block_table, q_start, meta.seq_lens, d, decode=not meta.is_prefill, num_splits=meta.num_splits or 1)
+    o = attend(ql, cache, meta.block_table, q_start, meta.seq_lens, d, decode=not meta.is_prefill, num_splits=meta.num_splits or 1, sink=sink)
     return absorb_out(o, w_ukv[d.heads * d.dim:].view(d.heads, d.vdim, d.rank), gate, d)

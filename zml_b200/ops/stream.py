@@ -1,5 +1,5 @@
-"""Layer glue of decoders with an fp32 residual stream: embedding, the norms behind and in front of a sublayer, and the
-convolution in front of a mixer (libzb_cuda.so: stream_f32.cu).
+"""Layer glue of decoders with an fp32 residual stream: embedding, the norms behind and in front of a sublayer, the
+convolution in front of a mixer, and hyper-connections (several streams) (libzb_cuda.so: stream_f32.cu).
 
 All of it works on the flattened varlen batch of the engine (`q_start`, `seq_lens`, `slots`, as in
 `ops.linear_attn`).  Activations that a projection reads are written in the model's dtype (bf16 or fp32); the stream,
@@ -16,13 +16,15 @@ import torch
 from . import _lib
 
 _p, _i, _ll, _f = C.c_void_p, C.c_int, C.c_longlong, C.c_float
-_lib.register_signature("zb_embedding_f32", _i, [_p, _p, _i, _p, _i, _i, _i, _f, _p])
+_lib.register_signature("zb_embedding_f32", _i, [_p, _p, _i, _p, _i, _i, _i, _f, _i, _p])
+_lib.register_signature("zb_hyper_norm", _i, [_p, _ll, _i, _p, _p, _i, _p, _i, _p, _p, _p, _p, _f, _p, _p, _ll, _i, _i, _i, _p])
 _lib.register_signature("zb_sandwich_norm", _i, [_p, _ll, _i, _p, _p, _i, _p, _f, _p, _p, _f, _p, _p, _ll, _i, _i, _i, _p])
 _lib.register_signature("zb_stream_conv", _i, [_p, _p, _p, _p, _p, _p, _i, _ll, _ll, _i, _i, _i, _i, _p, _p, _i, _i, _p])
 _lib.register_signature("zb_post_norm", _i, [_p, _ll, _i, _p, _f, _p, _f, _p, _p, _ll, _i, _i, _i, _p, _p, _p, _p, _p, _ll, _ll,
                                              _i, _i, _i, _p, _p])
 
 MAX_TAPS = 8
+MAX_STREAMS = 8
 CONV_BLOCK = 32          # tokens per block of the convolution kernel
 
 
@@ -30,14 +32,16 @@ def _ptr(t: Optional[torch.Tensor]):
     return None if t is None else t.data_ptr()
 
 
-def embedding_f32(ids, table, scale: float = 1.0):
-    """Rows of `table` (bf16 or fp32) times `scale`, as fp32 [T, d]."""
+def embedding_f32(ids, table, scale: float = 1.0, streams: int = 0):
+    """Rows of `table` (bf16 or fp32) times `scale`, as fp32 [T, d]; with `streams` as [T, streams, d], equal copies."""
+    shape = (ids.shape[0], streams, table.shape[1]) if streams else (ids.shape[0], table.shape[1])
     if not table.is_cuda:
-        return table[ids.long()].float() * scale
+        x = table[ids.long()].float() * scale
+        return x[:, None].expand(shape).contiguous() if streams else x
     assert ids.dtype == torch.int32 and table.is_contiguous()
-    out = torch.empty((ids.shape[0], table.shape[1]), dtype=torch.float32, device=table.device)
+    out = torch.empty(shape, dtype=torch.float32, device=table.device)
     _lib.check(_lib.lib().zb_embedding_f32(_ptr(ids), _ptr(table), int(table.dtype == torch.float32), _ptr(out), ids.shape[0],
-                                           table.shape[1], table.shape[0], float(scale), _lib.stream_ptr()), "zb_embedding_f32")
+                                           table.shape[1], table.shape[0], float(scale), max(1, streams), _lib.stream_ptr()), "zb_embedding_f32")
     return out
 
 
@@ -199,3 +203,44 @@ def sandwich_norm(x, y=None, w=None, mult: float = 1.0, w_next=None, eps: float 
         _ptr(x), float(mult), _ptr(w), _ptr(w_next), float(eps), _ptr(x) if keep_x and rows is not None else None, _ptr(act), pad8(d),
         int(act_dtype == torch.float32), t, d, _lib.stream_ptr()), "zb_sandwich_norm")
     return (x if keep_x else None), act
+
+
+# ------------------------------------------------------------------ hyper-connections
+@dataclass
+class HyperMix:
+    """Coefficients of one sublayer with hyper-connections, fp32: it reads sum_s inp[s] x_s, and its output y gives
+    x_t <- sum_s mix[s, t] x_s + out[t] * y."""
+    inp: torch.Tensor                     # [streams]
+    mix: torch.Tensor                     # [streams, streams]
+    out: torch.Tensor                     # [streams]
+
+
+def hyper_norm(x, y=None, behind: Optional[HyperMix] = None, inp=None, w=None, eps: float = 1e-6, act_dtype=None):
+    """The update of the streams behind a sublayer (`behind`) and the norm in front of the next one, which reads the mix `inp`
+    [streams] of them, in one launch: act = rmsnorm(sum_s inp[s] x_s) * w in `act_dtype` ([T, d] with zero columns up to a
+    multiple of 8).  x fp32 [T, streams, d]; y [T, >= d] (bf16 or fp32) or `ExpertRows`; without y, act of x itself; without w,
+    no act.  Returns (x_new, act or None); x is overwritten on CUDA."""
+    t, s, d = x.shape
+    if not x.is_cuda:
+        if y is not None:
+            v = y.sum(d) if isinstance(y, ExpertRows) else y[:, :d].float()
+            x = torch.einsum("st,nsd->ntd", behind.mix, x) + behind.out[None, :, None] * v[:, None]
+        act = None
+        if w is not None:
+            act = rms_norm_reference(torch.einsum("s,nsd->nd", inp, x), w, eps)
+            act = torch.nn.functional.pad(act, (0, pad8(d) - d)).to(act_dtype)
+        return x, act
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    rows, pos, pw, k = y, None, None, 0
+    if isinstance(y, ExpertRows):
+        rows, pos, pw, k = y.rows, y.pair_pos, y.weights, y.weights.shape[1]
+        assert pw.dtype == torch.float32 and pw.is_contiguous()
+    assert rows is None or (rows.stride(1) == 1 and rows.shape[1] >= d and rows.dtype in (torch.float32, torch.bfloat16))
+    assert w is None or (w.dtype == inp.dtype == torch.float32 and inp.numel() == s and w.numel() == d)
+    act = torch.empty((t, pad8(d)), dtype=act_dtype, device=x.device) if w is not None else None
+    mix, out = (behind.mix, behind.out) if y is not None else (None, None)
+    _lib.check(_lib.lib().zb_hyper_norm(
+        _ptr(rows), rows.stride(0) if rows is not None else 0, int(rows is not None and rows.dtype == torch.float32), _ptr(pos), _ptr(pw), k,
+        _ptr(x), s, _ptr(mix), _ptr(out), _ptr(inp if w is not None else None), _ptr(w), float(eps), _ptr(x) if rows is not None else None,
+        _ptr(act), pad8(d), int(act_dtype == torch.float32), t, d, _lib.stream_ptr()), "zb_hyper_norm")
+    return x, act
