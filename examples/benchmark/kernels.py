@@ -61,6 +61,7 @@ class Args:
     splits: int = 0          # decode_attention: KV chunks per sequence (0: the planner's choice)
     w4: int = 0              # moe: 1 = NVFP4 expert weights de-quantised inside the grouped GEMM
     window: int = 4096       # latent and gated attention: keys a position sees; differential attention: its chunk
+    sink: int = 0            # latent attention: 1 = a sink per head and no output gate
     copies: int = 0          # operand copies to rotate through (0: enough to exceed the L2)
     help = __doc__
 
@@ -239,17 +240,18 @@ def bench_latent_prefill(a: Args) -> None:
     meta = SimpleNamespace(is_prefill=True, q_start_host=qs, seq_lens_host=sl, q_start=i32(qs), seq_lens=i32(sl), plans={}, block_table=bt,
                            positions=torch.arange(a.seqlen, dtype=torch.int32, device="cuda").repeat(a.batch))
     q = torch.randn(t, d.heads * 192, device="cuda").bfloat16()
-    gate = torch.randn(t, d.heads * 128, device="cuda").bfloat16()
+    gate = None if a.sink else torch.randn(t, d.heads * 128, device="cuda").bfloat16()
+    sink = torch.randn(d.heads, device="cuda") if a.sink else None
     w = torch.randn(d.heads * 256, 512, device="cuda").bfloat16() * 0.05
     inv = d.inv_freq("cuda")
     pairs = sum(min(i + 1, a.window) for i in range(a.seqlen)) * a.batch
     flops = 2.0 * pairs * d.heads * (192 + 128)
-    ms = timed([lambda c=c: lat.prefill(q, gate, w, inv, c, meta, d) for c in caches], a.iters, a.warmup)
+    ms = timed([lambda c=c: lat.prefill(q, gate, w, inv, c, meta, d, sink) for c in caches], a.iters, a.warmup)
     report(a, ms, t * d.heads * (192 + 256) * 2, flops + 2.0 * t * 512 * d.heads * 256, {"part": "whole", "batch": a.batch, "seqlen": a.seqlen, "heads": a.hq, "window": a.window})
     shape = {"batch": a.batch, "seqlen": a.seqlen, "heads": a.hq, "window": a.window}
     x, kv, rot_out, plan = lat.expand(caches[0], w, meta, d)
     qp = lat.pack_q(q, inv, meta.positions, d)
-    ms = timed([lambda: lat.attend_expanded(qp, gate, x, kv, rot_out, plan, meta, d)], a.iters, a.warmup)
+    ms = timed([lambda: lat.attend_expanded(qp, gate, x, kv, rot_out, plan, meta, d, sink)], a.iters, a.warmup)
     report(a, ms, t * d.heads * (192 + 192 + 128 + 128) * 2, flops, dict(shape, part="attention kernel"))
     ms = timed([lambda: lat.pack_q(q, inv, meta.positions, d)], a.iters, a.warmup)
     report(a, ms, t * d.heads * 192 * 4, 0, dict(shape, part="query packing"))
@@ -260,7 +262,8 @@ def bench_latent_prefill(a: Args) -> None:
 def bench_latent_decode(a: Args) -> None:
     lat, d, bt, caches = _latent(a)
     q = torch.randn(a.batch, d.heads * 192, device="cuda").bfloat16()
-    gate = torch.randn(a.batch, d.heads * 128, device="cuda").bfloat16()
+    gate = None if a.sink else torch.randn(a.batch, d.heads * 128, device="cuda").bfloat16()
+    sink = torch.randn(d.heads, device="cuda") if a.sink else None
     uk = [torch.randn(d.heads, 512, 128, device="cuda").bfloat16() for _ in range(8)]
     uv = [torch.randn(d.heads, 128, 512, device="cuda").bfloat16() for _ in range(8)]
     inv, pos = d.inv_freq("cuda"), torch.full((a.batch,), a.seqlen - 1, dtype=torch.int32, device="cuda")
@@ -269,9 +272,9 @@ def bench_latent_decode(a: Args) -> None:
     splits = a.splits or lat.decode_plan_splits(a.batch, d, a.seqlen)
     keys = a.batch * min(a.seqlen, a.window)
     shape = {"batch": a.batch, "seqlen": a.seqlen, "heads": a.hq, "window": a.window, "splits": splits}
-    ms = timed_graph([lambda c=c: lat.attend(ql, c, bt, qs, sl, d, decode=True, num_splits=splits) for c in caches], a.iters, a.warmup)
+    ms = timed_graph([lambda c=c: lat.attend(ql, c, bt, qs, sl, d, decode=True, num_splits=splits, sink=sink) for c in caches], a.iters, a.warmup)
     report(a, ms, keys * d.row * 2, 2.0 * keys * d.heads * (576 + 512), dict(shape, part="attention kernel"))
-    o = lat.attend(ql, caches[0], bt, qs, sl, d, decode=True, num_splits=splits)
+    o = lat.attend(ql, caches[0], bt, qs, sl, d, decode=True, num_splits=splits, sink=sink)
     wb = d.heads * 512 * 128 * 2
     ms = timed_graph([lambda w=w: lat.absorb_q(q, w, inv, pos, d) for w in uk], a.iters, a.warmup)
     report(a, ms, wb, 2.0 * a.batch * d.heads * 512 * 128, dict(shape, part="queries into the latent space"))

@@ -11,7 +11,7 @@ import torch
 
 sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
 import sodotar_oracle as oracle  # noqa: E402
-from sodotar_util import CONFIGS, TOL, attn, checkpoint, config, engine, run_portions, tokens  # noqa: E402
+from sodotar_util import CONFIGS, TOL, attn, case_for, checkpoint, config, engine, run_portions, tokens  # noqa: E402
 from zml_b200 import safetensors  # noqa: E402
 from zml_b200.models import hub  # noqa: E402
 from zml_b200.models.common import SamplingStrategy, detect_model_type  # noqa: E402
@@ -53,16 +53,16 @@ def row_errors(got, want):
 
 
 def check(got, want, dtype, what=""):
-    """Every row in fp32.  In bf16 a close call between two experts may fall the other way: one row in ten may be off."""
     e = row_errors(np.asarray(got, dtype=np.float64), want)
     over = np.nonzero(e > TOL[dtype])[0]
-    assert len(over) <= (len(e) // 10 if dtype == torch.bfloat16 else 0), (what, len(over), over[:5], e[over[:5]], e.max())
+    assert len(over) == 0 and np.median(e) < TOL[dtype] / 2, (what, len(over), over[:5], e[over[:5]], e.max(), np.median(e))
 
 
 @pytest.mark.parametrize("target", TARGETS)
-@pytest.mark.parametrize("name", sorted(CONFIGS))
+@pytest.mark.parametrize("name", [n for n in sorted(CONFIGS) if "," not in n])
 def test_whole_decode_and_portions_agree_with_the_oracle(repos, name, target):
     device, dtype = target
+    name = case_for(name, dtype)
     path, _, _ = repos(name)
     toks, want = expected(repos, name, 150, 1)
     eng = engine(path, device, dtype, max_tokens=192)
@@ -91,6 +91,7 @@ def test_stream_behind_every_layer(repos, name, target):
 @pytest.mark.parametrize("name", ["mixed", "odd"])
 def test_token_by_token_from_the_first_one(repos, name, target):
     device, dtype = target
+    name = case_for(name, dtype)
     path, _, _ = repos(name)
     toks, want = expected(repos, name, 80, 2)
     eng = engine(path, device, dtype, max_tokens=128)
@@ -102,8 +103,9 @@ def test_token_by_token_from_the_first_one(repos, name, target):
 def test_mixed_batches_equal_each_request_alone(repos, target):
     """Unequal requests in one batch, portions beside single tokens, requests that pause, end and hand on pages."""
     device, dtype = target
-    path, cfg, _ = repos("mixed")
-    reqs = {i: expected(repos, "mixed", n, 10 + i) for i, n in enumerate((131, 40, 1, 97, 70, 3))}
+    name = case_for("mixed", dtype)
+    path, cfg, _ = repos(name)
+    reqs = {i: expected(repos, name, n, 10 + i) for i, n in enumerate((131, 40, 1, 97, 70, 3))}
     eng = engine(path, device, dtype, max_tokens=384)
     rng = np.random.default_rng(5)
     live, at, got, waiting, pages0 = {}, {}, {i: [] for i in reqs}, list(reqs), eng.pool.num_free
@@ -136,8 +138,9 @@ def test_mixed_batches_equal_each_request_alone(repos, target):
 @pytest.mark.parametrize("target", TARGETS)
 def test_long_decoding_passes_chunks_and_pages(repos, target):
     device, dtype = target
-    path, _, _ = repos("mixed")
-    toks, want = expected(repos, "mixed", 300, 3)
+    name = case_for("mixed", dtype)
+    path, _, _ = repos(name)
+    toks, want = expected(repos, name, 300, 3)
     eng = engine(path, device, dtype, max_tokens=320)
     check(run_portions(eng, toks, [5, 1]), want, dtype)
 

@@ -67,17 +67,18 @@ ZB_DEVICE void st_elems(float* p, const float (&v)[V]) {
   else *p = v[0];
 }
 
-// One CTA per token, one warp per head; NR groups of V neighbouring elements per lane.
+// One CTA per token, L lanes (a warp or half of one) per head; NR groups of V neighbouring elements per lane.
 constexpr int kPrepThreads = 256;
 
-template <typename A, int NR, int V>
+template <typename A, int NR, int V, int L>
 __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrepArgs p) {
   extern __shared__ __align__(16) float prep_smem[];      // [rot / 2] (cos, sin) | [warps][rot] the rotated part's elements
   zb_pdl_launch();
   zb_pdl_wait();
-  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot / 2;
+  const int t = blockIdx.x, team = threadIdx.x / L, lane = threadIdx.x % L, half = p.rot / 2;
+  const uint32_t members = L == 32 ? 0xffffffffu : 0xffffu << (threadIdx.x & 16);
   float2* cs = reinterpret_cast<float2*>(prep_smem);
-  float* row = prep_smem + p.rot + warp * p.rot;
+  float* row = prep_smem + p.rot + team * p.rot;
   const float pos = static_cast<float>(p.positions[t]);
   for (int i = threadIdx.x; i < half; i += kPrepThreads) {
     float sn, c;
@@ -90,7 +91,7 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
   const bool slot_ok = slot >= 0 && slot < p.num_rows;
   const A* in = reinterpret_cast<const A*>(p.in) + t * p.ld_in;
   const int keys = p.hkv * p.maps, heads = p.hq + keys + p.hkv;
-  for (int h = warp; h < heads; h += kPrepThreads / 32) {
+  for (int h = team; h < heads; h += kPrepThreads / L) {
     const bool is_q = h < p.hq, is_v = h >= p.hq + keys;
     if (!is_q && !slot_ok) continue;
     const int u = is_q ? h : (is_v ? h - p.hq - keys : h - p.hq);        // row among its kind
@@ -104,7 +105,7 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
     float ss = 0.f;
 #pragma unroll
     for (int r = 0; r < NR; ++r) {
-      const int i = (lane + 32 * r) * V;
+      const int i = (lane + L * r) * V;
 #pragma unroll
       for (int e = 0; e < V; ++e) v[r][e] = 0.f;
       if (i < n) ld_elems<V>(v[r], src + i);
@@ -113,11 +114,16 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
     }
     if (!is_v) {
       const float* nw = is_q ? p.q_norm : p.k_norm;
-      const float inv = nw != nullptr ? 1.f / sqrtf(zb_warp_sum(ss) / static_cast<float>(n) + p.eps) : 1.f;
-      __syncwarp();
+      float inv = 1.f;
+      if (nw != nullptr) {
+#pragma unroll
+        for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(members, ss, o);
+        inv = 1.f / sqrtf(ss / static_cast<float>(n) + p.eps);
+      }
+      __syncwarp(members);
 #pragma unroll
       for (int r = 0; r < NR; ++r) {
-        const int i = (lane + 32 * r) * V;
+        const int i = (lane + L * r) * V;
         if (i >= n) continue;
 #pragma unroll
         for (int e = 0; e < V; ++e) {
@@ -125,10 +131,10 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
           if (i + e < p.rot) row[i + e] = v[r][e];
         }
       }
-      __syncwarp();
+      __syncwarp(members);
 #pragma unroll
       for (int r = 0; r < NR; ++r) {
-        const int i = (lane + 32 * r) * V;
+        const int i = (lane + L * r) * V;
 #pragma unroll
         for (int e = 0; e < V; ++e) {
           const int j = i + e;
@@ -142,7 +148,7 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
     }
 #pragma unroll
     for (int r = 0; r < NR; ++r) {
-      const int i = (lane + 32 * r) * V;
+      const int i = (lane + L * r) * V;
       if (i >= ld) continue;
       st_elems<V>(dst + i, v[r]);                          // elements n .. ld are zero
       if (is_q && p.maps == 2) {
@@ -156,13 +162,15 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
 template <typename A, int V>
 cudaError_t launch_prep(const GqaPrepArgs& p, int tokens, cudaStream_t s) {
   const int widest = max(max(p.ldq, p.hkv > 0 ? p.ldk : 0) / p.maps, p.hkv > 0 ? p.ldv : 0);
-  const size_t smem = static_cast<size_t>(p.rot) * (1 + kPrepThreads / 32) * sizeof(float);
+  const bool narrow = max(p.dk, p.hkv > 0 ? p.ldk / p.maps : 0) <= 16 * V && widest <= 32 * V;      // keys in half a warp, values in two rounds
+  const size_t smem = static_cast<size_t>(p.rot) * (1 + kPrepThreads / (narrow ? 16 : 32)) * sizeof(float);
   if (smem > 48 * 1024) return cudaErrorInvalidValue;
   const int nr = (widest + 32 * V - 1) / (32 * V);
-  if (nr <= 1) return zb_launch(zb_gqa_prep_kernel<A, 1, V>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
-  if (nr <= 2) return zb_launch(zb_gqa_prep_kernel<A, 2, V>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
-  if (nr <= 8) return zb_launch(zb_gqa_prep_kernel<A, 8, V>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
-  if (nr <= 32) return zb_launch(zb_gqa_prep_kernel<A, 32, V>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
+  if (narrow) return zb_launch(zb_gqa_prep_kernel<A, 2, V, 16>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
+  if (nr <= 1) return zb_launch(zb_gqa_prep_kernel<A, 1, V, 32>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
+  if (nr <= 2) return zb_launch(zb_gqa_prep_kernel<A, 2, V, 32>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
+  if (nr <= 8) return zb_launch(zb_gqa_prep_kernel<A, 8, V, 32>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
+  if (nr <= 32) return zb_launch(zb_gqa_prep_kernel<A, 32, V, 32>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
   return cudaErrorInvalidValue;
 }
 template <typename A>
