@@ -111,7 +111,21 @@ struct AttnParams {
   int out_f32;                  // out is fp32
   int pair;                     // decode: heads 2 h and 2 h + 1 are combined (ZbAttnExt)
   float pair_lambda, pair_scale, pair_eps;
+  int pool, pool_rows;          // pooled blocks (ZbAttnExt)
+  const __nv_bfloat16* pool_k;
+  const __nv_bfloat16* pool_v;
+  long long ldo;                // elements between output rows
+  float out_scale;
 };
+
+// Elements in front of one KV head's row of pooled block b.
+template <int HD>
+ZB_DEVICE size_t attn_pool_offset(const AttnParams& p, const int32_t* bt, int b, int kvh, uint32_t kernel) {
+  const int index = zb_pool_page_index(b, p.pool, p.page_size);
+  int page = bt[index];
+  if (!ZB_BC_OK(page, ZB_BC_PAGES, kernel, 12)) page = 0;
+  return (static_cast<size_t>(zb_pool_row(page, index, b, p.pool, p.page_size, p.pool_rows)) * p.num_kv_heads + kvh) * HD;
+}
 
 // First key in a position's window or chunk.
 template <bool EXT>
@@ -140,7 +154,8 @@ ZB_DEVICE void attn_store(const AttnParams& p, size_t tok, int head, int c, floa
       const float g = __bfloat162float(p.gate[tok * p.ldg + static_cast<size_t>(head) * p.vdim + c]);
       v *= __fdividef(1.f, 1.f + __expf(-g));
     }
-    const size_t at = (tok * p.num_q_heads + head) * p.vdim + c;
+    v *= p.out_scale;
+    const size_t at = tok * p.ldo + static_cast<size_t>(head) * p.vdim + c;
     if (p.out_f32) reinterpret_cast<float*>(p.out)[at] = v;
     else p.out[at] = __float2bfloat16(v);
   } else {
@@ -401,8 +416,9 @@ __global__ void __launch_bounds__(128) zb_paged_decode_kernel(const AttnParams p
   const int group = p.num_q_heads / p.num_kv_heads;
   const int len = p.seq_lens[seq];
   const int first_visible = attn_first_key<EXT>(p, len - 1);
-  ZbTileList tiles = {0, 0, (len + 15) >> 4};
-  if constexpr (EXT) tiles = zb_visible_tiles(first_visible, p.keep, tiles.count, 16);
+  ZbTileList tiles = {0, 0, (len + 15) >> 4, 0};
+  const int pooled = EXT && p.pool > 0 ? zb_pooled_visible(len - 1, p.window, p.pool) : 0;
+  if constexpr (EXT) tiles = zb_visible_tiles(first_visible, p.keep, tiles.count, 16, pooled);
   const int nblk = tiles.count;
   // the sequence is cut into chunks of `chunk_blocks` 16-key blocks; CTAs beyond the
   // last chunk of a short sequence have nothing to do
@@ -440,7 +456,16 @@ __global__ void __launch_bounds__(128) zb_paged_decode_kernel(const AttnParams p
   if (EXT && p.sink && split == 0 && warp == 0) m[0] = m[1] = 0.f, l[0] = l[1] = 1.f;
 
   auto issue = [&](int blk, int stage) {
-    if (blk < blk1) {
+    if (EXT && blk < blk1 && tiles.is_pooled(blk)) {
+      const uint32_t ks = wbase + stage * 2 * kBlkBytes, vs = ks + kBlkBytes;
+#pragma unroll
+      for (int i = 0; i < (16 * kChunks) / 32; ++i) {
+        const int idx = lane + 32 * i, row = idx / kChunks, chunk = idx % kChunks, b = blk * 16 + row;
+        const size_t goff = attn_pool_offset<HD>(p, bt, min(b, pooled - 1), kvh, kKernelDecode) + chunk * 8;
+        cp_async16(ks + tile_off<HD>(row, chunk), p.pool_k + goff, b < pooled ? 16u : 0u);
+        cp_async16(vs + tile_off<HD>(row, chunk), p.pool_v + goff, b < pooled ? 16u : 0u);
+      }
+    } else if (blk < blk1) {
       const int tok0 = tiles.at(blk) << 4;
       int page = bt[tok0 / p.page_size];
       if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelDecode, 10)) page = 0;      // checking build: reported, page 0 read instead
@@ -482,10 +507,12 @@ __global__ void __launch_bounds__(128) zb_paged_decode_kernel(const AttnParams p
     nxt += 4;
     const uint32_t ks = wbase + stage * 2 * kBlkBytes;
     const int tok0 = tiles.at(blk) << 4;
+    const bool in_pool = EXT && tiles.is_pooled(blk);
+    const int lo = in_pool ? 0 : first_visible, hi = in_pool ? pooled : len;
     attn_block16<HD, 0>(qf, ks, ks + kBlkBytes, 0, o, m, l, [&](float v) { return attn_score<EXT>(p, v); },
                         [&](int /*half*/, int col) {
                           const int kidx = tok0 + col;
-                          return kidx < len && (kidx >= first_visible || (EXT && kidx < p.keep));
+                          return kidx < hi && (kidx >= lo || (EXT && kidx < p.keep));
                         });
     __syncwarp();
     if (++stage == kDecStages) stage = 0;
@@ -534,7 +561,7 @@ __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_c
   const int group = p.num_q_heads / p.num_kv_heads;
   const int len = p.seq_lens[seq];
   const int first_visible = attn_first_key<EXT>(p, len - 1);
-  ZbTileList tiles = {0, 0, (len + 63) >> 6};
+  ZbTileList tiles = {0, 0, (len + 63) >> 6, 0};
   if constexpr (EXT) tiles = zb_visible_tiles(first_visible, p.keep, tiles.count, 64);
   const int nblk = EXT ? tiles.count * 4 : (len + 15) >> 4;
   const int per = p.chunk_blocks;                          // a multiple of 4 (64 keys)
@@ -666,7 +693,8 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
   const int rows_valid = min(64, q_len - row_base);
   const int last_key = min(len, ctx + row_base + 64);  // exclusive
   const int first_key = attn_first_key<EXT>(p, ctx + row_base);
-  const ZbTileList tiles = zb_visible_tiles(first_key, EXT ? p.keep : 0, (last_key + 63) >> 6, 64);
+  const int pooled = EXT && p.pool > 0 ? zb_pooled_visible(last_key - 1, p.window, p.pool) : 0;
+  const ZbTileList tiles = zb_visible_tiles(first_key, EXT ? p.keep : 0, (last_key + 63) >> 6, 64, pooled);
 
   const uint32_t q_s = zb_smem_u32(smem);
   const uint32_t kv_s = q_s + kTileBytes;             // 2 stages x (K tile, V tile)
@@ -681,9 +709,19 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
                                static_cast<size_t>(head) * HD + chunk * 8;
     cp_async16(q_s + tile_off<HD>(row, chunk), src, nbytes);
   }
-  auto issue_kv = [&](int tile, int stage) {
+  auto issue_kv = [&](int it, int stage) {
+    const int tile = tiles.at(it);
     const uint32_t ks = kv_s + stage * 2 * kTileBytes;
     const uint32_t vs = ks + kTileBytes;
+    if (EXT && tiles.is_pooled(it)) {
+      for (int idx = threadIdx.x; idx < 64 * kChunks; idx += 128) {
+        const int row = idx / kChunks, chunk = idx % kChunks, b = tile * 64 + row;
+        const size_t goff = attn_pool_offset<HD>(p, bt, min(b, pooled - 1), kvh, kKernelPrefill) + chunk * 8;
+        cp_async16(ks + tile_off<HD>(row, chunk), p.pool_k + goff, b < pooled ? 16u : 0u);
+        cp_async16(vs + tile_off<HD>(row, chunk), p.pool_v + goff, b < pooled ? 16u : 0u);
+      }
+      return;
+    }
     for (int idx = threadIdx.x; idx < 64 * kChunks; idx += 128) {
       const int row = idx / kChunks, chunk = idx % kChunks;
       const int tok = tile * 64 + row;
@@ -697,7 +735,7 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
       cp_async16(vs + tile_off<HD>(row, chunk), p.v_cache + goff, valid ? 16u : 0u);
     }
   };
-  issue_kv(tiles.at(0), 0);
+  issue_kv(0, 0);
   cp_async_commit();
 
   uint32_t qf[HD / 16][4];
@@ -709,6 +747,11 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
   const int g = lane >> 2;
   const int qpos0 = ctx + row_base + warp * 16 + g;   // key position limit of row g (row g+8: +8)
   const int from[2] = {attn_first_key<EXT>(p, qpos0), attn_first_key<EXT>(p, qpos0 + 8)};
+  int pool_end[2] = {0, 0};
+  if (EXT && p.pool > 0) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) pool_end[h] = min(pooled, zb_pooled_visible(qpos0 + 8 * h, p.window, p.pool));
+  }
 
   for (int it = 0; it < tiles.count; ++it) {
     const int tile = tiles.at(it), stage = it & 1;
@@ -722,12 +765,13 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
         ldmatrix_x4(qf[kk], q_s + tile_off<HD>(row, 2 * kk + (mi >> 1)));
       }
     }
-    if (it + 1 < tiles.count) issue_kv(tiles.at(it + 1), stage ^ 1);
+    if (it + 1 < tiles.count) issue_kv(it + 1, stage ^ 1);
     cp_async_commit();
     const uint32_t ks = kv_s + stage * 2 * kTileBytes;
     const uint32_t vs = ks + kTileBytes;
     // tiles entirely above the diagonal of this warp's rows contribute nothing
-    const int warp_max_q = ctx + row_base + warp * 16 + 15;
+    const bool in_pool = EXT && tiles.is_pooled(it);
+    const int warp_max_q = in_pool ? pooled - 1 : ctx + row_base + warp * 16 + 15;
 #pragma unroll
     for (int sub = 0; sub < 4; ++sub) {
       const int key0 = tile * 64 + sub * 16;
@@ -736,6 +780,7 @@ __global__ void __launch_bounds__(128) zb_paged_prefill_kernel(const AttnParams 
         const int kidx = key0 + col;
         const int qp = qpos0 + half * 8;
         const bool vis = kidx <= qp && kidx < len;
+        if (in_pool) return kidx < pool_end[half];
         return vis && (kidx >= from[half] || (EXT && kidx < p.keep));
       });
     }
@@ -843,6 +888,17 @@ void set_ext(AttnParams& p, const ZbAttnExt& x, float scale) {
   p.pair_lambda = x.pair_lambda;
   p.pair_scale = x.pair_scale;
   p.pair_eps = x.pair_eps;
+  p.pool = x.pool;
+  p.pool_rows = x.pool_rows;
+  p.pool_k = reinterpret_cast<const __nv_bfloat16*>(x.pool_k);
+  p.pool_v = reinterpret_cast<const __nv_bfloat16*>(x.pool_v);
+  p.ldo = x.ldo > 0 ? x.ldo : static_cast<long long>(p.num_q_heads) * x.vdim;
+  p.out_scale = x.scaled ? x.out_scale : 1.f;
+}
+
+bool ext_ok(const ZbAttnExt& x, int window) {
+  if (x.pair != 0 && (x.ldo != 0 || x.scaled)) return false;
+  return x.pool == 0 || (x.pool > 0 && window > 0 && x.chunk == 0 && x.pool_rows > 0 && x.pool_k != nullptr && x.pool_v != nullptr);
 }
 
 }  // namespace
@@ -914,12 +970,14 @@ int zb_paged_decode_ex(const void* q, const void* k_cache, const void* v_cache, 
     --num_splits;
   // chunk length that lets `num_splits` chunks cover the longest sequence the block table allows
   int max_blocks = (max_pages * page_size + 15) / 16;
+  if (ext != nullptr && !ext_ok(*ext, window)) return -35;
   if (ext != nullptr && ext->pair != 0 && ((num_q_heads / num_kv_heads) % 2 != 0 || ext->gate != nullptr || ext->out_f32 != 0)) return -35;
   if (ext != nullptr && (window > 0 || ext->chunk > 0)) {      // the longest list of visible tiles: the kept ones and a window that starts inside a tile
     const int tile = page_size == 64 ? 64 : 16;
     const int span = ext->chunk > 0 ? ext->chunk : window;
-    const int visible = ((ext->keep + tile - 1) / tile + (span + tile - 2) / tile + 1) * (tile / 16);
-    if (visible < max_blocks) max_blocks = visible;
+    int visible = ((ext->keep + tile - 1) / tile + (span + tile - 2) / tile + 1) * (tile / 16);
+    if (ext->pool > 0) visible += (max_pages * page_size / ext->pool + 15) / 16;
+    if (visible < max_blocks || ext->pool > 0) max_blocks = visible;
   }
   int chunk_blocks = (max_blocks + num_splits - 1) / num_splits;
   if (page_size == 64) chunk_blocks = (chunk_blocks + 3) / 4 * 4;      // whole pages per chunk (tensor-map fed kernel)
@@ -947,7 +1005,7 @@ int zb_paged_decode_ex(const void* q, const void* k_cache, const void* v_cache, 
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = status;
   // 64-token pages and chunks of whole pages: the tensor-map fed kernel; otherwise per-warp cp.async
-  const bool tma = g_decode_tma != 0 && page_size == 64 && (p.chunk_blocks % 4) == 0 &&
+  const bool tma = g_decode_tma != 0 && (ext == nullptr || ext->pool == 0) && page_size == 64 && (p.chunk_blocks % 4) == 0 &&
                    (reinterpret_cast<uintptr_t>(k_cache) & 15) == 0 && (reinterpret_cast<uintptr_t>(v_cache) & 15) == 0;
   if (ext == nullptr) return dispatch_decode<false>(p, head_dim, tma, stream);
   set_ext(p, *ext, scale);
@@ -997,7 +1055,7 @@ int zb_paged_prefill(const void* q, const void* k_cache, const void* v_cache, vo
   p.status = st->status;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (ext == nullptr) return dispatch_prefill<false>(p, head_dim, total_q_blocks, s);
-  if (ext->pair != 0) return -35;                 // the caller combines the maps (zb_pair_combine)
+  if (ext->pair != 0 || !ext_ok(*ext, window)) return -35;                 // the caller combines the maps (zb_pair_combine)
   set_ext(p, *ext, scale);
   return dispatch_prefill<true>(p, head_dim, total_q_blocks, s);
 }

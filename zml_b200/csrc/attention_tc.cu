@@ -22,6 +22,8 @@
 // where the running maximum goes: every score lies in [-c, c], so P = exp2(S') needs no reference and O no rescaling.  Kept
 // first keys join the window's tiles as one list, a chunk is a window whose start is the same for all its positions, a sink
 // is one more term of the sum, and the output gate is applied as the rows are stored.
+// Pooled blocks (ZbAttnExt.pool) are tiles in front of the window's.  Their rows lie a few to a page, so warp 8 gathers them with
+// cp.async into the layout that the tensor-map copies write, and makes them visible to the tensor core with a proxy fence.
 // Differential heads (ZbAttnExt.pair, kExt): the two pipelines are the two maps of one head.  A map's keys are one 64-column
 // sub-tile of the cached key, so its scores take half the products; at the end both warpgroups read both accumulators, the
 // upper and the lower 64 columns each, and exchange row sums and partial sums of squares through shared memory.
@@ -79,6 +81,11 @@ struct PrefillTcParams {
   long long ldg;
   int pair;                     // kExt
   float pair_lambda, pair_scale, pair_eps;
+  int pool, pool_rows;
+  const __nv_bfloat16* pool_k;
+  const __nv_bfloat16* pool_v;
+  long long ldo;                // elements between output rows
+  float out_scale;
 };
 
 // First key in a position's window or chunk.
@@ -100,9 +107,10 @@ ZB_DEVICE void pair_bar_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); 
 // Eight output values of one row at column c: gated, and cut at vdim.
 ZB_DEVICE void store_ext8(const PrefillTcParams& p, size_t tok, int head, int c, const uint32_t* o, float inv) {
   if (c >= p.vdim) return;
-  __nv_bfloat16* dst = p.out + (tok * p.num_q_heads + head) * p.vdim + c;
+  __nv_bfloat16* dst = p.out + tok * p.ldo + static_cast<size_t>(head) * p.vdim + c;
   const __nv_bfloat16* gate = p.gate != nullptr ? p.gate + tok * p.ldg + static_cast<size_t>(head) * p.vdim + c : nullptr;
-  const bool vec = (p.vdim & 7) == 0 && (p.ldg & 7) == 0 && (reinterpret_cast<uintptr_t>(p.gate) & 15) == 0;
+  const bool vec = (p.vdim & 7) == 0 && (p.ldg & 7) == 0 && (p.ldo & 7) == 0 &&
+                   ((reinterpret_cast<uintptr_t>(p.gate) | reinterpret_cast<uintptr_t>(p.out)) & 15) == 0;
   float v[8], g[8];
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
@@ -135,6 +143,27 @@ ZB_DEVICE void store_ext8(const PrefillTcParams& p, size_t tok, int head, int c,
     for (int i = 0; i < 8; ++i)
       if (c + i < p.vdim) dst[i] = __float2bfloat16(v[i]);
   }
+}
+
+// One 64-row tile of pooled keys and values by a warp, in the layout of a 128-byte-swizzled tensor-map copy; rows from `end` on are
+// zero.  Returns once the rows are in shared memory and visible to the tensor core.
+ZB_DEVICE void gather_pooled_tile(const PrefillTcParams& p, const int32_t* bt, int tile, int end, int kvh, uint8_t* k_dst, uint8_t* v_dst) {
+  const int lane = threadIdx.x & 31, chunk = lane & 15;
+#pragma unroll 4
+  for (int r = lane >> 4; r < kKeys; r += 2) {
+    const int b = tile * kKeys + r, have = min(b, end - 1);
+    const int index = zb_pool_page_index(have, p.pool, kKeys);
+    int page = bt[index];
+    if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelId, 12)) page = 0;
+    const size_t off = (static_cast<size_t>(zb_pool_row(page, index, have, p.pool, kKeys, p.pool_rows)) * p.num_kv_heads + kvh) * kHD + chunk * 8;
+    const uint32_t to = static_cast<uint32_t>((chunk >> 3) * (kKeys * 128) + r * 128 + (((chunk & 7) ^ (r & 7)) << 4));
+    const uint32_t bytes = b < end ? 16u : 0u;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(zb_smem_u32(k_dst) + to), "l"(p.pool_k + off), "r"(bytes) : "memory");
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(zb_smem_u32(v_dst) + to), "l"(p.pool_v + off), "r"(bytes) : "memory");
+  }
+  asm volatile("cp.async.wait_all;" ::: "memory");
+  zb_fence_proxy_async_smem();
+  __syncwarp();
 }
 
 template <Mode MODE>
@@ -193,7 +222,8 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
   const int rows_valid = min(kQRows, q_len - row_base);
   const int last_key = min(len, ctx + row_base + kQRows);     // exclusive
   const int first_key = first_key_of<EXT>(p, ctx + row_base);
-  const ZbTileList tiles = zb_visible_tiles(first_key, EXT ? p.keep : 0, (last_key + kKeys - 1) / kKeys, kKeys);
+  const int pooled = EXT && p.pool > 0 ? zb_pooled_visible(last_key - 1, p.window, p.pool) : 0;
+  const ZbTileList tiles = zb_visible_tiles(first_key, EXT ? p.keep : 0, (last_key + kKeys - 1) / kKeys, kKeys, pooled);
   const int n_tiles = tiles.count;
 
   if (threadIdx.x == 0) {
@@ -226,15 +256,38 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
 
   if (warp == 8) {
     // ------------------------------------------------------------------ TMA producer
+    const int32_t* bt = p.block_table + static_cast<size_t>(seq) * p.max_pages;
+    uint32_t stage = 0, phase = 0;
     if (lane == 0) {
       zb_mbar_expect_tx(q_full, pair ? kQBytes : 2 * kQBytes);
       for (int w = 0; w < 2; ++w)
         for (int c = 0; c < 2; ++c)
           if (!pair || c == w)
             zb_tma_load_2d(q_s + w * kQBytes + c * (kQRows * 128), &tmap_q, q_full, (head0 + w) * kHD + c * 64, tok_base);
-      const int32_t* bt = p.block_table + static_cast<size_t>(seq) * p.max_pages;
-      uint32_t stage = 0, phase = 0;
-      for (int j = 0; j < n_tiles; ++j) {
+    }
+    bool ok = true;
+    if constexpr (EXT) {
+      __syncwarp();
+      for (int j = 0; j < tiles.pooled; ++j) {             // the whole warp
+        if (j >= kStages) ok = zb_mbar_wait(&kv_empty[stage], phase ^ 1u, abort_flag);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) {
+          *abort_where = 1u;
+          break;
+        }
+        gather_pooled_tile(p, bt, tiles.at(j), pooled, kvh, k_s + stage * kKvBytes, v_s + stage * kKvBytes);
+        if (lane == 0) {
+          zb_mbar_arrive(&k_full[stage]);
+          zb_mbar_arrive(&v_full[stage]);
+        }
+        if (++stage == kStages) {
+          stage = 0;
+          phase ^= 1u;
+        }
+      }
+    }
+    if (lane == 0 && ok) {
+      for (int j = tiles.pooled; j < n_tiles; ++j) {
         if (j >= kStages) {
           if (!zb_mbar_wait(&kv_empty[stage], phase ^ 1u, abort_flag)) {
             *abort_where = 1u;
@@ -339,6 +392,9 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
     const uint32_t t_o = tmem_base + kColO + w * kHD + lane_off;
     float m = MODE == kExt && p.sink ? 0.f : -INFINITY, l = EXT && p.sink ? 1.f : 0.f;
     const int from = first_key_of<EXT>(p, qpos), from_last = first_key_of<EXT>(p, ctx + row_base + kQRows - 1);
+    // pooled blocks that this row sees, and those that every row of the block sees
+    const int pool_end = EXT && p.pool > 0 ? min(pooled, zb_pooled_visible(qpos, p.window, p.pool)) : 0;
+    const int pool_first = EXT && p.pool > 0 ? zb_pooled_visible(ctx + row_base, p.window, p.pool) : 0;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
       const uint32_t jj = static_cast<uint32_t>(j);
@@ -355,7 +411,15 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       const int key0 = tiles.at(j) * kKeys;
       // pages below the block's first row and inside every row's window need no mask (a branch per page, not a
       // predicate per score: predicated-off instructions still take issue slots, and this loop is issue-bound)
-      const bool full = (key0 + kKeys - 1 <= ctx + row_base) && (key0 + kKeys <= len) && key0 >= from_last;
+      bool full = (key0 + kKeys - 1 <= ctx + row_base) && (key0 + kKeys <= len) && key0 >= from_last;
+      int lo = from, hi = min(qpos + 1, len);              // visible: lo <= key < hi, and the kept ones in front
+      if constexpr (EXT) {
+        if (tiles.is_pooled(j)) {
+          full = key0 + kKeys <= pool_first;
+          lo = 0;
+          hi = pool_end;
+        }
+      }
       uint32_t pw[32];
       float sum0 = 0.f, sum1 = 0.f;
       if constexpr (MODE == kCapped) {
@@ -387,7 +451,7 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
 #pragma unroll
           for (int i = 0; i < 64; ++i) {
             const int kidx = key0 + i;
-            const bool vis = kidx <= qpos && kidx < len && (kidx >= from || kidx < p.keep);
+            const bool vis = kidx < hi && (kidx >= lo || kidx < p.keep);
             if (!vis) sr[i] = 0xff800000u;           // -inf
           }
         }
@@ -408,7 +472,7 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
 #pragma unroll
           for (int i = 0; i < 64; ++i) {
             const int kidx = key0 + i;
-            const bool vis = kidx <= qpos && kidx < len && (kidx >= from || (EXT && kidx < p.keep));
+            const bool vis = kidx < hi && (kidx >= lo || (EXT && kidx < p.keep));
             if (!vis) sr[i] = 0xff800000u;             // -inf
             mx_raw = fmaxf(mx_raw, __uint_as_float(sr[i]));
           }
@@ -507,7 +571,8 @@ zb_paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       const uint32_t last = static_cast<uint32_t>(n_tiles - 1);
       if (zb_mbar_wait(&o_ready[w], last & 1u, abort_flag)) {
         zb_tc_fence_after();
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        float inv = l > 0.f ? 1.f / l : 0.f;
+        if constexpr (EXT) inv *= p.out_scale;
         __nv_bfloat16* orow = p.out + (static_cast<size_t>(tok_base + r) * p.num_q_heads + head0 + w) * kHD;
 #pragma unroll 1
         for (int c0 = 0; c0 < kHD; c0 += 32) {
@@ -584,6 +649,10 @@ int zb_paged_prefill_tc(const void* q, const void* k_cache, const void* v_cache,
   if (!st) return -20;
   if (ext != nullptr && (!zb_paged_prefill_tc_ext_supported(ext->cap, ext->pair) || ext->out_f32 != 0 || (ext->pair != 0 && ext->gate != nullptr)))
     return -34;
+  if (ext != nullptr && ext->pair != 0 && (ext->ldo != 0 || ext->scaled)) return -34;
+  if (ext != nullptr && ext->pool != 0 &&
+      (ext->pool < 0 || window <= 0 || ext->chunk != 0 || ext->pool_rows <= 0 || ext->pool_k == nullptr || ext->pool_v == nullptr))
+    return -34;
   static bool configured[3][16] = {};
   const Mode mode = ext == nullptr ? kPlain : (ext->cap > 0.f ? kCapped : kExt);
   const auto kernel = mode == kPlain ? zb_paged_prefill_tc_kernel<kPlain> : (mode == kCapped ? zb_paged_prefill_tc_kernel<kCapped> : zb_paged_prefill_tc_kernel<kExt>);
@@ -627,6 +696,12 @@ int zb_paged_prefill_tc(const void* q, const void* k_cache, const void* v_cache,
     p.vdim = ext->vdim;
     p.gate = reinterpret_cast<const __nv_bfloat16*>(ext->gate);
     p.ldg = ext->ldg;
+    p.pool = ext->pool;
+    p.pool_rows = ext->pool_rows;
+    p.pool_k = reinterpret_cast<const __nv_bfloat16*>(ext->pool_k);
+    p.pool_v = reinterpret_cast<const __nv_bfloat16*>(ext->pool_v);
+    p.ldo = ext->ldo > 0 ? ext->ldo : static_cast<long long>(num_q_heads) * ext->vdim;
+    p.out_scale = ext->scaled ? ext->out_scale : 1.f;
   }
   const cudaError_t le = zb_launch(kernel, dim3(total_q_blocks128, num_q_heads / 2), dim3(kThreads), kSmemBytes,
                                    reinterpret_cast<cudaStream_t>(stream), tq, tk, tv, p);

@@ -1,23 +1,38 @@
 // Grouped-query attention whose heads are normalised, partly rotated, soft-capped, windowed with kept first tokens or chunked,
 // sunk and gated (any of these may be off), with key and value sizes of their own and one or two maps per head, bf16 or fp32:
 //
-//   zb_gqa_prep     per head RMS norm of q and k, rotation of the first `rot` dimensions (pairs (i, i + rot / 2)), cache write
+//   zb_gqa_prep     RMS norm of q and k (per head, or over all heads of a projection at once), rotation of the first `rot` dimensions (pairs (i, i + rot / 2)), cache write
 //                   of k and v.  Heads are written with a padded stride (zeros behind their elements), so that the
 //                   tensor-core kernels of attention.cu / attention_tc.cu take any size up to theirs.  With two maps a cached
 //                   key is [map 1 | map 2], and a head has two query rows, each zero where the other map's keys are
 //   zb_gqa_attend   attention over the paged cache for any sizes: the fp32 path and the fall-back for sizes the tensor-core
 //                   kernels do not take
+//   zb_gqa_pool     pooled blocks of a windowed cache: the mean of the cached keys and values of every `pool` positions whose last
+//                   one is new (for decode steps zb_gqa_prep does it behind its cache write)
 //   zb_pair_combine differential attention: the two maps' results a1, a2 of every head -> a1 - lambda a2 at unit root mean
 //                   square, times a constant (the kernels of attention.cu and attention_tc.cu do it as they store)
 //
-// Position i sees j when j <= i and (i - j < window or j < keep), or with chunks when floor(i / chunk) = floor(j / chunk).  score = q . k * scale, then cap * tanh(score / cap); with
+// Position i sees j when j <= i and (i - j < window or j < keep), or with chunks when floor(i / chunk) = floor(j / chunk); with
+// pooled blocks also the mean key and value of every block in front of its window.  score = q . k * scale, then cap * tanh(score / cap); with
 // a sink the softmax denominator has an additional exp(0).  Norms, angles, scores and softmax are fp32.
 #include "act.cuh"
+#include "attention_tiles.cuh"
 #include "host_api.h"
 
 namespace {
 constexpr uint32_t kKernelGqaPrep = 34;
 constexpr uint32_t kKernelGqaAttend = 35;
+constexpr uint32_t kKernelGqaPool = 37;
+
+// Pooled blocks of a cache (ZbAttnExt.pool).
+struct PoolArgs {
+  int pool;                  // positions per block, 0: none
+  int rows;                  // blocks per page at most
+  void* k;                   // [pages, rows, hkv, ldk]
+  void* v;                   // [pages, rows, hkv, ldv]
+  const int32_t* block_table;
+  int max_pages, page_size;
+};
 
 struct GqaPrepArgs {
   const void* in;            // [T, ld_in]: q heads | k heads | v heads
@@ -35,6 +50,11 @@ struct GqaPrepArgs {
   int hq, hkv, dk, dv, rot;  // hq: query rows, maps of a head counted one by one; hkv 0: queries only
   int maps;
   int ldq, ldk, ldv;         // elements per row where it is written
+  int whole;                 // 1: one norm over all query rows and one over all keys, weights [hq dk] and [hkv dk]
+  const float* sumsq;        // whole: [T, 2] sums of squares of q and k over all ranks, or null: those of `in`
+  int total_q, total_k;      // whole: elements that the sums cover
+  float amp;                 // factor on cosines and sines
+  PoolArgs pool;             // one token per sequence: blocks that the token completes are pooled
 };
 
 template <int V>
@@ -67,6 +87,39 @@ ZB_DEVICE void st_elems(float* p, const float (&v)[V]) {
   else *p = v[0];
 }
 
+// Mean key and value of block b of sequence s, by a CTA of NT threads; V elements at a time.
+template <typename A, int V>
+ZB_DEVICE void pool_block(const PoolArgs& p, const A* kc, const A* vc, int hkv, int ldk, int ldv, int s, int b, int threads) {
+  const int32_t* bt = p.block_table + static_cast<long long>(s) * p.max_pages;
+  const int index = min(zb_pool_page_index(b, p.pool, p.page_size), p.max_pages - 1);
+  int page = bt[index];
+  if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelGqaPool, 1)) page = 0;
+  const long long row = zb_pool_row(page, index, b, p.pool, p.page_size, p.rows);
+  const float scale = 1.f / static_cast<float>(p.pool);
+  const int nk = hkv * ldk, n = nk + hkv * ldv;
+  for (int i = threadIdx.x * V; i < n; i += threads * V) {
+    const bool is_k = i < nk;
+    const int c = is_k ? i : i - nk, ld = is_k ? nk : n - nk;
+    const A* src = (is_k ? kc : vc) + c;
+    float acc[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) acc[e] = 0.f;
+#pragma unroll 8
+    for (int j = 0; j < p.pool; ++j) {
+      const int tok = b * p.pool + j;
+      int pg = bt[min(tok / p.page_size, p.max_pages - 1)];
+      if (!ZB_BC_OK(pg, ZB_BC_PAGES, kKernelGqaPool, 2)) pg = 0;
+      float v[V];
+      ld_elems<V>(v, src + (static_cast<long long>(pg) * p.page_size + tok % p.page_size) * ld);
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] += v[e];
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) acc[e] *= scale;
+    st_elems<V>((is_k ? reinterpret_cast<A*>(p.k) : reinterpret_cast<A*>(p.v)) + row * ld + c, acc);
+  }
+}
+
 // One CTA per token, L lanes (a warp or half of one) per head; NR groups of V neighbouring elements per lane.
 constexpr int kPrepThreads = 256;
 
@@ -83,13 +136,50 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
   for (int i = threadIdx.x; i < half; i += kPrepThreads) {
     float sn, c;
     sincosf(pos * p.inv_freq[i], &sn, &c);
-    cs[i] = make_float2(c, sn);
+    cs[i] = make_float2(c * p.amp, sn * p.amp);
   }
-  __syncthreads();
+  const A* in = reinterpret_cast<const A*>(p.in) + t * p.ld_in;
+  __shared__ float whole_part[2][kPrepThreads / 32];
+  float whole_q = 1.f, whole_k = 1.f;
+  if (p.whole) {
+    float sq = 0.f, sk = 0.f;
+    if (p.sumsq != nullptr) {
+      sq = p.sumsq[2 * t];
+      sk = p.sumsq[2 * t + 1];
+      __syncthreads();
+    } else {
+      const int nq = p.hq * p.dk, nk = p.hkv * p.dk;
+#pragma unroll 4
+      for (int i = threadIdx.x * V; i < nq + nk; i += kPrepThreads * V) {
+        float v[V], s2 = 0.f;
+        ld_elems<V>(v, in + i);
+#pragma unroll
+        for (int e = 0; e < V; ++e) s2 = fmaf(v[e], v[e], s2);
+        if (i < nq) sq += s2;
+        else sk += s2;
+      }
+      sq = zb_warp_sum(sq);
+      sk = zb_warp_sum(sk);
+      if ((threadIdx.x & 31) == 0) {
+        whole_part[0][threadIdx.x >> 5] = sq;
+        whole_part[1][threadIdx.x >> 5] = sk;
+      }
+      __syncthreads();
+      sq = sk = 0.f;
+#pragma unroll
+      for (int i = 0; i < kPrepThreads / 32; ++i) {
+        sq += whole_part[0][i];
+        sk += whole_part[1][i];
+      }
+    }
+    whole_q = 1.f / sqrtf(sq / static_cast<float>(p.total_q) + p.eps);
+    whole_k = 1.f / sqrtf(sk / static_cast<float>(p.total_k) + p.eps);
+  } else {
+    __syncthreads();
+  }
   const long long slot = p.slots[t];
   if (slot >= p.num_rows) (void)ZB_BC_OK(slot, p.num_rows, kKernelGqaPrep, 1);
   const bool slot_ok = slot >= 0 && slot < p.num_rows;
-  const A* in = reinterpret_cast<const A*>(p.in) + t * p.ld_in;
   const int keys = p.hkv * p.maps, heads = p.hq + keys + p.hkv;
   for (int h = team; h < heads; h += kPrepThreads / L) {
     const bool is_q = h < p.hq, is_v = h >= p.hq + keys;
@@ -114,8 +204,10 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
     }
     if (!is_v) {
       const float* nw = is_q ? p.q_norm : p.k_norm;
-      float inv = 1.f;
-      if (nw != nullptr) {
+      float inv = is_q ? whole_q : whole_k;
+      if (p.whole) {
+        nw += u * p.dk;
+      } else if (nw != nullptr) {
 #pragma unroll
         for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(members, ss, o);
         inv = 1.f / sqrtf(ss / static_cast<float>(n) + p.eps);
@@ -157,6 +249,31 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
       }
     }
   }
+  if (p.pool.pool > 0 && slot_ok) {
+    const int done = p.positions[t] + 1;
+    if (done % p.pool.pool == 0) {
+      __syncthreads();                                     // this token's rows are written
+      pool_block<A, V>(p.pool, reinterpret_cast<const A*>(p.k_cache), reinterpret_cast<const A*>(p.v_cache), p.hkv, p.ldk, p.ldv, t,
+                       done / p.pool.pool - 1, kPrepThreads);
+    }
+  }
+}
+
+// The blocks that a varlen batch completes, one CTA each.
+template <typename A, int V>
+__global__ void __launch_bounds__(128) zb_gqa_pool_kernel(const PoolArgs p, const void* k_cache, const void* v_cache, int hkv, int ldk, int ldv,
+                                                          const ZbVarlen b) {
+  zb_pdl_launch();
+  zb_pdl_wait();
+  int idx = blockIdx.x;
+  for (int s = 0; s < b.num_seqs; ++s) {
+    const int len = b.seq_lens[s], first = (len - (b.q_start[s + 1] - b.q_start[s])) / p.pool, n = len / p.pool - first;
+    if (idx < n) {
+      pool_block<A, V>(p, reinterpret_cast<const A*>(k_cache), reinterpret_cast<const A*>(v_cache), hkv, ldk, ldv, s, first + idx, 128);
+      return;
+    }
+    idx -= n;
+  }
 }
 
 template <typename A, int V>
@@ -197,6 +314,8 @@ struct GqaArgs {
   int window, keep, chunk;
   float scale, cap;          // cap 0: none
   int sink;
+  PoolArgs pool;             // block_table and page size as above
+  float out_scale;
 };
 
 constexpr int kGqaKeys = 64;
@@ -227,26 +346,31 @@ __global__ void __launch_bounds__(128) zb_gqa_attend_kernel(const GqaArgs p, con
   const int kept = min(p.keep, first);
   const A* q = reinterpret_cast<const A*>(p.q) + (static_cast<long long>(t) * p.hq + h) * p.ldq;
   for (int i = threadIdx.x; i < p.dk; i += 128) gqa_smem[i] = zb_ld_act(q + i);
+  const int pooled = p.pool.pool > 0 ? zb_pooled_visible(pos, p.window, p.pool.pool) : 0;      // first in the list of keys
   const int32_t* bt = p.block_table + static_cast<long long>(s) * p.max_pages;
   const A* kc = reinterpret_cast<const A*>(p.k_cache) + static_cast<long long>(g) * p.ldk;
   const A* vc = reinterpret_cast<const A*>(p.v_cache) + static_cast<long long>(g) * p.ldv;
+  const A* pk = reinterpret_cast<const A*>(p.pool.k) + static_cast<long long>(g) * p.ldk;
+  const A* pv = reinterpret_cast<const A*>(p.pool.v) + static_cast<long long>(g) * p.ldv;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float m = p.sink ? 0.f : -INFINITY, l = p.sink ? 1.f : 0.f, acc[RC];
 #pragma unroll
   for (int i = 0; i < RC; ++i) acc[i] = 0.f;
-  const int total = kept + pos + 1 - first;
+  const int total = pooled + kept + pos + 1 - first;
   for (int k0 = 0; k0 < total; k0 += kGqaKeys) {
     const int nk = min(kGqaKeys, total - k0);
     __syncthreads();
     if (threadIdx.x < nk) {
-      const int i = k0 + threadIdx.x, key = i < kept ? i : first + i - kept;
-      int page = bt[key / p.page_size];
+      const int at = k0 + threadIdx.x, i = at - pooled, key = i < kept ? i : first + i - kept;
+      const int index = i < 0 ? zb_pool_page_index(at, p.pool.pool, p.page_size) : key / p.page_size;
+      int page = bt[index];
       if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelGqaAttend, 1)) page = 0;
-      srow[threadIdx.x] = (static_cast<long long>(page) * p.page_size + key % p.page_size) * p.hkv;
+      srow[threadIdx.x] = (i < 0 ? zb_pool_row(page, index, at, p.pool.pool, p.page_size, p.pool.rows)
+                                 : static_cast<long long>(page) * p.page_size + key % p.page_size) * p.hkv;
     }
     __syncthreads();
     for (int j = warp; j < nk; j += 4) {
-      const A* row = kc + srow[j] * p.ldk;
+      const A* row = (k0 + j < pooled ? pk : kc) + srow[j] * p.ldk;
       float d = 0.f;
       for (int i = lane; i < p.dk; i += 32) d = fmaf(gqa_smem[i], zb_ld_act(row + i), d);
       d = zb_warp_sum(d) * p.scale;
@@ -264,7 +388,7 @@ __global__ void __launch_bounds__(128) zb_gqa_attend_kernel(const GqaArgs p, con
     for (int j = 0; j < nk; ++j) {
       const float pj = expf(sc[j] - m);
       l += pj;
-      const A* row = vc + srow[j] * p.ldv;
+      const A* row = (k0 + j < pooled ? pv : vc) + srow[j] * p.ldv;
 #pragma unroll
       for (int i = 0; i < RC; ++i) {
         const int c = threadIdx.x + 128 * i;
@@ -280,7 +404,7 @@ __global__ void __launch_bounds__(128) zb_gqa_attend_kernel(const GqaArgs p, con
     if (c >= p.dv) continue;
     float o = acc[i] * inv;
     if (gate != nullptr) o *= 1.f / (1.f + expf(-zb_ld_act(gate + c)));
-    store(c, o);
+    store(c, o * p.out_scale);
   }
 }
 
@@ -319,26 +443,49 @@ extern "C" {
 
 int zb_gqa_prep(const void* in, long long ld_in, const float* q_norm, const float* k_norm, const float* inv_freq, const int32_t* positions,
                 const int32_t* slots, void* q, void* k_cache, void* v_cache, long long num_rows, float eps, int hq, int hkv, int dk, int dv,
-                int rot, int maps, int ldq, int ldk, int ldv, int act_f32, int tokens, void* stream) {
+                int rot, int maps, int ldq, int ldk, int ldv, int whole, const float* sumsq, int total_q, int total_k, float amp, int pool, int pool_rows,
+                void* pool_k, void* pool_v, const int32_t* block_table, int max_pages, int page_size, int act_f32, int tokens, void* stream) {
   if (tokens <= 0) return 0;
+  if (whole && (maps != 1 || q_norm == nullptr || k_norm == nullptr || total_q < 1 || total_k < 1)) return -70;
+  if (pool < 0 || (pool > 0 && (hkv < 1 || pool_rows * pool < page_size || pool_k == nullptr || pool_v == nullptr || block_table == nullptr))) return -70;
   if ((maps != 1 && maps != 2) || hq % maps != 0 || ldq % maps != 0 || ldk % maps != 0) return -70;
   if (rot % 2 != 0 || rot > dk || ldq < maps * dk || (hkv > 0 && (ldk < maps * dk || ldv < dv))) return -70;
   const GqaPrepArgs p = {in, ld_in, q_norm, k_norm, inv_freq, positions, slots, q, k_cache, v_cache, num_rows, eps,
-                         hq, hkv, dk, dv, rot, maps, ldq, ldk, ldv};
+                         hq, hkv, dk, dv, rot, maps, ldq, ldk, ldv, whole, sumsq, total_q, total_k, amp,
+                         {pool, pool_rows, pool_k, pool_v, block_table, max_pages, page_size}};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const cudaError_t e = act_f32 ? launch_prep<float>(p, tokens, s) : launch_prep<__nv_bfloat16>(p, tokens, s);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }
 
+// Pools the blocks that a varlen batch completes; num_blocks >= their number.
+int zb_gqa_pool(const void* k_cache, const void* v_cache, void* pool_k, void* pool_v, int pool, int pool_rows, const int32_t* block_table, int max_pages,
+                int page_size, int hkv, int ldk, int ldv, const int32_t* q_start, const int32_t* seq_lens, int num_seqs, int num_blocks, int act_f32,
+                void* stream) {
+  if (num_seqs <= 0 || num_blocks <= 0) return 0;
+  if (pool < 1 || hkv < 1 || pool_rows * pool < page_size) return -70;
+  const PoolArgs p = {pool, pool_rows, pool_k, pool_v, block_table, max_pages, page_size};
+  const ZbVarlen b = {q_start, seq_lens, num_seqs};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const bool vec = ldk % 4 == 0 && ldv % 4 == 0;
+  const auto kernel = act_f32 ? (vec ? zb_gqa_pool_kernel<float, 4> : zb_gqa_pool_kernel<float, 1>)
+                              : (vec ? zb_gqa_pool_kernel<__nv_bfloat16, 4> : zb_gqa_pool_kernel<__nv_bfloat16, 1>);
+  const cudaError_t e = zb_launch(kernel, dim3(num_blocks), dim3(128), 0, s, p, k_cache, v_cache, hkv, ldk, ldv, b);
+  zb_count_launch(1);
+  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+}
+
 int zb_gqa_attend(const void* q, int ldq, const void* k_cache, int ldk, const void* v_cache, int ldv, const void* gate, long long ld_gate, void* out,
                   long long ld_out, int out_f32, const int32_t* block_table, int max_pages, int page_size, int hq, int hkv, int dk, int dv,
-                  int window, int keep, int chunk, float scale, float cap, int sink, const int32_t* q_start, const int32_t* seq_lens, int num_seqs, int tokens, int act_f32,
-                  void* stream) {
+                  int window, int keep, int chunk, float scale, float cap, int sink, int pool, int pool_rows, const void* pool_k, const void* pool_v,
+                  float out_scale, const int32_t* q_start, const int32_t* seq_lens, int num_seqs, int tokens, int act_f32, void* stream) {
   if (tokens <= 0) return 0;
+  if (pool < 0 || (pool > 0 && (window <= 0 || chunk != 0 || pool_rows * pool < page_size || pool_k == nullptr || pool_v == nullptr))) return -70;
   if (hkv <= 0 || hq % hkv != 0) return -30;
   const GqaArgs p = {q, k_cache, v_cache, ldq, ldk, ldv, gate, ld_gate, out, ld_out, out_f32, block_table, max_pages, page_size,
-                     hq, hkv, dk, dv, window, keep, chunk, scale, cap, sink};
+                     hq, hkv, dk, dv, window, keep, chunk, scale, cap, sink,
+                     {pool, pool_rows, const_cast<void*>(pool_k), const_cast<void*>(pool_v), block_table, max_pages, page_size}, out_scale};
   const ZbVarlen b = {q_start, seq_lens, num_seqs};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const cudaError_t e = act_f32 ? launch_attend<float>(p, b, tokens, s) : launch_attend<__nv_bfloat16>(p, b, tokens, s);

@@ -113,6 +113,16 @@ struct ZbAttnExt {
   // a1 - pair_lambda * a2 at unit root mean square (pair_eps inside the root) times pair_scale.
   int pair;
   float pair_lambda, pair_scale, pair_eps;
+  // Pooled blocks beside a window: block b, the positions b * pool .. b * pool + pool - 1, is one more key and value for a
+  // position i when its last position is <= i - window.  pool_k / pool_v: [pages, pool_rows, kv_heads, head_dim] as
+  // zb_pool_row addresses them.  0: off
+  int pool;
+  int pool_rows;
+  const void* pool_k;
+  const void* pool_v;
+  long long ldo;               // elements between the rows of the output, 0: heads * vdim
+  int scaled;                  // 1: the output times out_scale
+  float out_scale;
 };
 
 ZbDeviceState* zb_device_state();       // state of the current device, or nullptr before zb_init

@@ -90,15 +90,21 @@ __global__ void __launch_bounds__(128) zb_moe_router_topk_kernel(const float* __
   }
 }
 
-// One warp per token: scores s = softmax of the first `experts` logits; the k largest s + correction are chosen and weighted by
-// their s, divided by the sum.  Behind the routed choices come `shared` always-on experts (ids 0 .. shared - 1), weighted by the
-// sigmoid of the logit in column `experts`; routed expert e has id shared + (e - e0) mod experts, so that the experts of the
+struct RouteScores {
+  int sigmoid;             // scores: 1 sigmoid, 0 softmax of the logits
+  int normalize;           // weights: 1 divided by the sum of the chosen scores
+  int gated;               // weight of the shared experts: 1 the sigmoid of the logit in column `experts`, 0 one
+  float scale;             // factor on the routed experts' weights
+};
+
+// One warp per token: scores s of the first `experts` logits; the k largest s + correction are chosen and weighted by
+// their s (`RouteScores`).  Behind the routed choices come `shared` always-on experts (ids 0 .. shared - 1); routed expert e has id shared + (e - e0) mod experts, so that the experts of the
 // rank that starts at e0 directly follow its shared ones.
 template <int MAX_PER_LANE>
 __global__ void __launch_bounds__(128) zb_moe_route_kernel(const float* __restrict__ logits, long long stride,
                                                            const float* __restrict__ correction, int32_t* __restrict__ ids,
                                                            float* __restrict__ weights, int tokens, int experts, int k, int shared,
-                                                           int e0) {
+                                                           int e0, const RouteScores how) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   float corr[MAX_PER_LANE];
@@ -108,23 +114,29 @@ __global__ void __launch_bounds__(128) zb_moe_route_kernel(const float* __restri
   zb_pdl_wait();
   if (warp >= tokens) return;
   const float* row = logits + static_cast<size_t>(warp) * stride;
-  const float gate = shared > 0 ? row[experts] : 0.f;
+  const float gate = shared > 0 && how.gated ? row[experts] : 0.f;
   float s[MAX_PER_LANE], v[MAX_PER_LANE], mx = -INFINITY, sum = 0.f;
 #pragma unroll
   for (int i = 0; i < MAX_PER_LANE; ++i) {
     s[i] = lane + 32 * i < experts ? row[lane + 32 * i] : -INFINITY;
     mx = fmaxf(mx, s[i]);
   }
-  mx = zb_warp_max(mx);
+  if (how.sigmoid) {
 #pragma unroll
-  for (int i = 0; i < MAX_PER_LANE; ++i) {
-    s[i] = lane + 32 * i < experts ? expf(s[i] - mx) : 0.f;
-    sum += s[i];
+    for (int i = 0; i < MAX_PER_LANE; ++i) s[i] = 1.f / (1.f + expf(-s[i]));
+  } else {
+    mx = zb_warp_max(mx);
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i) {
+      s[i] = lane + 32 * i < experts ? expf(s[i] - mx) : 0.f;
+      sum += s[i];
+    }
+    sum = zb_warp_sum(sum);
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i) s[i] /= sum;
   }
-  sum = zb_warp_sum(sum);
 #pragma unroll
   for (int i = 0; i < MAX_PER_LANE; ++i) {
-    s[i] /= sum;
     v[i] = lane + 32 * i < experts ? s[i] + corr[i] : -INFINITY;
   }
   float my_s = 0.f, total = 0.f;
@@ -164,9 +176,9 @@ __global__ void __launch_bounds__(128) zb_moe_route_kernel(const float* __restri
   const size_t at = static_cast<size_t>(warp) * (k + shared);
   if (lane < k) {
     ids[at + lane] = shared + (my_e >= e0 ? my_e - e0 : my_e - e0 + experts);
-    weights[at + lane] = my_s / (total + 1e-20f);
+    weights[at + lane] = how.scale * (how.normalize ? my_s / (total + 1e-20f) : my_s);
   }
-  const float on = 1.f / (1.f + expf(-gate));
+  const float on = how.gated ? 1.f / (1.f + expf(-gate)) : 1.f;
   for (int j = lane; j < shared; j += 32) {
     ids[at + k + j] = j;
     weights[at + k + j] = on;
@@ -841,17 +853,18 @@ int zb_moe_router_topk(const float* logits, int32_t* ids, float* weights, int to
   return static_cast<int>(cudaGetLastError());
 }
 
-// ids, weights [tokens, k + shared]; logits [tokens, >= experts (+ 1 with shared experts)]; see the kernel.
+// ids, weights [tokens, k + shared]; logits [tokens, >= experts (+ 1 with gated shared experts)]; see the kernel.
 int zb_moe_route(const float* logits, long long stride, const float* correction, int32_t* ids, float* weights, int tokens, int experts,
-                 int k, int shared, int e0, void* stream) {
+                 int k, int shared, int e0, int sigmoid, int normalize, int gated, float scale, void* stream) {
   if (tokens <= 0) return 0;
+  const RouteScores how = {sigmoid, normalize, gated, scale};
   if (k < 1 || k > 32 || experts < k || experts > 512 || shared < 0 || e0 < 0 || e0 >= experts) return -60;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid((tokens + 3) / 4), block(128);
   cudaError_t e;
-  if (experts <= 32) e = zb_launch(zb_moe_route_kernel<1>, grid, block, 0, s, logits, stride, correction, ids, weights, tokens, experts, k, shared, e0);
-  else if (experts <= 128) e = zb_launch(zb_moe_route_kernel<4>, grid, block, 0, s, logits, stride, correction, ids, weights, tokens, experts, k, shared, e0);
-  else e = zb_launch(zb_moe_route_kernel<16>, grid, block, 0, s, logits, stride, correction, ids, weights, tokens, experts, k, shared, e0);
+  if (experts <= 32) e = zb_launch(zb_moe_route_kernel<1>, grid, block, 0, s, logits, stride, correction, ids, weights, tokens, experts, k, shared, e0, how);
+  else if (experts <= 128) e = zb_launch(zb_moe_route_kernel<4>, grid, block, 0, s, logits, stride, correction, ids, weights, tokens, experts, k, shared, e0, how);
+  else e = zb_launch(zb_moe_route_kernel<16>, grid, block, 0, s, logits, stride, correction, ids, weights, tokens, experts, k, shared, e0, how);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }

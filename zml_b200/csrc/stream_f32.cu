@@ -8,6 +8,9 @@
 //   zb_sandwich_norm   x <- x + m * rmsnorm(y) * w, the residual sum of a sublayer with a norm behind it, and in the same
 //                      launch rmsnorm(x) * w_next, what the next sublayer reads.  y is a row, or the weighted sum of a
 //                      token's expert rows
+//   zb_add_norm        x <- x + y, the residual sum of a sublayer with a norm in front (y as above), and in the same launch what
+//                      the next sublayer reads: layernorm(x) * w + b, for decode steps on through its input convolution, or x
+//                      itself in the activation type
 //   zb_hyper_norm      hyper-connections: S streams per token instead of one.  x_t <- sum_s mix[s, t] x_s + out[t] y behind a
 //                      sublayer (y as above), and in the same launch rmsnorm(sum_s in[s] x_s) * w, what the next one reads
 //   zb_stream_conv     that input convolution over a varlen batch: h = x + conv(x), causal and per channel, and for
@@ -597,6 +600,196 @@ cudaError_t launch_sandwich(const SandwichArgs& p, int act_f32, int tokens, cuda
   return vec ? launch_sandwich<Y, __nv_bfloat16, 4>(p, tokens, s) : launch_sandwich<Y, __nv_bfloat16, 1>(p, tokens, s);
 }
 
+// ------------------------------------------------------------------------------------------ residual sum and layer norm
+struct AddNormArgs {
+  const void* y;               // as SandwichArgs
+  long long ldy;
+  const int32_t* pair_pos;
+  const float* pair_w;
+  int k;
+  const float* x;              // [T, d]
+  float* x_out;                // [T, d] or null (may be x)
+  const float* w;              // [d]: weight and bias of the norm; null: act is x_out itself
+  const float* b;
+  float eps;
+  void* act;                   // [T, ld_act] or null: columns d .. ld_act are zero
+  long long ld_act;
+  int d;
+};
+
+// T > 0: one token per sequence, and the normed row goes on through the convolution `a` with a.taps <= T (its output is `act`).
+template <typename Y, typename A, int NT, int NG, int V, int T>
+__global__ void __launch_bounds__(NT) zb_add_norm_kernel(const AddNormArgs p, const ConvArgs a, const int32_t* __restrict__ seq_lens) {
+  constexpr int kSlots = 32;                             // expert slots read through shared memory at a time
+  constexpr int R = T > 1 ? T - 1 : 1;                   // rows of state the convolution can need
+  __shared__ float red[2][NT / 32];
+  __shared__ float sw[kSlots];
+  __shared__ int spos[kSlots];
+  zb_pdl_launch();
+  const int d = p.d;
+  float w[NG][V], b[NG][V], cw[NG][T > 0 ? T : 1][V];    // parameters: on their way before the input is there
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + NT * i) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) w[i][e] = b[i][e] = 0.f;
+    if (c < d && p.w != nullptr) {
+      ld_vec<V>(w[i], p.w + c);
+      ld_vec<V>(b[i], p.b + c);
+    }
+    if constexpr (T > 0) {
+#pragma unroll
+      for (int j = 0; j < T; ++j) {                      // the last taps of the window count
+#pragma unroll
+        for (int e = 0; e < V; ++e) cw[i][j][e] = 0.f;
+        if (c < d && j >= T - a.taps) ld_vec<V>(cw[i][j], a.w + static_cast<size_t>(j - (T - a.taps)) * d + c);
+      }
+    }
+  }
+  zb_pdl_wait();
+  const long long t = blockIdx.x;
+  float x[NG][V], hist[NG][R][V];                        // hist[R - 1]: the newest past input
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + NT * i) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[i][e] = 0.f;
+    if (c < d) ld_vec<V>(x[i], p.x + t * d + c);
+  }
+  float* st0 = nullptr;
+  const int rows = a.rows;
+  if constexpr (T > 0) {
+    const int slot = a.slots[t];
+    const bool slot_ok = ZB_BC_OK(slot, ZB_BC_STATE_SLOTS, kKernelStreamConv, 3);
+    if (slot_ok) st0 = a.state + static_cast<size_t>(slot) * rows * d;
+    const bool fresh = !slot_ok || seq_lens[t] - 1 <= 0;
+#pragma unroll
+    for (int i = 0; i < NG; ++i) {
+      const int c = (threadIdx.x + NT * i) * V;
+#pragma unroll
+      for (int j = 0; j < R; ++j) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) hist[i][j][e] = 0.f;
+        if (c < d && !fresh && j >= R - rows) ld_vec<V>(hist[i][j], st0 + static_cast<size_t>(j - (R - rows)) * d + c);
+      }
+    }
+  }
+  if (p.y != nullptr) {
+    const Y* ys = reinterpret_cast<const Y*>(p.y);
+    auto add = [&](long long row, float wt) {
+#pragma unroll
+      for (int i = 0; i < NG; ++i) {
+        const int c = (threadIdx.x + NT * i) * V;
+        if (c >= d) continue;
+        float v[V];
+        if constexpr (V == 4) ld_row4(v, ys + row * p.ldy + c);
+        else v[0] = zb_ld_act(ys + row * p.ldy + c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[i][e] = fmaf(wt, v[e], x[i][e]);
+      }
+    };
+    if (p.pair_pos == nullptr) {
+      add(t, 1.f);
+    } else {
+      for (int j0 = 0; j0 < p.k; j0 += kSlots) {
+        const int n = min(kSlots, p.k - j0);
+        __syncthreads();
+        if (threadIdx.x < n) {
+          spos[threadIdx.x] = p.pair_pos[t * p.k + j0 + threadIdx.x];
+          sw[threadIdx.x] = p.pair_w[t * p.k + j0 + threadIdx.x];
+        }
+        __syncthreads();
+#pragma unroll 4
+        for (int j = 0; j < n; ++j)
+          if (spos[j] >= 0) add(spos[j], sw[j]);
+      }
+    }
+  }
+  if (p.x_out != nullptr) {
+#pragma unroll
+    for (int i = 0; i < NG; ++i) {
+      const int c = (threadIdx.x + NT * i) * V;
+      if (c < d) st_vec<float, V>(p.x_out + t * d + c, x[i]);
+    }
+  }
+  if (p.act == nullptr) return;
+  if (p.w != nullptr) {
+    float sum = 0.f, sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < NG; ++i)
+#pragma unroll
+      for (int e = 0; e < V; ++e) sum += x[i][e];
+    const float mean = block_sum_warps<NT / 32>(sum, red[0]) / static_cast<float>(d);
+#pragma unroll
+    for (int i = 0; i < NG; ++i) {
+      if ((threadIdx.x + NT * i) * V >= d) continue;     // columns past d stay zero
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        x[i][e] -= mean;
+        sq = fmaf(x[i][e], x[i][e], sq);
+      }
+    }
+    const float inv = 1.f / sqrtf(block_sum_warps<NT / 32>(sq, red[1]) / static_cast<float>(d) + p.eps);
+#pragma unroll
+    for (int i = 0; i < NG; ++i)
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[i][e] = fmaf(inv * x[i][e], w[i][e], b[i][e]);
+  }
+  A* act = reinterpret_cast<A*>(p.act) + t * p.ld_act;
+#pragma unroll
+  for (int i = 0; i < NG; ++i) {
+    const int c = (threadIdx.x + NT * i) * V;
+    if (c >= p.ld_act) continue;
+    if constexpr (T > 0) {
+      float h[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        float acc = cw[i][T - 1][e] * x[i][e];
+#pragma unroll
+        for (int j = 0; j + 1 < T; ++j) acc = fmaf(cw[i][j][e], hist[i][j][e], acc);
+        h[e] = x[i][e] + acc;
+      }
+      st_vec<A, V>(act + c, h);
+      if (st0 == nullptr || c >= d) continue;
+#pragma unroll
+      for (int j = 0; j < R; ++j) {
+        if (j < R - rows) continue;
+        float* dst = st0 + static_cast<size_t>(j - (R - rows)) * d + c;
+        if (j + 1 < R) st_vec<float, V>(dst, hist[i][j + 1 < R ? j + 1 : j]);
+        else st_vec<float, V>(dst, x[i]);
+      }
+    } else {
+      st_vec<A, V>(act + c, x[i]);
+    }
+  }
+}
+
+template <typename Y, typename A, int V, int T>
+cudaError_t launch_add_norm(const AddNormArgs& p, const ConvArgs& a, const int32_t* seq_lens, int tokens, cudaStream_t s) {
+  const long long groups = ((p.act != nullptr && p.ld_act > p.d ? p.ld_act : p.d) + V - 1) / V;
+  if (groups <= 128) return zb_launch(zb_add_norm_kernel<Y, A, 128, 1, V, T>, dim3(tokens), dim3(128), 0, s, p, a, seq_lens);
+  if (groups <= 512) return zb_launch(zb_add_norm_kernel<Y, A, 512, 1, V, T>, dim3(tokens), dim3(512), 0, s, p, a, seq_lens);
+  if (groups <= 1024) return zb_launch(zb_add_norm_kernel<Y, A, 512, 2, V, T>, dim3(tokens), dim3(512), 0, s, p, a, seq_lens);
+  if constexpr (T == 0)
+    if (groups <= 4096) return zb_launch(zb_add_norm_kernel<Y, A, 512, 8, V, T>, dim3(tokens), dim3(512), 0, s, p, a, seq_lens);
+  return cudaErrorInvalidValue;
+}
+template <typename Y, typename A, int V>
+cudaError_t launch_add_norm(const AddNormArgs& p, const ConvArgs& a, const int32_t* seq_lens, int tokens, cudaStream_t s) {
+  if (a.w == nullptr) return launch_add_norm<Y, A, V, 0>(p, a, seq_lens, tokens, s);
+  if (a.taps <= 4) return launch_add_norm<Y, A, V, 4>(p, a, seq_lens, tokens, s);
+  return launch_add_norm<Y, A, V, kMaxTaps>(p, a, seq_lens, tokens, s);
+}
+bool add_norm_vec(int d, long long ldy, const void* y) {
+  return d % 4 == 0 && (y == nullptr || (ldy % 4 == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0));
+}
+template <typename Y>
+cudaError_t launch_add_norm(const AddNormArgs& p, const ConvArgs& a, const int32_t* seq_lens, int act_f32, int tokens, cudaStream_t s) {
+  const bool vec = add_norm_vec(p.d, p.ldy, p.y) && (p.act == nullptr || p.ld_act % 4 == 0);
+  if (act_f32) return vec ? launch_add_norm<Y, float, 4>(p, a, seq_lens, tokens, s) : launch_add_norm<Y, float, 1>(p, a, seq_lens, tokens, s);
+  return vec ? launch_add_norm<Y, __nv_bfloat16, 4>(p, a, seq_lens, tokens, s) : launch_add_norm<Y, __nv_bfloat16, 1>(p, a, seq_lens, tokens, s);
+}
+
 // ------------------------------------------------------------------------------------------ hyper-connections
 constexpr int kMaxStreams = 8;
 
@@ -880,6 +1073,33 @@ int zb_hyper_norm(const void* y, long long ldy, int y_f32, const int32_t* pair_p
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const bool vec = d % 4 == 0 && (act == nullptr || ld_act % 4 == 0) && (y == nullptr || (ldy % 4 == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0));
   const cudaError_t e = vec ? launch_hyper<4>(p, tokens, s) : launch_hyper<1>(p, tokens, s);
+  zb_count_launch(1);
+  return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
+}
+
+// 1 when zb_add_norm takes a convolution for rows of d channels with these inputs: it holds a row in 512 threads.
+int zb_add_norm_conv_supported(const void* y, long long ldy, int d, long long ld_act) {
+  const int v = add_norm_vec(d, ldy, y) && ld_act % 4 == 0 ? 4 : 1;
+  return (ld_act > d ? ld_act : d) <= 1024ll * v ? 1 : 0;
+}
+
+// x_out = x + y; act = layernorm(x_out) * w + b, or x_out itself without w.  y as in zb_sandwich_norm; null: nothing to add.
+// `conv_w` non-null: one token per sequence, and act is what zb_stream_conv (without interpolations) makes of the normed rows.
+// d as in zb_sandwich_norm.
+int zb_add_norm(const void* y, long long ldy, int y_f32, const int32_t* pair_pos, const float* pair_w, int k, const float* x, float* x_out,
+                const float* w, const float* b, float eps, void* act, long long ld_act, int act_f32, int tokens, int d, const float* conv_w,
+                float* state, const int32_t* slots, int taps, const int32_t* seq_lens, void* stream) {
+  if (tokens <= 0) return 0;
+  if ((w == nullptr) != (b == nullptr) || (act != nullptr && ld_act < d)) return -70;
+  const AddNormArgs p = {y, ldy, pair_pos, pair_w, k, x, x_out, w, b, eps, act, ld_act, d};
+  ConvArgs a = {};
+  if (conv_w != nullptr) {
+    if (!conv_ok(taps, taps - 1, 0) || w == nullptr || act == nullptr || !zb_add_norm_conv_supported(y, ldy, d, ld_act)) return -70;
+    a = conv_args(conv_w, state, slots, nullptr, act, ld_act, 0, taps, taps - 1, 0, d);
+  }
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const cudaError_t e = y_f32 ? launch_add_norm<float>(p, a, seq_lens, act_f32, tokens, s)
+                              : launch_add_norm<__nv_bfloat16>(p, a, seq_lens, act_f32, tokens, s);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }

@@ -60,7 +60,7 @@ MODEL_TYPES = {
     "llama": "llama", "qwen3_5": "qwen3_5", "qwen3_5_text": "qwen3_5", "qwen3_5_moe": "qwen3_5_moe",
     "qwen3_5_moe_text": "qwen3_5_moe", "lfm2": "lfm2", "qwen3": "qwen3", "qwen2": "qwen3",
     "qwen3_moe": "qwen3_moe", "mistral": "llama", "dopurax": "dopurax", "kirisun": "kirisun",
-    "sodotar": "sodotar",
+    "sodotar": "sodotar", "dogidra": "dogidra",
 }
 
 

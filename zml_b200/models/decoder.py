@@ -3,6 +3,7 @@ the output head, sampling, and the cache / plan hooks a model may override.
 """
 from __future__ import annotations
 
+import dataclasses
 from dataclasses import dataclass, field
 from typing import Optional
 
@@ -68,6 +69,17 @@ class DecoderModel:
     def decode_splits(self, batch: int, max_seq_len: int) -> int:
         """KV chunks per sequence of a decode step (part of the key of captured graphs)."""
         return ops.decode_plan_splits(batch, self.hkv, max_seq_len)
+
+    def layer_plan(self, meta: AttnMeta, splits) -> AttnMeta:
+        """The metadata of a decode step with a layer's own number of key chunks, at most the step's: a layer that sees a part of
+        the sequence is cut into fewer pieces than one that sees all of it.  `splits(max_seq_len)`: that number."""
+        if meta.is_prefill or meta.num_splits is None or meta.max_seq_len is None or self.device.type != "cuda":
+            return meta
+        n = min(meta.num_splits, splits(meta.max_seq_len))
+        plan = meta.plans.get(("splits", n))
+        if plan is None:
+            plan = meta.plans[("splits", n)] = dataclasses.replace(meta, num_splits=n)
+        return plan
 
     # ------------------------------------------------------------------ output head
     def _pad_lm_head(self) -> None:

@@ -15,6 +15,7 @@ from .llama import PRESETS as LLAMA_PRESETS, LlamaConfig, LlamaModel
 
 def _families():
     """(presets, config class, model class) of every model family, imported lazily."""
+    from .dogidra import PRESETS as P_DOG, DogidraConfig, DogidraModel
     from .dopurax import PRESETS as P_DOP, DopuraxConfig, DopuraxModel
     from .kirisun import PRESETS as P_KIR, KirisunConfig, KirisunModel
     from .lfm2 import PRESETS as P_LFM2, Lfm2Config, Lfm2Model
@@ -25,7 +26,8 @@ def _families():
     return [(LLAMA_PRESETS, LlamaConfig, LlamaModel), (P_MOE, Qwen3MoeConfig, Qwen3MoeModel),
             (P_Q35, Qwen35Config, Qwen35Model), (P_Q35M, Qwen35MoeConfig, Qwen35MoeModel),
             (P_LFM2, Lfm2Config, Lfm2Model), (P_DOP, DopuraxConfig, DopuraxModel),
-            (P_KIR, KirisunConfig, KirisunModel), (P_SOD, SodotarConfig, SodotarModel)]
+            (P_KIR, KirisunConfig, KirisunModel), (P_SOD, SodotarConfig, SodotarModel),
+            (P_DOG, DogidraConfig, DogidraModel)]
 
 
 def preset_names() -> list[str]:
@@ -80,4 +82,7 @@ def model_class_for(config: dict):
     if kind == "sodotar":
         from .sodotar import SodotarConfig, SodotarModel
         return SodotarConfig, SodotarModel
+    if kind == "dogidra":
+        from .dogidra import DogidraConfig, DogidraModel
+        return DogidraConfig, DogidraModel
     raise ValueError(kind)

@@ -17,7 +17,6 @@ mixture.  Tensor parallelism splits heads, experts and the shared expert's hidde
 """
 from __future__ import annotations
 
-import dataclasses
 from dataclasses import dataclass, field
 from typing import Optional
 
@@ -464,19 +463,14 @@ class SodotarModel(DecoderModel):
         return max((self._layer_splits(L, batch, max_seq_len) for L in self.layers), default=1)
 
     def _plan(self, i: int, batch: int, meta: AttnMeta) -> AttnMeta:
-        """The step's metadata with this layer's own number of key chunks: a layer that sees one chunk of the sequence is cut
-        into fewer pieces than one that sees all of it."""
-        if meta.is_prefill or meta.num_splits is None or meta.max_seq_len is None or self.device.type != "cuda":
-            return meta
         L = self.layers[i]
-        key = (L.latent or L.attn, batch, meta.max_seq_len)
-        n = self._splits.get(key)
-        if n is None:
-            n = self._splits[key] = min(meta.num_splits, self._layer_splits(L, batch, meta.max_seq_len))
-        plan = meta.plans.get(("splits", n))
-        if plan is None:
-            plan = meta.plans[("splits", n)] = dataclasses.replace(meta, num_splits=n)
-        return plan
+
+        def splits(max_seq_len):
+            key = (L.latent or L.attn, batch, max_seq_len)
+            if key not in self._splits:
+                self._splits[key] = self._layer_splits(L, batch, max_seq_len)
+            return self._splits[key]
+        return self.layer_plan(meta, splits)
 
     # ------------------------------------------------------------------ forward
     def _out_proj(self, a, w):

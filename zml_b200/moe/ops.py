@@ -22,7 +22,7 @@ _lib.register_signature("zb_moe_grouped_gemm", C.c_int, [C.c_void_p, C.c_void_p,
 _lib.register_signature("zb_moe_grouped_f32", C.c_int, [C.c_void_p, C.c_longlong, C.c_void_p, C.c_int, C.c_void_p, C.c_void_p, C.c_longlong,
                                                          C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_int, C.c_int, C.c_void_p, C.c_void_p])
 _lib.register_signature("zb_moe_route", C.c_int, [C.c_void_p, C.c_longlong, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_int,
-                                                  C.c_int, C.c_void_p])
+                                                  C.c_int, C.c_int, C.c_int, C.c_int, C.c_float, C.c_void_p])
 
 
 class Backend(enum.Enum):
@@ -58,29 +58,35 @@ def router_topk(logits: torch.Tensor, k: int, renormalize: bool = True):
     return ids, w
 
 
-def route(logits: torch.Tensor, k: int, experts: int, correction: Optional[torch.Tensor] = None, shared: int = 0, e0: int = 0):
-    """Routing by softmax scores: s = softmax(logits[:, :experts]); the k experts with the largest s + correction, weighted by
-    their s divided by the sum (+ 1e-20).  `shared` experts run for every token, weighted by sigmoid(logits[:, experts]).
+def route(logits: torch.Tensor, k: int, experts: int, correction: Optional[torch.Tensor] = None, shared: int = 0, e0: int = 0,
+          scores: str = "softmax", normalize: bool = True, scale: float = 1.0, shared_gate: bool = True):
+    """Routing by scores: s = softmax or sigmoid (`scores`) of logits[:, :experts]; the k experts with the largest s + correction,
+    weighted by their s, with `normalize` divided by the sum (+ 1e-20), times `scale`.  `shared` experts run for every token,
+    weighted by sigmoid(logits[:, experts]) or, without `shared_gate`, by one.
     Returns (ids int32 [T, k + shared], weights float32): the choices first, then the shared ones.  Shared experts have the ids
     0 .. shared - 1, expert e has shared + (e - e0) mod experts: the local experts of the rank that starts at e0 follow its
     shared ones, so `moe_align(ids, 0, shared + local)` takes both."""
     t = logits.shape[0]
-    assert logits.shape[1] >= experts + (1 if shared else 0)
+    shared_gate = shared_gate and shared > 0
+    assert logits.shape[1] >= experts + int(shared_gate) and scores in ("softmax", "sigmoid")
     if not logits.is_cuda:
-        s = torch.softmax(logits[:, :experts].float(), -1)
+        z = logits[:, :experts].float()
+        s = torch.sigmoid(z) if scores == "sigmoid" else torch.softmax(z, -1)
         i = torch.topk(s if correction is None else s + correction.float(), k, dim=-1).indices
         w = s.gather(1, i)
-        ids, w = shared + (i - e0) % experts, w / (w.sum(-1, keepdim=True) + 1e-20)
+        ids, w = shared + (i - e0) % experts, scale * (w / (w.sum(-1, keepdim=True) + 1e-20) if normalize else w)
         if shared:
             ids = torch.cat([ids, torch.arange(shared).expand(t, shared)], 1)
-            w = torch.cat([w, torch.sigmoid(logits[:, experts:experts + 1].float()).expand(t, shared)], 1)
+            on = torch.sigmoid(logits[:, experts:experts + 1].float()) if shared_gate else torch.ones((t, 1))
+            w = torch.cat([w, on.expand(t, shared)], 1)
         return ids.to(torch.int32).contiguous(), w.contiguous()
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     assert correction is None or (correction.dtype == torch.float32 and correction.numel() == experts)
     ids = torch.empty((t, k + shared), dtype=torch.int32, device=logits.device)
     w = torch.empty((t, k + shared), dtype=torch.float32, device=logits.device)
     _lib.check(_lib.lib().zb_moe_route(logits.data_ptr(), logits.stride(0), correction.data_ptr() if correction is not None else None, ids.data_ptr(),
-                                       w.data_ptr(), t, experts, k, shared, e0, _lib.stream_ptr()), "zb_moe_route")
+                                       w.data_ptr(), t, experts, k, shared, e0, int(scores == "sigmoid"), int(normalize), int(shared_gate),
+                                       float(scale), _lib.stream_ptr()), "zb_moe_route")
     return ids, w
 
 
@@ -517,6 +523,24 @@ def pad_experts(gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor):
     _, f, d = gate.shape
     fp, d8, dp = -f % 64, -d % 8, -d % 128
     return interleave_gate_up(pad(gate, (0, d8, 0, fp)), pad(up, (0, d8, 0, fp))), pad(down, (0, fp, 0, dp)).contiguous()
+
+
+def pad_plain_experts(up: torch.Tensor, down: torch.Tensor):
+    """The same for experts without a gate (up [E, F, D], down [E, D, F]): zero hidden units up to a multiple of 128."""
+    pad = torch.nn.functional.pad
+    _, f, d = up.shape
+    fp, d8, dp = -f % 128, -d % 8, -d % 128
+    return pad(up, (0, d8, 0, fp)).contiguous(), pad(down, (0, fp, 0, dp)).contiguous()
+
+
+def shared_pieces(up: torch.Tensor, down: torch.Tensor, size: int):
+    """A shared expert (up [F, D], down [D, F], or several stacked as up [n, F, D]) cut into pieces of `size` hidden units, zero
+    units behind the last: (up [.., pieces, size, D], down [pieces, D, size]).  Every token is routed to all pieces."""
+    f = up.shape[-2]
+    n = (f + size - 1) // size
+    pad = torch.nn.functional.pad
+    up = pad(up, (0, 0, 0, n * size - f))
+    return up.reshape(*up.shape[:-2], n, size, up.shape[-1]), pad(down, (0, n * size - f)).reshape(down.shape[0], n, size).transpose(0, 1)
 
 
 def expert_rows(x: torch.Tensor, topk_ids: torch.Tensor, w_gate_up_il: torch.Tensor, w_down: torch.Tensor, e0: int = 0,

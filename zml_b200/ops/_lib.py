@@ -159,7 +159,8 @@ KERNEL_NAMES = {1: "gemm_bf16", 2: "paged_decode", 3: "paged_prefill", 4: "gemm_
                 10: "moe_combine", 11: "allreduce_ll", 12: "allreduce_mm", 13: "paged_prefill_tc", 14: "gemm_2cta", 15: "argmax_tp",
                 20: "rope_kvwrite", 21: "embedding", 22: "decode_advance", 24: "causal_conv1d", 25: "gated_delta_scan",
                 26: "embedding_f32", 27: "stream_conv", 28: "latent_prep", 29: "latent_attend", 30: "latent_gather", 31: "wkv_scan",
-                32: "latent_prefill_tc", 33: "latent_decode", 34: "gqa_prep", 35: "gqa_attend", 36: "channel_delta"}
+                32: "latent_prefill_tc", 33: "latent_decode", 34: "gqa_prep", 35: "gqa_attend", 36: "channel_delta",
+                37: "gqa_pool", 38: "gated_scan"}
 
 
 class BoundsError(KernelError):

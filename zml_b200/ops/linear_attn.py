@@ -1,7 +1,8 @@
 """Ops of the hybrid decoder layers: depthwise causal conv with a rolling cache, the gated
 delta rule scan, and the sigmoid output gate (libzb_cuda.so: linear_attn.cu); the WKV
 recurrence with its low-rank decay (wkv.cu); the delta rule with a decay per key channel, with its
-convolutions, norms and gate (channel_delta.cu).
+convolutions, norms and gate (channel_delta.cu); the recurrence whose gates read the current token only
+(gated_scan.cu).
 
 All of them run over the flattened varlen token batch the engine uses everywhere else:
 `q_start[S+1]` gives every sequence's token range in this launch, `seq_lens[S]` its length
@@ -343,4 +344,55 @@ def channel_delta(proj, beta_col: int, low, m: ChannelDelta, q_start, seq_lens, 
         _ptr(proj), proj.stride(0), beta_col, _ptr(low), low.stride(0), _ptr(m.conv_w), m.taps, _ptr(m.a_log), _ptr(m.dt_bias), _ptr(m.norm),
         float(m.eps), _ptr(m.ring), _ptr(m.state), _ptr(slots), _ptr(blocks), _ptr(o), _ptr(out), out.stride(0), m.heads, m.kv_heads, m.dim,
         m.vdim, int(proj.dtype == torch.float32), _ptr(q_start), _ptr(seq_lens), seq_lens.shape[0], t, nb, _lib.stream_ptr()), "zb_channel_delta")
+    return out
+
+
+# ---------------------------------------------------------------------------- recurrence with gates of the current token
+_lib.register_signature("zb_gated_scan_rows", _i, [])
+_lib.register_signature("zb_gated_scan", _i, [_p, _p, _p, _ll, _p, _p, _p, _p, _p, _p, _ll, _f, _i, _i, _p, _p, _i, _i, _p])
+
+GATED_ROWS = 64          # tokens per block of the kernel
+
+
+def gated_scan_reference(z, x, gate, z_bias, x_bias, state, q_start, seq_lens, slots, scale):
+    g, u, f = torch.sigmoid(z.float() + z_bias), x.float() + x_bias, gate.float()
+    c = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+    out = torch.zeros(z.shape)
+    qs, sl, so = q_start.tolist(), seq_lens.tolist(), slots.tolist()
+    for s in range(len(sl)):
+        a, b = qs[s], qs[s + 1]
+        if b <= a:
+            continue
+        st = torch.zeros(z.shape[1]) if sl[s] - (b - a) <= 0 else state[so[s]].clone()
+        for i in range(a, b):
+            st = (1 - g[i]) * st + g[i] * c[i]
+            out[i] = st
+        state[so[s]] = st
+    return (out * f * torch.sigmoid(f) * scale).to(z.dtype)
+
+
+def gated_scan(z, x, gate, z_bias, x_bias, state, q_start, seq_lens, slots, scale: float = 1.0, out=None, decode: bool = False,
+               num_blocks: Optional[int] = None):
+    """minGRU by channel: with g = sigmoid(z + z_bias), u = x + x_bias and the candidate c = u + 1/2 where u >= 0, else
+    sigmoid(u): S <- (1 - g) S + g c, out = S * silu(gate) * scale.  z, x, gate [T, width] (equal row strides), biases fp32
+    [width], state fp32 [slots, width] updated in place.  `decode`: one token per sequence; else `num_blocks` (optional) is the
+    sum of ceil(tokens / 64) over the sequences.  `out`: [T, width] columns of a wider buffer to write to."""
+    if not z.is_cuda:
+        y = gated_scan_reference(z, x, gate, z_bias, x_bias, state, q_start, seq_lens, slots, scale)
+        return y if out is None else out.copy_(y)
+    t, n = z.shape
+    l = _lib.lib()
+    assert z.stride(0) == x.stride(0) == gate.stride(0) and z.stride(1) == 1 and z.dtype == x.dtype == gate.dtype
+    assert state.dtype == z_bias.dtype == x_bias.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == n
+    if out is None:
+        out = torch.empty((t, n), dtype=z.dtype, device=z.device)
+    assert out.shape == (t, n) and out.stride(1) == 1 and out.dtype == z.dtype
+    maps, nb = None, 0
+    if not decode:
+        rows = l.zb_gated_scan_rows()
+        nb = num_blocks if num_blocks is not None and rows == GATED_ROWS else t // rows + seq_lens.shape[0]
+        maps = torch.empty((nb, n, 2), dtype=torch.float32, device=z.device)
+    _lib.check(l.zb_gated_scan(
+        _ptr(z), _ptr(x), _ptr(gate), z.stride(0), _ptr(z_bias), _ptr(x_bias), _ptr(state), _ptr(slots), _ptr(maps), _ptr(out), out.stride(0),
+        float(scale), n, int(z.dtype == torch.float32), _ptr(q_start), _ptr(seq_lens), seq_lens.shape[0], nb, _lib.stream_ptr()), "zb_gated_scan")
     return out

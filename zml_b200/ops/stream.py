@@ -19,6 +19,8 @@ _p, _i, _ll, _f = C.c_void_p, C.c_int, C.c_longlong, C.c_float
 _lib.register_signature("zb_embedding_f32", _i, [_p, _p, _i, _p, _i, _i, _i, _f, _i, _p])
 _lib.register_signature("zb_hyper_norm", _i, [_p, _ll, _i, _p, _p, _i, _p, _i, _p, _p, _p, _p, _f, _p, _p, _ll, _i, _i, _i, _p])
 _lib.register_signature("zb_sandwich_norm", _i, [_p, _ll, _i, _p, _p, _i, _p, _f, _p, _p, _f, _p, _p, _ll, _i, _i, _i, _p])
+_lib.register_signature("zb_add_norm_conv_supported", _i, [_p, _ll, _i, _ll])
+_lib.register_signature("zb_add_norm", _i, [_p, _ll, _i, _p, _p, _i, _p, _p, _p, _p, _f, _p, _ll, _i, _i, _i, _p, _p, _p, _i, _p, _p])
 _lib.register_signature("zb_stream_conv", _i, [_p, _p, _p, _p, _p, _p, _i, _ll, _ll, _i, _i, _i, _i, _p, _p, _i, _i, _p])
 _lib.register_signature("zb_post_norm", _i, [_p, _ll, _i, _p, _f, _p, _f, _p, _p, _ll, _i, _i, _i, _p, _p, _p, _p, _p, _ll, _ll,
                                              _i, _i, _i, _p, _p])
@@ -77,6 +79,12 @@ class InputConv:
         shape = (tokens, self.w.shape[1]) if self.mu is None else (self.nmix(), tokens, self.w.shape[1])
         return torch.empty(shape, dtype=dtype, device=device)
 
+    def alloc_padded(self, tokens: int, dtype, device):
+        """h with zero columns up to a multiple of 8."""
+        d = self.w.shape[1]
+        make = torch.empty if d % 8 == 0 else torch.zeros
+        return make((tokens, pad8(d)), dtype=dtype, device=device)
+
     def args(self, out):
         """The trailing kernel arguments: out pointer, row stride, plane stride, taps, rows, nmix."""
         return (_ptr(out), out.stride(-2), out.stride(0) if self.mu is not None else 0, self.w.shape[0], self.state.shape[1], self.nmix())
@@ -103,14 +111,16 @@ def _stream_conv_reference(x, conv: InputConv, q_start, seq_lens, slots, dtype):
     return out
 
 
-def stream_conv(x, conv: InputConv, q_start, seq_lens, slots, dtype, num_blocks: Optional[int] = None):
-    """x [T, d] fp32 -> h [T, d] or the interpolations [nmix, T, d], in `dtype`; updates `conv.state`."""
+def stream_conv(x, conv: InputConv, q_start, seq_lens, slots, dtype, num_blocks: Optional[int] = None, padded: bool = False):
+    """x [T, d] fp32 -> h [T, d] or the interpolations [nmix, T, d], in `dtype`; updates `conv.state`.  `padded` (h only): with
+    zero columns up to a multiple of 8."""
     conv.check()
     if not x.is_cuda:
-        return _stream_conv_reference(x, conv, q_start, seq_lens, slots, dtype)
+        h = _stream_conv_reference(x, conv, q_start, seq_lens, slots, dtype)
+        return torch.nn.functional.pad(h, (0, pad8(h.shape[1]) - h.shape[1])) if padded else h
     t, d = x.shape
     assert x.is_contiguous() and x.dtype == torch.float32
-    out = conv.alloc(t, dtype, x.device)
+    out = conv.alloc_padded(t, dtype, x.device) if padded else conv.alloc(t, dtype, x.device)
     nb = num_blocks if num_blocks is not None else t // CONV_BLOCK + seq_lens.shape[0]
     ptr, ld, plane, taps, rows, nmix = conv.args(out)
     _lib.check(_lib.lib().zb_stream_conv(_ptr(x), _ptr(conv.w), _ptr(conv.state), _ptr(slots), _ptr(conv.mu), ptr,
@@ -203,6 +213,58 @@ def sandwich_norm(x, y=None, w=None, mult: float = 1.0, w_next=None, eps: float 
         _ptr(x), float(mult), _ptr(w), _ptr(w_next), float(eps), _ptr(x) if keep_x and rows is not None else None, _ptr(act), pad8(d),
         int(act_dtype == torch.float32), t, d, _lib.stream_ptr()), "zb_sandwich_norm")
     return (x if keep_x else None), act
+
+
+# ------------------------------------------------------------------ norm in front of a sublayer
+def _rows_of(y):
+    """(rows, pair_pos, weights, k) of a sublayer's output, a tensor or `ExpertRows`."""
+    if not isinstance(y, ExpertRows):
+        return y, None, None, 0
+    assert y.weights.dtype == torch.float32 and y.weights.is_contiguous()
+    return y.rows, y.pair_pos, y.weights, y.weights.shape[1]
+
+
+def add_norm(x, y=None, w=None, b=None, eps: float = 1e-6, act_dtype=None, conv: Optional[InputConv] = None, seq_lens=None, slots=None,
+             inplace: bool = True, keep_x: bool = True, padded: bool = True):
+    """The residual sum of a sublayer with a norm in front, and what the next one reads, in one launch: x_new = x + y and
+    act = layernorm(x_new) * w + b in `act_dtype` ([T, d], `padded` with zero columns up to a multiple of 8) - for a decode step, one token
+    per sequence, what `stream_conv` makes of that when `conv` is given.  Without w, act is x_new itself; without `act_dtype`, no
+    act.  x fp32 [T, d]; y [T, >= d] (bf16 or fp32) or `ExpertRows`.  Returns (x_new or None, act or None); on CUDA x is
+    overwritten unless `inplace` is off."""
+    t, d = x.shape
+    if not x.is_cuda:
+        if y is not None:
+            x = x + (y.sum(d) if isinstance(y, ExpertRows) else y[:, :d].float())
+        act = None
+        if act_dtype is not None:
+            n = x if w is None else layer_norm_reference(x, w, eps) + b
+            if conv is not None:
+                n = _stream_conv_reference(n, conv, torch.arange(t + 1, dtype=torch.int32), seq_lens, slots, act_dtype)
+            act = torch.nn.functional.pad(n, (0, pad8(d) - d if padded else 0)).to(act_dtype)
+        return (x if keep_x else None), act
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    rows, pos, pw, k = _rows_of(y)
+    assert rows is None or (rows.stride(1) == 1 and rows.shape[1] >= d and rows.dtype in (torch.float32, torch.bfloat16))
+    assert w is None or (w.dtype == b.dtype == torch.float32 and w.numel() == b.numel() == d)
+    ldy, ptr, l = rows.stride(0) if rows is not None else 0, _ptr(rows), _lib.lib()
+    apart = None
+    if conv is not None:
+        conv.check()
+        if not l.zb_add_norm_conv_supported(ptr, ldy, d, pad8(d)):
+            apart, conv, dtype, act_dtype = conv, None, act_dtype, torch.float32             # norm and convolution in two launches
+    ld = d if apart is not None or not padded else pad8(d)
+    act = torch.empty((t, ld), dtype=act_dtype, device=x.device) if act_dtype is not None else None
+    x_new = None if not keep_x or (rows is None and inplace) else (x if inplace else torch.empty_like(x))
+    c = conv
+    _lib.check(l.zb_add_norm(
+        ptr, ldy, int(rows is not None and rows.dtype == torch.float32), _ptr(pos), _ptr(pw), k, _ptr(x), _ptr(x_new), _ptr(w), _ptr(b), float(eps),
+        _ptr(act), ld, int(act_dtype == torch.float32), t, d, _ptr(c.w) if c else None, _ptr(c.state) if c else None, _ptr(slots) if c else None,
+        c.w.shape[0] if c else 0, _ptr(seq_lens) if c else None, _lib.stream_ptr()), "zb_add_norm")
+    if apart is not None:
+        act = stream_conv(act, apart, torch.arange(t + 1, dtype=torch.int32, device=x.device), seq_lens, slots, dtype, t, padded=True)
+    if not keep_x:
+        return None, act
+    return (x if inplace else x_new), act
 
 
 # ------------------------------------------------------------------ hyper-connections
