@@ -297,7 +297,7 @@ c.finish(0)
 
 @pytest.mark.parametrize("world,families", [
     (2, "tiny-llama-test,tiny-moe-test,tiny-qwen35-test,tiny-qwen35-moe-test,tiny-lfm2-test,tiny-dopurax-test,tiny-kirisun-test,"
-        "tiny-sodotar-test"),
+        "tiny-sodotar-test,tiny-dogidra-test"),
     (4, "tiny-llama-test,tiny-moe-test,tiny-dopurax-test"),           # the tiny hybrids have 2 linear-attention heads: not divisible by 4
 ])
 def test_every_model_family_under_two_way_parallelism_on_cpu(tmp_path, world, families):
@@ -316,7 +316,7 @@ def test_every_model_family_under_two_way_parallelism_on_cpu(tmp_path, world, fa
     assert r.stdout.count("TP_CPU_OK") == world
 
 
-@pytest.mark.parametrize("name", ["tiny-llama-test", "tiny-qwen35-test", "tiny-dopurax-test", "tiny-kirisun-test", "tiny-sodotar-test"])
+@pytest.mark.parametrize("name", ["tiny-llama-test", "tiny-qwen35-test", "tiny-dopurax-test", "tiny-kirisun-test", "tiny-sodotar-test", "tiny-dogidra-test"])
 def test_continuous_admission_matches_one_at_a_time_generation(name):
     """Seven prompts through three batch rows: sequences leave and join between decode blocks (also with staggered
     arrivals); every prompt gets the tokens it gets alone, and all pages and state slots come back."""
