@@ -51,6 +51,9 @@ WORKLOADS = {
     "sodotar-3b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
     "sodotar-10b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
     "tiny-sodotar-test": dict(batch=4, prompt=(16, 64), new_tokens=8),
+    "dogidra-3b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
+    "dogidra-10b": dict(batch=32, prompt=(128, 2048), new_tokens=512),
+    "tiny-dogidra-test": dict(batch=4, prompt=(16, 64), new_tokens=8),
 }
 
 
@@ -222,7 +225,8 @@ def run_workload(name: str, comm, args, steps: int, warmup: int, sample_clocks: 
 # depth, vocabulary, head sizes of the recurrent layers and feed-forward parameters (Dopurax: three matrices of 2/3 the
 # units; Kirisun: the same experts, and the shared expert that the family always has at its smallest size).  Sodotar, which
 # has no recurrence, stands beside the same family with gated full attention in every layer and the same routed and shared
-# experts.
+# experts.  Dogidra stands beside Kirisun: attention with the same heads and window and the delta rule in turn, a layer for every
+# run of one, and gated experts of two thirds the units, one more of them and one more choice for the shared one.
 COMPARE_SHAPES = [dict(batch=1, prompt=4096), dict(batch=8, prompt=1024), dict(batch=32, prompt=1024), dict(batch=64, prompt=2048)]
 
 
@@ -236,6 +240,19 @@ def moe_hybrid_twin(cfg) -> dict:
                 linear_key_head_dim=rec.dim, linear_num_key_heads=rec.kv_heads, linear_value_head_dim=rec.vdim, linear_num_value_heads=rec.heads,
                 layer_types=["full_attention" if s.kind == ATTENTION else "linear_attention" for s in cfg.layers], num_experts=att.experts,
                 num_experts_per_tok=att.top, moe_intermediate_size=att.ff, shared_expert_intermediate_size=64, tie_word_embeddings=False)
+
+
+def kirisun_twin(cfg) -> dict:
+    s = cfg.layers[0]
+    e = s.moe
+    head = dict(heads=s.heads, kv_heads=s.kv_heads, dim=s.dim, vdim=s.vdim)
+    att = dict(head, rot={"base": s.base, "dims": s.rot, "scaling": {"factor": s.yarn.factor}}, scale=s.scale, softcap=s.cap,
+               mask={"size": s.window, "keep_first": 16})
+    rec = dict(heads=s.width // s.vdim, kv_heads=s.width // s.vdim, dim=s.dim, vdim=s.vdim, conv=cfg.taps)
+    mlp = {"kind": "moe", "expert": {"ff": e.ff * 2 // 3}, "router": {"experts": e.experts + 1, "top": e.top + 1}}
+    layers = [{"type": "channel_delta" if i % 2 else "attention", "mixer": rec if i % 2 else att, "mlp": mlp} for i in range(len(cfg.runs()))]
+    return dict(architecture="Kirisun", width=cfg.hidden_size, vocab=cfg.vocab_size, layers=layers, norm={"eps": cfg.norm_eps}, embedding={"scale": 1.0},
+                residual_mult=0.5, decay_rank=128, gate_rank=128)
 
 
 def moe_attention_twin(cfg) -> dict:
@@ -278,6 +295,10 @@ def compare(name: str, args) -> None:
         from zml_b200.models.sodotar import PRESETS, SodotarConfig as Config, SodotarModel as Model
         from zml_b200.models.qwen3_5_moe import Qwen35MoeConfig as TwinConfig, Qwen35MoeModel as TwinModel
         to_twin = moe_attention_twin
+    elif name.startswith("dogidra"):
+        from zml_b200.models.dogidra import PRESETS, DogidraConfig as Config, DogidraModel as Model
+        from zml_b200.models.kirisun import KirisunConfig as TwinConfig, KirisunModel as TwinModel
+        to_twin = kirisun_twin
     else:
         from zml_b200.models.dopurax import PRESETS, DopuraxConfig as Config, DopuraxModel as Model
         from zml_b200.models.qwen3_5 import Qwen35Config as TwinConfig, Qwen35Model as TwinModel
@@ -286,7 +307,8 @@ def compare(name: str, args) -> None:
     twin = TwinConfig.from_hf(to_twin(cfg))
     sampler = ClockSampler(True)
     new, out = args.new_tokens or 128, {}
-    for label, build in ((name, lambda: Model(cfg, device="cuda:0")), ("other family at equal size" if to_twin is moe_attention_twin else "hybrid of equal size", lambda: TwinModel(twin, device="cuda:0"))):
+    for label, build in ((name, lambda: Model(cfg, device="cuda:0")),
+                         ("hybrid of equal size" if to_twin in (hybrid_twin, moe_hybrid_twin) else "other family at equal size", lambda: TwinModel(twin, device="cuda:0"))):
         model = build().init_random(args.seed)
         model.SERIAL_PREFILL = True                  # the same launch mode for both
         rows = []
@@ -336,7 +358,7 @@ def main() -> None:
     ap.add_argument("--headline", default="auto", choices=["auto", "none"],
                     help="auto: after the scaling configuration also measure the headline configurations that fit this "
                          "number of GPUs (Llama-3.1-70B and the NVFP4 MoE at 8, the MoE at 2 and 4), 3 timed jobs each")
-    ap.add_argument("--compare", default="", choices=["", "dopurax-1b", "dopurax-8b", "kirisun-3b", "kirisun-10b", "sodotar-3b", "sodotar-10b"],
+    ap.add_argument("--compare", default="", choices=["", "dopurax-1b", "dopurax-8b", "kirisun-3b", "kirisun-10b", "sodotar-3b", "sodotar-10b", "dogidra-3b", "dogidra-10b"],
                     help="instead of the benchmark: prefill and decode throughput of this design beside the closest other family at equal "
                          "size, at a few batch shapes (1 GPU)")
     args = ap.parse_args()

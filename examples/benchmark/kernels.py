@@ -12,6 +12,11 @@
     python examples/benchmark/kernels.py --op=stream --tokens=4096 --k=4096
     python examples/benchmark/kernels.py --op=gqa_prefill --batch=2 --seqlen=2048 --window=4096
     python examples/benchmark/kernels.py --op=gqa_decode --batch=32 --seqlen=1344 --window=4096
+    python examples/benchmark/kernels.py --op=pool_prefill --batch=2 --seqlen=8192 --window=1024 --pool=16
+    python examples/benchmark/kernels.py --op=pool_decode --batch=32 --seqlen=8192 --window=1024 --pool=16
+    python examples/benchmark/kernels.py --op=gated_scan --batch=8 --seqlen=512 --k=4096
+    python examples/benchmark/kernels.py --op=add_norm --tokens=4096 --k=4096
+    python examples/benchmark/kernels.py --op=relu_mixture --tokens=32 --experts=32 --topk=4 --n=1536 --k=2048
     python examples/benchmark/kernels.py --op=channel_delta --batch=8 --seqlen=512 --hq=32 --hd=128
     python examples/benchmark/kernels.py --op=mixture --tokens=32 --experts=32 --topk=4 --n=1024 --k=2048
     python examples/benchmark/kernels.py --op=decode_layers --model=llama-3.1-8b --batch=32 --seqlen=1344
@@ -61,6 +66,7 @@ class Args:
     splits: int = 0          # decode_attention: KV chunks per sequence (0: the planner's choice)
     w4: int = 0              # moe: 1 = NVFP4 expert weights de-quantised inside the grouped GEMM
     window: int = 4096       # latent and gated attention: keys a position sees; differential attention: its chunk
+    pool: int = 16           # windowed attention with pooled blocks: tokens per block
     sink: int = 0            # latent attention: 1 = a sink per head and no output gate
     copies: int = 0          # operand copies to rotate through (0: enough to exceed the L2)
     help = __doc__
@@ -343,6 +349,137 @@ def bench_gqa_decode(a: Args) -> None:
     ms = timed_graph([lambda c=c: ops.paged_decode(q, *c, meta.block_table, sl, num_splits=meta.num_splits, max_seq_len=a.seqlen) for c in caches], a.iters, a.warmup)
     kvb = a.batch * a.seqlen * a.hkv * a.hd * 4
     report(a, ms, kvb, 4.0 * a.batch * a.hq * a.seqlen * a.hd, {"batch": a.batch, "seqlen": a.seqlen, "part": "the plain kernel"})
+
+
+def _pool(a: Args, n: int):
+    """A capped attention over a window and the pooled blocks in front of it, and the same without blocks, with filled caches."""
+    from types import SimpleNamespace
+    from zml_b200.ops import gqa
+    s = gqa.GqaSpec(a.hq, a.hkv, a.hd, a.hd, a.hd // 2, scale=a.hd ** -0.5, cap=50.0, window=a.window, pool=a.pool, whole_norm=True,
+                    yarn=gqa.Yarn(4.0, 4096, 32.0, 1.0))
+    plain = gqa.GqaSpec(a.hq, a.hkv, a.hd, a.hd, a.hd // 2, scale=a.hd ** -0.5, cap=50.0, window=a.window)
+    caches, bt = _kv(a, n_copies(a, a.batch * min(a.seqlen, a.window) * a.hkv * a.hd * 4) if n == 1 else 2)
+    rows = gqa.pool_rows(a.pool, 64)
+    caches = [(k, v, *(torch.randn(k.shape[0], rows, a.hkv, a.hd, device="cuda").bfloat16() for _ in range(2))) for k, v in caches]
+    t = a.batch * n
+    qs = (torch.arange(a.batch + 1, dtype=torch.int32, device="cuda") * n).int()
+    sl = torch.full((a.batch,), a.seqlen, dtype=torch.int32, device="cuda")
+    pos = (a.seqlen - n + torch.arange(t, device="cuda") % n).int()
+    metas = [SimpleNamespace(is_prefill=n > 1, q_start=qs, seq_lens=sl, block_table=bt, positions=pos, total_q_blocks=a.batch * ((n + 63) // 64),
+                             num_splits=a.splits or ops.decode_plan_splits(a.batch, a.hkv, x.visible(a.seqlen)), max_seq_len=a.seqlen) for x in (s, plain)]
+    proj = torch.randn(t, s.columns(), device="cuda").bfloat16()
+    shape = {"batch": a.batch, "seqlen": a.seqlen, "hq": a.hq, "hkv": a.hkv, "hd": a.hd, "window": a.window, "pool": a.pool}
+    return gqa, (s, plain), caches, metas, proj, bt, shape, t
+
+
+def bench_pool_prefill(a: Args) -> None:
+    gqa, specs, caches, metas, proj, bt, shape, t = _pool(a, a.seqlen)
+    q = torch.randn(t, a.hq, a.hd, device="cuda").bfloat16()
+    w = min(a.window, a.seqlen)
+    pairs = w * (a.seqlen - (w - 1) / 2)
+    blocks = sum((i - w + 1) // a.pool for i in range(w, a.seqlen))
+    nbytes = (2 * t * a.hq * a.hd + 2 * t * a.hkv * a.hd) * 2
+    for s, meta, n, part in ((specs[0], metas[0], pairs + blocks, "window and pooled blocks"), (specs[1], metas[1], pairs, "window alone")):
+        ms = timed([lambda c=c: gqa.attention(q, None, c if s.pool else c[:2], meta, s) for c in caches], a.iters, a.warmup)
+        report(a, ms, nbytes, 4.0 * a.batch * a.hq * a.hd * n, dict(shape, part=part))
+    slots = (bt[:, :, None] * 64 + torch.arange(64, dtype=torch.int32, device="cuda")).reshape(a.batch, -1)[:, :a.seqlen].reshape(-1).int().contiguous()
+    qn, kn = torch.ones(a.hq * a.hd, device="cuda"), torch.ones(a.hkv * a.hd, device="cuda")
+    freq, pos = specs[0].inv_freq("cuda"), metas[0].positions
+    kept = specs[1]
+    for part, fn in (("norms over the projections, rotation, cache write", lambda c: gqa.prep(proj, qn, kn, freq, pos, slots, c, 1e-6, specs[0])),
+                     ("norms per head, rotation, cache write", lambda c: gqa.prep(proj, qn[:a.hd], kn[:a.hd], freq, pos, slots, c[:2], 1e-6, kept))):
+        ms = timed([lambda c=c: fn(c) for c in caches], a.iters, a.warmup)
+        report(a, ms, 2 * t * proj.shape[1] * 2, 0, dict(shape, part=part))
+    ms = timed([lambda c=c: gqa.pool_new(c, metas[0], specs[0]) for c in caches], a.iters, a.warmup)
+    report(a, ms, t * a.hkv * a.hd * 4 * (1 + 1 / a.pool), 0, dict(shape, part="pooled blocks"))
+
+
+def bench_pool_decode(a: Args) -> None:
+    gqa, specs, caches, metas, proj, bt, shape, t = _pool(a, 1)
+    q = torch.randn(t, a.hq, a.hd, device="cuda").bfloat16()
+    w = min(a.window, a.seqlen)
+    for s, meta, n, part in ((specs[0], metas[0], w + (a.seqlen - w) // a.pool, "window and pooled blocks"), (specs[1], metas[1], w, "window alone")):
+        ms = timed_graph([lambda c=c: gqa.attention(q, None, c if s.pool else c[:2], meta, s) for c in caches], a.iters, a.warmup)
+        report(a, ms, a.batch * n * a.hkv * a.hd * 4, 4.0 * a.batch * a.hq * n * a.hd, dict(shape, part=part, splits=meta.num_splits))
+    slots = (bt[:, (a.seqlen - 1) // 64] * 64 + (a.seqlen - 1) % 64).int()
+    qn, kn = torch.ones(a.hq * a.hd, device="cuda"), torch.ones(a.hkv * a.hd, device="cuda")
+    freq, pos = specs[0].inv_freq("cuda"), metas[0].positions
+    for part, fn in (("norms over the projections, rotation, cache write, a block per sequence", lambda c: gqa.prep(proj, qn, kn, freq, pos, slots, c, 1e-6, specs[0], step_table=bt)),
+                     ("norms per head, rotation, cache write", lambda c: gqa.prep(proj, qn[:a.hd], kn[:a.hd], freq, pos, slots, c[:2], 1e-6, specs[1]))):
+        ms = timed_graph([lambda c=c: fn(c) for c in caches], a.iters, a.warmup)
+        report(a, ms, 2 * t * proj.shape[1] * 2, 0, dict(shape, part=part))
+
+
+def bench_gated_scan(a: Args) -> None:
+    from zml_b200.ops import _lib
+    from zml_b200.ops import linear_attn as la
+    n, t, decode = a.k, a.batch * a.seqlen, a.seqlen == 1
+    qs = (torch.arange(a.batch + 1, dtype=torch.int32, device="cuda") * a.seqlen).int()
+    sl = torch.full((a.batch,), a.seqlen + decode, dtype=torch.int32, device="cuda")
+    slots, zb, xb = torch.arange(a.batch, dtype=torch.int32, device="cuda"), torch.randn(n, device="cuda") - 2, torch.randn(n, device="cuda")
+    projs = [torch.randn(t, 3 * n, device="cuda").bfloat16() for _ in range(n_copies(a, t * n * 6))]
+    state = torch.zeros(a.batch, n, device="cuda")
+    nb = a.batch * ((a.seqlen + la.GATED_ROWS - 1) // la.GATED_ROWS)
+    fns = [lambda p=p: la.gated_scan(p[:, :n], p[:, n:2 * n], p[:, 2 * n:], zb, xb, state, qs, sl, slots, 0.7, decode=decode, num_blocks=nb) for p in projs]
+    with contextlib.nullcontext() if decode else _lib.serial_launches():          # as the engine launches them
+        ms = (timed_graph if decode else timed)(fns, a.iters, a.warmup)
+    report(a, ms, t * n * 8 + a.batch * n * 8, 0, {"batch": a.batch, "seqlen": a.seqlen, "width": n})
+
+
+def bench_add_norm(a: Args) -> None:
+    """The residual sum with the norm in front of the next sublayer and its convolution: two launches for prompts, one for a step."""
+    from zml_b200.ops import stream
+    t, d = a.tokens, a.k
+    c = max(2, min(64, math.ceil(256e6 / (t * d * 8)) + 1))
+    xs = [torch.randn(t, d, device="cuda") for _ in range(c)]
+    y, w, b = torch.randn(t, d, device="cuda"), torch.ones(d, device="cuda"), torch.zeros(d, device="cuda")
+    conv = stream.InputConv(torch.randn(4, d, device="cuda"), torch.zeros(t, 3, d, device="cuda"))
+    qs, sl, slots = torch.tensor([0, t], dtype=torch.int32, device="cuda"), torch.tensor([t], dtype=torch.int32, device="cuda"), torch.arange(t, dtype=torch.int32, device="cuda")
+    kw = dict(w=w, b=b, eps=1e-5)
+    ms = timed_graph([lambda x=x: stream.add_norm(x, y, act_dtype=torch.float32, **kw) for x in xs], a.iters, a.warmup)
+    report(a, ms, t * d * 16, 0, {"part": "residual sum and norm", "tokens": t, "d": d})
+    ms = timed_graph([lambda x=x: stream.stream_conv(x, conv, qs, sl, slots, torch.bfloat16) for x in xs], a.iters, a.warmup)
+    report(a, ms, t * d * 6, 0, {"part": "convolution", "tokens": t, "d": d})
+    lens = torch.full((t,), 9, dtype=torch.int32, device="cuda")
+    ms = timed_graph([lambda x=x: stream.add_norm(x, y, act_dtype=torch.bfloat16, conv=conv, seq_lens=lens, slots=slots, **kw) for x in xs], a.iters, a.warmup)
+    report(a, ms, t * d * (14 + 24), 0, {"part": "step: residual sum, norm, convolution", "tokens": t, "d": d})
+    ms = timed_graph([lambda x=x: stream.post_norm(x, w, 1e-5, y, 2.0, act_dtype=torch.bfloat16, conv=conv, seq_lens=lens, slots=slots) for x in xs], a.iters, a.warmup)
+    report(a, ms, t * d * (14 + 24), 0, {"part": "step: norm behind a sublayer, convolution", "tokens": t, "d": d})
+    ms = timed_graph([lambda x=x: stream.sandwich_norm(x, y, w, 0.5, w, 1e-5, act_dtype=torch.bfloat16) for x in xs], a.iters, a.warmup)
+    report(a, ms, t * d * 14, 0, {"part": "norms on both sides of a sublayer", "tokens": t, "d": d})
+
+
+def bench_relu_mixture(a: Args) -> None:
+    """Router by sigmoid scores, routed and shared experts with squared units, and the residual sum with the norm that follows; beside
+    it a gated mixture with the same active parameters and its norms."""
+    from zml_b200.moe import ops as mops
+    from zml_b200.ops import stream
+    e, k, f, d, t = a.experts, a.topk, a.n, a.k, a.tokens
+    c = max(2, min(8, math.ceil(300e6 / (e * f * d * 4)) + 1))
+    rand = lambda *s: torch.randn(*s, device="cuda").bfloat16() * 0.02
+    ws = [mops.pad_plain_experts(rand(e + 1, f, d), rand(e + 1, d, f)) for _ in range(c)]
+    fg = f * 2 // 3
+    gated = [mops.pad_experts(rand(e + 1, fg, d), rand(e + 1, fg, d), rand(e + 1, d, fg)) for _ in range(c)]
+    router, bias = rand(e + 1, d), torch.zeros(e + 1, device="cuda").bfloat16()
+    corr, w, b = torch.zeros(e, device="cuda"), torch.ones(d, device="cuda"), torch.zeros(d, device="cuda")
+    h, x = torch.randn(t, d, device="cuda").bfloat16(), torch.randn(t, d, device="cuda")
+
+    def mine(i):
+        z = ops.gemm(h, router[:e], out_dtype=torch.float32, static_w=True)
+        ids, wt = mops.route(z, k, e, corr, 1, 0, "sigmoid", False, 1.0, False)
+        rows, pos = mops.expert_rows(h, ids, *ws[i], 0, e + 1, "relu2")
+        return stream.add_norm(x, stream.ExpertRows(rows, pos, wt), w, b, 1e-6, torch.float32)
+
+    def theirs(i):
+        z = ops.gemm(h, router, bias=bias, out_dtype=torch.float32, static_w=True)
+        ids, wt = mops.router_topk(z, k + 1)
+        rows, pos = mops.expert_rows(h, ids, *gated[i], 0, e + 1)
+        return stream.sandwich_norm(x, stream.ExpertRows(rows, pos, wt), w, 0.5, w, 1e-6, act_dtype=torch.bfloat16)
+
+    active = min(e, t * k) + 1
+    for part, fn in (("squared units, shared expert", mine), ("gated units, one more choice", theirs)):
+        ms = timed_graph([lambda i=i, fn=fn: fn(i) for i in range(c)], a.iters, a.warmup)
+        report(a, ms, active * 2 * f * d * 2, 4.0 * t * (k + 1) * f * d, {"part": part, "tokens": t, "experts": e, "top": k, "ff": f, "d": d})
 
 
 def _diff(a: Args, n: int):
@@ -677,7 +814,9 @@ OPS = {"moe_w4_timeline": bench_moe_w4_timeline, "gemm_chain_timeline": bench_ge
        "moe": bench_moe, "gated_delta_scan": bench_gated_delta_scan, "decode_layers": bench_decode_layers,
        "latent_prefill": bench_latent_prefill, "latent_decode": bench_latent_decode, "wkv_scan": bench_wkv_scan, "stream": bench_stream,
        "diff_prefill": bench_diff_prefill, "diff_decode": bench_diff_decode, "hyper": bench_hyper, "shared_mixture": bench_shared_mixture,
-       "gqa_prefill": bench_gqa_prefill, "gqa_decode": bench_gqa_decode, "channel_delta": bench_channel_delta, "mixture": bench_mixture}
+       "gqa_prefill": bench_gqa_prefill, "gqa_decode": bench_gqa_decode, "channel_delta": bench_channel_delta, "mixture": bench_mixture,
+       "pool_prefill": bench_pool_prefill, "pool_decode": bench_pool_decode, "gated_scan": bench_gated_scan, "add_norm": bench_add_norm,
+       "relu_mixture": bench_relu_mixture}
 
 
 def main(argv=None) -> int:

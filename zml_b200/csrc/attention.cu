@@ -562,7 +562,8 @@ __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_c
   const int len = p.seq_lens[seq];
   const int first_visible = attn_first_key<EXT>(p, len - 1);
   ZbTileList tiles = {0, 0, (len + 63) >> 6, 0};
-  if constexpr (EXT) tiles = zb_visible_tiles(first_visible, p.keep, tiles.count, 64);
+  const int pooled = EXT && p.pool > 0 ? zb_pooled_visible(len - 1, p.window, p.pool) : 0;
+  if constexpr (EXT) tiles = zb_visible_tiles(first_visible, p.keep, tiles.count, 64, pooled);
   const int nblk = EXT ? tiles.count * 4 : (len + 15) >> 4;
   const int per = p.chunk_blocks;                          // a multiple of 4 (64 keys)
   const int my_splits = max(1, (nblk + per - 1) / per);
@@ -579,9 +580,53 @@ __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_c
   if (EXT && p.sink && split == 0 && warp == 0) m[0] = m[1] = 0.f, l[0] = l[1] = 1.f;
 
   if (warp == 4) {
+    uint32_t stage = 0, phase = 0;
+    int first_tile = tile0;
+    if constexpr (EXT) {
+      // Pooled rows lie a few to a page: the whole warp gathers a tile of them into the layout of the tensor-map copies, and
+      // signals it one tile later, when its copies have landed behind those of the next one.
+      const int pool_end = min(tile1, tiles.pooled);
+      constexpr int chunks = HD / 8;
+      auto signal = [&](uint32_t st) {
+        zb_fence_proxy_async_smem();                       // a later tensor-map copy may overwrite the stage
+        __syncwarp();
+        if (lane == 0) zb_mbar_arrive(&full_bar[st]);
+      };
+      bool ok = true;
+      int pending = -1;
+      for (; first_tile < pool_end; ++first_tile) {
+        ok = __all_sync(0xffffffffu, zb_mbar_wait(&empty_bar[stage], phase ^ 1u, abort_flag));
+        if (!ok) break;
+        const uint32_t ks = zb_smem_u32(smem + stage * 2 * kTileBytes), vs = ks + kTileBytes;
+        const int chunk = lane % chunks;
+        size_t at[2];                                      // rows lane and lane + 32
+#pragma unroll
+        for (int i = 0; i < 2; ++i) at[i] = attn_pool_offset<HD>(p, bt, min(first_tile * 64 + lane + 32 * i, pooled - 1), kvh, kKernelDecode);
+#pragma unroll 8
+        for (int i = 0; i < 64 / (32 / chunks); ++i) {
+          const int row = i * (32 / chunks) + lane / chunks, b = first_tile * 64 + row;
+          const size_t goff = __shfl_sync(0xffffffffu, i * (32 / chunks) < 32 ? at[0] : at[1], row & 31) + chunk * 8;
+          const uint32_t to = tile_off_tma<HD>(row, chunk), bytes = b < pooled ? 16u : 0u;
+          cp_async16(ks + to, p.pool_k + goff, bytes);
+          cp_async16(vs + to, p.pool_v + goff, bytes);
+        }
+        cp_async_commit();
+        if (pending >= 0) {
+          cp_async_wait<1>();
+          signal(pending);
+        }
+        pending = stage;
+        if (++stage == kStages) {
+          stage = 0;
+          phase ^= 1u;
+        }
+      }
+      cp_async_wait<0>();
+      if (pending >= 0) signal(pending);
+      if (!ok) first_tile = tile1;
+    }
     if (lane == 0) {
-      uint32_t stage = 0, phase = 0;
-      for (int t = tile0; t < tile1; ++t) {
+      for (int t = first_tile; t < tile1; ++t) {
         if (!zb_mbar_wait(&empty_bar[stage], phase ^ 1u, abort_flag)) break;
         int page = bt[tiles.at(t)];
         if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelDecode, 11)) page = 0;
@@ -615,10 +660,12 @@ __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_c
     for (int t = tile0; t < tile1; ++t) {
       if (!zb_mbar_wait(&full_bar[stage], phase, abort_flag)) break;
       const int key0 = tiles.at(t) * 64, tok0 = key0 + warp * 16;      // the tile's first key, this warp's 16 keys of it
-      if (tok0 < len && (EXT || ((tok0 >> 4) >= blk0 && (tok0 >> 4) < blk1))) {
+      const bool in_pool = EXT && tiles.is_pooled(t);
+      const int lo = in_pool ? 0 : first_visible, hi = in_pool ? pooled : len;
+      if (tok0 < hi && (EXT || ((tok0 >> 4) >= blk0 && (tok0 >> 4) < blk1))) {
         const uint32_t ks = zb_smem_u32(smem + stage * 2 * kTileBytes);
         const uint32_t vs = ks + kTileBytes;
-        if (tok0 + 16 > len) {
+        if (tok0 + 16 > len && !in_pool) {
           // rows past the end of the sequence hold whatever the page held before: their
           // probabilities are zero, but 0 x NaN would still poison the sum - clear those V rows
           for (int idx = lane; idx < 16 * (HD / 8); idx += 32) {
@@ -632,7 +679,7 @@ __global__ void __launch_bounds__(160) zb_paged_decode_tma_kernel(const __grid_c
         attn_block16<HD, 1>(qf, ks, vs, warp * 16, o, m, l, [&](float v) { return attn_score<EXT>(p, v); },
                             [&](int /*half*/, int col) {
                               const int kidx = tok0 + col;
-                              return kidx < len && (kidx >= first_visible || (EXT && kidx < p.keep));
+                              return kidx < hi && (kidx >= lo || (EXT && kidx < p.keep));
                             });
       }
       __syncwarp();
@@ -1005,7 +1052,7 @@ int zb_paged_decode_ex(const void* q, const void* k_cache, const void* v_cache, 
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = status;
   // 64-token pages and chunks of whole pages: the tensor-map fed kernel; otherwise per-warp cp.async
-  const bool tma = g_decode_tma != 0 && (ext == nullptr || ext->pool == 0) && page_size == 64 && (p.chunk_blocks % 4) == 0 &&
+  const bool tma = g_decode_tma != 0 && page_size == 64 && (p.chunk_blocks % 4) == 0 &&
                    (reinterpret_cast<uintptr_t>(k_cache) & 15) == 0 && (reinterpret_cast<uintptr_t>(v_cache) & 15) == 0;
   if (ext == nullptr) return dispatch_decode<false>(p, head_dim, tma, stream);
   set_ext(p, *ext, scale);

@@ -149,13 +149,18 @@ ZB_DEVICE void store_ext8(const PrefillTcParams& p, size_t tok, int head, int c,
 // zero.  Returns once the rows are in shared memory and visible to the tensor core.
 ZB_DEVICE void gather_pooled_tile(const PrefillTcParams& p, const int32_t* bt, int tile, int end, int kvh, uint8_t* k_dst, uint8_t* v_dst) {
   const int lane = threadIdx.x & 31, chunk = lane & 15;
-#pragma unroll 4
-  for (int r = lane >> 4; r < kKeys; r += 2) {
-    const int b = tile * kKeys + r, have = min(b, end - 1);
-    const int index = zb_pool_page_index(have, p.pool, kKeys);
+  size_t at[2];                                      // rows lane and lane + 32
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int b = min(tile * kKeys + lane + 32 * i, end - 1), index = zb_pool_page_index(b, p.pool, kKeys);
     int page = bt[index];
     if (!ZB_BC_OK(page, ZB_BC_PAGES, kKernelId, 12)) page = 0;
-    const size_t off = (static_cast<size_t>(zb_pool_row(page, index, have, p.pool, kKeys, p.pool_rows)) * p.num_kv_heads + kvh) * kHD + chunk * 8;
+    at[i] = (static_cast<size_t>(zb_pool_row(page, index, b, p.pool, kKeys, p.pool_rows)) * p.num_kv_heads + kvh) * kHD;
+  }
+#pragma unroll 8
+  for (int i = 0; i < kKeys / 2; ++i) {
+    const int r = 2 * i + (lane >> 4), b = tile * kKeys + r;
+    const size_t off = __shfl_sync(0xffffffffu, i < 16 ? at[0] : at[1], r & 31) + chunk * 8;
     const uint32_t to = static_cast<uint32_t>((chunk >> 3) * (kKeys * 128) + r * 128 + (((chunk & 7) ^ (r & 7)) << 4));
     const uint32_t bytes = b < end ? 16u : 0u;
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(zb_smem_u32(k_dst) + to), "l"(p.pool_k + off), "r"(bytes) : "memory");

@@ -87,9 +87,9 @@ ZB_DEVICE void st_elems(float* p, const float (&v)[V]) {
   else *p = v[0];
 }
 
-// Mean key and value of block b of sequence s, by a CTA of NT threads; V elements at a time.
+// Mean key and value of block b of sequence s, by a CTA; V elements at a time.
 template <typename A, int V>
-ZB_DEVICE void pool_block(const PoolArgs& p, const A* kc, const A* vc, int hkv, int ldk, int ldv, int s, int b, int threads) {
+ZB_DEVICE void pool_block(const PoolArgs& p, const A* kc, const A* vc, int hkv, int ldk, int ldv, int s, int b) {
   const int32_t* bt = p.block_table + static_cast<long long>(s) * p.max_pages;
   const int index = min(zb_pool_page_index(b, p.pool, p.page_size), p.max_pages - 1);
   int page = bt[index];
@@ -97,7 +97,7 @@ ZB_DEVICE void pool_block(const PoolArgs& p, const A* kc, const A* vc, int hkv, 
   const long long row = zb_pool_row(page, index, b, p.pool, p.page_size, p.rows);
   const float scale = 1.f / static_cast<float>(p.pool);
   const int nk = hkv * ldk, n = nk + hkv * ldv;
-  for (int i = threadIdx.x * V; i < n; i += threads * V) {
+  for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {
     const bool is_k = i < nk;
     const int c = is_k ? i : i - nk, ld = is_k ? nk : n - nk;
     const A* src = (is_k ? kc : vc) + c;
@@ -120,10 +120,10 @@ ZB_DEVICE void pool_block(const PoolArgs& p, const A* kc, const A* vc, int hkv, 
   }
 }
 
-// One CTA per token, L lanes (a warp or half of one) per head; NR groups of V neighbouring elements per lane.
+// One CTA per token (STEP: several, which share its heads, and blocks are pooled), L lanes (a warp or half of one) per head; NR groups of V neighbouring elements per lane.
 constexpr int kPrepThreads = 256;
 
-template <typename A, int NR, int V, int L>
+template <typename A, int NR, int V, int L, bool STEP>
 __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrepArgs p) {
   extern __shared__ __align__(16) float prep_smem[];      // [rot / 2] (cos, sin) | [warps][rot] the rotated part's elements
   zb_pdl_launch();
@@ -181,7 +181,9 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
   if (slot >= p.num_rows) (void)ZB_BC_OK(slot, p.num_rows, kKernelGqaPrep, 1);
   const bool slot_ok = slot >= 0 && slot < p.num_rows;
   const int keys = p.hkv * p.maps, heads = p.hq + keys + p.hkv;
-  for (int h = team; h < heads; h += kPrepThreads / L) {
+  const int done = STEP && p.pool.pool > 0 && slot_ok ? p.positions[t] + 1 : 0;
+  const bool pool_now = STEP && done > 0 && done % p.pool.pool == 0;     // this token completes a block
+  for (int h = team + (STEP ? kPrepThreads / L * blockIdx.y : 0); h < heads; h += kPrepThreads / L * (STEP ? gridDim.y : 1)) {
     const bool is_q = h < p.hq, is_v = h >= p.hq + keys;
     if (!is_q && !slot_ok) continue;
     const int u = is_q ? h : (is_v ? h - p.hq - keys : h - p.hq);        // row among its kind
@@ -248,13 +250,44 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
         st_elems<V>(dst + i + (map == 0 ? ld : -ld), zero);
       }
     }
-  }
-  if (p.pool.pool > 0 && slot_ok) {
-    const int done = p.positions[t] + 1;
-    if (done % p.pool.pool == 0) {
-      __syncthreads();                                     // this token's rows are written
-      pool_block<A, V>(p.pool, reinterpret_cast<const A*>(p.k_cache), reinterpret_cast<const A*>(p.v_cache), p.hkv, p.ldk, p.ldv, t,
-                       done / p.pool.pool - 1, kPrepThreads);
+    if (STEP && pool_now && !is_q) {                               // every lane averages the elements that it has written
+      const A* cache = reinterpret_cast<const A*>(is_v ? p.v_cache : p.k_cache) + static_cast<long long>(u) * ld;
+      const long long step = static_cast<long long>(p.hkv) * ld;
+      const int32_t* bt = p.pool.block_table + static_cast<long long>(t) * p.pool.max_pages;
+#pragma unroll
+      for (int r = 0; r < NR; ++r)
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[r][e] = 0.f;
+      auto page_of = [&](int index) {
+        const int page = bt[min(index, p.pool.max_pages - 1)];
+        return ZB_BC_OK(page, ZB_BC_PAGES, kKernelGqaPool, 3) ? page : 0;
+      };
+#pragma unroll 8
+      for (int j = 0; j < p.pool.pool; ++j) {
+        const int tok = done - p.pool.pool + j;
+        const A* row_j = cache + (static_cast<long long>(page_of(tok / p.pool.page_size)) * p.pool.page_size + tok % p.pool.page_size) * step;
+#pragma unroll
+        for (int r = 0; r < NR; ++r) {
+          const int i = (lane + L * r) * V;
+          float w[V];
+#pragma unroll
+          for (int e = 0; e < V; ++e) w[e] = 0.f;
+          if (i < ld) ld_elems<V>(w, row_j + i);
+#pragma unroll
+          for (int e = 0; e < V; ++e) v[r][e] += w[e];
+        }
+      }
+      const int b = done / p.pool.pool - 1, index = min(zb_pool_page_index(b, p.pool.pool, p.pool.page_size), p.pool.max_pages - 1);
+      A* out = reinterpret_cast<A*>(is_v ? p.pool.v : p.pool.k) +
+               zb_pool_row(page_of(index), index, b, p.pool.pool, p.pool.page_size, p.pool.rows) * step + static_cast<long long>(u) * ld;
+      const float scale = 1.f / static_cast<float>(p.pool.pool);
+#pragma unroll
+      for (int r = 0; r < NR; ++r) {
+        const int i = (lane + L * r) * V;
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[r][e] *= scale;
+        if (i < ld) st_elems<V>(out + i, v[r]);
+      }
     }
   }
 }
@@ -269,32 +302,36 @@ __global__ void __launch_bounds__(128) zb_gqa_pool_kernel(const PoolArgs p, cons
   for (int s = 0; s < b.num_seqs; ++s) {
     const int len = b.seq_lens[s], first = (len - (b.q_start[s + 1] - b.q_start[s])) / p.pool, n = len / p.pool - first;
     if (idx < n) {
-      pool_block<A, V>(p, reinterpret_cast<const A*>(k_cache), reinterpret_cast<const A*>(v_cache), hkv, ldk, ldv, s, first + idx, 128);
+      pool_block<A, V>(p, reinterpret_cast<const A*>(k_cache), reinterpret_cast<const A*>(v_cache), hkv, ldk, ldv, s, first + idx);
       return;
     }
     idx -= n;
   }
 }
 
-template <typename A, int V>
+template <typename A, int V, bool STEP>
 cudaError_t launch_prep(const GqaPrepArgs& p, int tokens, cudaStream_t s) {
   const int widest = max(max(p.ldq, p.hkv > 0 ? p.ldk : 0) / p.maps, p.hkv > 0 ? p.ldv : 0);
   const bool narrow = max(p.dk, p.hkv > 0 ? p.ldk / p.maps : 0) <= 16 * V && widest <= 32 * V;      // keys in half a warp, values in two rounds
   const size_t smem = static_cast<size_t>(p.rot) * (1 + kPrepThreads / (narrow ? 16 : 32)) * sizeof(float);
   if (smem > 48 * 1024) return cudaErrorInvalidValue;
+  // few tokens: several CTAs per token, so that a decode step does not wait for one CTA to walk over all heads
+  const int teams = kPrepThreads / (narrow ? 16 : 32), heads = p.hq + p.hkv * (p.maps + 1);
+  const dim3 grid(tokens, STEP ? min((heads + teams - 1) / teams, 8) : 1);
   const int nr = (widest + 32 * V - 1) / (32 * V);
-  if (narrow) return zb_launch(zb_gqa_prep_kernel<A, 2, V, 16>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
-  if (nr <= 1) return zb_launch(zb_gqa_prep_kernel<A, 1, V, 32>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
-  if (nr <= 2) return zb_launch(zb_gqa_prep_kernel<A, 2, V, 32>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
-  if (nr <= 8) return zb_launch(zb_gqa_prep_kernel<A, 8, V, 32>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
-  if (nr <= 32) return zb_launch(zb_gqa_prep_kernel<A, 32, V, 32>, dim3(tokens), dim3(kPrepThreads), smem, s, p);
+  if (narrow) return zb_launch(zb_gqa_prep_kernel<A, 2, V, 16, STEP>, grid, dim3(kPrepThreads), smem, s, p);
+  if (nr <= 1) return zb_launch(zb_gqa_prep_kernel<A, 1, V, 32, STEP>, grid, dim3(kPrepThreads), smem, s, p);
+  if (nr <= 2) return zb_launch(zb_gqa_prep_kernel<A, 2, V, 32, STEP>, grid, dim3(kPrepThreads), smem, s, p);
+  if (nr <= 8) return zb_launch(zb_gqa_prep_kernel<A, 8, V, 32, STEP>, grid, dim3(kPrepThreads), smem, s, p);
+  if (nr <= 32) return zb_launch(zb_gqa_prep_kernel<A, 32, V, 32, STEP>, grid, dim3(kPrepThreads), smem, s, p);
   return cudaErrorInvalidValue;
 }
 template <typename A>
 cudaError_t launch_prep(const GqaPrepArgs& p, int tokens, cudaStream_t s) {
   const bool vec = p.dk % 4 == 0 && p.dv % 4 == 0 && p.ld_in % 4 == 0 && p.ldq / p.maps % 4 == 0 && p.ldk / p.maps % 4 == 0 && p.ldv % 4 == 0 &&
                    (reinterpret_cast<uintptr_t>(p.in) & (4 * sizeof(A) - 1)) == 0;
-  return vec ? launch_prep<A, 4>(p, tokens, s) : launch_prep<A, 1>(p, tokens, s);
+  if (p.pool.pool > 0 || tokens <= 128) return vec ? launch_prep<A, 4, true>(p, tokens, s) : launch_prep<A, 1, true>(p, tokens, s);
+  return vec ? launch_prep<A, 4, false>(p, tokens, s) : launch_prep<A, 1, false>(p, tokens, s);
 }
 
 // ------------------------------------------------------------------------------------------ attention, any sizes
