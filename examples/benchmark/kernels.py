@@ -422,7 +422,7 @@ def bench_gated_scan(a: Args) -> None:
     nb = a.batch * ((a.seqlen + la.GATED_ROWS - 1) // la.GATED_ROWS)
     fns = [lambda p=p: la.gated_scan(p[:, :n], p[:, n:2 * n], p[:, 2 * n:], zb, xb, state, qs, sl, slots, 0.7, decode=decode, num_blocks=nb) for p in projs]
     with contextlib.nullcontext() if decode else _lib.serial_launches():          # as the engine launches them
-        ms = (timed_graph if decode else timed)(fns, a.iters, a.warmup)
+        ms = timed_graph(fns, a.iters, a.warmup)
     report(a, ms, t * n * 8 + a.batch * n * 8, 0, {"batch": a.batch, "seqlen": a.seqlen, "width": n})
 
 

@@ -87,7 +87,7 @@ ZB_DEVICE void st_elems(float* p, const float (&v)[V]) {
   else *p = v[0];
 }
 
-// Mean key and value of block b of sequence s, by a CTA; V elements at a time.
+// Mean key and value of block b of sequence s: V elements per thread of a row of CTAs.
 template <typename A, int V>
 ZB_DEVICE void pool_block(const PoolArgs& p, const A* kc, const A* vc, int hkv, int ldk, int ldv, int s, int b) {
   const int32_t* bt = p.block_table + static_cast<long long>(s) * p.max_pages;
@@ -97,7 +97,8 @@ ZB_DEVICE void pool_block(const PoolArgs& p, const A* kc, const A* vc, int hkv, 
   const long long row = zb_pool_row(page, index, b, p.pool, p.page_size, p.rows);
   const float scale = 1.f / static_cast<float>(p.pool);
   const int nk = hkv * ldk, n = nk + hkv * ldv;
-  for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {
+  const int i = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (i < n) {
     const bool is_k = i < nk;
     const int c = is_k ? i : i - nk, ld = is_k ? nk : n - nk;
     const A* src = (is_k ? kc : vc) + c;
@@ -292,7 +293,7 @@ __global__ void __launch_bounds__(kPrepThreads) zb_gqa_prep_kernel(const GqaPrep
   }
 }
 
-// The blocks that a varlen batch completes, one CTA each.
+// The blocks that a varlen batch completes, a row of CTAs each.
 template <typename A, int V>
 __global__ void __launch_bounds__(128) zb_gqa_pool_kernel(const PoolArgs p, const void* k_cache, const void* v_cache, int hkv, int ldk, int ldv,
                                                           const ZbVarlen b) {
@@ -508,7 +509,8 @@ int zb_gqa_pool(const void* k_cache, const void* v_cache, void* pool_k, void* po
   const bool vec = ldk % 4 == 0 && ldv % 4 == 0;
   const auto kernel = act_f32 ? (vec ? zb_gqa_pool_kernel<float, 4> : zb_gqa_pool_kernel<float, 1>)
                               : (vec ? zb_gqa_pool_kernel<__nv_bfloat16, 4> : zb_gqa_pool_kernel<__nv_bfloat16, 1>);
-  const cudaError_t e = zb_launch(kernel, dim3(num_blocks), dim3(128), 0, s, p, k_cache, v_cache, hkv, ldk, ldv, b);
+  const int threads = (hkv * (ldk + ldv) + (vec ? 3 : 0)) / (vec ? 4 : 1);
+  const cudaError_t e = zb_launch(kernel, dim3(num_blocks, (threads + 127) / 128), dim3(128), 0, s, p, k_cache, v_cache, hkv, ldk, ldv, b);
   zb_count_launch(1);
   return static_cast<int>(e != cudaSuccess ? e : cudaGetLastError());
 }
