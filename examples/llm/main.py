@@ -12,7 +12,7 @@ models, one conversation).  --system puts a system message in front of the first
 Without --prompt an interactive chat loop starts (history in ~/.llm_chat_history).  For
 tensor / expert parallelism launch one process per GPU:
     python -m torch.distributed.run --nproc-per-node=8 --master-addr 127.0.0.1 examples/llm/main.py --model=...
-Supported `model_type`s: llama, mistral, qwen2, qwen3, qwen3_moe, qwen3_5, qwen3_5_moe, lfm2, dopurax, kirisun, sodotar (the last three by `architecture`).
+Supported `model_type`s: llama, mistral, qwen2, qwen3, qwen3_moe, qwen3_5, qwen3_5_moe, lfm2, dopurax, kirisun, sodotar, dogidra (the last four by `architecture`).
 """
 from __future__ import annotations
 

@@ -187,7 +187,7 @@ def test_stretched_frequencies(yarn, rot, base):
 #       heads kv dim vdim window pool cap
 POOL = {
     "tensor cores": (4, 2, 128, 128, 70, 6, 20.0),
-    "tensor cores, narrower": (6, 1, 96, 64, 100, 8, 50.0),
+    "tensor cores, narrower": (6, 1, 88, 72, 100, 8, 40.0),
     "tensor cores, odd values": (2, 1, 90, 101, 64, 16, 20.0),
     "tensor cores, no cap": (4, 2, 128, 120, 33, 5, 0.0),
     "tensor cores, one token": (2, 1, 128, 128, 1, 1, 20.0),
